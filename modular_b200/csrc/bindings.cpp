@@ -8,6 +8,7 @@
 #include <stdexcept>
 #include <string>
 
+#include "bindings.h"
 #include "common/api.h"
 #include "engine/decoder_executor.h"
 #include "runtime/runtime.h"
@@ -15,7 +16,8 @@
 namespace py = pybind11;
 using torch::Tensor;
 
-namespace {
+namespace mb {
+namespace bind {
 
 cudaStream_t cur_stream() { return at::cuda::getCurrentCUDAStream().stream(); }
 
@@ -61,6 +63,13 @@ int num_sms() {
   if (!n) n = at::cuda::getCurrentDeviceProperties()->multiProcessorCount;
   return n;
 }
+
+}  // namespace bind
+}  // namespace mb
+
+using namespace mb::bind;
+
+namespace {
 
 // y = x @ w.T with optional fusions; see mb_gemm_bf16.
 void gemm_bf16(const Tensor& x, const Tensor& w, Tensor& y, const c10::optional<Tensor>& residual,
@@ -1023,7 +1032,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
                                 cache.stride(0), cache.size(0), block_table.data_ptr<int32_t>(),
                                 block_table.stride(0), q_start.data_ptr<int32_t>(), q_len.data_ptr<int32_t>(),
                                 kv_len.data_ptr<int32_t>(), q_lat.size(0), block_table.size(0), q_lat.size(1),
-                                cache.size(1), scale, error_flag(), cur_stream()),
+                                cache.size(1), scale, nullptr, 64, error_flag(), cur_stream()),
                "mla_decode_tc");
       return;
     }
@@ -1034,7 +1043,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
                                  cache.stride(0), cache.size(0), block_table.data_ptr<int32_t>(),
                                  block_table.stride(0), q_start.data_ptr<int32_t>(), q_len.data_ptr<int32_t>(),
                                  kv_len.data_ptr<int32_t>(), q_lat.size(0), block_table.size(0), q_lat.size(1),
-                                 cache.size(1), scale, scratch.data_ptr<int32_t>(), error_flag(), cur_stream()),
+                                 cache.size(1), scale, nullptr, 64, scratch.data_ptr<int32_t>(), error_flag(),
+                                 cur_stream()),
                "mla_prefill_tc");
       return;
     }
@@ -1241,4 +1251,5 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
       .def("set_profiling", &PyDecoderExecutor::set_profiling)
       .def("profile", &PyDecoderExecutor::profile);
   mb::bind_runtime(m);
+  mb::bind_layers(m);
 }

@@ -1,0 +1,281 @@
+// Bindings of the layer kernels that exist in bf16 and fp32: the fp32 residual seam, latent attention of any size, the
+// gated delta rule, token-id expert routing and the fp32 products.
+#include "bindings.h"
+
+#include "common/api.h"
+
+namespace py = pybind11;
+using torch::Tensor;
+using namespace mb::bind;
+typedef c10::optional<Tensor> Opt;
+
+namespace {
+
+int dtype_of(const Tensor& t, const char* what) {
+  TORCH_CHECK(t.scalar_type() == at::kBFloat16 || t.scalar_type() == at::kFloat, what, ": bf16 or fp32 expected");
+  return t.scalar_type() == at::kFloat ? 1 : 0;
+}
+bool given(const Opt& t) { return t.has_value() && t->defined(); }
+// a CUDA matrix with unit column stride of `dtype`; returns its row stride
+int ld_of(const Tensor& t, at::ScalarType dtype, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.dim() == 2 && t.stride(1) == 1 && t.scalar_type() == dtype, what,
+              ": CUDA matrix of the expected dtype with unit column stride");
+  return static_cast<int>(t.stride(0));
+}
+const int32_t* i32(const Tensor& t, int64_t n, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.is_contiguous() && t.scalar_type() == at::kInt && t.numel() >= n, what, ": int32 CUDA tensor");
+  return t.data_ptr<int32_t>();
+}
+const float* f32(const Tensor& t, int64_t n, const char* what) {
+  TORCH_CHECK(t.is_cuda() && t.is_contiguous() && t.scalar_type() == at::kFloat && t.numel() >= n, what, ": fp32 CUDA tensor");
+  return t.data_ptr<float>();
+}
+
+void residual_norm(Tensor& x, const Opt& ids, const Opt& table, double scale, const Opt& a, const Opt& b, const Opt& e,
+                   const Opt& inverse, int top_k, double pair_w, const Opt& rows, const Opt& w1, const Opt& n1,
+                   const Opt& w2, const Opt& n2, const Opt& scatter, int cols, bool store_x, double eps, int n_rows) {
+  MbResidualNorm p = {};
+  p.ldx = ld_of(x, at::kFloat, "x");
+  p.x = x.data_ptr<float>();
+  p.cols = cols; p.cols_pad = static_cast<int>(x.size(1)); p.store_x = store_x; p.eps = static_cast<float>(eps);
+  p.n_rows = n_rows;
+  const int64_t T = x.size(0);
+  at::ScalarType dt = given(w1) ? w1->scalar_type() : given(a) ? a->scalar_type() : at::kBFloat16;
+  if (given(table)) {
+    TORCH_CHECK(given(ids) && ids->scalar_type() == at::kLong && ids->numel() >= T, "residual_norm: ids");
+    p.ld_table = ld_of(*table, dt, "table");
+    TORCH_CHECK(table->size(1) == p.cols_pad, "residual_norm: table width");
+    p.table = table->data_ptr(); p.ids = ids->data_ptr<int64_t>(); p.scale = static_cast<float>(scale);
+    p.vocab = static_cast<int>(table->size(0));
+  }
+  auto branch = [&](const Opt& t, const char* what, int64_t min_rows) {
+    const int ld = ld_of(*t, dt, what);
+    TORCH_CHECK(t->size(1) >= p.cols_pad && t->size(0) >= min_rows, "residual_norm: ", what, " shape");
+    return ld;
+  };
+  if (given(a)) { p.lda = branch(a, "a", T); p.a = a->data_ptr(); }
+  if (given(b)) { p.ldb = branch(b, "b", T); p.b = b->data_ptr(); }
+  if (given(e)) {
+    p.lde = branch(e, "e", T * top_k); p.e = e->data_ptr();
+    TORCH_CHECK(given(inverse), "residual_norm: inverse");
+    p.inverse = i32(*inverse, T * top_k, "inverse"); p.top_k = top_k; p.pair_w = static_cast<float>(pair_w);
+  }
+  if (given(rows)) p.rows = i32(*rows, n_rows, "rows");
+  else TORCH_CHECK(n_rows <= T, "residual_norm: rows");
+  if (given(w1)) {
+    TORCH_CHECK(given(n1) && w1->is_contiguous() && w1->numel() >= p.cols_pad, "residual_norm: w1 / n1");
+    p.w1 = w1->data_ptr(); p.ld1 = branch(n1, "n1", n_rows); p.n1 = n1->data_ptr();
+  }
+  if (given(w2)) {
+    TORCH_CHECK(given(n2) && w2->is_contiguous() && w2->scalar_type() == dt && w2->numel() >= p.cols_pad, "residual_norm: w2 / n2");
+    p.w2 = w2->data_ptr(); p.n2 = n2->data_ptr();
+    if (given(scatter)) {
+      TORCH_CHECK(scatter->dim() == 2, "residual_norm: scatter");
+      p.k2 = static_cast<int>(scatter->size(1));
+      p.scatter = i32(*scatter, T * p.k2, "scatter");
+      p.ld2 = branch(n2, "n2", T * p.k2);
+    } else {
+      p.ld2 = branch(n2, "n2", n_rows);
+    }
+  }
+  check_rc(mb_residual_norm(&p, dt == at::kFloat ? 1 : 0, cur_stream()), "residual_norm");
+}
+
+void latent_post_down(const Tensor& x, int q_rank, const Opt& gamma_q, const Opt& q_out, int kv_off, int R, int Rp,
+                      const Opt& gamma_kv, int rot_dim, int Dp, int dims, bool interleaved, double eps,
+                      const Tensor& positions, const Tensor& cos_sin, const Tensor& slots, const Opt& cache) {
+  const int dt = dtype_of(x, "x"), ld = ld_of(x, x.scalar_type(), "x");
+  const int64_t T = x.size(0);
+  TORCH_CHECK(slots.scalar_type() == at::kLong && slots.numel() >= T && cos_sin.dim() == 2 && cos_sin.size(1) == dims &&
+                  q_rank <= x.size(1) && kv_off + (kv_off >= 0 ? R + rot_dim : 0) <= x.size(1),
+              "latent_post_down: slots / cos_sin / columns");
+  int ld_q = 0, q_pad = 0;
+  if (q_rank > 0) {
+    TORCH_CHECK(given(gamma_q) && given(q_out) && gamma_q->numel() >= q_rank && gamma_q->scalar_type() == x.scalar_type() &&
+                    q_out->size(0) >= T, "latent_post_down: query latent");
+    ld_q = ld_of(*q_out, x.scalar_type(), "q_out"); q_pad = static_cast<int>(q_out->size(1));
+  }
+  int page = 1, ld_cache = 0;
+  int64_t page_stride = 0;
+  if (kv_off >= 0) {
+    TORCH_CHECK(given(gamma_kv) && gamma_kv->numel() >= R && gamma_kv->scalar_type() == x.scalar_type() && given(cache) &&
+                    cache->dim() == 3 && cache->stride(2) == 1 && cache->size(2) >= Rp + Dp && cache->scalar_type() == x.scalar_type(),
+                "latent_post_down: cache");
+    page = static_cast<int>(cache->size(1)); ld_cache = static_cast<int>(cache->stride(1)); page_stride = cache->stride(0);
+  }
+  check_rc(mb_latent_post_down(x.data_ptr(), ld, static_cast<int>(T), q_rank, q_pad, optptr(gamma_q),
+                               const_cast<void*>(optptr(q_out)), ld_q, kv_off, R, Rp, optptr(gamma_kv), rot_dim, Dp, dims,
+                               interleaved ? 1 : 0, static_cast<float>(eps), i32(positions, T, "positions"),
+                               f32(cos_sin, 0, "cos_sin"), slots.data_ptr<int64_t>(), const_cast<void*>(optptr(cache)), page,
+                               page_stride, ld_cache, dt, cur_stream()),
+           "latent_post_down");
+}
+
+// q_lat [T, h, Rp], q_rope [T, h, Dp] (any token stride, heads contiguous blocks), cache [pages, page, >= Rp + Dp]
+void latent_attention(const Tensor& q_lat, const Tensor& q_rope, const Tensor& cache, const Tensor& block_table,
+                      const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, Tensor& out, double scale,
+                      const Opt& sink, bool one_token, const Opt& ws, bool allow_tc) {
+  const int dt = dtype_of(q_lat, "q_lat");
+  TORCH_CHECK(q_lat.is_cuda() && q_lat.dim() == 3 && q_lat.stride(2) == 1 && q_rope.dim() == 3 && q_rope.stride(2) == 1 &&
+                  out.is_contiguous() && out.sizes() == q_lat.sizes() && q_rope.size(0) == q_lat.size(0) &&
+                  q_rope.size(1) == q_lat.size(1) && q_rope.scalar_type() == q_lat.scalar_type() &&
+                  out.scalar_type() == q_lat.scalar_type() && cache.scalar_type() == q_lat.scalar_type() && cache.dim() == 3 &&
+                  cache.stride(2) == 1 && cache.size(2) >= q_lat.size(2) + q_rope.size(2) && block_table.stride(1) == 1 &&
+                  block_table.scalar_type() == at::kInt,
+              "latent_attention layout");
+  const int T = q_lat.size(0), h = q_lat.size(1), R = q_lat.size(2), D = q_rope.size(2), B = q_len.numel();
+  const float* sk = given(sink) ? f32(*sink, h, "sink") : nullptr;
+  const int32_t *qs = i32(q_start, B, "q_start"), *ql = i32(q_len, B, "q_len"), *kl = i32(kv_len, B, "kv_len");
+  const int32_t* bt = block_table.data_ptr<int32_t>();
+  const int page = cache.size(1), bts = block_table.stride(0), ldc = cache.stride(1);
+  TORCH_CHECK(block_table.size(0) >= B, "latent_attention: block table rows");
+  const bool mma = dt == 0 && D == 64 && (R == 64 || R == 128 || R == 192 || R == 256 || R == 384 || R == 512) &&
+                   q_lat.stride(1) == R;
+  // 512-wide latents with a multiple of 128 heads: tcgen05 kernel, which addresses contiguous query rows
+  if (mma && allow_tc && q_lat.is_contiguous() && q_rope.stride(0) == h * q_rope.stride(1) && ldc == R + D && cache.stride(0) % (R + D) == 0 &&
+      mb_mla_tc_usable(T, T, h, R, page)) {
+    if (one_token) {
+      check_rc(mb_mla_decode_tc(q_lat.data_ptr(), q_rope.data_ptr(), out.data_ptr(), cache.data_ptr(), cache.stride(0),
+                                cache.size(0), bt, bts, qs, ql, kl, T, B, h, page, scale, sk,
+                                static_cast<int>(q_rope.stride(1)), error_flag(), cur_stream()),
+               "mla_decode_tc");
+    } else {
+      auto scratch = at::empty({2 * static_cast<int64_t>(T)}, q_start.options());
+      check_rc(mb_mla_prefill_tc(q_lat.data_ptr(), q_rope.data_ptr(), out.data_ptr(), cache.data_ptr(), cache.stride(0),
+                                 cache.size(0), bt, bts, qs, ql, kl, T, B, h, page, scale, sk,
+                                 static_cast<int>(q_rope.stride(1)), scratch.data_ptr<int32_t>(),
+                                 error_flag(), cur_stream()),
+               "mla_prefill_tc");
+    }
+    return;
+  }
+  if (mma) {
+    check_rc(mb_mla_paged_attention_ex(q_lat.data_ptr(), q_lat.stride(0), q_rope.data_ptr(), q_rope.stride(0), q_rope.stride(1),
+                                       out.data_ptr(), cache.data_ptr(), cache.stride(0), ldc, bt, bts, qs, ql, kl, T, B, h, R, page, scale, sk,
+                                       given(ws) ? ws->data_ptr() : nullptr, given(ws) ? ws->nbytes() : 0, num_sms(),
+                                       cur_stream()),
+             "mla_paged_attention");
+    return;
+  }
+  check_rc(mb_latent_attention(q_lat.data_ptr(), q_lat.stride(0), q_lat.stride(1), q_rope.data_ptr(), q_rope.stride(0),
+                               q_rope.stride(1), out.data_ptr(), out.stride(0), out.stride(1), cache.data_ptr(),
+                               cache.stride(0), ldc, page, bt, bts, qs, ql, kl, T, B, h, R, D, scale, sk, dt, cur_stream()),
+           "latent_attention");
+}
+
+// x: projection rows with the column blocks of q, k, v and beta at the given offsets; see MbDelta for the rest
+void delta_rule(const Tensor& x, int q_off, int k_off, int v_off, int b_off, const Tensor& conv_w, const Tensor& z,
+                const Tensor& A_log, const Tensor& dt_bias, const Tensor& gate, const Tensor& norm_w, double eps,
+                std::vector<Tensor>& scratch, Tensor& out, Tensor& state, Tensor& conv_state, const Tensor& state_idx,
+                const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, int heads, int kv_heads, int dim, int vdim,
+                bool one_token) {
+  MbDelta p = {};
+  const int dt = dtype_of(x, "x");
+  const at::ScalarType st = x.scalar_type();
+  p.T = x.size(0); p.B = q_len.numel();
+  p.heads = heads; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim; p.one_token = one_token;
+  p.dim_pad = mb_delta_dim_pad(dim);
+  TORCH_CHECK(p.dim_pad > 0, "delta_rule: key width ", dim, " is beyond the supported maximum");
+  const int64_t T = p.T, C = 2ll * kv_heads * dim + static_cast<int64_t>(heads) * vdim;
+  p.x = x.data_ptr(); p.ldx = ld_of(x, st, "x");
+  p.q_off = q_off; p.k_off = k_off; p.v_off = v_off; p.b_off = b_off;
+  TORCH_CHECK(q_off + kv_heads * dim <= x.size(1) && k_off + kv_heads * dim <= x.size(1) &&
+                  v_off + heads * vdim <= x.size(1) && b_off + heads <= x.size(1), "delta_rule: columns");
+  TORCH_CHECK(conv_w.is_contiguous() && conv_w.scalar_type() == st && conv_w.dim() == 2 && conv_w.size(0) == C, "delta_rule: conv_w");
+  p.conv_w = conv_w.data_ptr(); p.taps = conv_w.size(1);
+  p.ldz = ld_of(z, at::kFloat, "z"); p.z = z.data_ptr<float>();
+  TORCH_CHECK(z.size(0) >= T && z.size(1) >= heads * dim, "delta_rule: z");
+  p.A_log = f32(A_log, heads, "A_log"); p.dt_bias = f32(dt_bias, static_cast<int64_t>(heads) * dim, "dt_bias");
+  p.ld_gate = ld_of(gate, st, "gate"); p.gate = gate.data_ptr();
+  TORCH_CHECK(gate.size(0) >= T && gate.size(1) >= heads * vdim, "delta_rule: gate");
+  TORCH_CHECK(norm_w.is_contiguous() && norm_w.scalar_type() == st && norm_w.numel() >= vdim, "delta_rule: norm_w");
+  p.norm_w = norm_w.data_ptr(); p.eps = static_cast<float>(eps);
+  TORCH_CHECK(scratch.size() == 7, "delta_rule: scratch is {q, k, g, v, beta, kq, o}");
+  const int64_t need[7] = {T * kv_heads * p.dim_pad, T * kv_heads * p.dim_pad, T * heads * p.dim_pad, T * heads * vdim,
+                           T * heads, T * kv_heads, T * heads * vdim};
+  float** dst[7] = {&p.q, &p.k, &p.g, &p.v, &p.beta, &p.kq, &p.o};
+  for (int i = 0; i < 7; ++i) *dst[i] = const_cast<float*>(f32(scratch[i], need[i], "delta_rule scratch"));
+  p.ld_out = ld_of(out, st, "out"); p.out = out.data_ptr();
+  TORCH_CHECK(out.size(0) >= T && out.size(1) >= heads * vdim, "delta_rule: out");
+  TORCH_CHECK(state.is_contiguous() && state.scalar_type() == at::kFloat && state.dim() == 4 && state.size(1) == heads &&
+                  state.size(2) == vdim && state.size(3) == p.dim_pad, "delta_rule: state [slots, heads, vdim, dim_pad]");
+  TORCH_CHECK(conv_state.is_contiguous() && conv_state.scalar_type() == at::kFloat && conv_state.dim() == 3 &&
+                  conv_state.size(1) == C && conv_state.size(2) == p.taps - 1, "delta_rule: conv_state [slots, channels, taps - 1]");
+  p.state = state.data_ptr<float>(); p.conv_state = conv_state.data_ptr<float>();
+  p.state_idx = i32(state_idx, p.B, "state_idx"); p.q_start = i32(q_start, p.B, "q_start");
+  p.q_len = i32(q_len, p.B, "q_len"); p.kv_len = i32(kv_len, p.B, "kv_len");
+  check_rc(mb_delta_rule(&p, dt, num_sms(), cur_stream()), "delta_rule");
+}
+
+}  // namespace
+
+void mb::bind_layers(py::module_& m) {
+  const auto none = py::none();
+  m.def("residual_norm", &residual_norm, py::arg("x"), py::arg("ids") = none, py::arg("table") = none, py::arg("scale") = 1.0,
+        py::arg("a") = none, py::arg("b") = none, py::arg("e") = none, py::arg("inverse") = none, py::arg("top_k") = 0,
+        py::arg("pair_w") = 1.0, py::arg("rows") = none, py::arg("w1") = none, py::arg("n1") = none, py::arg("w2") = none,
+        py::arg("n2") = none, py::arg("scatter") = none, py::arg("cols") = 0, py::arg("store_x") = true, py::arg("eps") = 1e-6,
+        py::arg("n_rows") = 0);
+  m.def("gelu_tanh", [](Tensor& x) {
+    TORCH_CHECK(x.is_cuda() && x.is_contiguous(), "gelu_tanh: contiguous CUDA tensor");
+    check_rc(mb_gelu_tanh(x.data_ptr(), x.numel(), dtype_of(x, "x"), cur_stream()), "gelu_tanh");
+  });
+  m.def("sigmoid_gate", [](Tensor& o, const Tensor& g, int cols) {
+    const int ldo = ld_of(o, o.scalar_type(), "o"), ldg = ld_of(g, o.scalar_type(), "g");
+    TORCH_CHECK(o.size(1) >= cols && g.size(1) >= cols && g.size(0) >= o.size(0), "sigmoid_gate shapes");
+    check_rc(mb_sigmoid_gate(o.data_ptr(), ldo, g.data_ptr(), ldg, o.size(0), cols, dtype_of(o, "o"), cur_stream()), "sigmoid_gate");
+  });
+  m.def("latent_post_down", &latent_post_down);
+  m.def("rotate_heads", [](Tensor& x, int heads, int head_stride, int dims, bool interleaved, const Tensor& positions,
+                           const Tensor& cos_sin) {
+    const int ld = ld_of(x, x.scalar_type(), "x");
+    TORCH_CHECK(static_cast<int64_t>(heads - 1) * head_stride + dims <= x.size(1) && cos_sin.dim() == 2 && cos_sin.size(1) == dims,
+                "rotate_heads shapes");
+    check_rc(mb_rotate_heads(x.data_ptr(), ld, x.size(0), heads, head_stride, dims, interleaved ? 1 : 0,
+                             i32(positions, x.size(0), "positions"), f32(cos_sin, 0, "cos_sin"), dtype_of(x, "x"), cur_stream()),
+             "rotate_heads");
+  });
+  m.def("latent_attention", &latent_attention, py::arg("q_lat"), py::arg("q_rope"), py::arg("cache"), py::arg("block_table"),
+        py::arg("q_start"), py::arg("q_len"), py::arg("kv_len"), py::arg("out"), py::arg("scale"), py::arg("sink") = none,
+        py::arg("one_token") = false, py::arg("ws") = none, py::arg("allow_tc") = true);
+  m.def("delta_dim_pad", [](int dim) { return mb_delta_dim_pad(dim); });
+  m.def("delta_rule", &delta_rule);
+  m.def("moe_table_route", [](const Tensor& ids, const Tensor& tables, const Tensor& desc, int max_experts, Tensor& inverse,
+                              Tensor& offsets) {
+    TORCH_CHECK(ids.is_cuda() && ids.is_contiguous() && ids.scalar_type() == at::kLong && desc.is_cuda() && desc.is_contiguous() &&
+                    desc.scalar_type() == at::kLong && desc.dim() == 2 && desc.size(1) == 6, "moe_table_route layout");
+    check_rc(mb_moe_table_route(ids.data_ptr<int64_t>(), ids.numel(), i32(tables, 0, "tables"), desc.data_ptr<int64_t>(),
+                                desc.size(0), max_experts, const_cast<int32_t*>(i32(inverse, 0, "inverse")),
+                                const_cast<int32_t*>(i32(offsets, 0, "offsets")), cur_stream()),
+             "moe_table_route");
+  });
+  m.def("gemm_f32", [](const Tensor& x, const Tensor& w, Tensor& y, const Opt& r) {
+    const int ldx = ld_of(x, at::kFloat, "x"), ldw = ld_of(w, at::kFloat, "w"), ldy = ld_of(y, at::kFloat, "y");
+    TORCH_CHECK(w.size(1) == x.size(1) && y.size(0) == x.size(0) && y.size(1) == w.size(0), "gemm_f32 shapes");
+    int ldr = 0;
+    if (given(r)) { ldr = ld_of(*r, at::kFloat, "residual"); TORCH_CHECK(r->sizes() == y.sizes(), "gemm_f32 residual"); }
+    check_rc(mb_gemm_f32(x.data_ptr<float>(), w.data_ptr<float>(), y.data_ptr<float>(), static_cast<const float*>(optptr(r)),
+                         x.size(0), w.size(0), x.size(1), ldx, ldw, ldy, ldr, cur_stream()), "gemm_f32");
+  }, py::arg("x"), py::arg("w"), py::arg("y"), py::arg("residual") = none);
+  m.def("batched_gemm_f32", [](const Tensor& x, const Tensor& w, Tensor& y, int x_off, int y_off) {
+    const int ldx = ld_of(x, at::kFloat, "x"), ldy = ld_of(y, at::kFloat, "y");
+    TORCH_CHECK(w.dim() == 3 && w.is_contiguous() && w.scalar_type() == at::kFloat, "batched_gemm_f32: w [B, N, K]");
+    const int B = w.size(0), N = w.size(1), K = w.size(2);
+    TORCH_CHECK(static_cast<int64_t>(B - 1) * x_off + K <= x.size(1) && static_cast<int64_t>(B - 1) * y_off + N <= y.size(1) &&
+                    y.size(0) == x.size(0), "batched_gemm_f32: column blocks out of range");
+    check_rc(mb_batched_gemm_f32(x.data_ptr<float>(), w.data_ptr<float>(), y.data_ptr<float>(), B, x.size(0), N, K, ldx, x_off,
+                                 ldy, y_off, cur_stream()), "batched_gemm_f32");
+  });
+  m.def("grouped_gemm_f32", [](const Tensor& x, const Tensor& w, Tensor& y, const Tensor& offsets) {
+    TORCH_CHECK(x.is_cuda() && x.is_contiguous() && w.is_contiguous() && y.is_contiguous() && w.dim() == 3 &&
+                    x.scalar_type() == at::kFloat && w.scalar_type() == at::kFloat && y.scalar_type() == at::kFloat &&
+                    x.size(1) == w.size(2) && y.size(1) == w.size(1) && y.size(0) == x.size(0), "grouped_gemm_f32 layout");
+    check_rc(mb_grouped_gemm_f32(x.data_ptr<float>(), w.data_ptr<float>(), y.data_ptr<float>(), i32(offsets, w.size(0) + 1, "offsets"),
+                                 w.size(0), x.size(0), w.size(1), w.size(2), cur_stream()), "grouped_gemm_f32");
+  });
+  m.def("silu_mul_f32", [](const Tensor& gu, Tensor& out) {
+    TORCH_CHECK(gu.is_cuda() && gu.is_contiguous() && out.is_contiguous() && gu.scalar_type() == at::kFloat &&
+                    out.scalar_type() == at::kFloat && gu.size(1) == 2 * out.size(1) && gu.size(0) == out.size(0), "silu_mul_f32");
+    check_rc(mb_silu_mul_f32(gu.data_ptr<float>(), out.data_ptr<float>(), out.size(0), out.size(1), cur_stream()), "silu_mul_f32");
+  });
+}

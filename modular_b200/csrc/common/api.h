@@ -108,7 +108,7 @@ size_t mb_mla_split_workspace_bytes(int num_sms);
 int mb_mla_prefill_tc(const void* q_lat, const void* q_rope, void* out, const void* cache, long long page_stride,
                       long long n_pages, const int32_t* block_table, int bt_stride, const int32_t* q_start,
                       const int32_t* q_len, const int32_t* kv_len, int T, int B, int n_heads, int page_size, float scale,
-                      int32_t* tok_scratch, int* err, cudaStream_t stream);
+                      const float* sink, int ld_rope, int32_t* tok_scratch, int* err, cudaStream_t stream);
 int mb_mla_post_down(const void* qkv_a, int ld, int q_lora, int R, const void* gamma_q, const void* gamma_kv, float eps,
                      const int32_t* positions, const float* cos_sin, const int64_t* slots, void* q_a_out, void* cache,
                      int T, int page_size, long long page_stride, cudaStream_t stream);
@@ -195,13 +195,78 @@ int mb_mla_tc_usable(int T, int B, int n_heads, int R, int page_size);
 int mb_mla_decode_tc(const void* q_lat, const void* q_rope, void* out, const void* cache, long long page_stride,
                      long long n_pages, const int32_t* block_table, int bt_stride, const int32_t* q_start,
                      const int32_t* q_len, const int32_t* kv_len, int T, int B, int n_heads, int page_size,
-                     float scale, int* err, cudaStream_t stream);
+                     float scale, const float* sink, int ld_rope, int* err, cudaStream_t stream);
+// any latent width of {64, 128, 192, 256, 384, 512}, row strides, an optional softmax sink per head and a KV split
+int mb_mla_paged_attention_ex(const void* q_lat, long long ld_ql, const void* q_rope, long long ld_qr, int hs_qr, void* out,
+                              const void* cache, long long page_stride, int ld_cache, const int32_t* block_table,
+                              int bt_stride, const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len, int T,
+                              int B, int n_heads, int R, int page_size, float scale, const float* sink, void* ws,
+                              size_t ws_bytes, int num_sms, cudaStream_t stream);
 int mb_mla_paged_attention(const void* q_lat, const void* q_rope, void* out, const void* cache,
                            long long page_stride, const int32_t* block_table, int bt_stride,
                            const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len, int T,
                            int B, int n_heads, int R, int page_size, float scale, cudaStream_t stream);
 int mb_mla_kv_store(const void* c_kv, const void* k_rope, const int64_t* slots, void* cache, int T, int R,
                     int ld_c, int ld_r, int page_size, long long page_stride, cudaStream_t stream);
+
+// ---- latent attention of any size, bf16 (dtype 0) and fp32 (1) (mla_ragged.cu) ---------------
+int mb_latent_post_down(const void* x, int ld, int T, int q_rank, int q_rank_pad, const void* gamma_q, void* q_out,
+                        int ld_q, int kv_off, int R, int Rp, const void* gamma_kv, int rot_dim, int Dp, int dims,
+                        int interleaved, float eps, const int32_t* positions, const float* cos_sin, const int64_t* slots,
+                        void* cache, int page_size, long long page_stride, int ld_cache, int dtype, cudaStream_t stream);
+int mb_rotate_heads(void* x, int ld, int T, int heads, int head_stride, int dims, int interleaved,
+                    const int32_t* positions, const float* cos_sin, int dtype, cudaStream_t stream);
+int mb_latent_attention(const void* q_lat, int ld_ql, int hs_ql, const void* q_rope, int ld_qr, int hs_qr, void* out,
+                        int ld_out, int hs_out, const void* cache, long long page_stride, int ld_cache, int page_size,
+                        const int32_t* block_table, int bt_stride, const int32_t* q_start, const int32_t* q_len,
+                        const int32_t* kv_len, int T, int B, int n_heads, int Rp, int Dp, float scale, const float* sink,
+                        int dtype, cudaStream_t stream);
+
+// ---- seams of an fp32 residual stream (residual_norm.cu); null pointers switch parts off -----
+typedef struct {
+  float* x; int ldx;                                                     // residual rows, updated when store_x
+  const int64_t* ids; const void* table; float scale; int vocab, ld_table;  // x = table[ids] * scale
+  const void* a; int lda;                                                // x += a
+  const void* b; int ldb;                                                // x += b
+  const void* e; int lde; const int32_t* inverse; int top_k; float pair_w;  // x += pair_w * sum_k e[inverse[., k]]
+  const int32_t* rows;                                                   // rows of x to work on (all otherwise)
+  const void* w1; void* n1; int ld1;                                     // normalised rows * w1
+  const void* w2; void* n2; int ld2; const int32_t* scatter; int k2;     // normalised rows * w2, optionally scattered
+  int n_rows, cols, cols_pad, store_x;
+  float eps;
+} MbResidualNorm;
+int mb_residual_norm(const MbResidualNorm* p, int dtype, cudaStream_t stream);
+int mb_gelu_tanh(void* x, long long n, int dtype, cudaStream_t stream);
+int mb_sigmoid_gate(void* o, int ldo, const void* g, int ldg, int rows, int cols, int dtype, cudaStream_t stream);
+
+// ---- gated delta rule with per-channel decay (delta_rule.cu) ---------------------------------
+typedef struct {
+  const void* x; int ldx, q_off, k_off, v_off, b_off;    // projection rows [T, ldx]: column blocks of q, k, v, beta
+  const void* conv_w; int taps;                          // [q | k | v channels, taps]
+  const float* z; int ldz;                               // decay projection [T, heads * dim]
+  const float *A_log, *dt_bias;                          // [heads], [heads * dim]
+  const void* gate; int ld_gate;                         // output gate projection [T, heads * vdim]
+  const void* norm_w; float eps;                         // [vdim]
+  float *q, *k, *g, *v, *beta, *kq, *o;                  // fp32 scratch (q, k, g rows are dim_pad wide)
+  void* out; int ld_out;                                 // [T, heads * vdim]
+  float* state;                                          // [slots, heads, vdim, dim_pad]
+  float* conv_state;                                     // [slots, channels, taps - 1]
+  const int32_t *state_idx, *q_start, *q_len, *kv_len;
+  int T, B, heads, kv_heads, dim, dim_pad, vdim, one_token;
+} MbDelta;
+int mb_delta_dim_pad(int dim);
+int mb_delta_rule(const MbDelta* p, int dtype, int num_sms, cudaStream_t stream);
+
+// ---- fp32 products (gemm_simt.cu) ------------------------------------------------------------
+int mb_gemm_f32(const float* x, const float* w, float* y, const float* r, int M, int N, int K, int ldx, int ldw, int ldy,
+                int ldr, cudaStream_t stream);
+int mb_batched_gemm_f32(const float* x, const float* w, float* y, int B, int M, int N, int K, int ldx, int x_off, int ldy,
+                        int y_off, cudaStream_t stream);
+int mb_grouped_gemm_f32(const float* x, const float* w, float* y, const int32_t* offsets, int E, int max_rows, int N, int K,
+                        cudaStream_t stream);
+int mb_silu_mul_f32(const float* gu, float* out, int rows, int inter, cudaStream_t stream);
+int mb_moe_table_route(const int64_t* ids, int T, const int32_t* tables, const int64_t* desc, int n_layers,
+                       int max_experts, int32_t* inverse, int32_t* offsets, cudaStream_t stream);
 
 // ---- mixture of experts (moe.cu, grouped mode of gemm_tcgen05.cu) ---------------------------
 int mb_moe_router_group_limited(const float* logits, const float* bias, int32_t* topk_ids, float* topk_w,

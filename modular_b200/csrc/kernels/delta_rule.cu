@@ -1,0 +1,359 @@
+// Gated delta rule with a decay per key channel, for ragged batches. Per head, with a state S [dim, vdim] in fp32:
+//   S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+// q, k and v pass a short causal convolution and silu first, q and k are unit vectors per head, and o is RMS-normed over
+// vdim, scaled by a weight and gated.
+//
+//   delta_prep_kernel   one warp per (token, piece): convolution + silu of q, k, v (inputs before the step come from the
+//                       sequence's convolution state), unit norms, decays g = exp(-exp(A_log) softplus(z + dt_bias)),
+//                       beta, k . q. Everything leaves in fp32.
+//   delta_scan_kernel   columns of S are independent, so a warp owns eight of them: eight lanes share the rows of a
+//                       column (each 4 * RL4 of them, in registers), four lane groups hold two columns each. A token
+//                       costs one pass of decay, two dot products reduced together over eight lanes with four
+//                       shuffles (o = (gS)^T q + u (k . q) needs no second reduction), and the rank-one update. Token rows
+//                       are staged through shared memory with cp.async. The state is read once and written once per
+//                       launch, [slot, head, column, row]; sequences of one token are a decode step, for which one CTA
+//                       owns a whole head and also applies the output norm and gate. The convolution state is advanced
+//                       at the end of this kernel, after every read of it by the first one.
+//   delta_out_kernel    output norm and gate for longer sequences, one warp per (token, head)
+//
+// A chunked formulation on the tensor cores would round what enters the recurrence to 16 bits; this one keeps it in fp32.
+#include <cuda_runtime.h>
+
+#include "../common/api.h"
+#include "../common/launch.h"
+#include "../common/ptx.cuh"
+#include "../common/scalar.cuh"
+
+namespace mb {
+namespace delta {
+
+__device__ __forceinline__ void cp_async4(void* dst, const void* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(dst))), "l"(src)
+               : "memory");
+}
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(dst))), "l"(src)
+               : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+__device__ __forceinline__ float softplusf(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+
+template <typename T>
+__global__ void __launch_bounds__(256) delta_prep_kernel(const MbDelta p) {
+  pdl_wait();
+  pdl_trigger();
+  const int t = blockIdx.x, lane = threadIdx.x & 31;
+  const int unit = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int KH = p.kv_heads, H = p.heads, D = p.dim, V = p.vdim, DP = p.dim_pad;
+  const int qkC = KH * D, vC = H * V, C = 2 * qkC + vC, W = p.taps;
+  const int v_units = (vC + 127) / 128;
+  if (unit >= KH + H + v_units) return;
+  int s = t;
+  if (!p.one_token) {
+    int lo = 0, hi = p.B - 1;
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (p.q_start[mid] <= t) lo = mid; else hi = mid - 1;
+    }
+    s = lo;
+  }
+  const int off = t - p.q_start[s];
+  if (off < 0 || off >= p.q_len[s]) return;      // a row of no sequence
+  const T* row = static_cast<const T*>(p.x) + static_cast<size_t>(t) * p.ldx;
+  const int slot = p.state_idx[s];
+  const float* hist = (slot >= 0 && W > 1 && p.kv_len[s] > p.q_len[s])
+                          ? p.conv_state + static_cast<size_t>(slot) * C * (W - 1) : nullptr;
+  // channel `ch` of the convolution state, read from column `col` of the projection rows
+  auto conv_silu = [&](int ch, int col) {
+    const T* w = static_cast<const T*>(p.conv_w) + static_cast<size_t>(ch) * W;
+    float acc = 0.f;
+    for (int j = 0; j < W; ++j) {
+      const int src = off - (W - 1) + j;
+      float xv = 0.f;
+      if (src >= 0) xv = ldf(row - static_cast<ptrdiff_t>(W - 1 - j) * p.ldx + col);
+      else if (hist) xv = hist[static_cast<size_t>(ch) * (W - 1) + (W - 1 + src)];
+      acc = fmaf(ldf(w + j), xv, acc);
+    }
+    return siluf(acc);
+  };
+  if (unit < KH) {
+    float* qo = p.q + (static_cast<size_t>(t) * KH + unit) * DP;
+    float* ko = p.k + (static_cast<size_t>(t) * KH + unit) * DP;
+    float qq = 0.f, kk = 0.f, kq = 0.f;
+    for (int c = lane; c < D; c += 32) {
+      const float a = conv_silu(unit * D + c, p.q_off + unit * D + c);
+      const float b = conv_silu(qkC + unit * D + c, p.k_off + unit * D + c);
+      qq = fmaf(a, a, qq); kk = fmaf(b, b, kk); kq = fmaf(a, b, kq);
+      qo[c] = a; ko[c] = b;                        // rescaled below by the same lane
+    }
+    qq = warp_allsum(qq); kk = warp_allsum(kk); kq = warp_allsum(kq);
+    const float iq = 1.f / sqrtf(qq + 1e-6f) / sqrtf(static_cast<float>(D)), ik = 1.f / sqrtf(kk + 1e-6f);
+    for (int c = lane; c < DP; c += 32) {
+      qo[c] = c < D ? qo[c] * iq : 0.f;
+      ko[c] = c < D ? ko[c] * ik : 0.f;
+    }
+    if (lane == 0) p.kq[static_cast<size_t>(t) * KH + unit] = kq * iq * ik;
+  } else if (unit < KH + H) {
+    const int h = unit - KH;
+    const float a = expf(p.A_log[h]);
+    const float* z = p.z + static_cast<size_t>(t) * p.ldz + h * D;
+    float* go = p.g + (static_cast<size_t>(t) * H + h) * DP;
+    for (int c = lane; c < DP; c += 32) go[c] = c < D ? expf(-a * softplusf(z[c] + p.dt_bias[h * D + c])) : 0.f;
+    if (lane == 0) p.beta[static_cast<size_t>(t) * H + h] = sigmoidf(ldf(row + p.b_off + h));
+  } else {
+    const int c0 = (unit - KH - H) * 128;
+    for (int c = c0 + lane; c < min(c0 + 128, vC); c += 32)
+      p.v[static_cast<size_t>(t) * vC + c] = conv_silu(2 * qkC + c, p.v_off + c);
+  }
+}
+
+template <typename T, int RL4, int MAXT, bool FUSE>
+__global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int col_blocks, int chunk) {
+  constexpr int DP = 32 * RL4;
+  extern __shared__ __align__(16) float sm[];
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_trigger();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int rg = lane & 7, cg = lane >> 3;
+  const int KH = p.kv_heads, H = p.heads, V = p.vdim;
+  const int h = blockIdx.x / col_blocks, cols = (blockDim.x >> 5) * 8, cbase = (blockIdx.x % col_blocks) * cols;
+  const int kh = h / (H / KH), s = blockIdx.y;
+  const int t0 = p.q_start[s], n = p.q_len[s], slot = p.state_idx[s];
+  const bool resume = slot >= 0 && p.kv_len[s] > n;
+  if (n > 0) {
+    const int row_floats = 3 * DP + cols;          // q | k | g | v columns, then beta and k . q per token
+    float* stage[2] = {sm, sm + chunk * (row_floats + 2)};
+    float* so = sm + 2 * chunk * (row_floats + 2); // FUSE: outputs of one token
+    auto fetch = [&](int c0, float* dst) {
+      const int m = min(chunk, n - c0);
+      float* sc = dst + chunk * row_floats;
+      for (int i = tid; i < m * (3 * DP / 4); i += blockDim.x) {
+        const int j = i / (3 * DP / 4), v = i % (3 * DP / 4);
+        const size_t t = static_cast<size_t>(t0 + c0 + j);
+        const int which = v / (DP / 4), c = (v % (DP / 4)) * 4;
+        const float* src = which == 0 ? p.q + (t * KH + kh) * DP : which == 1 ? p.k + (t * KH + kh) * DP : p.g + (t * H + h) * DP;
+        cp_async16(dst + j * row_floats + v * 4, src + c);
+      }
+      for (int i = tid; i < m * cols; i += blockDim.x) {
+        const int j = i / cols, c = i % cols;
+        if (cbase + c < V) cp_async4(dst + j * row_floats + 3 * DP + c, p.v + (static_cast<size_t>(t0 + c0 + j) * H + h) * V + cbase + c);
+      }
+      for (int i = tid; i < 2 * m; i += blockDim.x) {
+        const size_t t = static_cast<size_t>(t0 + c0 + (i >> 1));
+        cp_async4(sc + i, (i & 1) ? p.kq + t * KH + kh : p.beta + t * H + h);
+      }
+      cp_async_commit();
+    };
+    fetch(0, stage[0]);
+    const int col0 = cbase + warp * 8 + cg * 2;
+    const bool ok0 = col0 < V, ok1 = col0 + 1 < V;
+    float* st = p.state + ((static_cast<size_t>(slot >= 0 ? slot : 0) * H + h) * V + col0) * DP;
+    float4 S0[RL4], S1[RL4];
+#pragma unroll
+    for (int i = 0; i < RL4; ++i) {
+      const int r = (i * 8 + rg) * 4;
+      S0[i] = (resume && ok0) ? *reinterpret_cast<const float4*>(st + r) : make_float4(0.f, 0.f, 0.f, 0.f);
+      S1[i] = (resume && ok1) ? *reinterpret_cast<const float4*>(st + DP + r) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    const bool hi_col = (lane & 4) != 0, is_q = (lane & 2) != 0;
+    for (int c0 = 0, it = 0; c0 < n; c0 += chunk, ++it) {
+      const int m = min(chunk, n - c0);
+      if (c0 + chunk < n) { fetch(c0 + chunk, stage[(it + 1) & 1]); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
+      __syncthreads();
+      const float* buf = stage[it & 1];
+      const float* sc = buf + chunk * row_floats;
+      for (int j = 0; j < m; ++j) {
+        const float* rowp = buf + j * row_floats;
+        float4 kr[RL4];
+        float a0[4] = {}, a1[4] = {}, b0[4] = {}, b1[4] = {};
+#pragma unroll
+        for (int i = 0; i < RL4; ++i) {
+          const int r = (i * 8 + rg) * 4;
+          const float4 q4 = *reinterpret_cast<const float4*>(rowp + r);
+          const float4 k4 = *reinterpret_cast<const float4*>(rowp + DP + r);
+          const float4 g4 = *reinterpret_cast<const float4*>(rowp + 2 * DP + r);
+          kr[i] = k4;
+          S0[i].x *= g4.x; S0[i].y *= g4.y; S0[i].z *= g4.z; S0[i].w *= g4.w;
+          S1[i].x *= g4.x; S1[i].y *= g4.y; S1[i].z *= g4.z; S1[i].w *= g4.w;
+          a0[0] = fmaf(S0[i].x, k4.x, a0[0]); a0[1] = fmaf(S0[i].y, k4.y, a0[1]);
+          a0[2] = fmaf(S0[i].z, k4.z, a0[2]); a0[3] = fmaf(S0[i].w, k4.w, a0[3]);
+          a1[0] = fmaf(S1[i].x, k4.x, a1[0]); a1[1] = fmaf(S1[i].y, k4.y, a1[1]);
+          a1[2] = fmaf(S1[i].z, k4.z, a1[2]); a1[3] = fmaf(S1[i].w, k4.w, a1[3]);
+          b0[0] = fmaf(S0[i].x, q4.x, b0[0]); b0[1] = fmaf(S0[i].y, q4.y, b0[1]);
+          b0[2] = fmaf(S0[i].z, q4.z, b0[2]); b0[3] = fmaf(S0[i].w, q4.w, b0[3]);
+          b1[0] = fmaf(S1[i].x, q4.x, b1[0]); b1[1] = fmaf(S1[i].y, q4.y, b1[1]);
+          b1[2] = fmaf(S1[i].z, q4.z, b1[2]); b1[3] = fmaf(S1[i].w, q4.w, b1[3]);
+        }
+        const float A0 = (a0[0] + a0[1]) + (a0[2] + a0[3]), A1 = (a1[0] + a1[1]) + (a1[2] + a1[3]);
+        const float B0 = (b0[0] + b0[1]) + (b0[2] + b0[3]), B1 = (b1[0] + b1[1]) + (b1[2] + b1[3]);
+        // eight partial sums of four values: lanes with bit 2 take column 1, lanes with bit 1 the q product
+        float a = (hi_col ? A1 : A0) + __shfl_xor_sync(0xffffffffu, hi_col ? A0 : A1, 4);
+        float b = (hi_col ? B1 : B0) + __shfl_xor_sync(0xffffffffu, hi_col ? B0 : B1, 4);
+        float r = (is_q ? b : a) + __shfl_xor_sync(0xffffffffu, is_q ? a : b, 2);
+        r += __shfl_xor_sync(0xffffffffu, r, 1);
+        const float beta = sc[2 * j], kq = sc[2 * j + 1];
+        const float vv = rowp[3 * DP + warp * 8 + cg * 2 + (hi_col ? 1 : 0)];
+        const float u = beta * (vv - r);           // meaningful in the lanes that hold a key product
+        const float u0 = __shfl_sync(0xffffffffu, u, lane & 24), u1 = __shfl_sync(0xffffffffu, u, (lane & 24) | 4);
+#pragma unroll
+        for (int i = 0; i < RL4; ++i) {
+          S0[i].x = fmaf(kr[i].x, u0, S0[i].x); S0[i].y = fmaf(kr[i].y, u0, S0[i].y);
+          S0[i].z = fmaf(kr[i].z, u0, S0[i].z); S0[i].w = fmaf(kr[i].w, u0, S0[i].w);
+          S1[i].x = fmaf(kr[i].x, u1, S1[i].x); S1[i].y = fmaf(kr[i].y, u1, S1[i].y);
+          S1[i].z = fmaf(kr[i].z, u1, S1[i].z); S1[i].w = fmaf(kr[i].w, u1, S1[i].w);
+        }
+        const float o = fmaf(hi_col ? u1 : u0, kq, r);
+        if ((lane & 3) == 2) {
+          const int c = warp * 8 + cg * 2 + (hi_col ? 1 : 0);
+          if (FUSE) so[c] = cbase + c < V ? o : 0.f;
+          else if (cbase + c < V) p.o[(static_cast<size_t>(t0 + c0 + j) * H + h) * V + cbase + c] = o;
+        }
+        if (FUSE) {                                // one CTA holds the whole head (cbase = 0)
+          __syncthreads();
+          float ss = 0.f;
+          for (int c = tid; c < V; c += blockDim.x) ss = fmaf(so[c], so[c], ss);
+          ss = warp_allsum(ss);
+          if (lane == 0) red[warp] = ss;
+          __syncthreads();
+          float tot = 0.f;
+          for (int i = 0; i < static_cast<int>(blockDim.x >> 5); ++i) tot += red[i];
+          const float inv = 1.f / sqrtf(tot / static_cast<float>(V) + p.eps);
+          const size_t t = static_cast<size_t>(t0 + c0 + j);
+          for (int c = tid; c < V; c += blockDim.x) {
+            const float gate = sigmoidf(ldf(static_cast<const T*>(p.gate) + t * p.ld_gate + h * V + c));
+            stf(static_cast<T*>(p.out) + t * p.ld_out + h * V + c, so[c] * inv * ldf(static_cast<const T*>(p.norm_w) + c) * gate);
+          }
+          __syncthreads();
+        }
+      }
+      __syncthreads();                             // the stage is free again
+    }
+    if (slot >= 0) {
+#pragma unroll
+      for (int i = 0; i < RL4; ++i) {
+        const int r = (i * 8 + rg) * 4;
+        if (ok0) *reinterpret_cast<float4*>(st + r) = S0[i];
+        if (ok1) *reinterpret_cast<float4*>(st + DP + r) = S1[i];
+      }
+    }
+  }
+  // the last taps - 1 convolution inputs of the sequence; this CTA's share of the channels
+  const int W = p.taps;
+  if (n > 0 && slot >= 0 && W > 1) {
+    const int qkC = KH * p.dim, C = 2 * qkC + H * V;
+    for (int c = blockIdx.x * blockDim.x + tid; c < C; c += gridDim.x * blockDim.x) {
+      const int col = c < qkC ? p.q_off + c : c < 2 * qkC ? p.k_off + (c - qkC) : p.v_off + (c - 2 * qkC);
+      float* cs = p.conv_state + (static_cast<size_t>(slot) * C + c) * (W - 1);
+      // ascending order only overwrites entries that have been read: entry i comes from entry i + n
+      for (int i = 0; i < W - 1; ++i) {
+        const int src = n - (W - 1) + i;           // position within the step
+        float x = 0.f;
+        if (src >= 0) x = ldf(static_cast<const T*>(p.x) + static_cast<size_t>(t0 + src) * p.ldx + col);
+        else if (resume) x = cs[W - 1 + src];
+        cs[i] = x;
+      }
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) delta_out_kernel(const MbDelta p) {
+  pdl_wait();
+  pdl_trigger();
+  const int V = p.vdim, lane = threadIdx.x & 31;
+  const long long unit = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (unit >= static_cast<long long>(p.T) * p.heads) return;
+  const size_t t = static_cast<size_t>(unit / p.heads);
+  const int h = static_cast<int>(unit % p.heads);
+  const float* o = p.o + unit * V;
+  float ss = 0.f;
+  for (int c = lane; c < V; c += 32) ss = fmaf(o[c], o[c], ss);
+  const float inv = 1.f / sqrtf(warp_allsum(ss) / static_cast<float>(V) + p.eps);
+  for (int c = lane; c < V; c += 32) {
+    const float gate = sigmoidf(ldf(static_cast<const T*>(p.gate) + t * p.ld_gate + h * V + c));
+    stf(static_cast<T*>(p.out) + t * p.ld_out + h * V + c, o[c] * inv * ldf(static_cast<const T*>(p.norm_w) + c) * gate);
+  }
+}
+
+template <typename T, int RL4>
+static int scan(const MbDelta& p, int num_sms, cudaStream_t stream) {
+  constexpr int MAXT = RL4 <= 8 ? 512 : 256;
+  const int head_warps = (p.vdim + 7) / 8;
+  const bool fuse = p.one_token && head_warps * 32 <= MAXT;
+  int warps;
+  if (fuse) {
+    warps = head_warps;
+  } else {                         // fewer columns per CTA until the step fills the machine
+    warps = MAXT / 32 < 4 ? MAXT / 32 : 4;
+    while (warps > 1 && static_cast<long long>(p.B) * p.heads * ((head_warps + warps - 1) / warps) < 2ll * num_sms) warps >>= 1;
+    if (warps > head_warps) warps = head_warps;
+  }
+  const int col_blocks = (head_warps + warps - 1) / warps;
+  const int per_token = (3 * 32 * RL4 + warps * 8 + 2) * 4;
+  int chunk = p.one_token ? 1 : 40 * 1024 / (2 * per_token);
+  if (chunk > 16) chunk = 16;
+  if (chunk >= 4) chunk &= ~3;      // whole float4 rows keep the second stage 16-byte aligned
+  else if (chunk > 1) chunk = 2;
+  if (chunk < 1) chunk = 1;
+  // the second stage starts chunk * per_token bytes in: 16-byte aligned when chunk * 2 floats are a multiple of 4
+  if (chunk == 1 && !p.one_token) chunk = 2;
+  const size_t smem = static_cast<size_t>(2) * chunk * per_token + (fuse ? warps * 8 * 4 : 0) + 16;
+  const dim3 grid(p.heads * col_blocks, p.B);
+  cudaError_t e;
+  if (fuse) {
+    e = launch_k(delta_scan_kernel<T, RL4, MAXT, true>, grid, dim3(warps * 32), smem, stream, p, col_blocks, chunk);
+  } else {
+    e = launch_k(delta_scan_kernel<T, RL4, MAXT, false>, grid, dim3(warps * 32), smem, stream, p, col_blocks, chunk);
+    if (e == cudaSuccess) {
+      const long long units = static_cast<long long>(p.T) * p.heads;
+      e = launch_k(delta_out_kernel<T>, dim3(static_cast<unsigned>((units + 7) / 8)), dim3(256), 0, stream, p);
+    }
+  }
+  return e == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
+}
+
+template <typename T>
+static int run(const MbDelta& p, int num_sms, cudaStream_t stream) {
+  const int vC = p.heads * p.vdim;
+  const int units = p.kv_heads + p.heads + (vC + 127) / 128;
+  if (launch_k(delta_prep_kernel<T>, dim3(p.T, (units + 7) / 8), dim3(256), 0, stream, p) != cudaSuccess)
+    return MB_ERR_LAUNCH;
+  switch (p.dim_pad / 32) {
+    case 1: return scan<T, 1>(p, num_sms, stream);
+    case 2: return scan<T, 2>(p, num_sms, stream);
+    case 3: return scan<T, 3>(p, num_sms, stream);
+    case 4: return scan<T, 4>(p, num_sms, stream);
+    case 6: return scan<T, 6>(p, num_sms, stream);
+    case 8: return scan<T, 8>(p, num_sms, stream);
+    case 16: return scan<T, 16>(p, num_sms, stream);
+    default: return MB_ERR_SHAPE;
+  }
+}
+
+}  // namespace delta
+}  // namespace mb
+
+using namespace mb;
+
+// Rows of the state per column: the smallest size the scan kernel is built for (0 = too large).
+extern "C" int mb_delta_dim_pad(int dim) {
+  const int sizes[] = {32, 64, 96, 128, 192, 256, 512};
+  for (int s : sizes)
+    if (dim <= s) return s;
+  return 0;
+}
+
+extern "C" int mb_delta_rule(const MbDelta* p, int dtype, int num_sms, cudaStream_t stream) {
+  if (p->T <= 0 || p->B <= 0) return MB_OK;
+  if (p->heads <= 0 || p->kv_heads <= 0 || p->heads % p->kv_heads || p->dim <= 0 || p->vdim <= 0 || p->taps < 1 ||
+      p->dim_pad != mb_delta_dim_pad(p->dim))
+    return MB_ERR_SHAPE;
+  if ((reinterpret_cast<uintptr_t>(p->q) | reinterpret_cast<uintptr_t>(p->k) | reinterpret_cast<uintptr_t>(p->g) |
+       reinterpret_cast<uintptr_t>(p->state)) & 15)
+    return MB_ERR_ALIGN;
+  return dtype == kF32 ? delta::run<float>(*p, num_sms, stream) : delta::run<__nv_bfloat16>(*p, num_sms, stream);
+}

@@ -23,6 +23,7 @@
 
 #include "../common/api.h"
 #include "../common/launch.h"
+#include "../common/ptx.cuh"
 
 namespace mb {
 namespace mla {
@@ -35,7 +36,14 @@ struct Params {
   const bf16* q_lat;   // [T, h, R]
   const bf16* q_rope;  // [T, h, DR]
   bf16* out;           // [T, h, R]
-  const bf16* cache;   // page p, slot s at cache + p * page_stride + s * (R + DR)
+  const bf16* cache;   // page p, slot s at cache + p * page_stride + s * ld_cache
+  const float* sink;   // per head: a score without key or value that joins the softmax denominator (nullptr: none)
+  // KV split: grid z parts walk equal shares of the 64-token tiles and leave (O, m, l) of their valid rows in `ws`,
+  // [part][T * h][R] then [part][T * h][2]; a second kernel combines them
+  float* ws;
+  int nsplit, ld_cache, T;
+  int64_t ld_ql, ld_qr;  // elements between tokens of q_lat (heads are R apart) and q_rope (heads are hs_qr apart)
+  int hs_qr;
   const int32_t* block_table;
   const int32_t* q_start;
   const int32_t* q_len;
@@ -92,7 +100,7 @@ __device__ __forceinline__ void load_kv_tile(bf16* sK, const Params& p, const in
     const bool valid = tok < kv_end;
     const int pg = valid ? bt[tok / p.page_size] : 0;
     const int off = valid ? tok % p.page_size : 0;
-    const bf16* src = p.cache + static_cast<int64_t>(pg) * p.page_stride + static_cast<int64_t>(off) * LD + chunk * 8;
+    const bf16* src = p.cache + static_cast<int64_t>(pg) * p.page_stride + static_cast<int64_t>(off) * p.ld_cache + chunk * 8;
     cp_async16(sK + swz<LD>(row, chunk), src, valid);
   }
 }
@@ -106,7 +114,10 @@ __global__ void __launch_bounds__(256, 1) mla_kernel(const Params p) {
   bf16* sK = sQ + 64 * LD;                       // [2][64][LD]
   __shared__ int s_seq, s_tq0;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  pdl_wait();
+  pdl_trigger();
   const int tokens_per_tile = 64 / p.HB;
+  const int rows = tokens_per_tile * p.HB;   // query rows of a full tile (below 64 when HB does not divide it)
 
   // locate this CTA's (sequence, first query token): tiles are enumerated sequence by sequence
   if (tid == 0) {
@@ -128,18 +139,21 @@ __global__ void __launch_bounds__(256, 1) mla_kernel(const Params p) {
   for (int idx = tid; idx < 64 * CH; idx += 256) {
     const int row = idx / CH, chunk = idx % CH;
     const int tq = tq0 + row / p.HB, head = head0 + row % p.HB;
-    const bool valid = tq < ql;
+    const bool valid = row < rows && tq < ql;
     const int64_t tok = qs + (valid ? tq : 0);
     const bf16* src = chunk < R / 8
-                          ? p.q_lat + (tok * p.n_heads + head) * R + chunk * 8
-                          : p.q_rope + (tok * p.n_heads + head) * DR + (chunk - R / 8) * 8;
+                          ? p.q_lat + tok * p.ld_ql + static_cast<int64_t>(head) * R + chunk * 8
+                          : p.q_rope + tok * p.ld_qr + static_cast<int64_t>(head) * p.hs_qr + (chunk - R / 8) * 8;
     cp_async16(sQ + swz<LD>(row, chunk), src, valid);
   }
   int last_tq = tq0 + tokens_per_tile;
   if (last_tq > ql) last_tq = ql;
   const int kv_hi = kl - ql + last_tq;  // exclusive bound of the KV positions any row here may see
-  const int ntiles = (kv_hi + 63) / 64;
-  load_kv_tile<R>(sK, p, bt, 0, kv_hi, tid);
+  const int tiles_all = (kv_hi + 63) / 64;
+  const int tiles_per = (tiles_all + p.nsplit - 1) / p.nsplit;
+  const int t_begin = static_cast<int>(blockIdx.z) * tiles_per;
+  const int t_end = min(tiles_all, t_begin + tiles_per);     // trailing parts may be empty
+  load_kv_tile<R>(sK, p, bt, t_begin * 64, kv_hi, tid);
   cp_async_commit();
   cp_async_wait_all();
   __syncthreads();
@@ -155,16 +169,18 @@ __global__ void __launch_bounds__(256, 1) mla_kernel(const Params p) {
   for (int h = 0; h < 2; ++h) {
     const int r = rb * 16 + (lane >> 2) + h * 8;
     const int tq = tq0 + r / p.HB;
-    limit[h] = tq < ql ? kl - ql + tq : -1;
+    limit[h] = (r < rows && tq < ql) ? kl - ql + tq : -1;
   }
+  const bool active = __any_sync(0xffffffffu, limit[0] >= 0 || limit[1] >= 0);   // this warp's block has valid rows
 
-  for (int it = 0; it < ntiles; ++it) {
-    const int buf = it & 1;
-    if (it + 1 < ntiles) {
+  for (int it = t_begin; it < t_end; ++it) {
+    const int buf = (it - t_begin) & 1;
+    if (it + 1 < t_end) {
       load_kv_tile<R>(sK + (buf ^ 1) * 64 * LD, p, bt, (it + 1) * 64, kv_hi, tid);
       cp_async_commit();
     }
     const bf16* tK = sK + buf * 64 * LD;
+    if (active) {
     float s[8][4];
 #pragma unroll
     for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
@@ -236,6 +252,7 @@ __global__ void __launch_bounds__(256, 1) mla_kernel(const Params p) {
         mma_bf16(o[2 * dp + 1], a, b[2], b[3]);
       }
     }
+    }
     cp_async_wait_all();
     __syncthreads();
   }
@@ -244,15 +261,63 @@ __global__ void __launch_bounds__(256, 1) mla_kernel(const Params p) {
   for (int h = 0; h < 2; ++h) {
     l[h] += __shfl_xor_sync(0xffffffffu, l[h], 1);
     l[h] += __shfl_xor_sync(0xffffffffu, l[h], 2);
-    const float inv = l[h] > 0.f ? 1.f / l[h] : 0.f;
     const int r = rb * 16 + (lane >> 2) + h * 8;
     const int tq = tq0 + r / p.HB, head = head0 + r % p.HB;
-    if (tq < ql) {
+    if (r >= rows || tq >= ql) continue;
+    if (p.nsplit > 1) {
+      const int64_t row = static_cast<int64_t>(blockIdx.z) * p.T * p.n_heads + static_cast<int64_t>(qs + tq) * p.n_heads + head;
+      float* orow = p.ws + row * R + chalf * HALF + 2 * (lane & 3);
+#pragma unroll
+      for (int dt = 0; dt < DT; ++dt) *reinterpret_cast<float2*>(orow + dt * 8) = make_float2(o[dt][2 * h], o[dt][2 * h + 1]);
+      if (chalf == 0 && (lane & 3) == 0)
+        *reinterpret_cast<float2*>(p.ws + static_cast<int64_t>(p.nsplit) * p.T * p.n_heads * R + row * 2) = make_float2(m[h], l[h]);
+      continue;
+    }
+    float inv = l[h] > 0.f ? 1.f / l[h] : 0.f;
+    if (p.sink) {       // the running maximum and the sink share one reference, so neither exponential overflows
+      const float sk = p.sink[head] * 1.4426950408889634f, mm = fmaxf(m[h], sk);
+      const float f = exp2f(m[h] - mm);
+      inv = f / (l[h] * f + exp2f(sk - mm));
+    }
+    {
       bf16* orow = p.out + (static_cast<int64_t>(qs + tq) * p.n_heads + head) * R + chalf * HALF + 2 * (lane & 3);
 #pragma unroll
       for (int dt = 0; dt < DT; ++dt)
         *reinterpret_cast<uint32_t*>(orow + dt * 8) = pack_bf16(o[dt][2 * h] * inv, o[dt][2 * h + 1] * inv);
     }
+  }
+}
+
+// Combines the parts of a KV-split launch: one warp per (token, head), part weights exp2(m - max).
+__global__ void __launch_bounds__(256)
+mla_combine_kernel(const float* __restrict__ ws, bf16* __restrict__ out, const float* __restrict__ sink, int n_rows,
+                   int n_heads, int R, int nsplit) {
+  pdl_wait();
+  pdl_trigger();
+  const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= n_rows) return;
+  const float2* ml = reinterpret_cast<const float2*>(ws + static_cast<int64_t>(nsplit) * n_rows * R);
+  float2 mine = lane < nsplit ? ml[static_cast<int64_t>(lane) * n_rows + row] : make_float2(-INFINITY, 0.f);
+  const float sk = sink ? sink[row % n_heads] * 1.4426950408889634f : -INFINITY;
+  float M = fmaxf(mine.x, sk);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
+  const float f = mine.x == -INFINITY ? 0.f : exp2f(mine.x - M);
+  float den = mine.y * f;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
+  if (sink) den += exp2f(sk - M);
+  const float inv = den > 0.f ? 1.f / den : 0.f;
+  for (int c = lane * 2; c < R; c += 64) {
+    float2 acc = make_float2(0.f, 0.f);
+    for (int q = 0; q < nsplit; ++q) {
+      const float fq = __shfl_sync(0xffffffffu, f, q);
+      if (fq == 0.f) continue;         // also a part without tiles, whose rows hold zeros
+      const float2 v = *reinterpret_cast<const float2*>(ws + (static_cast<int64_t>(q) * n_rows + row) * R + c);
+      acc.x = fmaf(fq, v.x, acc.x);
+      acc.y = fmaf(fq, v.y, acc.y);
+    }
+    *reinterpret_cast<uint32_t*>(out + static_cast<int64_t>(row) * R + c) = pack_bf16(acc.x * inv, acc.y * inv);
   }
 }
 
@@ -378,9 +443,15 @@ static int launch(const Params& p, int grid_x, cudaStream_t stream) {
       return MB_ERR_LAUNCH;
     configured.done();
   }
-  dim3 grid(grid_x, p.n_heads / p.HB);
-  kern<<<grid, 256, smem, stream>>>(p);
-  return cudaGetLastError() == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
+  dim3 grid(grid_x, p.n_heads / p.HB, p.nsplit);
+  if (launch_k(kern, grid, dim3(256), smem, stream, p) != cudaSuccess) return MB_ERR_LAUNCH;
+  if (p.nsplit > 1) {
+    const int n_rows = p.T * p.n_heads;
+    if (launch_k(mla_combine_kernel, dim3((n_rows + 7) / 8), dim3(256), 0, stream, static_cast<const float*>(p.ws), p.out,
+                 p.sink, n_rows, p.n_heads, R, p.nsplit) != cudaSuccess)
+      return MB_ERR_LAUNCH;
+  }
+  return MB_OK;
 }
 
 }  // namespace mla
@@ -414,32 +485,70 @@ extern "C" int mb_mla_q_rope(const void* q, int n_heads, int nope, const int32_t
   return cudaGetLastError() == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
 }
 
-// T = total query tokens, B = sequences. kv_lora_rank R in {128, 256, 512}; rope width 64.
-extern "C" int mb_mla_paged_attention(const void* q_lat, const void* q_rope, void* out, const void* cache,
-                                      long long page_stride, const int32_t* block_table, int bt_stride,
-                                      const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
-                                      int T, int B, int n_heads, int R, int page_size, float scale,
-                                      cudaStream_t stream) {
+// The largest number of heads per 64-row tile: a divisor of the head count.
+static int heads_per_tile(int n_heads) {
+  int hb = n_heads < 64 ? n_heads : 64;
+  while (n_heads % hb) --hb;
+  return hb;
+}
+
+// T = total query tokens, B = sequences. Latent width R in {64, 128, 192, 256, 384, 512}; rotated part 64 wide (both may
+// be zero-padded). `max_kv` bounds the cache rows of a sequence. `ws` (optional): fp32 scratch for splitting the KV range
+// of steps that would leave SMs idle.
+extern "C" int mb_mla_paged_attention_ex(const void* q_lat, long long ld_ql, const void* q_rope, long long ld_qr, int hs_qr,
+                                         void* out, const void* cache, long long page_stride, int ld_cache,
+                                         const int32_t* block_table, int bt_stride, const int32_t* q_start,
+                                         const int32_t* q_len, const int32_t* kv_len, int T, int B, int n_heads, int R,
+                                         int page_size, float scale, const float* sink, void* ws, size_t ws_bytes,
+                                         int num_sms, cudaStream_t stream) {
   if (T <= 0 || B <= 0) return MB_OK;
-  int HB = 64;
-  while (HB > 1 && n_heads % HB) HB >>= 1;
+  if (ld_cache < R + mla::DR || ld_cache % 8 || page_stride % 8 || ld_ql % 8 || ld_qr % 8 || hs_qr % 8) return MB_ERR_SHAPE;
+  if ((reinterpret_cast<uintptr_t>(q_lat) | reinterpret_cast<uintptr_t>(q_rope) | reinterpret_cast<uintptr_t>(cache) |
+       reinterpret_cast<uintptr_t>(out)) & 15)
+    return MB_ERR_ALIGN;
   mla::Params p;
   p.q_lat = static_cast<const mla::bf16*>(q_lat);
   p.q_rope = static_cast<const mla::bf16*>(q_rope);
   p.out = static_cast<mla::bf16*>(out);
   p.cache = static_cast<const mla::bf16*>(cache);
   p.block_table = block_table; p.q_start = q_start; p.q_len = q_len; p.kv_len = kv_len;
-  p.page_stride = page_stride; p.B = B; p.bt_stride = bt_stride; p.n_heads = n_heads; p.HB = HB;
+  p.page_stride = page_stride; p.B = B; p.bt_stride = bt_stride; p.n_heads = n_heads; p.HB = heads_per_tile(n_heads);
   p.page_size = page_size;
   p.scale_log2 = scale * 1.4426950408889634f;
-  const int tpt = 64 / HB;
+  p.sink = sink; p.ld_cache = ld_cache; p.T = T; p.ld_ql = ld_ql; p.ld_qr = ld_qr; p.hs_qr = hs_qr;
+  p.ws = static_cast<float*>(ws); p.nsplit = 1;
+  const int tpt = 64 / p.HB;
   const int grid_x = (T + tpt - 1) / tpt + B;  // >= sum over sequences of ceil(q_len / tpt)
+  if (ws != nullptr) {
+    // decode-sized steps: tiles of the batch that really exist are at most T, so count those
+    const long long ctas = static_cast<long long>(T < grid_x ? T : grid_x) * (n_heads / p.HB);
+    const long long max_tiles = static_cast<long long>(bt_stride) * page_size / 64;
+    long long ns = ctas > 0 ? num_sms / ctas : 1;
+    if (ns > max_tiles / 2) ns = max_tiles / 2;      // at least two tiles per part
+    if (ns > 32) ns = 32;
+    while (ns > 1 && static_cast<size_t>(ns) * T * n_heads * (R + 2) * sizeof(float) > ws_bytes) --ns;
+    if (ns > 1) p.nsplit = static_cast<int>(ns);
+  }
   switch (R) {
+    case 64: return mla::launch<64>(p, grid_x, stream);
     case 128: return mla::launch<128>(p, grid_x, stream);
+    case 192: return mla::launch<192>(p, grid_x, stream);
     case 256: return mla::launch<256>(p, grid_x, stream);
+    case 384: return mla::launch<384>(p, grid_x, stream);
     case 512: return mla::launch<512>(p, grid_x, stream);
     default: return MB_ERR_SHAPE;
   }
+}
+
+extern "C" int mb_mla_paged_attention(const void* q_lat, const void* q_rope, void* out, const void* cache,
+                                      long long page_stride, const int32_t* block_table, int bt_stride,
+                                      const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
+                                      int T, int B, int n_heads, int R, int page_size, float scale,
+                                      cudaStream_t stream) {
+  return mb_mla_paged_attention_ex(q_lat, static_cast<long long>(n_heads) * R, q_rope,
+                                   static_cast<long long>(n_heads) * mla::DR, mla::DR, out, cache, page_stride, R + mla::DR,
+                                   block_table, bt_stride, q_start, q_len, kv_len, T, B, n_heads, R, page_size, scale,
+                                   nullptr, nullptr, 0, 0, stream);
 }
 
 extern "C" int mb_mla_kv_store(const void* c_kv, const void* k_rope, const int64_t* slots, void* cache, int T,

@@ -70,6 +70,7 @@ struct Params {
   long long page_rows;             // rows of the [rows, 576] view between consecutive pages
   int bt_stride, n_heads, page_size;
   float scale_log2;
+  const float* sink;               // per head: a score without key or value in the softmax denominator (nullptr: none)
 };
 
 struct Bars {
@@ -333,7 +334,12 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap tmQl, const __grid_constant__ 
     // ---- epilogue: O / l -> bf16, 256 columns of this CTA's half
     bf16* orow = p.out + (static_cast<int64_t>(q_row) + r) * R + half * 256;
     if (n_parts <= 1) {
-      const float inv = (ok && ntiles > 0 && l > 0.f) ? 1.f / l : 0.f;
+      float inv = (ok && ntiles > 0 && l > 0.f) ? 1.f / l : 0.f;
+      if (p.sink != nullptr && inv > 0.f) {
+        const float sk = p.sink[hb * 128 + r] * 1.4426950408889634f, M = fmaxf(m_ref, sk);
+        const float f = exp2f(m_ref - M);
+        inv = f / (l * f + exp2f(sk - M));
+      }
       if (ntiles > 0 && ok) {
 #pragma unroll 1
         for (int q8 = 0; q8 < 8; ++q8) {
@@ -376,13 +382,14 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap tmQl, const __grid_constant__ 
       asm volatile("bar.sync 1, 128;" ::: "memory");
       if (bars->last_flag != 0) {
         __threadfence();
-        float M = -INFINITY;
+        const float sk = p.sink != nullptr ? p.sink[hb * 128 + r] * 1.4426950408889634f : -INFINITY;
+        float M = sk;
         for (int q = 0; q < n_parts; ++q) {
           const float* pp = base + static_cast<size_t>(q) * kPartFloats;
           if (__ldcg(pp + 256 * 128 + 128 + r) > 0.f) M = fmaxf(M, __ldcg(pp + 256 * 128 + r));
         }
         float wq[16];                                         // nsplit <= 16
-        float L = 0.f;
+        float L = p.sink != nullptr ? exp2f(sk - M) : 0.f;
         for (int q = 0; q < n_parts; ++q) {
           const float* pp = base + static_cast<size_t>(q) * kPartFloats;
           const float lq = __ldcg(pp + 256 * 128 + 128 + r);
@@ -468,18 +475,21 @@ extern "C" int mb_mla_tc_usable(int T, int B, int n_heads, int R, int page_size)
 
 // Decode-only absorbed MLA: T == B (one query token per sequence; sequences with q_len 0 are skipped),
 // R = 512, n_heads % 128 == 0, page_size % 64 == 0. `cache` is one layer's [pages, page_size, 576] view with
+// `ld_rope` elements from one (token, head) row of q_rope to the next (64 when they are contiguous).
 // `page_stride` elements between pages (a multiple of 576); `n_pages` bounds the tensor map.
 static int mla_tc_launch(const void* q_lat, const void* q_rope, void* out, const void* cache, long long page_stride,
                          long long n_pages, const int32_t* block_table, int bt_stride, const int32_t* q_start,
                          const int32_t* q_len, const int32_t* kv_len, int T, int B, int n_heads, int page_size,
-                         float scale, int32_t* tok_scratch, int* err, cudaStream_t stream);
+                         float scale, const float* sink, int ld_rope, int32_t* tok_scratch, int* err,
+                         cudaStream_t stream);
 
 extern "C" int mb_mla_decode_tc(const void* q_lat, const void* q_rope, void* out, const void* cache,
                                 long long page_stride, long long n_pages, const int32_t* block_table, int bt_stride,
                                 const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len, int T, int B,
-                                int n_heads, int page_size, float scale, int* err, cudaStream_t stream) {
+                                int n_heads, int page_size, float scale, const float* sink, int ld_rope, int* err,
+                                cudaStream_t stream) {
   return mla_tc_launch(q_lat, q_rope, out, cache, page_stride, n_pages, block_table, bt_stride, q_start, q_len, kv_len,
-                       T, B, n_heads, page_size, scale, nullptr, err, stream);
+                       T, B, n_heads, page_size, scale, sink, ld_rope, nullptr, err, stream);
 }
 
 // Any ragged batch (prefill, chunks, mixed steps) on the same tensor-core kernel: every query token is one CTA
@@ -488,19 +498,21 @@ extern "C" int mb_mla_decode_tc(const void* q_lat, const void* q_rope, void* out
 extern "C" int mb_mla_prefill_tc(const void* q_lat, const void* q_rope, void* out, const void* cache,
                                  long long page_stride, long long n_pages, const int32_t* block_table, int bt_stride,
                                  const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len, int T, int B,
-                                 int n_heads, int page_size, float scale, int32_t* tok_scratch, int* err,
-                                 cudaStream_t stream) {
+                                 int n_heads, int page_size, float scale, const float* sink, int ld_rope,
+                                 int32_t* tok_scratch, int* err, cudaStream_t stream) {
   if (tok_scratch == nullptr) return MB_ERR_SHAPE;
   return mla_tc_launch(q_lat, q_rope, out, cache, page_stride, n_pages, block_table, bt_stride, q_start, q_len, kv_len,
-                       T, B, n_heads, page_size, scale, tok_scratch, err, stream);
+                       T, B, n_heads, page_size, scale, sink, ld_rope, tok_scratch, err, stream);
 }
 
 static int mla_tc_launch(const void* q_lat, const void* q_rope, void* out, const void* cache, long long page_stride,
                          long long n_pages, const int32_t* block_table, int bt_stride, const int32_t* q_start,
                          const int32_t* q_len, const int32_t* kv_len, int T, int B, int n_heads, int page_size,
-                         float scale, int32_t* tok_scratch, int* err, cudaStream_t stream) {
+                         float scale, const float* sink, int ld_rope, int32_t* tok_scratch, int* err,
+                         cudaStream_t stream) {
   using namespace mb::mlatc;
   if (T <= 0 || B <= 0) return MB_OK;
+  if (ld_rope < DR || ld_rope % 8) return MB_ERR_SHAPE;
   if (n_heads % 128 || page_size % 64 || page_stride % LD || n_pages <= 0) return MB_ERR_SHAPE;
   if ((reinterpret_cast<uintptr_t>(q_lat) | reinterpret_cast<uintptr_t>(q_rope) | reinterpret_cast<uintptr_t>(out) |
        reinterpret_cast<uintptr_t>(cache)) & 15)
@@ -536,10 +548,11 @@ static int mla_tc_launch(const void* q_lat, const void* q_rope, void* out, const
   p.err = err;
   p.page_rows = page_rows; p.bt_stride = bt_stride; p.n_heads = n_heads; p.page_size = page_size;
   p.scale_log2 = scale * 1.4426950408889634f;
+  p.sink = sink;
   CUtensorMap tql, tqr, tkv;
   int rc = cached_tmap(&tql, q_lat, static_cast<uint64_t>(T) * n_heads, R, R, 128, 2);
   if (rc != MB_OK) return rc;
-  rc = cached_tmap(&tqr, q_rope, static_cast<uint64_t>(T) * n_heads, DR, DR, 128, 2);
+  rc = cached_tmap(&tqr, q_rope, static_cast<uint64_t>(T) * n_heads, DR, ld_rope, 128, 2);
   if (rc != MB_OK) return rc;
   rc = cached_tmap(&tkv, cache, static_cast<uint64_t>(total_rows), LD, LD, 64, 2);
   if (rc != MB_OK) return rc;

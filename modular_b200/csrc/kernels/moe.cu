@@ -5,6 +5,8 @@
 //                             best `topk_group` groups, top-k experts inside them, weights from
 //                             the un-biased scores, optional normalisation, times a scaling factor.
 //   moe_router_softmax_topk   plain softmax top-k routing (Mixtral / Qwen style).
+//   moe_table_route           routing by token id: a table names every id's experts, so the expert order of
+//                             all layers of a step is known before the first layer runs (one launch).
 //   moe_create_indices        counting sort of (token, slot) pairs by expert: CSR offsets per
 //                             expert, the permutation and its inverse.
 //   moe_permute_rows          gather token rows into expert order (optionally fused with the
@@ -19,6 +21,8 @@
 #include <stdint.h>
 
 #include "../common/api.h"
+#include "../common/launch.h"
+#include "../common/ptx.cuh"
 
 namespace mb {
 
@@ -178,6 +182,60 @@ __global__ void moe_scatter_kernel(const int32_t* __restrict__ ids, int n, int32
   }
 }
 
+// Routing by token id for all mixture-of-experts layers of a step. One CTA per layer sorts the layer's (token, slot)
+// pairs by expert: desc[l] = {first element of the layer's table in `tables`, experts per token, experts, sum of the
+// earlier layers' experts per token, sum of the earlier layers' (experts + 1), vocabulary rows of the table}.
+// inverse[T * desc[3] + t * top + k] = row of the pair in expert order (-1 for an id outside the table),
+// offsets[desc[4] ...] = CSR offsets per expert.
+__global__ void __launch_bounds__(1024)
+moe_table_route_kernel(const int64_t* __restrict__ ids, int T, const int32_t* __restrict__ tables,
+                       const int64_t* __restrict__ desc, int32_t* __restrict__ inverse, int32_t* __restrict__ offsets) {
+  extern __shared__ int32_t cnt[];       // counts, then cursors
+  pdl_wait();
+  pdl_trigger();
+  const int64_t* d = desc + static_cast<size_t>(blockIdx.x) * 6;
+  const int32_t* tab = tables + d[0];
+  const int top = static_cast<int>(d[1]), E = static_cast<int>(d[2]);
+  const int64_t vocab = d[5];
+  int32_t* inv = inverse + static_cast<size_t>(T) * d[3];
+  int32_t* off = offsets + d[4];
+  for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
+  __syncthreads();
+  const int n = T * top;
+  auto expert = [&](int i) {
+    const int64_t id = ids[i / top];
+    if (id < 0 || id >= vocab) return -1;
+    const int e = tab[id * top + i % top];
+    return e >= 0 && e < E ? e : -1;
+  };
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const int e = expert(i);
+    if (e >= 0) atomicAdd(&cnt[e], 1);
+  }
+  __syncthreads();
+  if (threadIdx.x < 32) {                // exclusive scan of the counts by one warp
+    int base = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + threadIdx.x;
+      const int c = e < E ? cnt[e] : 0;
+      int s = c;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int u = __shfl_up_sync(0xffffffffu, s, o);
+        if (static_cast<int>(threadIdx.x) >= o) s += u;
+      }
+      if (e < E) { cnt[e] = base + s - c; off[e] = base + s - c; }
+      base += __shfl_sync(0xffffffffu, s, 31);
+    }
+    if (threadIdx.x == 0) off[E] = base;
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const int e = expert(i);
+    inv[i] = e >= 0 ? atomicAdd(&cnt[e], 1) : -1;
+  }
+}
+
 // dst[p] = src[order[p] / top_k]  (16 bytes per thread)
 __global__ void moe_permute_rows_kernel(const uint8_t* __restrict__ src, const int32_t* __restrict__ order,
                                         const int32_t* __restrict__ n_rows_dev, uint8_t* __restrict__ dst,
@@ -270,6 +328,14 @@ extern "C" int mb_moe_create_indices(const int32_t* topk_ids, int n_pairs, int e
     moe_scatter_kernel<<<(n_pairs + 255) / 256, 256, 0, stream>>>(topk_ids, n_pairs, cursor, order, inverse,
                                                                  e_begin, e_end);
   return MB_OK_OR_LAUNCH();
+}
+
+extern "C" int mb_moe_table_route(const int64_t* ids, int T, const int32_t* tables, const int64_t* desc, int n_layers,
+                                  int max_experts, int32_t* inverse, int32_t* offsets, cudaStream_t stream) {
+  if (T <= 0 || n_layers <= 0) return MB_OK;
+  if (max_experts <= 0 || max_experts > 8192) return MB_ERR_SHAPE;
+  return launch_k(moe_table_route_kernel, dim3(n_layers), dim3(1024), static_cast<size_t>(max_experts) * 4, stream, ids,
+                  T, tables, desc, inverse, offsets) == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
 }
 
 extern "C" int mb_moe_permute_rows(const void* src, const int32_t* order, const int32_t* n_rows_dev,

@@ -87,12 +87,14 @@ class LLM:
                  disk_kvcache_dir: Optional[str] = None, disk_kvcache_space_gb: float = 0.0,
                  step_token_alignment: Optional[int] = None, weights_are_sharded: bool = False,
                  ep_size: int = 1, ep_rank: int = 0, ep_fp8_dispatch: bool = False, speculative=None,
-                 draft_model_config=None, draft_weights=None):
+                 draft_model_config=None, draft_weights=None, num_state_slots: Optional[int] = None,
+                 max_logit_rows: int = 0):
         """``speculative``: a :class:`pipelines.speculative.SpeculativeConfig`; decode steps of greedy requests
         then verify proposals (several tokens per step, same output as plain greedy decoding): n-gram look-ups in
         the request's own history, or with ``method="draft_model"`` the greedy continuation of a smaller model of
         the same vocabulary (``draft_model_config`` / ``draft_weights``; random weights when none are given),
-        which gets its own paged cache and drafts for all requests of a step at once."""
+        which gets its own paged cache and drafts for all requests of a step at once.
+        ``num_state_slots``: recurrent-state slots of families that keep some (default: one per request of a batch)."""
         from ..models import family_for
 
         fam = family_for(model_config)
@@ -137,7 +139,8 @@ class LLM:
                 weights = fam.weights_class.random_init_ep(model_config, ep_rank, ep_size, self.device, dtype, seed=seed)
         elif weights is None:
             weights = fam.weights_class.random_init(model_config, self.device, dtype, seed=seed)
-        if speculative is not None and fam.name in ("mamba", "lfm2"):
+        recurrent = fam.name in ("mamba", "lfm2") or bool(fam.kv_params(model_config, page_size, dtype, False).state_specs)
+        if speculative is not None and recurrent:
             # verifying a draft runs the rejected tokens through the recurrence too, and a state cannot be rolled back
             raise ValueError("speculative decoding is not implemented for state-space models")
         self.weights = weights
@@ -155,6 +158,8 @@ class LLM:
             if draft_weights is None:
                 draft_weights = dfam.weights_class.random_init(draft_model_config, self.device, dtype, seed=seed + 1)
             dkvp = dfam.kv_params(draft_model_config, page_size, dtype, False)   # no prefix cache: drafts get rewritten
+            if dfam.name in ("mamba", "lfm2") or dkvp.state_specs:
+                raise ValueError("a draft model with recurrent state cannot take back rejected tokens")
             if on_gpu:
                 free, total = torch.cuda.mem_get_info(self.device)
                 d_budget = int(0.1 * (free - (1.0 - device_memory_utilization) * total))
@@ -179,8 +184,11 @@ class LLM:
         host_pages = int(host_kvcache_swap_space_gb * (1 << 30) // kvp.bytes_per_page)
         disk_pages = int(disk_kvcache_space_gb * (1 << 30) // kvp.bytes_per_page) if disk_kvcache_dir else 0
         self.kv = PagedKVCacheManager(kvp, num_kv_pages, self.device, max_seq_len=max_length,
-                                      host_pages=host_pages, disk_pages=disk_pages, disk_dir=disk_kvcache_dir)
+                                      host_pages=host_pages, disk_pages=disk_pages, disk_dir=disk_kvcache_dir,
+                                      state_slots=(num_state_slots or max_batch_size) if kvp.state_specs else 0)
         extra = {"tp": self.tp} if fam.supports_tp else {}
+        if kvp.state_specs:
+            extra["state"] = self.kv.state
         if ep_size > 1:
             from ..parallel.ep import EPContext
 
@@ -207,7 +215,8 @@ class LLM:
             self.model, self.kv, max_batch_input_tokens, max_batch_size, overlap=overlap,
             graph_batch_sizes=graph_batch_sizes if (device_graph_capture and on_gpu) else (),
             eos_token_ids=eos_token_ids, speculative=speculative, draft=self._draft_proposer(max_batch_input_tokens,
-                                                                                             max_batch_size))
+                                                                                             max_batch_size),
+            max_logit_rows=max_logit_rows)
         if device_graph_capture and on_gpu:
             self.pipeline.warmup_graph_capture()
             if hasattr(self.model, "capture_decode_graphs"):

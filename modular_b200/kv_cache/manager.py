@@ -18,6 +18,10 @@ so a (page, plane, layer, head) slice is one contiguous ``page_size x head_dim``
 bulk copy or a TMA box can fetch in one piece, and a whole page (all layers) is contiguous
 for offload and transfer.
 
+Families with recurrent layers add *state slots*: fixed-size tensors per request (``KVCacheParams.state_specs``), one
+slot per live request, taken with its first pages and given back when it is released. A state cannot be shared or
+restored by prefix, so such caches run without prefix caching.
+
 Block hashes are chained: ``h_i = H(h_{i-1} || tokens of page i)`` with the request's salt
 folded into the seed; the final token of a prompt is never hashed, so a full-prompt hit
 still leaves one token to run (reference: block_manager.py:62, :91-98).
@@ -70,6 +74,17 @@ class KVCacheParams:
     dtype: torch.dtype = torch.bfloat16
     is_mla: bool = False
     enable_prefix_caching: bool = True
+    # recurrent state per request: (name, shape of one slot, dtype)
+    state_specs: tuple = ()
+
+    def __post_init__(self):
+        if self.state_specs and self.enable_prefix_caching:
+            raise ValueError("a recurrent state cannot be restored by prefix: prefix caching must be off")
+
+    @property
+    def state_bytes_per_slot(self) -> int:
+        return sum(int(np.prod(shape, dtype=np.int64)) * torch.empty(0, dtype=dt).element_size()
+                   for _, shape, dt in self.state_specs)
 
     @property
     def kv_dim(self) -> int:
@@ -100,12 +115,13 @@ class _ReqState:
     salt: int = 0
     prefix_hit_tokens: int = 0
     prefix_checked: bool = False
+    state_slot: int = -1
 
 
 class PagedKVCacheManager:
     def __init__(self, params: KVCacheParams, num_pages: int, device="cpu", max_seq_len: int = 0,
                  allocate: bool = True, host_pages: int = 0, disk_pages: int = 0,
-                 disk_dir: Optional[str] = None):
+                 disk_dir: Optional[str] = None, state_slots: int = 0):
         self.params = params
         self.page_size = params.page_size
         self.num_pages = num_pages
@@ -116,6 +132,12 @@ class PagedKVCacheManager:
         self.kv = (torch.zeros(params.shape(num_pages), dtype=params.dtype, device=self.device)
                    if allocate else None)
         self._req: dict[str, _ReqState] = {}
+        # recurrent state, one slot per live request: name -> [slots, *shape]
+        if params.state_specs and state_slots < 1:
+            raise ValueError("this cache holds recurrent state: state_slots must be at least 1")
+        self.state = ({name: torch.zeros((state_slots, *shape), dtype=dt, device=self.device)
+                       for name, shape, dt in params.state_specs} if allocate else {})
+        self._free_slots = list(range(state_slots - 1, -1, -1)) if params.state_specs else []
         # lower tiers for evicted prefix pages (pinned host memory, then a file); see tiers.py
         self.tiers = None
         if allocate and params.enable_prefix_caching and host_pages > 0:
@@ -144,6 +166,19 @@ class PagedKVCacheManager:
         # release in reverse so that leaf pages are evicted before their parents
         for bid in reversed(st.blocks):
             self.pool.release(bid)
+        if st.state_slot >= 0:
+            self._free_slots.append(st.state_slot)
+
+    def state_slot_of(self, request_id: str) -> int:
+        """The request's slot in the state tensors (-1 for families without recurrent state)."""
+        return self._req[request_id].state_slot
+
+    @property
+    def free_state_slots(self) -> int:
+        return len(self._free_slots)
+
+    def _needs_slot(self, st: Optional[_ReqState]) -> bool:
+        return bool(self.params.state_specs) and (st is None or st.state_slot < 0)
 
     def reset_prefix_cache(self) -> bool:
         if self.tiers is not None:
@@ -231,6 +266,8 @@ class PagedKVCacheManager:
         (+ ``extra_tokens`` look-ahead). Raises InsufficientBlocksError without side effects
         on the request's existing pages."""
         st = self._req[ctx.request_id]
+        if self._needs_slot(st) and not self._free_slots:
+            raise InsufficientBlocksError(f"request {ctx.request_id} needs a state slot; all are in use")
         self.lookup_prefix(ctx)
         need_tokens = ctx.tokens.active_end + extra_tokens
         need = (need_tokens + self.page_size - 1) // self.page_size - len(st.blocks)
@@ -240,12 +277,14 @@ class PagedKVCacheManager:
                     f"request {ctx.request_id} needs {len(st.blocks) + need} pages; the per-sequence "
                     f"limit is {self.max_pages_per_seq}")
             st.blocks.extend(self.pool.allocate(need))
+        if self._needs_slot(st):
+            st.state_slot = self._free_slots.pop()
 
     def can_alloc(self, ctx: TextContext, extra_tokens: int = 0) -> bool:
         st = self._req.get(ctx.request_id)
         have = len(st.blocks) if st else 0
         need = (ctx.tokens.active_end + extra_tokens + self.page_size - 1) // self.page_size - have
-        return need <= self.pool.free_blocks
+        return need <= self.pool.free_blocks and not (self._needs_slot(st) and not self._free_slots)
 
     # ------------------------------------------------------------ after a forward pass
     def step(self, ctx: TextContext) -> None:

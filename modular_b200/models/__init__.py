@@ -87,6 +87,33 @@ def _lfm2_family() -> ModelFamily:
     return ModelFamily("lfm2", Lfm2Config, Lfm2Weights, Lfm2Model, kv, act)
 
 
+def _gotunex_family() -> ModelFamily:
+    from ..kv_cache import KVCacheParams
+    from .gotunex import GotunexConfig, GotunexModel, GotunexWeights
+
+    def kv(cfg, page, dtype, prefix):
+        # one plane of latent rows per layer that stores any; recurrent state lives in slots and rules out prefix sharing
+        state = cfg.state_specs()
+        return KVCacheParams(max(len(cfg.cache_layers), 1), 1, cfg.cache_width, page, dtype, True, prefix and not state, state)
+
+    def act(cfg, T, B):
+        per_tok = 4 * cfg.width_pad
+        for i, l in enumerate(cfg.layers):
+            m, ff = l["mixer"], l.get("mlp")
+            if cfg.is_attention(i):
+                a = cfg.attention(i)
+                n = a.heads * (a.head_width + 2 * a.cache_width + 2 * a.vdim_pad) + a.q_rank
+            else:
+                n = 8 * m["heads"] * (m["dim"] + m["vdim"])
+            if ff is not None:
+                n += ff["ff"] if ff["kind"] == "dense" else ff["router"]["top"] * (2 * cfg.width_pad + ff["expert"]["ff"])
+            per_tok = max(per_tok, 4 * cfg.width_pad + n)
+        state = kv(cfg, 64, torch.bfloat16, False).state_bytes_per_slot
+        return T * per_tok * 4 + B * cfg.vocab_size * 4 + B * state + (256 << 20)
+
+    return ModelFamily("gotunex", GotunexConfig, GotunexWeights, GotunexModel, kv, act)
+
+
 def _bert_family() -> ModelFamily:
     from ..kv_cache import KVCacheParams
     from .bert import BertConfig, BertModel, BertWeights
@@ -103,7 +130,7 @@ def _bert_family() -> ModelFamily:
 
 def family_for(config) -> ModelFamily:
     """The family that serves `config` (matched on the config class)."""
-    for make in (_llama_family, _deepseek_family, _mamba_family, _lfm2_family, _bert_family):
+    for make in (_llama_family, _deepseek_family, _mamba_family, _lfm2_family, _gotunex_family, _bert_family):
         fam = make()
         if isinstance(config, fam.config_class):
             return fam

@@ -255,3 +255,76 @@ class MoE:
         return self.experts_forward(x, ids, w, self.shared_forward(x))
 
     __call__ = forward
+
+
+# ---------------------------------------------------------------------- routing by token id
+class TableRouter:
+    """Experts chosen by a table of token ids (no scores: the ``top`` experts of an id weigh ``1 / top`` each) for all the
+    mixture-of-experts layers of a model. Since the choice does not depend on activations, one kernel sorts the pairs of
+    every layer before the first layer runs, and the layers' norm and residual kernels read and write expert order
+    directly. ``tables``: one int tensor [vocab, top] and the expert count per layer."""
+
+    def __init__(self, tables: list, experts: list, device):
+        dev = torch.device(device)
+        self.experts = list(experts)
+        self.tops = [int(t.shape[1]) for t in tables]
+        self.tables = [t.to(dev, torch.int32).contiguous() for t in tables]
+        self._flat = torch.cat([t.reshape(-1) for t in self.tables]) if tables else None
+        desc, first, pairs, offs = [], 0, 0, 0
+        for t, e in zip(self.tables, self.experts):
+            desc.append([first, t.shape[1], e, pairs, offs, t.shape[0]])
+            first, pairs, offs = first + t.numel(), pairs + t.shape[1], offs + e + 1
+        self._desc = torch.tensor(desc, dtype=torch.int64, device=dev).view(-1, 6)
+        self._pairs, self._offs = pairs, offs
+
+    def route(self, ids: torch.Tensor) -> list:
+        """Per layer: (inverse int32 [T, top]: row of every pair in expert order, offsets int32 [experts + 1])."""
+        if not self.tables:
+            return []
+        T = ids.numel()
+        if not ids.is_cuda:
+            return [self._route_ref(ids, t, e) for t, e in zip(self.tables, self.experts)]
+        inverse = torch.empty(T * self._pairs, dtype=torch.int32, device=ids.device)
+        offsets = torch.empty(self._offs, dtype=torch.int32, device=ids.device)
+        _lib().moe_table_route(ids, self._flat, self._desc, max(self.experts), inverse, offsets)
+        out, p, o = [], 0, 0
+        for top, e in zip(self.tops, self.experts):
+            out.append((inverse[T * p: T * (p + top)].view(T, top), offsets[o: o + e + 1]))
+            p, o = p + top, o + e + 1
+        return out
+
+    @staticmethod
+    def _route_ref(ids, table, experts):
+        flat = table[ids.long()].reshape(-1).long()
+        order = torch.argsort(flat, stable=True)
+        inverse = torch.empty_like(order)
+        inverse[order] = torch.arange(order.numel())
+        offsets = torch.zeros(experts + 1, dtype=torch.int32)
+        offsets[1:] = torch.cumsum(torch.bincount(flat, minlength=experts), 0)
+        return inverse.view(-1, table.shape[1]).int(), offsets
+
+
+def expert_mlp(xp, offsets, w_gate_up, w_down, max_rows: int):
+    """SwiGLU experts on rows already in expert order: xp [rows, H] -> [rows, H]; w_gate_up [E, 2I, H], w_down [E, H, I].
+    ``max_rows`` bounds the rows of one expert (the step's tokens when a token's experts differ)."""
+    n, I = xp.shape[0], w_gate_up.shape[1] // 2
+    out = torch.empty(n, w_down.shape[1], dtype=xp.dtype, device=xp.device)
+    if not xp.is_cuda:
+        out.zero_()
+        off = offsets.tolist()
+        for e in range(w_down.shape[0]):
+            if off[e + 1] > off[e]:
+                out[off[e]: off[e + 1]] = ops.reference.linear(
+                    ops.reference.linear_swiglu(xp[off[e]: off[e + 1]], w_gate_up[e]), w_down[e])
+        return out
+    act = torch.empty(n, I, dtype=xp.dtype, device=xp.device)
+    L = _lib()
+    if xp.dtype == torch.float32:
+        gu = torch.empty(n, 2 * I, dtype=xp.dtype, device=xp.device)
+        L.grouped_gemm_f32(xp, w_gate_up, gu, offsets)
+        L.silu_mul_f32(gu, act)
+        L.grouped_gemm_f32(act, w_down, out, offsets)
+    else:
+        L.grouped_gemm_bf16(xp, w_gate_up, act, offsets, max_rows, True, 0)
+        L.grouped_gemm_bf16(act, w_down, out, offsets, max_rows, False, 0)
+    return out

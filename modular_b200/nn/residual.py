@@ -1,0 +1,62 @@
+"""The seam between two layers of a decoder whose residual stream is kept in fp32.
+
+``residual_norm`` adds what the branches of the last layer produced and writes the normalised input of every branch of
+the next one in a single kernel (``csrc/kernels/residual_norm.cu``); the PyTorch form below runs on CPU tensors.
+
+* ``table`` / ``ids`` / ``scale``: the stream starts as scaled embedding rows instead of what ``x`` holds;
+* ``a``, ``b``: branch outputs; ``e`` with ``inverse`` [T, k] and ``pair_w``: expert outputs in expert order, summed per
+  token (a mixture-of-experts branch without a combine kernel);
+* ``w1``/``n1`` and ``w2``/``n2``: norm weights and outputs of up to two parallel branches; ``scatter`` [T, k] writes
+  the second one to the rows a token occupies in expert order (no permute kernel);
+* ``rows``: work on these rows of ``x`` only (the ones whose logits are wanted), outputs compacted.
+
+The norm is computed in fp32 and rounded once.
+"""
+
+from __future__ import annotations
+
+import torch
+
+from .._native import lib as _lib
+
+
+def residual_norm_reference(x, ids=None, table=None, scale=1.0, a=None, b=None, e=None, inverse=None, pair_w=1.0, rows=None,
+                            w1=None, n1=None, w2=None, n2=None, scatter=None, cols=0, store_x=True, eps=1e-6):
+    cols = cols or x.shape[1]
+    idx = torch.arange(x.shape[0]) if rows is None else rows.long()
+    h = x[idx] if table is None else table[ids[idx]].float() * scale
+    s = torch.zeros_like(h)
+    if e is not None:
+        inv = inverse.view(x.shape[0], -1)[idx].long()
+        got = e[inv.clamp(min=0)].float() * (inv >= 0).unsqueeze(-1)
+        s = got.sum(1) * pair_w
+    elif b is not None:
+        s = b[idx, : x.shape[1]].float()
+    if a is not None:
+        s = s + a[idx, : x.shape[1]].float()
+    h = h + s
+    if store_x:
+        x[idx] = h
+    if w1 is None:
+        return
+    n = h * torch.rsqrt((h * h).sum(-1, keepdim=True) / cols + eps)
+    n1[: idx.numel()] = (n * w1.float()).to(n1.dtype)
+    if w2 is not None:
+        y = (n * w2.float()).to(n2.dtype)
+        if scatter is None:
+            n2[: idx.numel()] = y
+        else:
+            for k in range(scatter.shape[1]):
+                pos = scatter[idx, k].long()
+                n2[pos[pos >= 0]] = y[pos >= 0]
+
+
+def residual_norm(x, ids=None, table=None, scale=1.0, a=None, b=None, e=None, inverse=None, pair_w=1.0, rows=None, w1=None,
+                  n1=None, w2=None, n2=None, scatter=None, cols=0, store_x=True, eps=1e-6):
+    """x: fp32 [T, width], width padded to a multiple of 4 with zeros; ``cols`` is the true width (the norm's divisor)."""
+    if not x.is_cuda:
+        return residual_norm_reference(x, ids, table, scale, a, b, e, inverse, pair_w, rows, w1, n1, w2, n2, scatter, cols,
+                                       store_x, eps)
+    _lib().residual_norm(x, ids, table, float(scale), a, b, e, inverse, 0 if inverse is None else inverse.numel() // x.shape[0],
+                         float(pair_w), rows, w1, n1, w2, n2, scatter, cols or x.shape[1], store_x, float(eps),
+                         x.shape[0] if rows is None else rows.numel())

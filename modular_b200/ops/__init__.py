@@ -22,7 +22,7 @@ from . import reference as ref
 __all__ = [
     "linear", "linear_swiglu", "rms_norm", "add_rms_norm", "silu_mul", "embedding",
     "rope_kv_store", "paged_attention", "build_attention_plan", "argmax", "sample",
-    "apply_penalties", "gemm_workspace", "check_device_error", "linear_decode", "decode_gemm_workspace",
+    "apply_penalties", "gelu_tanh", "sigmoid_gate", "gemm_workspace", "check_device_error", "linear_decode", "decode_gemm_workspace",
 ]
 
 _WORKSPACES: dict[int, torch.Tensor] = {}
@@ -148,6 +148,9 @@ def batched_linear_heads(x, w, out, x_off, y_off):
         for b in range(B):
             out[:, b * y_off: b * y_off + N] = ref.linear(x[:, b * x_off: b * x_off + K], w[b])
         return out
+    if x.dtype == torch.float32:
+        _lib().batched_gemm_f32(x, w, out, x_off, y_off)
+        return out
     if HEADS_ON_DECODE_GEMM and x.shape[0] <= DECODE_GEMM_MAX_TOKENS and w.shape[1] % 128 == 0 and w.shape[2] % 64 == 0:
         ws, state = decode_gemm_workspace(x.device)
         _lib().gemm_dec_batched(x, w, out, x_off, y_off, ws, state)
@@ -158,13 +161,18 @@ def batched_linear_heads(x, w, out, x_off, y_off):
 
 def linear(x, w, residual=None, out=None, out_dtype=None, bn=0, splits=0, stages=0, impl=None,
            mode=-1, pdl=False):
-    """``x @ w.T`` (+ residual). x: [M, K] bf16, w: [N, K] bf16."""
+    """``x @ w.T`` (+ residual). x: [M, K] bf16, w: [N, K] bf16; fp32 operands run in true 32-bit arithmetic."""
     if not x.is_cuda:
         y = ref.linear(x, w, residual, out_dtype)
         if out is not None:
             out.copy_(y)
             return out
         return y
+    if x.dtype == torch.float32:
+        if out is None:
+            out = torch.empty(x.shape[0], w.shape[0], dtype=torch.float32, device=x.device)
+        _lib().gemm_f32(x, w, out, residual)
+        return out
     if out is None:
         out = torch.empty(x.shape[0], w.shape[0], dtype=out_dtype or x.dtype, device=x.device)
     sel = impl or GEMM_IMPL
@@ -242,13 +250,33 @@ def add_rms_norm(x, residual, w, eps, weight_offset=0.0, multiply_before_cast=Fa
 
 
 def silu_mul(gate_up, out=None):
-    if not gate_up.is_cuda or gate_up.dtype != torch.bfloat16:
+    if not gate_up.is_cuda or gate_up.dtype not in (torch.bfloat16, torch.float32):
         return ref.silu_mul(gate_up)
     if out is None:
         out = torch.empty(gate_up.shape[0], gate_up.shape[1] // 2, dtype=gate_up.dtype,
                           device=gate_up.device)
-    _lib().silu_mul(gate_up, out)
+    if gate_up.dtype == torch.float32:
+        _lib().silu_mul_f32(gate_up, out)
+    else:
+        _lib().silu_mul(gate_up, out)
     return out
+
+
+def gelu_tanh(x):
+    """tanh-form GELU, in place."""
+    if not x.is_cuda:
+        return x.copy_(ref.gelu_tanh(x))
+    _lib().gelu_tanh(x)
+    return x
+
+
+def sigmoid_gate(o, g, cols):
+    """``o[:, :cols] *= sigmoid(g[:, :cols])`` in place (the output gate of an attention layer)."""
+    if not o.is_cuda:
+        o[:, :cols] = (o[:, :cols].float() * torch.sigmoid(g[:, :cols].float())).to(o.dtype)
+        return o
+    _lib().sigmoid_gate(o, g, cols)
+    return o
 
 
 def embedding(ids, table, vocab_start=0, out=None):

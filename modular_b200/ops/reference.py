@@ -46,6 +46,10 @@ def silu_mul(gate_up):
     return (F.silu(g) * u).to(gate_up.dtype)
 
 
+def gelu_tanh(x):
+    return F.gelu(x.float(), approximate="tanh").to(x.dtype)
+
+
 def embedding(ids, table, vocab_start=0):
     local = ids - vocab_start
     ok = (local >= 0) & (local < table.shape[0])

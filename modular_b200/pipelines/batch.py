@@ -27,7 +27,7 @@ from .context import FUTURE_TOKEN, TextContext
 _FIELDS = [
     ("tokens", 2, "T"), ("slots", 2, "T"), ("seeds", 2, "R"),
     ("positions", 1, "T"), ("future_src", 1, "T"),
-    ("q_start", 1, "B"), ("q_len", 1, "B"), ("kv_len", 1, "B"), ("decode_seq", 1, "B"),
+    ("q_start", 1, "B"), ("q_len", 1, "B"), ("kv_len", 1, "B"), ("decode_seq", 1, "B"), ("state_slot", 1, "B"),
     ("logit_rows", 1, "R"), ("temperature", 1, "R"), ("top_k", 1, "R"), ("top_p", 1, "R"),
     ("min_p", 1, "R"), ("tile_seq", 1, "tile"), ("tile_q0", 1, "tile"), ("block_table", 1, "bt"),
 ]
@@ -99,14 +99,15 @@ class BatchPacker:
         return i
 
     def pack(self, ctxs: Sequence[TextContext], kv, fixed: Optional[tuple] = None,
-             pad_to: int = 0, all_logits: bool = False) -> StepBatch:
+             pad_to: int = 0, all_logits: bool = False, want: Optional[Sequence[Sequence[int]]] = None) -> StepBatch:
         """Build the metadata for ``ctxs`` (each contributes its active window).
 
         ``fixed = (T_cap, B_cap, bt_stride, tiles_cap)`` pins the layout (CUDA-graph replay);
         ``pad_to`` pads the batch with dummy single-token sequences on the null page;
         ``all_logits`` asks for the logits of every row of a window that reaches the last known token
         (verification of draft tokens), not only of its last row: the per-row sampling arrays are then laid
-        out for one entry per token.
+        out for one entry per token; ``want`` instead names, per context, the places of its window whose logits are
+        asked for (any places, possibly none).
         """
         B_real = len(ctxs)
         B = max(B_real, pad_to)
@@ -118,11 +119,16 @@ class BatchPacker:
             raise ValueError(f"batch ({T} tokens, {B} sequences) exceeds limits "
                              f"({self.max_tokens}, {self.max_seqs})")
         tile_seq, tile_q0, decode_seq = build_attention_plan(q_lens, self.n_q, self.n_kv)
+        if want is not None and (fixed is not None or all_logits):
+            raise ValueError("want cannot be combined with a fixed layout or all_logits")
         if fixed is None:
             bt_stride = max([len(kv.blocks_of(c.request_id)) for c in ctxs] + [1])
             if all_logits and T > self.max_logit_rows:
                 raise ValueError(f"{T} rows ask for logits; the pipeline was built for {self.max_logit_rows}")
-            off, words = meta_layout(T, B, bt_stride, len(tile_seq), T if all_logits else 0)
+            n_want = 0 if want is None else sum(len(w) for w in want)
+            if n_want > self.max_logit_rows:
+                raise ValueError(f"{n_want} rows ask for logits; the pipeline was built for {self.max_logit_rows}")
+            off, words = meta_layout(T, B, bt_stride, len(tile_seq), max(T if all_logits else 0, n_want))
         else:
             T_cap, B_cap, bt_stride, tiles_cap = fixed
             off, words = meta_layout(T_cap, B_cap, bt_stride, tiles_cap)
@@ -138,8 +144,9 @@ class BatchPacker:
         q_start = sb.arr("q_start", np.int32, B)
         q_len = sb.arr("q_len", np.int32, B)
         kv_len = sb.arr("kv_len", np.int32, B)
+        state_slot = sb.arr("state_slot", np.int32, B)
         bt = sb.arr("block_table", np.int32, B * bt_stride).reshape(B, bt_stride)
-        n_rows_cap = max(B, T) if all_logits else B
+        n_rows_cap = max(B, T) if all_logits else max(B, n_want) if fixed is None else B
         logit_rows = sb.arr("logit_rows", np.int32, n_rows_cap)
         temperature = sb.arr("temperature", np.float32, n_rows_cap)
         top_k = sb.arr("top_k", np.int32, n_rows_cap)
@@ -152,6 +159,7 @@ class BatchPacker:
         if B > 1:
             np.cumsum(q_lens[:-1], out=q_start[1:])
         future_src[:] = -1
+        state_slot[:] = -1
         bt[:] = 0
         n_logits = 0
         ps = self.page_size
@@ -165,6 +173,7 @@ class BatchPacker:
             blocks = kv.blocks_of(c.request_id)
             nb = len(blocks)
             bt[i, :nb] = blocks
+            state_slot[i] = kv.state_slot_of(c.request_id)
             if n == 1:
                 slots[row] = blocks[p0 // ps] * ps + p0 % ps
                 if tokens[row] == FUTURE_TOKEN:
@@ -174,10 +183,13 @@ class BatchPacker:
                 pos = positions[row : row + n].astype(np.int64)
                 slots[row : row + n] = bt[i, pos // ps].astype(np.int64) * ps + pos % ps
             kv_len[i] = tb.active_end
-            if tb.active_end == len(tb):
+            places = None if want is None else [row + int(w) for w in want[i]]
+            if places is not None and any(r < row or r >= row + n for r in places):
+                raise ValueError(f"request {c.request_id} wants logits outside its window of {n} tokens")
+            if places if places is not None else tb.active_end == len(tb):
                 # the window reaches the last known token: this pass produces a new token
                 sp = c.sampling_params
-                for r in (range(row, row + n) if all_logits else (row + n - 1,)):
+                for r in places or (range(row, row + n) if all_logits else (row + n - 1,)):
                     logit_rows[n_logits] = r
                     temperature[n_logits] = 0.0 if sp.is_greedy else sp.temperature
                     top_k[n_logits] = sp.top_k if sp.top_k > 0 else 0
@@ -218,6 +230,27 @@ class BatchPacker:
         self._events[si] = ev
         return self.meta_dev
 
+    def step_tensors(self, sb: StepBatch) -> dict:
+        """Per-array tensors of a step for models that run op by op: on the GPU, views of the packed buffer after its
+        single upload."""
+        if self.meta_dev is None:
+            return self.tensors(sb, self.device)
+        meta = self.upload(sb)
+
+        def view(name, dt, n):
+            o = sb.offsets[name]
+            words = 2 * n if dt is torch.int64 else n
+            v = meta[o: o + words]
+            return v if dt is torch.int32 else v.view(dt)
+
+        i32, i64, f32 = torch.int32, torch.int64, torch.float32
+        out = {n: view(n, dt, sb.T) for n, dt in (("tokens", i64), ("slots", i64), ("positions", i32), ("future_src", i32))}
+        out.update({n: view(n, i32, sb.B) for n in ("q_start", "q_len", "kv_len", "state_slot")})
+        out["block_table"] = view("block_table", i32, sb.B * sb.bt_stride).view(sb.B, sb.bt_stride)
+        out.update({n: view(n, dt, sb.n_logits) for n, dt in (("logit_rows", i32), ("temperature", f32), ("top_k", i32),
+                                                               ("top_p", f32), ("min_p", f32), ("seeds", i64))})
+        return out
+
     @staticmethod
     def tensors(sb: StepBatch, device="cpu") -> dict:
         """Per-array torch tensors (CPU op-by-op path and tests)."""
@@ -226,6 +259,7 @@ class BatchPacker:
             tokens=t("tokens", np.int64, sb.T), positions=t("positions", np.int32, sb.T),
             slots=t("slots", np.int64, sb.T), q_start=t("q_start", np.int32, sb.B),
             q_len=t("q_len", np.int32, sb.B), kv_len=t("kv_len", np.int32, sb.B),
+            state_slot=t("state_slot", np.int32, sb.B),
             block_table=t("block_table", np.int32, sb.B * sb.bt_stride).view(sb.B, sb.bt_stride),
             logit_rows=t("logit_rows", np.int32, sb.n_logits),
             temperature=t("temperature", np.float32, sb.n_logits),

@@ -165,6 +165,17 @@ class TokenBuffer:
         self._len += 1
         self.active_end = self._len
 
+    def extend(self, tokens: Sequence[int] | np.ndarray) -> None:
+        """Append known tokens (a prompt that arrives in portions); they join the active window."""
+        new = np.asarray(tokens, dtype=np.int64).reshape(-1)
+        n = self._len + new.size
+        if n > self._arr.size:
+            arr = np.empty(max(2 * self._arr.size, n), dtype=np.int64)
+            arr[: self._len] = self._arr[: self._len]
+            self._arr = arr
+        self._arr[self._len: n] = new
+        self._len = self.prompt_len = self.active_end = n
+
     def set_token(self, index: int, token: int) -> None:
         self._arr[index] = token
 

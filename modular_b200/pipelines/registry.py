@@ -58,10 +58,12 @@ class PipelineRegistry:
 
     def retrieve_architecture(self, hf_config: dict) -> SupportedArchitecture:
         self._materialise()
-        for name in hf_config.get("architectures", []):
+        # most checkpoints name their architecture in a list, some in a single string
+        names = list(hf_config.get("architectures") or ([hf_config["architecture"]] if hf_config.get("architecture") else []))
+        for name in names:
             if name in self.architectures:
                 return self.architectures[name]
-        raise ValueError(f"no registered architecture among {hf_config.get('architectures')}; "
+        raise ValueError(f"no registered architecture among {names}; "
                          f"known: {sorted(self.architectures)}")
 
     # ------------------------------------------------------------ config resolution
@@ -346,6 +348,13 @@ def _register_builtin() -> None:
         name="Lfm2ForCausalLM", config_class=Lfm2Config, weights_class=Lfm2Weights, model_class=Lfm2Model,
         default_encoding="bfloat16", supported_encodings=("bfloat16", "float32"),
         example_repo_ids=("LiquidAI/LFM2-1.2B",), preset_configs={"tiny-lfm2": Lfm2Config.tiny}), allow_override=True)
+    from ..models.gotunex import GotunexConfig, GotunexModel, GotunexWeights
+
+    # latent attention and gated delta-rule layers with parallel feed-forwards, experts chosen by token id
+    PIPELINE_REGISTRY.register(SupportedArchitecture(
+        name="Gotunex", config_class=GotunexConfig, weights_class=GotunexWeights, model_class=GotunexModel,
+        default_encoding="bfloat16", supported_encodings=("bfloat16", "float32"), example_repo_ids=(),
+        preset_configs={"tiny-gotunex": GotunexConfig.tiny}), allow_override=True)
     from ..models.bert import BertConfig, BertModel, BertWeights
 
     # encoder-only embedding models (bidirectional attention; MPNet adds relative-position biases); embeddings only

@@ -54,9 +54,11 @@ class PipelineStats:
 class TextGenerationPipeline:
     def __init__(self, model, kv_manager: PagedKVCacheManager, max_batch_tokens: int = 8192,
                  max_batch_size: int = 256, overlap: bool = False, graph_batch_sizes: Sequence[int] = (),
-                 eos_token_ids: Sequence[int] = (), speculative=None, draft=None):
+                 eos_token_ids: Sequence[int] = (), speculative=None, draft=None,
+                 max_logit_rows: int = 0):
         """``speculative``: a :class:`speculative.SpeculativeConfig` turns decode steps of greedy requests into
         propose-and-verify steps (the step runs synchronously: the proposals need the previous token values).
+        ``max_logit_rows``: most rows of a step that may ask for logits (default: one per request).
         ``draft``: the :class:`speculative.BatchedDraftProposer` of the ``draft_model`` method."""
         self.model = model
         self.kv = kv_manager
@@ -70,7 +72,7 @@ class TextGenerationPipeline:
         self.spec_stats = None
         self.proposer = None
         self.draft = None
-        rows = max_batch_size
+        rows = max(max_batch_size, max_logit_rows)
         if speculative is not None:
             from .speculative import NgramProposer, SpecStats
 
@@ -240,8 +242,7 @@ class TextGenerationPipeline:
             inflight = _InFlight(sb, ev, host, time.perf_counter(), step_logprobs)
         else:
             sb = self.packer.pack(batch, self.kv)
-            t = BatchPacker.tensors(sb, self.device)
-            toks = t["tokens"]
+            t = self.packer.step_tensors(sb)
             if sb.has_future:
                 raise RuntimeError("future tokens require the overlap (GPU) pipeline")
             extra = {}
@@ -251,8 +252,7 @@ class TextGenerationPipeline:
                 extra["lora"] = LoRABatch(self.lora_manager, token_slots_for(
                     self.lora_manager, [c.tokens.active_length for c in sb.ctxs], [c.lora_name for c in sb.ctxs],
                     self.device))
-            logits = model.forward_tensors(toks, t["positions"], t["slots"], t["block_table"],
-                                           t["q_start"], t["q_len"], t["kv_len"], t["logit_rows"], **extra)
+            logits = self._forward_step(t, **extra)
             mask = self._grammar_bitmask(sb) if self.structured is not None else None
             if mask is not None:
                 ops.apply_token_bitmask(logits, mask)
@@ -268,6 +268,28 @@ class TextGenerationPipeline:
         for c in sb.logit_ctx:
             c.update_with_future_token()
         return inflight
+
+    def _forward_step(self, t: dict, **extra) -> torch.Tensor:
+        """The model's op-by-op step on the tensors of a packed batch; fp32 logits of the rows that ask for them."""
+        if self.kv.params.state_specs:
+            extra["state_slot"] = t["state_slot"]
+        return self.model.forward_tensors(t["tokens"], t["positions"], t["slots"], t["block_table"], t["q_start"],
+                                          t["q_len"], t["kv_len"], t["logit_rows"], **extra)
+
+    def score(self, batch: Sequence[TextContext], want: Sequence[Sequence[int]]) -> torch.Tensor:
+        """One step without sampling: runs every context's active window (its pages must be allocated) and returns the
+        fp32 logits at the places ``want[i]`` of window i, in order. The windows become processed tokens."""
+        self._step += 1
+        self.stats.steps += 1
+        sb = self.packer.pack(batch, self.kv, want=want)
+        if self.on_gpu and self.model.use_executor:
+            raise NotImplementedError(f"{type(self.model).__name__} steps run in the native executor, which samples")
+        logits = self._forward_step(self.packer.step_tensors(sb))
+        self.stats.tokens_in += sb.T
+        for c in sb.ctxs:
+            c.tokens.advance_processed()
+            self.kv.step(c)
+        return logits
 
     def _penalties_and_sample(self, sb: StepBatch, meta: torch.Tensor) -> None:
         n, off = sb.n_logits, sb.offsets
@@ -325,15 +347,15 @@ class TextGenerationPipeline:
                     cnt.extend(counts.get(int(x), 0) for x in u.tolist())
                 offs.append(len(tok))
             sp = [c.sampling_params for c in sb.logit_ctx]
-            ops.apply_penalties(logits, torch.tensor(tok or [0], dtype=torch.int32),
-                                torch.tensor(cnt or [0], dtype=torch.int32), torch.tensor(offs, dtype=torch.int32),
-                                torch.tensor([s.frequency_penalty for s in sp]),
-                                torch.tensor([s.presence_penalty for s in sp]),
-                                torch.tensor([s.repetition_penalty for s in sp]))
+            i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=logits.device)
+            f32 = lambda v: torch.tensor(v, dtype=torch.float32, device=logits.device)
+            ops.apply_penalties(logits, i32(tok or [0]), i32(cnt or [0]), i32(offs),
+                                f32([s.frequency_penalty for s in sp]), f32([s.presence_penalty for s in sp]),
+                                f32([s.repetition_penalty for s in sp]))
         self._add_logit_bias(sb, logits)
         if sb.all_greedy:
             return ops.argmax(logits)
-        return ops.sample(logits, t["temperature"], t["top_k"], t["top_p"], t["min_p"],
+        return ops.sample(logits, t["temperature"], t["top_k"], t["top_p"], t["min_p"], seeds=t["seeds"], step=self._step,
                           generator=self._cpu_gen)
 
     @staticmethod
