@@ -21,7 +21,6 @@ model_config.py; HF ``DeepseekV3ForCausalLM`` naming for checkpoints.
 
 from __future__ import annotations
 
-import contextlib
 import math
 from dataclasses import dataclass, field
 from typing import Optional
@@ -31,25 +30,8 @@ import torch
 from .. import ops
 from ..nn.moe import Fp8ExpertWeights, MoE, MoEConfig
 from ..nn.rotary_embedding import RopeScaling, cos_sin_table
+from .decode_graphs import no_gc_during_capture as _no_gc_during_capture
 
-
-
-@contextlib.contextmanager
-def _no_gc_during_capture():
-    """Collect dead reference cycles now and keep the cyclic collector off while a CUDA graph is captured. The
-    step below runs as Python code that allocates many temporaries; a collection triggered in the middle of it
-    can destroy CUDA graphs of an engine that is no longer referenced, and destroying a graph is not permitted
-    while a stream captures (the capture is invalidated and the next launch fails)."""
-    import gc
-
-    gc.collect()
-    was_on = gc.isenabled()
-    gc.disable()
-    try:
-        yield
-    finally:
-        if was_on:
-            gc.enable()
 
 @dataclass
 class DeepseekV3Config:
