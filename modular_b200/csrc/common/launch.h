@@ -47,4 +47,12 @@ inline cudaError_t launch_k(void (*kern)(KArgs...), dim3 grid, dim3 block, size_
   return cudaLaunchKernelEx(&cfg, kern, static_cast<KArgs>(args)...);
 }
 
+// Ordinary launch: starts when everything before it on the stream has finished.
+template <typename... KArgs, typename... Args>
+inline cudaError_t launch_plain(void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
+                                Args&&... args) {
+  kern<<<grid, block, smem, stream>>>(static_cast<KArgs>(args)...);
+  return cudaGetLastError();
+}
+
 }  // namespace mb

@@ -21,7 +21,6 @@
 
 #include "../common/api.h"
 #include "../common/launch.h"
-#include "../common/ptx.cuh"
 #include "../common/scalar.cuh"
 
 namespace mb {
@@ -39,12 +38,35 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int N>
 __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
+// two fp32 lanes per 64-bit register: one instruction for two multiply-adds, each rounded like fmaf
+struct __align__(16) u64x2 { uint64_t x, y; };
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t pack2(float lo, float hi) {
+  uint64_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ float sum4(uint64_t a, uint64_t b) {
+  float x, y;
+  uint64_t c;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(c) : "l"(a), "l"(b));
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(c));
+  return x + y;
+}
+
 __device__ __forceinline__ float softplusf(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 template <typename T>
 __global__ void __launch_bounds__(256) delta_prep_kernel(const MbDelta p) {
-  pdl_wait();
-  pdl_trigger();
   const int t = blockIdx.x, lane = threadIdx.x & 31;
   const int unit = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int KH = p.kv_heads, H = p.heads, D = p.dim, V = p.vdim, DP = p.dim_pad;
@@ -110,13 +132,132 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const MbDelta p) {
   }
 }
 
+// The same for key widths up to 128 (a multiple of 4) and W taps known at compile time: a lane owns four neighbouring
+// channels, keeps its taps and the convolution window in registers and walks `tile` consecutive tokens.
+template <int W>
+struct ConvLane {
+  float w[W][4];
+  float4 win[W];                    // the last W - 1 inputs in win[1..]
+  template <typename T>
+  __device__ __forceinline__ void taps(const T* p) {     // [4 channels, W]
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+#pragma unroll
+      for (int j = 0; j < W; ++j) w[j][c] = ldf(p + c * W + j);
+  }
+  // inputs before token `off` of its sequence: rows of the step, then the state (`hist` [4 channels, W - 1] or none)
+  template <typename T>
+  __device__ __forceinline__ void start(const T* x, int ldx, int off, const float* hist) {
+#pragma unroll
+    for (int j = 0; j < W - 1; ++j) {
+      const int src = off - (W - 1) + j;
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (src >= 0) {
+        v = ld4(x - static_cast<ptrdiff_t>(W - 1 - j) * ldx);
+      } else if (hist) {
+        const float* h = hist + (W - 1 + src);
+        v = make_float4(h[0], h[W - 1], h[2 * (W - 1)], h[3 * (W - 1)]);
+      }
+      win[j + 1] = v;
+    }
+  }
+  __device__ __forceinline__ float4 step(float4 x) {
+#pragma unroll
+    for (int j = 0; j < W - 1; ++j) win[j] = win[j + 1];
+    win[W - 1] = x;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j < W; ++j) {
+      a.x = fmaf(w[j][0], win[j].x, a.x); a.y = fmaf(w[j][1], win[j].y, a.y);
+      a.z = fmaf(w[j][2], win[j].z, a.z); a.w = fmaf(w[j][3], win[j].w, a.w);
+    }
+    return make_float4(siluf(a.x), siluf(a.y), siluf(a.z), siluf(a.w));
+  }
+};
+
+template <typename T, int W>
+__global__ void __launch_bounds__(256) delta_prep_fast_kernel(const MbDelta p, int tile) {
+  const int lane = threadIdx.x & 31;
+  const int unit = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int KH = p.kv_heads, H = p.heads, D = p.dim, V = p.vdim, DP = p.dim_pad;
+  const int qkC = KH * D, vC = H * V, C = 2 * qkC + vC;
+  if (unit >= KH + H + (vC + 127) / 128) return;
+  const int tb = blockIdx.x * tile, te = min(tb + tile, p.T);
+  int s = tb;
+  if (!p.one_token) {
+    int lo = 0, hi = p.B - 1;
+    while (lo < hi) {
+      const int mid = (lo + hi + 1) >> 1;
+      if (p.q_start[mid] <= tb) lo = mid; else hi = mid - 1;
+    }
+    s = lo;
+  }
+  const bool is_qk = unit < KH, is_g = !is_qk && unit < KH + H;
+  const int c = lane * 4;
+  const int v0 = is_qk || is_g ? 0 : (unit - KH - H) * 128;
+  const bool on = is_qk || is_g ? c < D : v0 + c < vC;
+  const T* w = static_cast<const T*>(p.conv_w);
+  const T* xq = static_cast<const T*>(p.x) + (is_qk ? p.q_off + unit * D + c : p.v_off + v0 + c);
+  const T* xk = static_cast<const T*>(p.x) + p.k_off + unit * D + c;
+  const int ch_a = is_qk ? unit * D + c : 2 * qkC + v0 + c, ch_b = qkC + unit * D + c;
+  ConvLane<W> ca, cb;
+  if (on && !is_g) ca.taps(w + static_cast<size_t>(ch_a) * W);
+  if (on && is_qk) cb.taps(w + static_cast<size_t>(ch_b) * W);
+  const float a_log = is_g ? expf(p.A_log[unit - KH]) : 0.f;
+  float4 bias = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (is_g && on) bias = *reinterpret_cast<const float4*>(p.dt_bias + (unit - KH) * D + c);
+  const float scale = 1.f / sqrtf(static_cast<float>(D));
+  int end = 0;                       // first token behind the current sequence
+  for (int t = tb; t < te; ++t) {
+    if (t >= end) {                  // a new sequence (or the first token of the tile)
+      if (t > tb) ++s;
+      while (s < p.B && p.q_start[s] + p.q_len[s] <= t) ++s;
+      if (s >= p.B || p.q_start[s] > t) return;      // rows of no sequence
+      end = p.q_start[s] + p.q_len[s];
+      if (!is_g && on) {
+        const int off = t - p.q_start[s], slot = p.state_idx[s];
+        const float* hist = (slot >= 0 && W > 1 && p.kv_len[s] > p.q_len[s])
+                                ? p.conv_state + static_cast<size_t>(slot) * C * (W - 1) : nullptr;
+        ca.start(xq + static_cast<size_t>(t) * p.ldx, p.ldx, off, hist ? hist + static_cast<size_t>(ch_a) * (W - 1) : nullptr);
+        if (is_qk)
+          cb.start(xk + static_cast<size_t>(t) * p.ldx, p.ldx, off, hist ? hist + static_cast<size_t>(ch_b) * (W - 1) : nullptr);
+      }
+    }
+    const size_t row = static_cast<size_t>(t) * p.ldx;
+    if (is_qk) {
+      float4 q = make_float4(0.f, 0.f, 0.f, 0.f), k = q;
+      if (on) { q = ca.step(ld4(xq + row)); k = cb.step(ld4(xk + row)); }
+      float qq = q.x * q.x + q.y * q.y + q.z * q.z + q.w * q.w, kk = k.x * k.x + k.y * k.y + k.z * k.z + k.w * k.w;
+      float kq = q.x * k.x + q.y * k.y + q.z * k.z + q.w * k.w;
+      qq = warp_allsum(qq); kk = warp_allsum(kk); kq = warp_allsum(kq);
+      const float iq = scale / sqrtf(qq + 1e-6f), ik = 1.f / sqrtf(kk + 1e-6f);
+      const size_t o = (static_cast<size_t>(t) * KH + unit) * DP + c;
+      if (c < DP) {
+        *reinterpret_cast<float4*>(p.q + o) = make_float4(q.x * iq, q.y * iq, q.z * iq, q.w * iq);
+        *reinterpret_cast<float4*>(p.k + o) = make_float4(k.x * ik, k.y * ik, k.z * ik, k.w * ik);
+      }
+      if (lane == 0) p.kq[static_cast<size_t>(t) * KH + unit] = kq * iq * ik;
+    } else if (is_g) {
+      const int h = unit - KH;
+      float4 g = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (on) {
+        const float4 z = *reinterpret_cast<const float4*>(p.z + static_cast<size_t>(t) * p.ldz + h * D + c);
+        g = make_float4(expf(-a_log * softplusf(z.x + bias.x)), expf(-a_log * softplusf(z.y + bias.y)),
+                        expf(-a_log * softplusf(z.z + bias.z)), expf(-a_log * softplusf(z.w + bias.w)));
+      }
+      if (c < DP) *reinterpret_cast<float4*>(p.g + (static_cast<size_t>(t) * H + h) * DP + c) = g;
+      if (lane == 0) p.beta[static_cast<size_t>(t) * H + h] = sigmoidf(ldf(static_cast<const T*>(p.x) + row + p.b_off + h));
+    } else if (on) {
+      *reinterpret_cast<float4*>(p.v + static_cast<size_t>(t) * vC + v0 + c) = ca.step(ld4(xq + row));
+    }
+  }
+}
+
 template <typename T, int RL4, int MAXT, bool FUSE>
 __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int col_blocks, int chunk) {
   constexpr int DP = 32 * RL4;
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[32];
-  pdl_wait();
-  pdl_trigger();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int rg = lane & 7, cg = lane >> 3;
   const int KH = p.kv_heads, H = p.heads, V = p.vdim;
@@ -126,91 +267,91 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
   const bool resume = slot >= 0 && p.kv_len[s] > n;
   if (n > 0) {
     const int row_floats = 3 * DP + cols;          // q | k | g | v columns, then beta and k . q per token
-    float* stage[2] = {sm, sm + chunk * (row_floats + 2)};
-    float* so = sm + 2 * chunk * (row_floats + 2); // FUSE: outputs of one token
-    auto fetch = [&](int c0, float* dst) {
+    const int stage_floats = chunk * (row_floats + 2);
+    float* so = sm + 2 * stage_floats;             // FUSE: outputs of one token
+    auto fetch = [&](int c0, float* dst) {         // every thread walks the tokens of its piece of the row
       const int m = min(chunk, n - c0);
-      float* sc = dst + chunk * row_floats;
-      for (int i = tid; i < m * (3 * DP / 4); i += blockDim.x) {
-        const int j = i / (3 * DP / 4), v = i % (3 * DP / 4);
-        const size_t t = static_cast<size_t>(t0 + c0 + j);
-        const int which = v / (DP / 4), c = (v % (DP / 4)) * 4;
+      const size_t t = static_cast<size_t>(t0 + c0);
+      for (int pc = tid; pc < 3 * DP / 4; pc += blockDim.x) {
+        const int which = pc / (DP / 4), c = (pc % (DP / 4)) * 4;
         const float* src = which == 0 ? p.q + (t * KH + kh) * DP : which == 1 ? p.k + (t * KH + kh) * DP : p.g + (t * H + h) * DP;
-        cp_async16(dst + j * row_floats + v * 4, src + c);
+        src += c;
+        const int step = (which == 2 ? H : KH) * DP;
+        float* d = dst + pc * 4;
+        for (int j = 0; j < m; ++j, src += step, d += row_floats) cp_async16(d, src);
       }
-      for (int i = tid; i < m * cols; i += blockDim.x) {
-        const int j = i / cols, c = i % cols;
-        if (cbase + c < V) cp_async4(dst + j * row_floats + 3 * DP + c, p.v + (static_cast<size_t>(t0 + c0 + j) * H + h) * V + cbase + c);
+      if (tid < cols && cbase + tid < V) {
+        const float* src = p.v + (t * H + h) * V + cbase + tid;
+        float* d = dst + 3 * DP + tid;
+        for (int j = 0; j < m; ++j, src += H * V, d += row_floats) cp_async4(d, src);
       }
-      for (int i = tid; i < 2 * m; i += blockDim.x) {
-        const size_t t = static_cast<size_t>(t0 + c0 + (i >> 1));
-        cp_async4(sc + i, (i & 1) ? p.kq + t * KH + kh : p.beta + t * H + h);
-      }
+      float* sc = dst + chunk * row_floats;
+      for (int i = tid; i < 2 * m; i += blockDim.x)
+        cp_async4(sc + i, (i & 1) ? p.kq + (t + (i >> 1)) * KH + kh : p.beta + (t + (i >> 1)) * H + h);
       cp_async_commit();
     };
-    fetch(0, stage[0]);
+    fetch(0, sm);
     const int col0 = cbase + warp * 8 + cg * 2;
     const bool ok0 = col0 < V, ok1 = col0 + 1 < V;
     float* st = p.state + ((static_cast<size_t>(slot >= 0 ? slot : 0) * H + h) * V + col0) * DP;
-    float4 S0[RL4], S1[RL4];
+    u64x2 S0[RL4], S1[RL4];                        // four rows per entry, two packed fp32 pairs
 #pragma unroll
     for (int i = 0; i < RL4; ++i) {
       const int r = (i * 8 + rg) * 4;
-      S0[i] = (resume && ok0) ? *reinterpret_cast<const float4*>(st + r) : make_float4(0.f, 0.f, 0.f, 0.f);
-      S1[i] = (resume && ok1) ? *reinterpret_cast<const float4*>(st + DP + r) : make_float4(0.f, 0.f, 0.f, 0.f);
+      S0[i] = (resume && ok0) ? *reinterpret_cast<const u64x2*>(st + r) : u64x2{0ull, 0ull};
+      S1[i] = (resume && ok1) ? *reinterpret_cast<const u64x2*>(st + DP + r) : u64x2{0ull, 0ull};
     }
     const bool hi_col = (lane & 4) != 0, is_q = (lane & 2) != 0;
+    const int my_col = warp * 8 + cg * 2 + (hi_col ? 1 : 0);
+    float* optr = p.o + (static_cast<size_t>(t0) * H + h) * V + cbase + my_col;
+    const bool writes = (lane & 3) == 2 && cbase + my_col < V;
     for (int c0 = 0, it = 0; c0 < n; c0 += chunk, ++it) {
       const int m = min(chunk, n - c0);
-      if (c0 + chunk < n) { fetch(c0 + chunk, stage[(it + 1) & 1]); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
+      const float* buf = sm + (it & 1) * stage_floats;
+      if (c0 + chunk < n) { fetch(c0 + chunk, sm + ((it + 1) & 1) * stage_floats); cp_async_wait<1>(); } else { cp_async_wait<0>(); }
       __syncthreads();
-      const float* buf = stage[it & 1];
       const float* sc = buf + chunk * row_floats;
+#pragma unroll 2
       for (int j = 0; j < m; ++j) {
         const float* rowp = buf + j * row_floats;
-        float4 kr[RL4];
-        float a0[4] = {}, a1[4] = {}, b0[4] = {}, b1[4] = {};
+        u64x2 kr[RL4];
+        uint64_t a0 = 0ull, a1 = 0ull, b0 = 0ull, b1 = 0ull, a0h = 0ull, a1h = 0ull, b0h = 0ull, b1h = 0ull;
 #pragma unroll
         for (int i = 0; i < RL4; ++i) {
           const int r = (i * 8 + rg) * 4;
-          const float4 q4 = *reinterpret_cast<const float4*>(rowp + r);
-          const float4 k4 = *reinterpret_cast<const float4*>(rowp + DP + r);
-          const float4 g4 = *reinterpret_cast<const float4*>(rowp + 2 * DP + r);
+          const u64x2 q4 = *reinterpret_cast<const u64x2*>(rowp + r);
+          const u64x2 k4 = *reinterpret_cast<const u64x2*>(rowp + DP + r);
+          const u64x2 g4 = *reinterpret_cast<const u64x2*>(rowp + 2 * DP + r);
           kr[i] = k4;
-          S0[i].x *= g4.x; S0[i].y *= g4.y; S0[i].z *= g4.z; S0[i].w *= g4.w;
-          S1[i].x *= g4.x; S1[i].y *= g4.y; S1[i].z *= g4.z; S1[i].w *= g4.w;
-          a0[0] = fmaf(S0[i].x, k4.x, a0[0]); a0[1] = fmaf(S0[i].y, k4.y, a0[1]);
-          a0[2] = fmaf(S0[i].z, k4.z, a0[2]); a0[3] = fmaf(S0[i].w, k4.w, a0[3]);
-          a1[0] = fmaf(S1[i].x, k4.x, a1[0]); a1[1] = fmaf(S1[i].y, k4.y, a1[1]);
-          a1[2] = fmaf(S1[i].z, k4.z, a1[2]); a1[3] = fmaf(S1[i].w, k4.w, a1[3]);
-          b0[0] = fmaf(S0[i].x, q4.x, b0[0]); b0[1] = fmaf(S0[i].y, q4.y, b0[1]);
-          b0[2] = fmaf(S0[i].z, q4.z, b0[2]); b0[3] = fmaf(S0[i].w, q4.w, b0[3]);
-          b1[0] = fmaf(S1[i].x, q4.x, b1[0]); b1[1] = fmaf(S1[i].y, q4.y, b1[1]);
-          b1[2] = fmaf(S1[i].z, q4.z, b1[2]); b1[3] = fmaf(S1[i].w, q4.w, b1[3]);
+          S0[i].x = mul2(S0[i].x, g4.x); S0[i].y = mul2(S0[i].y, g4.y);
+          S1[i].x = mul2(S1[i].x, g4.x); S1[i].y = mul2(S1[i].y, g4.y);
+          a0 = fma2(S0[i].x, k4.x, a0); a0h = fma2(S0[i].y, k4.y, a0h);
+          a1 = fma2(S1[i].x, k4.x, a1); a1h = fma2(S1[i].y, k4.y, a1h);
+          b0 = fma2(S0[i].x, q4.x, b0); b0h = fma2(S0[i].y, q4.y, b0h);
+          b1 = fma2(S1[i].x, q4.x, b1); b1h = fma2(S1[i].y, q4.y, b1h);
         }
-        const float A0 = (a0[0] + a0[1]) + (a0[2] + a0[3]), A1 = (a1[0] + a1[1]) + (a1[2] + a1[3]);
-        const float B0 = (b0[0] + b0[1]) + (b0[2] + b0[3]), B1 = (b1[0] + b1[1]) + (b1[2] + b1[3]);
+        const float A0 = sum4(a0, a0h), A1 = sum4(a1, a1h), B0 = sum4(b0, b0h), B1 = sum4(b1, b1h);
         // eight partial sums of four values: lanes with bit 2 take column 1, lanes with bit 1 the q product
         float a = (hi_col ? A1 : A0) + __shfl_xor_sync(0xffffffffu, hi_col ? A0 : A1, 4);
         float b = (hi_col ? B1 : B0) + __shfl_xor_sync(0xffffffffu, hi_col ? B0 : B1, 4);
         float r = (is_q ? b : a) + __shfl_xor_sync(0xffffffffu, is_q ? a : b, 2);
         r += __shfl_xor_sync(0xffffffffu, r, 1);
         const float beta = sc[2 * j], kq = sc[2 * j + 1];
-        const float vv = rowp[3 * DP + warp * 8 + cg * 2 + (hi_col ? 1 : 0)];
+        const float vv = rowp[3 * DP + my_col];
         const float u = beta * (vv - r);           // meaningful in the lanes that hold a key product
         const float u0 = __shfl_sync(0xffffffffu, u, lane & 24), u1 = __shfl_sync(0xffffffffu, u, (lane & 24) | 4);
+        const uint64_t u0p = pack2(u0, u0), u1p = pack2(u1, u1);
 #pragma unroll
         for (int i = 0; i < RL4; ++i) {
-          S0[i].x = fmaf(kr[i].x, u0, S0[i].x); S0[i].y = fmaf(kr[i].y, u0, S0[i].y);
-          S0[i].z = fmaf(kr[i].z, u0, S0[i].z); S0[i].w = fmaf(kr[i].w, u0, S0[i].w);
-          S1[i].x = fmaf(kr[i].x, u1, S1[i].x); S1[i].y = fmaf(kr[i].y, u1, S1[i].y);
-          S1[i].z = fmaf(kr[i].z, u1, S1[i].z); S1[i].w = fmaf(kr[i].w, u1, S1[i].w);
+          S0[i].x = fma2(kr[i].x, u0p, S0[i].x); S0[i].y = fma2(kr[i].y, u0p, S0[i].y);
+          S1[i].x = fma2(kr[i].x, u1p, S1[i].x); S1[i].y = fma2(kr[i].y, u1p, S1[i].y);
         }
         const float o = fmaf(hi_col ? u1 : u0, kq, r);
-        if ((lane & 3) == 2) {
-          const int c = warp * 8 + cg * 2 + (hi_col ? 1 : 0);
-          if (FUSE) so[c] = cbase + c < V ? o : 0.f;
-          else if (cbase + c < V) p.o[(static_cast<size_t>(t0 + c0 + j) * H + h) * V + cbase + c] = o;
+        if (FUSE) {
+          if ((lane & 3) == 2) so[my_col] = cbase + my_col < V ? o : 0.f;
+        } else {
+          if (writes) *optr = o;
+          optr += H * V;
         }
         if (FUSE) {                                // one CTA holds the whole head (cbase = 0)
           __syncthreads();
@@ -236,8 +377,8 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
 #pragma unroll
       for (int i = 0; i < RL4; ++i) {
         const int r = (i * 8 + rg) * 4;
-        if (ok0) *reinterpret_cast<float4*>(st + r) = S0[i];
-        if (ok1) *reinterpret_cast<float4*>(st + DP + r) = S1[i];
+        if (ok0) *reinterpret_cast<u64x2*>(st + r) = S0[i];
+        if (ok1) *reinterpret_cast<u64x2*>(st + DP + r) = S1[i];
       }
     }
   }
@@ -262,8 +403,6 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
 
 template <typename T>
 __global__ void __launch_bounds__(256) delta_out_kernel(const MbDelta p) {
-  pdl_wait();
-  pdl_trigger();
   const int V = p.vdim, lane = threadIdx.x & 31;
   const long long unit = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (unit >= static_cast<long long>(p.T) * p.heads) return;
@@ -289,7 +428,7 @@ static int scan(const MbDelta& p, int num_sms, cudaStream_t stream) {
     warps = head_warps;
   } else {                         // fewer columns per CTA until the step fills the machine
     warps = MAXT / 32 < 4 ? MAXT / 32 : 4;
-    while (warps > 1 && static_cast<long long>(p.B) * p.heads * ((head_warps + warps - 1) / warps) < 2ll * num_sms) warps >>= 1;
+    while (warps > 1 && static_cast<long long>(p.B) * p.heads * ((head_warps + warps - 1) / warps) < num_sms) warps >>= 1;
     if (warps > head_warps) warps = head_warps;
   }
   const int col_blocks = (head_warps + warps - 1) / warps;
@@ -305,12 +444,12 @@ static int scan(const MbDelta& p, int num_sms, cudaStream_t stream) {
   const dim3 grid(p.heads * col_blocks, p.B);
   cudaError_t e;
   if (fuse) {
-    e = launch_k(delta_scan_kernel<T, RL4, MAXT, true>, grid, dim3(warps * 32), smem, stream, p, col_blocks, chunk);
+    e = launch_plain(delta_scan_kernel<T, RL4, MAXT, true>, grid, dim3(warps * 32), smem, stream, p, col_blocks, chunk);
   } else {
-    e = launch_k(delta_scan_kernel<T, RL4, MAXT, false>, grid, dim3(warps * 32), smem, stream, p, col_blocks, chunk);
+    e = launch_plain(delta_scan_kernel<T, RL4, MAXT, false>, grid, dim3(warps * 32), smem, stream, p, col_blocks, chunk);
     if (e == cudaSuccess) {
       const long long units = static_cast<long long>(p.T) * p.heads;
-      e = launch_k(delta_out_kernel<T>, dim3(static_cast<unsigned>((units + 7) / 8)), dim3(256), 0, stream, p);
+      e = launch_plain(delta_out_kernel<T>, dim3(static_cast<unsigned>((units + 7) / 8)), dim3(256), 0, stream, p);
     }
   }
   return e == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
@@ -320,8 +459,19 @@ template <typename T>
 static int run(const MbDelta& p, int num_sms, cudaStream_t stream) {
   const int vC = p.heads * p.vdim;
   const int units = p.kv_heads + p.heads + (vC + 127) / 128;
-  if (launch_k(delta_prep_kernel<T>, dim3(p.T, (units + 7) / 8), dim3(256), 0, stream, p) != cudaSuccess)
-    return MB_ERR_LAUNCH;
+  // vector loads: four channels per lane, every row and block start aligned to them
+  const bool fast = p.dim <= 128 && p.dim % 4 == 0 && vC % 4 == 0 && p.taps >= 2 && p.taps <= 4 && p.ldx % 8 == 0 &&
+                    p.q_off % 8 == 0 && p.k_off % 8 == 0 && p.v_off % 8 == 0 && p.ldz % 4 == 0 &&
+                    ((reinterpret_cast<uintptr_t>(p.x) | reinterpret_cast<uintptr_t>(p.z) | reinterpret_cast<uintptr_t>(p.v) |
+                      reinterpret_cast<uintptr_t>(p.dt_bias)) & 15) == 0;
+  const int tile = p.T <= 4 * p.B ? 1 : 16;
+  const dim3 grid((p.T + tile - 1) / tile, (units + 7) / 8);
+  cudaError_t e;
+  if (fast && p.taps == 4) e = launch_plain(delta_prep_fast_kernel<T, 4>, grid, dim3(256), 0, stream, p, tile);
+  else if (fast && p.taps == 3) e = launch_plain(delta_prep_fast_kernel<T, 3>, grid, dim3(256), 0, stream, p, tile);
+  else if (fast) e = launch_plain(delta_prep_fast_kernel<T, 2>, grid, dim3(256), 0, stream, p, tile);
+  else e = launch_plain(delta_prep_kernel<T>, dim3(p.T, (units + 7) / 8), dim3(256), 0, stream, p);
+  if (e != cudaSuccess) return MB_ERR_LAUNCH;
   switch (p.dim_pad / 32) {
     case 1: return scan<T, 1>(p, num_sms, stream);
     case 2: return scan<T, 2>(p, num_sms, stream);

@@ -8,7 +8,6 @@
 
 #include "../common/api.h"
 #include "../common/launch.h"
-#include "../common/ptx.cuh"
 
 namespace mb {
 namespace simt {
@@ -28,8 +27,6 @@ struct Params {
 __global__ void __launch_bounds__(256) gemm_simt_kernel(const Params p) {
   __shared__ __align__(16) float sx[kBK][kBM + kPad];
   __shared__ __align__(16) float sw[kBK][kBN + kPad];
-  pdl_wait();
-  pdl_trigger();
   const int z = blockIdx.z;
   int m_begin = 0, m_end = p.M;
   if (p.offsets) { m_begin = p.offsets[z]; m_end = p.offsets[z + 1]; }
@@ -77,8 +74,6 @@ __global__ void __launch_bounds__(256) gemm_simt_kernel(const Params p) {
 
 // out[r, i] = silu(gu[r, i]) * gu[r, inter + i]
 __global__ void silu_mul_f32_kernel(const float* __restrict__ gu, float* __restrict__ out, size_t n, int inter) {
-  pdl_wait();
-  pdl_trigger();
   const size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= n) return;
   const size_t r = i / inter, c = i % inter;
@@ -89,7 +84,7 @@ __global__ void silu_mul_f32_kernel(const float* __restrict__ gu, float* __restr
 static int launch(const Params& p, int m_rows, int batches, cudaStream_t stream) {
   const dim3 grid((p.N + kBN - 1) / kBN, (m_rows + kBM - 1) / kBM, batches);
   if (grid.y > 65535 || grid.z > 65535) return MB_ERR_TOO_LARGE;
-  return launch_k(gemm_simt_kernel, grid, dim3(256), 0, stream, p) == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
+  return launch_plain(gemm_simt_kernel, grid, dim3(256), 0, stream, p) == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
 }
 
 }  // namespace simt
@@ -121,6 +116,6 @@ extern "C" int mb_grouped_gemm_f32(const float* x, const float* w, float* y, con
 extern "C" int mb_silu_mul_f32(const float* gu, float* out, int rows, int inter, cudaStream_t stream) {
   if (rows <= 0 || inter <= 0) return MB_OK;
   const size_t n = static_cast<size_t>(rows) * inter;
-  return launch_k(simt::silu_mul_f32_kernel, dim3(static_cast<unsigned>((n + 255) / 256)), dim3(256), 0, stream, gu, out,
+  return launch_plain(simt::silu_mul_f32_kernel, dim3(static_cast<unsigned>((n + 255) / 256)), dim3(256), 0, stream, gu, out,
                   n, inter) == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
 }

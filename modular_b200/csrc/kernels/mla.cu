@@ -23,7 +23,6 @@
 
 #include "../common/api.h"
 #include "../common/launch.h"
-#include "../common/ptx.cuh"
 
 namespace mb {
 namespace mla {
@@ -114,8 +113,6 @@ __global__ void __launch_bounds__(256, 1) mla_kernel(const Params p) {
   bf16* sK = sQ + 64 * LD;                       // [2][64][LD]
   __shared__ int s_seq, s_tq0;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  pdl_wait();
-  pdl_trigger();
   const int tokens_per_tile = 64 / p.HB;
   const int rows = tokens_per_tile * p.HB;   // query rows of a full tile (below 64 when HB does not divide it)
 
@@ -292,8 +289,6 @@ __global__ void __launch_bounds__(256, 1) mla_kernel(const Params p) {
 __global__ void __launch_bounds__(256)
 mla_combine_kernel(const float* __restrict__ ws, bf16* __restrict__ out, const float* __restrict__ sink, int n_rows,
                    int n_heads, int R, int nsplit) {
-  pdl_wait();
-  pdl_trigger();
   const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (row >= n_rows) return;
   const float2* ml = reinterpret_cast<const float2*>(ws + static_cast<int64_t>(nsplit) * n_rows * R);
@@ -444,10 +439,10 @@ static int launch(const Params& p, int grid_x, cudaStream_t stream) {
     configured.done();
   }
   dim3 grid(grid_x, p.n_heads / p.HB, p.nsplit);
-  if (launch_k(kern, grid, dim3(256), smem, stream, p) != cudaSuccess) return MB_ERR_LAUNCH;
+  if (launch_plain(kern, grid, dim3(256), smem, stream, p) != cudaSuccess) return MB_ERR_LAUNCH;
   if (p.nsplit > 1) {
     const int n_rows = p.T * p.n_heads;
-    if (launch_k(mla_combine_kernel, dim3((n_rows + 7) / 8), dim3(256), 0, stream, static_cast<const float*>(p.ws), p.out,
+    if (launch_plain(mla_combine_kernel, dim3((n_rows + 7) / 8), dim3(256), 0, stream, static_cast<const float*>(p.ws), p.out,
                  p.sink, n_rows, p.n_heads, R, p.nsplit) != cudaSuccess)
       return MB_ERR_LAUNCH;
   }

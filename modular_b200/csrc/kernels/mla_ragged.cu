@@ -14,7 +14,6 @@
 
 #include "../common/api.h"
 #include "../common/launch.h"
-#include "../common/ptx.cuh"
 #include "../common/scalar.cuh"
 
 namespace mb {
@@ -44,32 +43,58 @@ struct PostDown {
   const int64_t* slots;
 };
 
+// RMS norm of one row by the CTA: dst[c] = src[c] / rms * gamma[c] for c < n, zeros up to n_pad. Rows whose pieces are
+// aligned go through registers four values at a time (one read of `src`), others element by element.
 template <typename T>
-__global__ void __launch_bounds__(128)
+__device__ __forceinline__ void norm_row(const T* src, const T* gamma, T* dst, int n, int n_pad, float eps, bool vec, float* scratch) {
+  const int tid = threadIdx.x;
+  float ss = 0.f;
+  if (vec) {                                 // n and n_pad are multiples of 4, n <= 4 * kVec * blockDim.x
+    constexpr int kVec = 2;
+    float4 x[kVec], g[kVec];
+#pragma unroll
+    for (int i = 0; i < kVec; ++i) {
+      const int c = (tid + i * blockDim.x) * 4;
+      x[i] = c < n ? ld4(src + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      g[i] = c < n ? ld4(gamma + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
+    }
+    const float inv = 1.f / sqrtf(block_allsum(ss, scratch) / static_cast<float>(n) + eps);
+#pragma unroll
+    for (int i = 0; i < kVec; ++i) {
+      const int c = (tid + i * blockDim.x) * 4;
+      if (c < n_pad) st4(dst + c, make_float4(x[i].x * inv * g[i].x, x[i].y * inv * g[i].y, x[i].z * inv * g[i].z, x[i].w * inv * g[i].w));
+    }
+    return;
+  }
+  for (int c = tid; c < n; c += blockDim.x) { const float v = ldf(src + c); ss += v * v; }
+  const float inv = 1.f / sqrtf(block_allsum(ss, scratch) / static_cast<float>(n) + eps);
+  for (int c = tid; c < n_pad; c += blockDim.x) stf(dst + c, c < n ? ldf(src + c) * inv * ldf(gamma + c) : 0.f);
+}
+
+__device__ __forceinline__ bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+template <typename T>
+__global__ void __launch_bounds__(256)
 post_down_kernel(const PostDown p, const T* __restrict__ x, const T* __restrict__ gamma_q, const T* __restrict__ gamma_kv,
                  T* __restrict__ q_out, T* __restrict__ cache) {
-  __shared__ float scratch[4];
-  pdl_wait();
-  pdl_trigger();
+  __shared__ float scratch[8];
   const int t = blockIdx.x, tid = threadIdx.x;
   const T* row = x + static_cast<size_t>(t) * p.ld;
   if (p.q_rank > 0) {
-    float ss = 0.f;
-    for (int c = tid; c < p.q_rank; c += blockDim.x) { const float v = ldf(row + c); ss += v * v; }
-    const float inv = 1.f / sqrtf(block_allsum(ss, scratch) / static_cast<float>(p.q_rank) + p.eps);
     T* o = q_out + static_cast<size_t>(t) * p.ld_q;
-    for (int c = tid; c < p.q_rank_pad; c += blockDim.x)
-      stf(o + c, c < p.q_rank ? ldf(row + c) * inv * ldf(gamma_q + c) : 0.f);
+    norm_row(row, gamma_q, o, p.q_rank, p.q_rank_pad, p.eps,
+             p.q_rank % 4 == 0 && p.q_rank_pad % 4 == 0 && p.q_rank_pad <= 8 * static_cast<int>(blockDim.x) && aligned16(row) &&
+                 aligned16(gamma_q) && aligned16(o), scratch);
   }
   if (p.kv_off < 0) return;
   const int64_t slot = p.slots[t];
   if (slot < 0) return;                    // uniform over the CTA
   const T* kv = row + p.kv_off;
-  float ss = 0.f;
-  for (int c = tid; c < p.R; c += blockDim.x) { const float v = ldf(kv + c); ss += v * v; }
-  const float inv = 1.f / sqrtf(block_allsum(ss, scratch) / static_cast<float>(p.R) + p.eps);
   T* dst = cache + (slot / p.page_size) * p.page_stride + (slot % p.page_size) * p.ld_cache;
-  for (int c = tid; c < p.Rp; c += blockDim.x) stf(dst + c, c < p.R ? ldf(kv + c) * inv * ldf(gamma_kv + c) : 0.f);
+  norm_row(kv, gamma_kv, dst, p.R, p.Rp, p.eps,
+           p.R % 4 == 0 && p.Rp % 4 == 0 && p.Rp <= 8 * static_cast<int>(blockDim.x) && aligned16(kv) && aligned16(gamma_kv) &&
+               aligned16(dst), scratch);
   const T* kr = kv + p.R;
   const float* cs = p.cos_sin + static_cast<size_t>(p.positions[t]) * p.dims;
   const int half = p.dims / 2;
@@ -85,8 +110,6 @@ post_down_kernel(const PostDown p, const T* __restrict__ x, const T* __restrict_
 template <typename T>
 __global__ void rotate_heads_kernel(T* __restrict__ x, int ld, int heads, int head_stride, int dims, int interleaved,
                                     const int32_t* __restrict__ positions, const float* __restrict__ cos_sin, int T_rows) {
-  pdl_wait();
-  pdl_trigger();
   const int half = dims / 2;
   const long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= static_cast<long long>(T_rows) * heads * half) return;
@@ -117,8 +140,6 @@ __global__ void __launch_bounds__(kWarps * 32)
 attention_kernel(const Attn p, const T* __restrict__ q_lat, const T* __restrict__ q_rope, const T* __restrict__ cache,
                  T* __restrict__ out) {
   extern __shared__ float sm[];                 // query row [Rp + Dp] | warp outputs [kWarps][Rp] | m, l
-  pdl_wait();
-  pdl_trigger();
   const int head = blockIdx.x, t = blockIdx.y;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int LD = p.Rp + p.Dp;
@@ -199,7 +220,7 @@ static int launch_attn(const Attn& p, const void* ql, const void* qr, const void
   if (smem > 200 * 1024) return MB_ERR_TOO_LARGE;
   // the grid's y dimension ends at 65535 rows; steps are far smaller
   if (T_rows > 65535) return MB_ERR_TOO_LARGE;
-  return launch_k(kern, dim3(p.n_heads, T_rows), dim3(kWarps * 32), smem, stream, p, static_cast<const T*>(ql),
+  return launch_plain(kern, dim3(p.n_heads, T_rows), dim3(kWarps * 32), smem, stream, p, static_cast<const T*>(ql),
                   static_cast<const T*>(qr), static_cast<const T*>(cache), static_cast<T*>(out)) == cudaSuccess
              ? MB_OK : MB_ERR_LAUNCH;
 }
@@ -230,11 +251,11 @@ extern "C" int mb_latent_post_down(const void* x, int ld, int T, int q_rank, int
                         page_stride, eps, positions, cos_sin, slots};
   cudaError_t e;
   if (dtype == kF32)
-    e = launch_k(latent::post_down_kernel<float>, dim3(T), dim3(128), 0, stream, p, static_cast<const float*>(x),
+    e = launch_plain(latent::post_down_kernel<float>, dim3(T), dim3(256), 0, stream, p, static_cast<const float*>(x),
                  static_cast<const float*>(gamma_q), static_cast<const float*>(gamma_kv), static_cast<float*>(q_out),
                  static_cast<float*>(cache));
   else
-    e = launch_k(latent::post_down_kernel<__nv_bfloat16>, dim3(T), dim3(128), 0, stream, p,
+    e = launch_plain(latent::post_down_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, p,
                  static_cast<const __nv_bfloat16*>(x), static_cast<const __nv_bfloat16*>(gamma_q),
                  static_cast<const __nv_bfloat16*>(gamma_kv), static_cast<__nv_bfloat16*>(q_out),
                  static_cast<__nv_bfloat16*>(cache));
@@ -248,9 +269,9 @@ extern "C" int mb_rotate_heads(void* x, int ld, int T, int heads, int head_strid
   const long long work = static_cast<long long>(T) * heads * (dims / 2);
   const dim3 grid(static_cast<unsigned>((work + 255) / 256));
   cudaError_t e = dtype == kF32
-                      ? launch_k(latent::rotate_heads_kernel<float>, grid, dim3(256), 0, stream, static_cast<float*>(x), ld,
+                      ? launch_plain(latent::rotate_heads_kernel<float>, grid, dim3(256), 0, stream, static_cast<float*>(x), ld,
                                  heads, head_stride, dims, interleaved, positions, cos_sin, T)
-                      : launch_k(latent::rotate_heads_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream,
+                      : launch_plain(latent::rotate_heads_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream,
                                  static_cast<__nv_bfloat16*>(x), ld, heads, head_stride, dims, interleaved, positions,
                                  cos_sin, T);
   return e == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;

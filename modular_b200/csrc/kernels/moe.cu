@@ -22,7 +22,6 @@
 
 #include "../common/api.h"
 #include "../common/launch.h"
-#include "../common/ptx.cuh"
 
 namespace mb {
 
@@ -191,8 +190,6 @@ __global__ void __launch_bounds__(1024)
 moe_table_route_kernel(const int64_t* __restrict__ ids, int T, const int32_t* __restrict__ tables,
                        const int64_t* __restrict__ desc, int32_t* __restrict__ inverse, int32_t* __restrict__ offsets) {
   extern __shared__ int32_t cnt[];       // counts, then cursors
-  pdl_wait();
-  pdl_trigger();
   const int64_t* d = desc + static_cast<size_t>(blockIdx.x) * 6;
   const int32_t* tab = tables + d[0];
   const int top = static_cast<int>(d[1]), E = static_cast<int>(d[2]);
@@ -334,7 +331,7 @@ extern "C" int mb_moe_table_route(const int64_t* ids, int T, const int32_t* tabl
                                   int max_experts, int32_t* inverse, int32_t* offsets, cudaStream_t stream) {
   if (T <= 0 || n_layers <= 0) return MB_OK;
   if (max_experts <= 0 || max_experts > 8192) return MB_ERR_SHAPE;
-  return launch_k(moe_table_route_kernel, dim3(n_layers), dim3(1024), static_cast<size_t>(max_experts) * 4, stream, ids,
+  return launch_plain(moe_table_route_kernel, dim3(n_layers), dim3(1024), static_cast<size_t>(max_experts) * 4, stream, ids,
                   T, tables, desc, inverse, offsets) == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
 }
 

@@ -15,7 +15,6 @@
 
 #include "../common/api.h"
 #include "../common/launch.h"
-#include "../common/ptx.cuh"
 #include "../common/scalar.cuh"
 
 namespace mb {
@@ -52,11 +51,10 @@ struct Params {
 };
 
 template <typename T>
-__global__ void __launch_bounds__(256) residual_norm_kernel(const Params<T> p) {
+__global__ void __launch_bounds__(1024) residual_norm_kernel(const Params<T> p) {
   extern __shared__ float4 row_cache[];   // the updated row
-  __shared__ float part[8];
-  pdl_wait();
-  pdl_trigger();
+  __shared__ float part[32];
+  __shared__ int32_t pos_in[32], pos_out[32];
   const int out_row = blockIdx.x;
   const int row = p.rows ? p.rows[out_row] : out_row;
   float* xr = p.x + static_cast<size_t>(row) * p.ldx;
@@ -69,6 +67,11 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const Params<T> p) {
   }
   const int nvec = p.cols_pad >> 2;
   float ss = 0.f;
+  // the expert rows of this token, read once
+  const bool cached_in = p.e && p.top_k <= 32, cached_out = p.scatter && p.k2 <= 32;
+  if (cached_in && threadIdx.x < p.top_k) pos_in[threadIdx.x] = p.inverse[static_cast<size_t>(row) * p.top_k + threadIdx.x];
+  if (cached_out && threadIdx.x < p.k2) pos_out[threadIdx.x] = p.scatter[static_cast<size_t>(row) * p.k2 + threadIdx.x];
+  if (cached_in || cached_out) __syncthreads();
   for (int v = threadIdx.x; v < nvec; v += blockDim.x) {
     const int c = v * 4;
     float4 x;
@@ -80,8 +83,9 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const Params<T> p) {
     }
     float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
     if (p.e) {
+#pragma unroll 4
       for (int k = 0; k < p.top_k; ++k) {
-        const int pos = p.inverse[static_cast<size_t>(row) * p.top_k + k];
+        const int pos = cached_in ? pos_in[k] : p.inverse[static_cast<size_t>(row) * p.top_k + k];
         if (pos < 0) continue;
         const float4 y = ld4(p.e + static_cast<size_t>(pos) * p.lde + c);
         s.x = fmaf(p.pair_w, y.x, s.x); s.y = fmaf(p.pair_w, y.y, s.y);
@@ -118,7 +122,7 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const Params<T> p) {
       const float4 y = make_float4(x.x * u.x, x.y * u.y, x.z * u.z, x.w * u.w);
       if (p.scatter) {
         for (int k = 0; k < p.k2; ++k) {
-          const int pos = p.scatter[static_cast<size_t>(row) * p.k2 + k];
+          const int pos = cached_out ? pos_out[k] : p.scatter[static_cast<size_t>(row) * p.k2 + k];
           if (pos >= 0) st4(p.n2 + static_cast<size_t>(pos) * p.ld2 + c, y);
         }
       } else {
@@ -142,15 +146,15 @@ static int run(const MbResidualNorm& q, cudaStream_t stream) {
   p.scatter = q.scatter; p.k2 = q.k2;
   p.cols = q.cols; p.cols_pad = q.cols_pad; p.store_x = q.store_x; p.eps = q.eps;
   const int nvec = p.cols_pad / 4;
-  const int threads = nvec >= 256 ? 256 : (nvec + 31) / 32 * 32;
-  return launch_k(residual_norm_kernel<T>, dim3(q.n_rows), dim3(threads), static_cast<size_t>(p.cols_pad) * 4, stream, p) ==
+  // few rows: one pass per row with as many threads as it has vectors; many rows: small CTAs, several per SM
+  const int most = q.n_rows <= 296 ? 1024 : 256;
+  const int threads = nvec >= most ? most : (nvec + 31) / 32 * 32;
+  return launch_plain(residual_norm_kernel<T>, dim3(q.n_rows), dim3(threads), static_cast<size_t>(p.cols_pad) * 4, stream, p) ==
                  cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
 }
 
 template <typename T>
 __global__ void gelu_tanh_kernel(T* __restrict__ x, size_t n4) {
-  pdl_wait();
-  pdl_trigger();
   const size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= n4) return;
   const float4 v = ld4(x + i * 4);
@@ -161,8 +165,6 @@ __global__ void gelu_tanh_kernel(T* __restrict__ x, size_t n4) {
 // o[r, c] *= sigmoid(g[r, c])
 template <typename T>
 __global__ void sigmoid_gate_kernel(T* __restrict__ o, int ldo, const T* __restrict__ g, int ldg, int rows, int cols4) {
-  pdl_wait();
-  pdl_trigger();
   const size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= static_cast<size_t>(rows) * cols4) return;
   const int r = static_cast<int>(i / cols4), c = static_cast<int>(i % cols4) * 4;
@@ -191,8 +193,8 @@ extern "C" int mb_gelu_tanh(void* x, long long n, int dtype, cudaStream_t stream
   if (n % 4) return MB_ERR_SHAPE;
   const size_t n4 = static_cast<size_t>(n) / 4;
   const dim3 grid(static_cast<unsigned>((n4 + 255) / 256));
-  cudaError_t e = dtype == kF32 ? launch_k(gelu_tanh_kernel<float>, grid, dim3(256), 0, stream, static_cast<float*>(x), n4)
-                                : launch_k(gelu_tanh_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream,
+  cudaError_t e = dtype == kF32 ? launch_plain(gelu_tanh_kernel<float>, grid, dim3(256), 0, stream, static_cast<float*>(x), n4)
+                                : launch_plain(gelu_tanh_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream,
                                            static_cast<__nv_bfloat16*>(x), n4);
   return e == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
 }
@@ -205,9 +207,9 @@ extern "C" int mb_sigmoid_gate(void* o, int ldo, const void* g, int ldg, int row
   const dim3 grid(static_cast<unsigned>((static_cast<size_t>(rows) * c4 + 255) / 256));
   cudaError_t e =
       dtype == kF32
-          ? launch_k(sigmoid_gate_kernel<float>, grid, dim3(256), 0, stream, static_cast<float*>(o), ldo,
+          ? launch_plain(sigmoid_gate_kernel<float>, grid, dim3(256), 0, stream, static_cast<float*>(o), ldo,
                      static_cast<const float*>(g), ldg, rows, c4)
-          : launch_k(sigmoid_gate_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, static_cast<__nv_bfloat16*>(o), ldo,
+          : launch_plain(sigmoid_gate_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, static_cast<__nv_bfloat16*>(o), ldo,
                      static_cast<const __nv_bfloat16*>(g), ldg, rows, c4);
   return e == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
 }

@@ -279,8 +279,8 @@ class GotunexWeights:
 
     @classmethod
     def random_init(cls, cfg: GotunexConfig, device="cpu", dtype=torch.bfloat16, seed: int = 0) -> "GotunexWeights":
-        return cls.from_state_dict(cfg, cls.random_state_dict(cfg, seed, torch.bfloat16 if dtype == torch.bfloat16 else
-                                                              torch.float32), device, dtype)
+        """Random weights, generated on ``device``."""
+        return cls.from_state_dict(cfg, cls.random_state_dict(cfg, seed, dtype, device), device, dtype)
 
 
 class GotunexModel:
@@ -349,7 +349,7 @@ class GotunexModel:
     def _linear(self, T: int):
         """The GEMM for a step's size: decode-sized bf16 steps on the GPU stream their weights once over all SMs."""
         small = self.device.type == "cuda" and self.dtype == torch.bfloat16 and T <= ops.DECODE_GEMM_MAX_TOKENS
-        return ops.linear_decode if small else ops.linear
+        return ops.linear_small if small else ops.linear
 
     @torch.no_grad()
     def _forward(self, tokens, positions, slots, block_table, q_start, q_len, kv_len, logit_rows, state_slot=None,

@@ -81,7 +81,7 @@ def pad_heads(w: torch.Tensor, heads: int, rows: int, rows_pad: int) -> torch.Te
     K = w.shape[1]
     if rows == rows_pad:
         return w
-    out = torch.zeros(heads, rows_pad, K, dtype=w.dtype)
+    out = torch.zeros(heads, rows_pad, K, dtype=w.dtype, device=w.device)
     out[:, :rows] = w.view(heads, rows, K)
     return out.view(heads * rows_pad, K)
 
@@ -107,14 +107,15 @@ class LatentAttention:
         self.q_norm = put(t["dq.norm"])
         self.kv_norm = put(t["dkv.norm"]) if c.own_cache else None
         uq = t["uq"].view(H, d + r, c.q_rank)
-        q = torch.zeros(H, c.head_width, self.q_pad, dtype=uq.dtype)
+        new = lambda *s: torch.zeros(*s, dtype=uq.dtype, device=uq.device)
+        q = new(H, c.head_width, self.q_pad)
         q[:, :d, : c.q_rank] = uq[:, :d]
         q[:, up64(d): up64(d) + r, : c.q_rank] = uq[:, d:]
         self.w_uq = put(q.view(H * c.head_width, self.q_pad))
-        uk = torch.zeros(H, Rp, up64(d), dtype=uq.dtype)
+        uk = new(H, Rp, up64(d))
         uk[:, : c.kv_rank, :d] = t["uk"].view(H, d, c.kv_rank).transpose(1, 2)
         self.w_uk = put(uk)                                          # [h, latent, dim]: queries into latent space
-        uv = torch.zeros(H, vp, Rp, dtype=uq.dtype)
+        uv = new(H, vp, Rp)
         uv[:, : c.vdim, : c.kv_rank] = t["uv"].view(H, c.vdim, c.kv_rank)
         self.w_uv = put(uv)                                          # [h, vdim, latent]: latent outputs to values
         self.sink = put(t["sink"], torch.float32)
