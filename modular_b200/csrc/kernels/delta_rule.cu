@@ -6,14 +6,14 @@
 //   delta_prep_kernel   one warp per (token, piece): convolution + silu of q, k, v (inputs before the step come from the
 //                       sequence's convolution state), unit norms, decays g = exp(-exp(A_log) softplus(z + dt_bias)),
 //                       beta, k . q. Everything leaves in fp32.
-//   delta_scan_kernel   columns of S are independent, so a warp owns eight of them: eight lanes share the rows of a
-//                       column (each 4 * RL4 of them, in registers), four lane groups hold two columns each. A token
-//                       costs one pass of decay, two dot products reduced together over eight lanes with four
-//                       shuffles (o = (gS)^T q + u (k . q) needs no second reduction), and the rank-one update. Token rows
-//                       are staged through shared memory with cp.async. The state is read once and written once per
-//                       launch, [slot, head, column, row]; sequences of one token are a decode step, for which one CTA
-//                       owns a whole head and also applies the output norm and gate. The convolution state is advanced
-//                       at the end of this kernel, after every read of it by the first one.
+//   delta_scan_kernel   columns of S are independent, so a warp owns 8 or 16 of them: eight lanes share the rows of a
+//                       column (each 4 * RL4 of them, in registers), four lane groups hold two or four columns each. A
+//                       token costs one pass of decay, two dot products per column reduced together over eight lanes
+//                       (o = (gS)^T q + u (k . q) needs no second reduction), and the rank-one update. Token rows are
+//                       staged through shared memory with cp.async. The state is read once and written once per launch,
+//                       [slot, head, column, row]; sequences of one token are a decode step, for which one CTA owns a
+//                       whole head and also applies the output norm and gate. The convolution state is advanced at the
+//                       end of this kernel, after every read of it by the first one.
 //   delta_out_kernel    output norm and gate for longer sequences, one warp per (token, head)
 //
 // A chunked formulation on the tensor cores would round what enters the recurrence to 16 bits; this one keeps it in fp32.
@@ -61,6 +61,13 @@ __device__ __forceinline__ float sum4(uint64_t a, uint64_t b) {
   asm("add.rn.f32x2 %0, %1, %2;" : "=l"(c) : "l"(a), "l"(b));
   asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(c));
   return x + y;
+}
+
+// silu of a convolution output: fp32 runs take the accurate exponential, 16-bit runs the fast one
+template <typename T>
+__device__ __forceinline__ float conv_act(float z) {
+  if constexpr (sizeof(T) == 4) return siluf(z);
+  return __fdividef(z, 1.f + __expf(-z));
 }
 
 __device__ __forceinline__ float softplusf(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
@@ -161,6 +168,7 @@ struct ConvLane {
       win[j + 1] = v;
     }
   }
+  template <typename T>
   __device__ __forceinline__ float4 step(float4 x) {
 #pragma unroll
     for (int j = 0; j < W - 1; ++j) win[j] = win[j + 1];
@@ -171,7 +179,7 @@ struct ConvLane {
       a.x = fmaf(w[j][0], win[j].x, a.x); a.y = fmaf(w[j][1], win[j].y, a.y);
       a.z = fmaf(w[j][2], win[j].z, a.z); a.w = fmaf(w[j][3], win[j].w, a.w);
     }
-    return make_float4(siluf(a.x), siluf(a.y), siluf(a.z), siluf(a.w));
+    return make_float4(conv_act<T>(a.x), conv_act<T>(a.y), conv_act<T>(a.z), conv_act<T>(a.w));
   }
 };
 
@@ -207,6 +215,9 @@ __global__ void __launch_bounds__(256) delta_prep_fast_kernel(const MbDelta p, i
   float4 bias = make_float4(0.f, 0.f, 0.f, 0.f);
   if (is_g && on) bias = *reinterpret_cast<const float4*>(p.dt_bias + (unit - KH) * D + c);
   const float scale = 1.f / sqrtf(static_cast<float>(D));
+  float4 fut_a = make_float4(0.f, 0.f, 0.f, 0.f), fut_b = fut_a;
+  if (on && !is_g) fut_a = ld4(xq + static_cast<size_t>(tb) * p.ldx);
+  if (on && is_qk) fut_b = ld4(xk + static_cast<size_t>(tb) * p.ldx);
   int end = 0;                       // first token behind the current sequence
   for (int t = tb; t < te; ++t) {
     if (t >= end) {                  // a new sequence (or the first token of the tile)
@@ -224,9 +235,14 @@ __global__ void __launch_bounds__(256) delta_prep_fast_kernel(const MbDelta p, i
       }
     }
     const size_t row = static_cast<size_t>(t) * p.ldx;
+    const float4 nxt_a = fut_a, nxt_b = fut_b;
+    if (on && t + 1 < te) {          // the next token's inputs travel while this one is worked on
+      if (!is_g) fut_a = ld4(xq + row + p.ldx);
+      if (is_qk) fut_b = ld4(xk + row + p.ldx);
+    }
     if (is_qk) {
       float4 q = make_float4(0.f, 0.f, 0.f, 0.f), k = q;
-      if (on) { q = ca.step(ld4(xq + row)); k = cb.step(ld4(xk + row)); }
+      if (on) { q = ca.template step<T>(nxt_a); k = cb.template step<T>(nxt_b); }
       float qq = q.x * q.x + q.y * q.y + q.z * q.z + q.w * q.w, kk = k.x * k.x + k.y * k.y + k.z * k.z + k.w * k.w;
       float kq = q.x * k.x + q.y * k.y + q.z * k.z + q.w * k.w;
       qq = warp_allsum(qq); kk = warp_allsum(kk); kq = warp_allsum(kq);
@@ -248,12 +264,12 @@ __global__ void __launch_bounds__(256) delta_prep_fast_kernel(const MbDelta p, i
       if (c < DP) *reinterpret_cast<float4*>(p.g + (static_cast<size_t>(t) * H + h) * DP + c) = g;
       if (lane == 0) p.beta[static_cast<size_t>(t) * H + h] = sigmoidf(ldf(static_cast<const T*>(p.x) + row + p.b_off + h));
     } else if (on) {
-      *reinterpret_cast<float4*>(p.v + static_cast<size_t>(t) * vC + v0 + c) = ca.step(ld4(xq + row));
+      *reinterpret_cast<float4*>(p.v + static_cast<size_t>(t) * vC + v0 + c) = ca.template step<T>(nxt_a);
     }
   }
 }
 
-template <typename T, int RL4, int MAXT, bool FUSE>
+template <typename T, int RL4, int NC, int MAXT, bool FUSE>
 __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int col_blocks, int chunk) {
   constexpr int DP = 32 * RL4;
   extern __shared__ __align__(16) float sm[];
@@ -261,7 +277,7 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int rg = lane & 7, cg = lane >> 3;
   const int KH = p.kv_heads, H = p.heads, V = p.vdim;
-  const int h = blockIdx.x / col_blocks, cols = (blockDim.x >> 5) * 8, cbase = (blockIdx.x % col_blocks) * cols;
+  const int h = blockIdx.x / col_blocks, cols = (blockDim.x >> 5) * 4 * NC, cbase = (blockIdx.x % col_blocks) * cols;
   const int kh = h / (H / KH), s = blockIdx.y;
   const int t0 = p.q_start[s], n = p.q_len[s], slot = p.state_idx[s];
   const bool resume = slot >= 0 && p.kv_len[s] > n;
@@ -291,20 +307,22 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
       cp_async_commit();
     };
     fetch(0, sm);
-    const int col0 = cbase + warp * 8 + cg * 2;
-    const bool ok0 = col0 < V, ok1 = col0 + 1 < V;
+    const int col0 = cbase + (warp * 4 + cg) * NC;
     float* st = p.state + ((static_cast<size_t>(slot >= 0 ? slot : 0) * H + h) * V + col0) * DP;
-    u64x2 S0[RL4], S1[RL4];                        // four rows per entry, two packed fp32 pairs
+    u64x2 S[NC][RL4];                              // four rows per entry, two packed fp32 pairs
 #pragma unroll
-    for (int i = 0; i < RL4; ++i) {
-      const int r = (i * 8 + rg) * 4;
-      S0[i] = (resume && ok0) ? *reinterpret_cast<const u64x2*>(st + r) : u64x2{0ull, 0ull};
-      S1[i] = (resume && ok1) ? *reinterpret_cast<const u64x2*>(st + DP + r) : u64x2{0ull, 0ull};
-    }
-    const bool hi_col = (lane & 4) != 0, is_q = (lane & 2) != 0;
-    const int my_col = warp * 8 + cg * 2 + (hi_col ? 1 : 0);
+    for (int i = 0; i < RL4; ++i)
+#pragma unroll
+      for (int c = 0; c < NC; ++c)
+        S[c][i] = (resume && col0 + c < V) ? *reinterpret_cast<const u64x2*>(st + c * DP + (i * 8 + rg) * 4) : u64x2{0ull, 0ull};
+    // which reduced value this lane ends up with: column `mine` of its group, key product or query product
+    const bool b4 = (lane & 4) != 0, b2 = (lane & 2) != 0, b1 = (lane & 1) != 0;
+    const int mine = NC == 4 ? (b4 ? 2 : 0) + (b2 ? 1 : 0) : (b4 ? 1 : 0);
+    const bool is_q = NC == 4 ? b1 : b2;
+    const int my_col = (warp * 4 + cg) * NC + mine;
     float* optr = p.o + (static_cast<size_t>(t0) * H + h) * V + cbase + my_col;
-    const bool writes = (lane & 3) == 2 && cbase + my_col < V;
+    const bool holds_o = NC == 4 ? b1 : (lane & 3) == 2;
+    const bool writes = holds_o && cbase + my_col < V;
     for (int c0 = 0, it = 0; c0 < n; c0 += chunk, ++it) {
       const int m = min(chunk, n - c0);
       const float* buf = sm + (it & 1) * stage_floats;
@@ -315,7 +333,9 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
       for (int j = 0; j < m; ++j) {
         const float* rowp = buf + j * row_floats;
         u64x2 kr[RL4];
-        uint64_t a0 = 0ull, a1 = 0ull, b0 = 0ull, b1 = 0ull, a0h = 0ull, a1h = 0ull, b0h = 0ull, b1h = 0ull;
+        uint64_t a[NC][2], b[NC][2];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) a[c][0] = a[c][1] = b[c][0] = b[c][1] = 0ull;
 #pragma unroll
         for (int i = 0; i < RL4; ++i) {
           const int r = (i * 8 + rg) * 4;
@@ -323,32 +343,52 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
           const u64x2 k4 = *reinterpret_cast<const u64x2*>(rowp + DP + r);
           const u64x2 g4 = *reinterpret_cast<const u64x2*>(rowp + 2 * DP + r);
           kr[i] = k4;
-          S0[i].x = mul2(S0[i].x, g4.x); S0[i].y = mul2(S0[i].y, g4.y);
-          S1[i].x = mul2(S1[i].x, g4.x); S1[i].y = mul2(S1[i].y, g4.y);
-          a0 = fma2(S0[i].x, k4.x, a0); a0h = fma2(S0[i].y, k4.y, a0h);
-          a1 = fma2(S1[i].x, k4.x, a1); a1h = fma2(S1[i].y, k4.y, a1h);
-          b0 = fma2(S0[i].x, q4.x, b0); b0h = fma2(S0[i].y, q4.y, b0h);
-          b1 = fma2(S1[i].x, q4.x, b1); b1h = fma2(S1[i].y, q4.y, b1h);
+#pragma unroll
+          for (int c = 0; c < NC; ++c) {
+            S[c][i].x = mul2(S[c][i].x, g4.x); S[c][i].y = mul2(S[c][i].y, g4.y);
+            a[c][0] = fma2(S[c][i].x, k4.x, a[c][0]); a[c][1] = fma2(S[c][i].y, k4.y, a[c][1]);
+            b[c][0] = fma2(S[c][i].x, q4.x, b[c][0]); b[c][1] = fma2(S[c][i].y, q4.y, b[c][1]);
+          }
         }
-        const float A0 = sum4(a0, a0h), A1 = sum4(a1, a1h), B0 = sum4(b0, b0h), B1 = sum4(b1, b1h);
-        // eight partial sums of four values: lanes with bit 2 take column 1, lanes with bit 1 the q product
-        float a = (hi_col ? A1 : A0) + __shfl_xor_sync(0xffffffffu, hi_col ? A0 : A1, 4);
-        float b = (hi_col ? B1 : B0) + __shfl_xor_sync(0xffffffffu, hi_col ? B0 : B1, 4);
-        float r = (is_q ? b : a) + __shfl_xor_sync(0xffffffffu, is_q ? a : b, 2);
-        r += __shfl_xor_sync(0xffffffffu, r, 1);
+        float A[NC], Bq[NC];
+#pragma unroll
+        for (int c = 0; c < NC; ++c) { A[c] = sum4(a[c][0], a[c][1]); Bq[c] = sum4(b[c][0], b[c][1]); }
+        // partial sums over the eight row lanes: every exchange halves the values a lane still carries
+        float r;
+        if (NC == 4) {
+          float a2[2], q2[2];
+#pragma unroll
+          for (int c = 0; c < 2; ++c) {
+            a2[c] = (b4 ? A[NC / 2 + c] : A[c]) + __shfl_xor_sync(0xffffffffu, b4 ? A[c] : A[NC / 2 + c], 4);
+            q2[c] = (b4 ? Bq[NC / 2 + c] : Bq[c]) + __shfl_xor_sync(0xffffffffu, b4 ? Bq[c] : Bq[NC / 2 + c], 4);
+          }
+          const float a1 = (b2 ? a2[1] : a2[0]) + __shfl_xor_sync(0xffffffffu, b2 ? a2[0] : a2[1], 2);
+          const float q1 = (b2 ? q2[1] : q2[0]) + __shfl_xor_sync(0xffffffffu, b2 ? q2[0] : q2[1], 2);
+          r = (b1 ? q1 : a1) + __shfl_xor_sync(0xffffffffu, b1 ? a1 : q1, 1);
+        } else {
+          const float a1 = (b4 ? A[1] : A[0]) + __shfl_xor_sync(0xffffffffu, b4 ? A[0] : A[1], 4);
+          const float q1 = (b4 ? Bq[1] : Bq[0]) + __shfl_xor_sync(0xffffffffu, b4 ? Bq[0] : Bq[1], 4);
+          r = (b2 ? q1 : a1) + __shfl_xor_sync(0xffffffffu, b2 ? a1 : q1, 2);
+          r += __shfl_xor_sync(0xffffffffu, r, 1);
+        }
         const float beta = sc[2 * j], kq = sc[2 * j + 1];
         const float vv = rowp[3 * DP + my_col];
         const float u = beta * (vv - r);           // meaningful in the lanes that hold a key product
-        const float u0 = __shfl_sync(0xffffffffu, u, lane & 24), u1 = __shfl_sync(0xffffffffu, u, (lane & 24) | 4);
-        const uint64_t u0p = pack2(u0, u0), u1p = pack2(u1, u1);
+        float uc[NC], u_mine = 0.f;
 #pragma unroll
-        for (int i = 0; i < RL4; ++i) {
-          S0[i].x = fma2(kr[i].x, u0p, S0[i].x); S0[i].y = fma2(kr[i].y, u0p, S0[i].y);
-          S1[i].x = fma2(kr[i].x, u1p, S1[i].x); S1[i].y = fma2(kr[i].y, u1p, S1[i].y);
+        for (int c = 0; c < NC; ++c) {
+          uc[c] = __shfl_sync(0xffffffffu, u, (lane & 24) | (NC == 4 ? (c >> 1) * 4 + (c & 1) * 2 : c * 4));
+          u_mine = mine == c ? uc[c] : u_mine;
         }
-        const float o = fmaf(hi_col ? u1 : u0, kq, r);
+#pragma unroll
+        for (int c = 0; c < NC; ++c) {
+          const uint64_t up = pack2(uc[c], uc[c]);
+#pragma unroll
+          for (int i = 0; i < RL4; ++i) { S[c][i].x = fma2(kr[i].x, up, S[c][i].x); S[c][i].y = fma2(kr[i].y, up, S[c][i].y); }
+        }
+        const float o = fmaf(u_mine, kq, r);       // in the lanes that hold a query product
         if (FUSE) {
-          if ((lane & 3) == 2) so[my_col] = cbase + my_col < V ? o : 0.f;
+          if (holds_o) so[my_col] = cbase + my_col < V ? o : 0.f;
         } else {
           if (writes) *optr = o;
           optr += H * V;
@@ -375,11 +415,10 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
     }
     if (slot >= 0) {
 #pragma unroll
-      for (int i = 0; i < RL4; ++i) {
-        const int r = (i * 8 + rg) * 4;
-        if (ok0) *reinterpret_cast<u64x2*>(st + r) = S0[i];
-        if (ok1) *reinterpret_cast<u64x2*>(st + DP + r) = S1[i];
-      }
+      for (int i = 0; i < RL4; ++i)
+#pragma unroll
+        for (int c = 0; c < NC; ++c)
+          if (col0 + c < V) *reinterpret_cast<u64x2*>(st + c * DP + (i * 8 + rg) * 4) = S[c][i];
     }
   }
   // the last taps - 1 convolution inputs of the sequence; this CTA's share of the channels
@@ -418,41 +457,44 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const MbDelta p) {
   }
 }
 
+template <typename T, int RL4, int NC>
+static int scan_launch(const MbDelta& p, int warps, bool fuse, cudaStream_t stream) {
+  constexpr int MAXT = RL4 <= 8 ? 512 : 256;
+  const int cols = warps * 4 * NC, col_blocks = (p.vdim + cols - 1) / cols;
+  const int per_token = (3 * 32 * RL4 + cols + 2) * 4;
+  // tokens per stage: even, so that the second stage stays 16-byte aligned (a one-token step has no second stage)
+  int chunk = p.one_token ? 1 : 40 * 1024 / (2 * per_token);
+  if (!p.one_token) chunk = chunk > 16 ? 16 : chunk < 2 ? 2 : chunk & ~1;
+  const size_t smem = static_cast<size_t>(2) * chunk * per_token + (fuse ? cols * 4 : 0) + 16;
+  const dim3 grid(p.heads * col_blocks, p.B);
+  if (fuse)
+    return launch_plain(delta_scan_kernel<T, RL4, NC, MAXT, true>, grid, dim3(warps * 32), smem, stream, p, col_blocks, chunk) ==
+                   cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
+  if (launch_plain(delta_scan_kernel<T, RL4, NC, MAXT, false>, grid, dim3(warps * 32), smem, stream, p, col_blocks, chunk) !=
+      cudaSuccess)
+    return MB_ERR_LAUNCH;
+  const long long units = static_cast<long long>(p.T) * p.heads;
+  return launch_plain(delta_out_kernel<T>, dim3(static_cast<unsigned>((units + 7) / 8)), dim3(256), 0, stream, p) == cudaSuccess
+             ? MB_OK : MB_ERR_LAUNCH;
+}
+
 template <typename T, int RL4>
 static int scan(const MbDelta& p, int num_sms, cudaStream_t stream) {
-  constexpr int MAXT = RL4 <= 8 ? 512 : 256;
+  constexpr int max_warps = (RL4 <= 8 ? 512 : 256) / 32;
   const int head_warps = (p.vdim + 7) / 8;
-  const bool fuse = p.one_token && head_warps * 32 <= MAXT;
-  int warps;
-  if (fuse) {
-    warps = head_warps;
-  } else {                         // fewer columns per CTA until the step fills the machine
-    warps = MAXT / 32 < 4 ? MAXT / 32 : 4;
-    while (warps > 1 && static_cast<long long>(p.B) * p.heads * ((head_warps + warps - 1) / warps) < num_sms) warps >>= 1;
-    if (warps > head_warps) warps = head_warps;
+  if (p.one_token && head_warps <= max_warps) return scan_launch<T, RL4, 2>(p, head_warps, true, stream);
+  // longer sequences: four columns per lane where the registers allow it (the rows are read once for all of them), and
+  // CTAs of up to four warps as long as the grid has one per SM
+  auto fit = [&](int per_warp) {
+    const int hw = (p.vdim + per_warp - 1) / per_warp;
+    int w = hw < 4 ? hw : 4;
+    while (w > 1 && static_cast<long long>(p.B) * p.heads * ((hw + w - 1) / w) < num_sms) w >>= 1;
+    return w;
+  };
+  if constexpr (RL4 <= 4) {
+    if (p.vdim >= 16) return scan_launch<T, RL4, 4>(p, fit(16), false, stream);
   }
-  const int col_blocks = (head_warps + warps - 1) / warps;
-  const int per_token = (3 * 32 * RL4 + warps * 8 + 2) * 4;
-  int chunk = p.one_token ? 1 : 40 * 1024 / (2 * per_token);
-  if (chunk > 16) chunk = 16;
-  if (chunk >= 4) chunk &= ~3;      // whole float4 rows keep the second stage 16-byte aligned
-  else if (chunk > 1) chunk = 2;
-  if (chunk < 1) chunk = 1;
-  // the second stage starts chunk * per_token bytes in: 16-byte aligned when chunk * 2 floats are a multiple of 4
-  if (chunk == 1 && !p.one_token) chunk = 2;
-  const size_t smem = static_cast<size_t>(2) * chunk * per_token + (fuse ? warps * 8 * 4 : 0) + 16;
-  const dim3 grid(p.heads * col_blocks, p.B);
-  cudaError_t e;
-  if (fuse) {
-    e = launch_plain(delta_scan_kernel<T, RL4, MAXT, true>, grid, dim3(warps * 32), smem, stream, p, col_blocks, chunk);
-  } else {
-    e = launch_plain(delta_scan_kernel<T, RL4, MAXT, false>, grid, dim3(warps * 32), smem, stream, p, col_blocks, chunk);
-    if (e == cudaSuccess) {
-      const long long units = static_cast<long long>(p.T) * p.heads;
-      e = launch_plain(delta_out_kernel<T>, dim3(static_cast<unsigned>((units + 7) / 8)), dim3(256), 0, stream, p);
-    }
-  }
-  return e == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
+  return scan_launch<T, RL4, 2>(p, fit(8), false, stream);
 }
 
 template <typename T>
