@@ -262,6 +262,6 @@ def run_kernels(s: dict, name: str, prefill: int = 2048, seqs: int = 4, batch: i
     return rows
 
 
-def main(sizes=("w2048", "w4096", "w7168")) -> dict:
-    return {"peaks": measured_peaks(), "fp32_tflops_nominal": FP32_TFLOPS, "models": list(run_models(sizes)),
+def main(sizes=("w2048", "w4096", "w7168"), steps: int = 20) -> dict:
+    return {"peaks": measured_peaks(), "fp32_tflops_nominal": FP32_TFLOPS, "models": list(run_models(sizes, steps=steps)),
             "kernels": [r for n in sizes for r in run_kernels(SIZES[n], n)]}
