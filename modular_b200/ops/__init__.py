@@ -134,21 +134,6 @@ def linear_decode(x, w, mode="plain", out=None, h=None, gamma=None, eps=1e-5, we
     return out
 
 
-_DEC_FITS: dict = {}
-
-
-def linear_small(x, w):
-    """``x @ w.T`` for a decode-sized step: the decode-step GEMM where it takes the shape, else the tiled one."""
-    if not x.is_cuda or x.dtype != torch.bfloat16:
-        return linear(x, w)
-    key = (x.shape[0], w.shape[0], w.shape[1])
-    ok = _DEC_FITS.get(key)
-    if ok is None:
-        ws, _ = decode_gemm_workspace(x.device)
-        ok = _DEC_FITS[key] = _lib().gemm_dec_plan(*key, 0, ws.nbytes) == 0
-    return linear_decode(x, w) if ok else linear(x, w)
-
-
 HEADS_ON_DECODE_GEMM = False
 
 

@@ -369,6 +369,19 @@ def test_gelu_and_rotation(device, dtype):
     assert rel(y, oracle.rotate(h.double().view(3, 4, 40), 24, 300.0, 5000).view(3, -1)) < TOL[dtype]
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("N,K", [(64, 64), (8192, 64), (896, 64), (1280, 72), (2048, 160), (256, 2048), (1408, 64)])
+def test_decode_sized_projection(N, K):
+    """Projections of few tokens, among them many rows over a single 64-wide block of the inner width."""
+    from modular_b200 import ops
+
+    g = torch.Generator().manual_seed(N + K)
+    w = torch.randn(N, K, generator=g).bfloat16()
+    for M in (1, 5, 64, 256):
+        x = torch.randn(M, K, generator=g).bfloat16()
+        assert rel(ops.linear(x.cuda(), w.cuda()), x.double() @ w.double().t()) < 1e-2
+
+
 # ---------------------------------------------------------------------------------- whole models
 def replay(llm, reqs, steps):
     """Runs ``steps`` (lists of (request, tokens)) and returns every request's logits [T, vocab]; all places are wanted. A
@@ -446,7 +459,9 @@ def test_schedules(mixed_model, name, device, dtype):
     config((latent(), None)), config((delta(), None)), config((delta(1, 1, 16, 8, 1), dense(8)), width=40, vocab=33),
     config((latent(heads=1, dim=4, rot_dim=2, vdim=4, kv_rank=8, q_rank=4), moe(2, 1, 8)), width=70, vocab=65),
     config((latent(heads=9, dim=64, rot_dim=64, vdim=128, kv_rank=256, q_rank=320), moe(9, 4, 200)), (delta(5, 5, 96, 64, 3), moe(3, 3, 48)),
-           width=264, vocab=258, eps=1e-3, scale=0.5)], ids=["latent only", "delta only", "tiny delta", "tiny latent", "wide"])
+           width=264, vocab=258, eps=1e-3, scale=0.5),
+    config((latent(heads=7, dim=56, rot_dim=40, q_rank=24), dense(72)), (delta(8, 2, 112, 48, 5), moe(6, 1, 56)), width=152, vocab=98)],
+    ids=["latent only", "delta only", "tiny delta", "tiny latent", "wide", "small query latent"])
 def test_other_sizes(cfg, device, dtype):
     t = weights_for(cfg, seed=11)
     toks = torch.randint(0, cfg["vocab"], (90,), generator=torch.Generator().manual_seed(1)).tolist()
