@@ -33,8 +33,11 @@ const float* f32(const Tensor& t, int64_t n, const char* what) {
 
 void residual_norm(Tensor& x, const Opt& ids, const Opt& table, double scale, const Opt& a, const Opt& b, const Opt& e,
                    const Opt& inverse, int top_k, double pair_w, const Opt& rows, const Opt& w1, const Opt& n1,
-                   const Opt& w2, const Opt& n2, const Opt& scatter, int cols, bool store_x, double eps, int n_rows) {
+                   const Opt& w2, const Opt& n2, const Opt& scatter, int cols, bool store_x, double eps, int n_rows,
+                   const Opt& norm_a, const Opt& norm_b, double ab_scale, const Opt& c, double mult, const Opt& inject,
+                   double inject_scale, const Opt& step) {
   MbResidualNorm p = {};
+  p.ab_scale = static_cast<float>(ab_scale); p.mult = static_cast<float>(mult);
   p.ldx = ld_of(x, at::kFloat, "x");
   p.x = x.data_ptr<float>();
   p.cols = cols; p.cols_pad = static_cast<int>(x.size(1)); p.store_x = store_x; p.eps = static_cast<float>(eps);
@@ -55,6 +58,21 @@ void residual_norm(Tensor& x, const Opt& ids, const Opt& table, double scale, co
   };
   if (given(a)) { p.lda = branch(a, "a", T); p.a = a->data_ptr(); }
   if (given(b)) { p.ldb = branch(b, "b", T); p.b = b->data_ptr(); }
+  auto weight = [&](const Opt& t, const char* what) {
+    TORCH_CHECK(t->is_cuda() && t->is_contiguous() && t->scalar_type() == dt && t->numel() >= p.cols_pad, "residual_norm: ", what);
+    return t->data_ptr();
+  };
+  if (given(norm_a)) { TORCH_CHECK(given(a), "residual_norm: norm_a without a"); p.norm_a = weight(norm_a, "norm_a"); }
+  if (given(norm_b)) { TORCH_CHECK(given(b), "residual_norm: norm_b without b"); p.norm_b = weight(norm_b, "norm_b"); }
+  if (given(c)) { p.ldc = branch(c, "c", T); p.c = c->data_ptr(); }
+  if (given(step)) p.step = weight(step, "step");
+  if (given(inject)) {
+    TORCH_CHECK(given(ids) && ids->scalar_type() == at::kLong && ids->numel() >= T, "residual_norm: ids");
+    p.ld_inject = ld_of(*inject, dt, "inject");
+    TORCH_CHECK(inject->size(1) == p.cols_pad && (!given(table) || table->size(0) == inject->size(0)), "residual_norm: inject shape");
+    p.inject = inject->data_ptr(); p.inject_scale = static_cast<float>(inject_scale);
+    p.ids = ids->data_ptr<int64_t>(); p.vocab = static_cast<int>(inject->size(0));
+  }
   if (given(e)) {
     p.lde = branch(e, "e", T * top_k); p.e = e->data_ptr();
     TORCH_CHECK(given(inverse), "residual_norm: inverse");
@@ -207,6 +225,98 @@ void delta_rule(const Tensor& x, int q_off, int k_off, int v_off, int b_off, con
   check_rc(mb_delta_rule(&p, dt, num_sms(), cur_stream()), "delta_rule");
 }
 
+// the cache [pages, 2, planes, kv heads, page, head width] at one plane
+struct CacheView {
+  char *k, *v;
+  long long page_stride, head_stride;
+  int page, hd;
+  CacheView(const Tensor& kv, int plane, int n_kv, const char* what) {
+    TORCH_CHECK(kv.is_cuda() && kv.dim() == 6 && kv.is_contiguous() && kv.size(1) == 2 && plane >= 0 && plane < kv.size(2) &&
+                    n_kv <= kv.size(3), what, ": cache [pages, 2, planes, kv heads, page, head width]");
+    k = static_cast<char*>(kv.data_ptr()) + plane * kv.stride(2) * kv.element_size();
+    v = k + kv.stride(1) * kv.element_size();
+    page_stride = kv.stride(0); head_stride = kv.stride(3); page = kv.size(4); hd = kv.size(5);
+  }
+};
+
+// x: projection rows; queries at column 0 .., see MbBlockPrep
+void block_prep(Tensor& x, int q_off, int heads, int k_off, int v_off, int kv_heads, int dims, const Tensor& positions,
+                const Opt& cos_sin, const Tensor& slots, Tensor& kv, int plane, int silu_off, int silu_n, int relu2_off, int relu2_n) {
+  MbBlockPrep p = {};
+  p.x = x.data_ptr(); p.ldx = ld_of(x, x.scalar_type(), "x"); p.T = x.size(0);
+  const CacheView c(kv, plane, kv_heads, "block_prep");
+  TORCH_CHECK(kv.scalar_type() == x.scalar_type(), "block_prep: cache dtype");
+  p.q_off = q_off; p.heads = heads; p.k_off = k_off; p.v_off = v_off; p.kv_heads = kv_heads; p.hd = c.hd; p.dims = dims;
+  const int64_t W = x.size(1);
+  TORCH_CHECK(q_off + static_cast<int64_t>(heads) * c.hd <= W && k_off + static_cast<int64_t>(kv_heads) * c.hd <= W &&
+                  v_off + static_cast<int64_t>(kv_heads) * c.hd <= W && silu_off + silu_n <= W && relu2_off + relu2_n <= W,
+              "block_prep: columns out of range");
+  if (dims > 0) {
+    TORCH_CHECK(given(cos_sin) && cos_sin->dim() == 2 && cos_sin->size(1) == dims, "block_prep: cos_sin");
+    p.cos_sin = f32(*cos_sin, 0, "cos_sin");
+  }
+  TORCH_CHECK(slots.is_cuda() && slots.scalar_type() == at::kLong && slots.numel() >= p.T, "block_prep: slots");
+  p.positions = i32(positions, p.T, "positions"); p.slots = slots.data_ptr<int64_t>();
+  p.k_cache = c.k; p.v_cache = c.v; p.page_size = c.page; p.page_stride = c.page_stride; p.head_stride = c.head_stride;
+  p.silu_off = silu_off; p.silu_n = silu_n; p.relu2_off = relu2_off; p.relu2_n = relu2_n;
+  check_rc(mb_block_prep(&p, dtype_of(x, "x"), cur_stream()), "block_prep");
+}
+
+// q [T, n_q * head width] (row stride free). Tensor cores: `decode_seq` (one row per sequence) or `tile_seq` / `tile_q0`;
+// none of them given: the kernel on the CUDA cores.
+void window_attention(const Tensor& q, Tensor& out, const Tensor& kv, int plane, const Tensor& block_table, const Tensor& q_start,
+                      const Tensor& q_len, const Tensor& kv_len, const Opt& tile_seq, const Opt& tile_q0, const Opt& decode_seq,
+                      int n_q, int n_kv, double scale, int window, const Opt& sink) {
+  const CacheView c(kv, plane, n_kv, "window_attention");
+  const int dt = dtype_of(q, "q"), ldq = ld_of(q, q.scalar_type(), "q"), ldo = ld_of(out, q.scalar_type(), "out");
+  const int B = q_len.numel(), T = q.size(0);
+  TORCH_CHECK(kv.scalar_type() == q.scalar_type() && q.size(1) >= static_cast<int64_t>(n_q) * c.hd && out.size(0) >= T &&
+                  out.size(1) >= static_cast<int64_t>(n_q) * c.hd && block_table.scalar_type() == at::kInt &&
+                  block_table.dim() == 2 && block_table.stride(1) == 1 && block_table.size(0) >= B, "window_attention layout");
+  const float* sk = given(sink) ? f32(*sink, n_q, "sink") : nullptr;
+  const int32_t *qs = i32(q_start, B, "q_start"), *ql = i32(q_len, B, "q_len"), *kl = i32(kv_len, B, "kv_len");
+  const int32_t* bt = block_table.data_ptr<int32_t>();
+  const int bts = block_table.stride(0);
+  if (!given(tile_seq) && !given(decode_seq)) {
+    check_rc(mb_window_attention(q.data_ptr(), ldq, out.data_ptr(), ldo, c.k, c.v, c.page_stride, c.head_stride, c.page, bt, bts, qs,
+                                 ql, kl, T, B, n_q, n_kv, c.hd, static_cast<float>(scale), window, sk, dt, cur_stream()),
+             "window_attention");
+    return;
+  }
+  TORCH_CHECK(dt == 0, "window_attention: the tensor-core kernels take bf16");
+  const int n_tiles = given(tile_seq) ? tile_seq->numel() : 0, n_dec = given(decode_seq) ? decode_seq->numel() : 0;
+  const long long hd = c.hd, rows_k = plane * kv.stride(2) / hd;
+  check_rc(mb_paged_attention_window(q.data_ptr(), ldq, out.data_ptr(), ldo, kv.data_ptr(), kv.numel() / hd, rows_k,
+                                     rows_k + kv.stride(1) / hd, kv.stride(0) / hd, bt, bts, qs, ql, kl,
+                                     n_tiles ? i32(*tile_seq, n_tiles, "tile_seq") : nullptr,
+                                     n_tiles ? i32(*tile_q0, n_tiles, "tile_q0") : nullptr, n_tiles, n_dec,
+                                     n_dec ? i32(*decode_seq, n_dec, "decode_seq") : nullptr, n_q, n_kv, c.hd, c.page,
+                                     static_cast<float>(scale), window, sk, error_flag(), cur_stream()),
+           "paged_attention_window");
+}
+
+// x: activated projection rows with the column blocks of q, k and v at the given offsets
+void lightning(const Tensor& x, int q_off, int k_off, int v_off, const Tensor& decay, const Tensor& decay_pow, Tensor& o,
+               Tensor& state, const Tensor& state_idx, const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, int heads,
+               int dim, int vdim, bool one_token) {
+  MbLightning p = {};
+  p.T = x.size(0); p.B = q_len.numel(); p.heads = heads; p.dim = dim; p.vdim = vdim; p.one_token = one_token;
+  p.dim_pad = mb_delta_dim_pad(dim);
+  TORCH_CHECK(p.dim_pad > 0, "lightning: key width ", dim, " is beyond the supported maximum");
+  p.x = x.data_ptr(); p.ldx = ld_of(x, x.scalar_type(), "x"); p.q_off = q_off; p.k_off = k_off; p.v_off = v_off;
+  TORCH_CHECK(q_off + heads * dim <= x.size(1) && k_off + heads * dim <= x.size(1) && v_off + heads * vdim <= x.size(1),
+              "lightning: columns");
+  p.decay = f32(decay, heads, "decay"); p.decay_pow = f32(decay_pow, 65ll * heads, "decay_pow");
+  p.o = o.data_ptr(); p.ldo = ld_of(o, x.scalar_type(), "o");
+  TORCH_CHECK(o.size(0) >= p.T && o.size(1) >= heads * vdim, "lightning: o");
+  TORCH_CHECK(state.is_contiguous() && state.scalar_type() == at::kFloat && state.dim() == 4 && state.size(1) == heads &&
+                  state.size(2) == vdim && state.size(3) == p.dim_pad, "lightning: state [slots, heads, vdim, dim_pad]");
+  p.state = state.data_ptr<float>();
+  p.state_idx = i32(state_idx, p.B, "state_idx"); p.q_start = i32(q_start, p.B, "q_start");
+  p.q_len = i32(q_len, p.B, "q_len"); p.kv_len = i32(kv_len, p.B, "kv_len");
+  check_rc(mb_lightning(&p, dtype_of(x, "x"), num_sms(), cur_stream()), "lightning");
+}
+
 }  // namespace
 
 void mb::bind_layers(py::module_& m) {
@@ -215,7 +325,12 @@ void mb::bind_layers(py::module_& m) {
         py::arg("a") = none, py::arg("b") = none, py::arg("e") = none, py::arg("inverse") = none, py::arg("top_k") = 0,
         py::arg("pair_w") = 1.0, py::arg("rows") = none, py::arg("w1") = none, py::arg("n1") = none, py::arg("w2") = none,
         py::arg("n2") = none, py::arg("scatter") = none, py::arg("cols") = 0, py::arg("store_x") = true, py::arg("eps") = 1e-6,
-        py::arg("n_rows") = 0);
+        py::arg("n_rows") = 0, py::arg("norm_a") = none, py::arg("norm_b") = none, py::arg("ab_scale") = 1.0, py::arg("c") = none,
+        py::arg("mult") = 1.0, py::arg("inject") = none, py::arg("inject_scale") = 1.0, py::arg("step") = none);
+  m.def("softcap", [](Tensor& x, double cap) {
+    TORCH_CHECK(x.is_cuda() && x.is_contiguous() && x.scalar_type() == at::kFloat, "softcap: contiguous fp32 CUDA tensor");
+    check_rc(mb_softcap(x.data_ptr<float>(), x.numel(), static_cast<float>(cap), cur_stream()), "softcap");
+  });
   m.def("gelu_tanh", [](Tensor& x) {
     TORCH_CHECK(x.is_cuda() && x.is_contiguous(), "gelu_tanh: contiguous CUDA tensor");
     check_rc(mb_gelu_tanh(x.data_ptr(), x.numel(), dtype_of(x, "x"), cur_stream()), "gelu_tanh");
@@ -238,6 +353,22 @@ void mb::bind_layers(py::module_& m) {
   m.def("latent_attention", &latent_attention, py::arg("q_lat"), py::arg("q_rope"), py::arg("cache"), py::arg("block_table"),
         py::arg("q_start"), py::arg("q_len"), py::arg("kv_len"), py::arg("out"), py::arg("scale"), py::arg("sink") = none,
         py::arg("one_token") = false, py::arg("ws") = none, py::arg("allow_tc") = true);
+  m.def("block_prep", &block_prep);
+  m.def("window_attention", &window_attention);
+  m.def("attention_plan", [](const Tensor& q_len, int tok_per_tile, Tensor& tile_seq, Tensor& tile_q0) {
+    const int n = tile_seq.numel();
+    check_rc(mb_attention_plan(i32(q_len, 1, "q_len"), q_len.numel(), tok_per_tile, n,
+                               const_cast<int32_t*>(i32(tile_seq, n, "tile_seq")), const_cast<int32_t*>(i32(tile_q0, n, "tile_q0")),
+                               cur_stream()), "attention_plan");
+  });
+  m.def("lightning", &lightning);
+  m.def("lightning_norm", [](Tensor& o, const Tensor& gate, const Tensor& w, int cols, int n, double eps) {
+    const int ldo = ld_of(o, o.scalar_type(), "o"), ldg = ld_of(gate, o.scalar_type(), "gate");
+    TORCH_CHECK(o.size(1) >= cols && gate.size(1) >= cols && gate.size(0) >= o.size(0) && w.is_contiguous() && w.numel() >= cols &&
+                    w.scalar_type() == o.scalar_type(), "lightning_norm shapes");
+    check_rc(mb_lightning_norm(o.data_ptr(), ldo, gate.data_ptr(), ldg, w.data_ptr(), o.size(0), cols, n, static_cast<float>(eps),
+                               dtype_of(o, "o"), cur_stream()), "lightning_norm");
+  });
   m.def("delta_dim_pad", [](int dim) { return mb_delta_dim_pad(dim); });
   m.def("delta_rule", &delta_rule);
   m.def("moe_table_route", [](const Tensor& ids, const Tensor& tables, const Tensor& desc, int max_experts, Tensor& inverse,

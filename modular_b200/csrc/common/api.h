@@ -168,6 +168,14 @@ int mb_paged_attention_tma(const void* q, int ldq, void* out, int ldo, const voi
                            const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, int n_decode,
                            const int32_t* decode_seq, int n_q, int n_kv, int head_dim, int page_size,
                            float scale, int* err, cudaStream_t stream);
+// ... with a sliding window and a sink score per query head; prompt tiles (128 / G tokens for head_dim 128, 64 / G for
+// 64) or one-token rows
+int mb_paged_attention_window(const void* q, int ldq, void* out, int ldo, const void* kv_base, long long total_rows,
+                              long long k_off_rows, long long v_off_rows, long long page_rows, const int32_t* block_table,
+                              int bt_stride, const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
+                              const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, int n_decode,
+                              const int32_t* decode_seq, int n_q, int n_kv, int head_dim, int page_size, float scale,
+                              int window, const float* sink, int* err, cudaStream_t stream);
 
 // Split-KV decode (attention_tma.cu): decode-only steps cut the KV tiles of all sequences into equal shares per
 // CTA once this process-wide workspace is set (partials + zeroed counters, one per KV head and sequence).
@@ -181,8 +189,8 @@ int mb_paged_attention_prefill_tc(const void* q, int ldq, void* out, int ldo, co
                                   long long page_rows, const int32_t* block_table, int bt_stride,
                                   const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
                                   const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, int n_q,
-                                  int n_kv, int head_dim, int page_size, float scale, int* err,
-                                  cudaStream_t stream);
+                                  int n_kv, int head_dim, int page_size, float scale, int window,
+                                  const float* sink, int* err, cudaStream_t stream);
 // Route the prefill tiles of mb_paged_attention_tma through the tcgen05 kernel when a step has at least
 // `min_tiles` 64-row tiles (process-wide; 0 = never).
 void mb_set_attn_tc(int min_tiles);
@@ -234,9 +242,16 @@ typedef struct {
   const void* w2; void* n2; int ld2; const int32_t* scatter; int k2;     // normalised rows * w2, optionally scattered
   int n_rows, cols, cols_pad, store_x;
   float eps;
+  // branches with an output norm (norm_a / norm_b given): x += mult * (ab_scale * (rms(a) norm_a + rms(b) norm_b) + c)
+  const void *norm_a, *norm_b; float ab_scale;
+  const void* c; int ldc; float mult;
+  const void* inject; int ld_inject; float inject_scale;                 // x += inject_scale * inject[ids] (vocab rows)
+  const void* step;                                                      // x += step, one row for every token
 } MbResidualNorm;
 int mb_residual_norm(const MbResidualNorm* p, int dtype, cudaStream_t stream);
 int mb_gelu_tanh(void* x, long long n, int dtype, cudaStream_t stream);
+// x[i] = cap * tanh(x[i] / cap) over fp32 logits
+int mb_softcap(float* x, long long n, float cap, cudaStream_t stream);
 int mb_sigmoid_gate(void* o, int ldo, const void* g, int ldg, int rows, int cols, int dtype, cudaStream_t stream);
 
 // ---- gated delta rule with per-channel decay (delta_rule.cu) ---------------------------------
@@ -256,6 +271,37 @@ typedef struct {
 } MbDelta;
 int mb_delta_dim_pad(int dim);
 int mb_delta_rule(const MbDelta* p, int dtype, int num_sms, cudaStream_t stream);
+
+// ---- sliding-window attention of any size, and what surrounds it (attention_window.cu) -------
+typedef struct {
+  void* x; int ldx, T;                                   // projection rows [T, ldx]; offsets and widths are multiples of 8
+  int q_off, heads, k_off, v_off, kv_heads, hd, dims;    // heads of hd columns, the first dims rotate (neighbours in pairs)
+  const int32_t* positions; const float* cos_sin;        // [positions, dims]: dims / 2 cosines, then as many sines
+  const int64_t* slots;                                  // cache slot per token (negative: not stored)
+  void *k_cache, *v_cache; int page_size; long long page_stride, head_stride;
+  int silu_off, silu_n, relu2_off, relu2_n;              // columns that become silu(x), relu(x)^2 (0: none)
+} MbBlockPrep;
+int mb_block_prep(const MbBlockPrep* p, int dtype, cudaStream_t stream);
+int mb_attention_plan(const int32_t* q_len, int B, int tok_per_tile, int n_tiles, int32_t* tile_seq, int32_t* tile_q0,
+                      cudaStream_t stream);
+int mb_window_attention(const void* q, int ldq, void* out, int ldo, const void* k_cache, const void* v_cache,
+                        long long page_stride, long long head_stride, int page_size, const int32_t* block_table, int bt_stride,
+                        const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len, int T, int B, int n_q, int n_kv,
+                        int hd, float scale, int window, const float* sink, int dtype, cudaStream_t stream);
+
+// ---- lightning attention: a constant decay per head (lightning.cu) ---------------------------
+typedef struct {
+  const void* x; int ldx, q_off, k_off, v_off;           // activated projection rows; heads of dim / vdim columns
+  const float* decay;                                    // [heads]
+  const float* decay_pow;                                // [heads, 65]: decay^0 .. decay^64 (tensor-core path)
+  void* o; int ldo;                                      // [T, heads * vdim]
+  float* state;                                          // [slots, heads, vdim, dim_pad]
+  const int32_t *state_idx, *q_start, *q_len, *kv_len;
+  int T, B, heads, dim, dim_pad, vdim, one_token;
+} MbLightning;
+int mb_lightning(const MbLightning* p, int dtype, int num_sms, cudaStream_t stream);
+int mb_lightning_norm(void* o, int ldo, const void* gate, int ldg, const void* w, int T, int cols, int n, float eps, int dtype,
+                      cudaStream_t stream);
 
 // ---- fp32 products (gemm_simt.cu) ------------------------------------------------------------
 int mb_gemm_f32(const float* x, const float* w, float* y, const float* r, int M, int N, int K, int ldx, int ldw, int ldy,

@@ -20,6 +20,9 @@
 //               normalisation, because P is always computed against that reference), so the common
 //               tile costs no read-modify-write of the accumulator
 //
+// A sliding window of W keys (itself and the W - 1 before it) starts the walk at the first tile any row of the CTA
+// sees and masks the edge; a sink score per head only adds exp(sink) to the denominator.
+//
 // All mbarrier waits are bounded; a timed-out wait raises the error word, and the CTA drains,
 // frees its TMEM and leaves. Decode rows (one token per sequence) stay on the mma.sync kernel of
 // attention_tma.cu: with one token only G of the 128 MMA rows would be used.
@@ -61,6 +64,8 @@ struct Params {
   long long k_off_rows, v_off_rows, page_rows;
   int ldq, ldo, bt_stride, page_size, n_tiles, G;
   float scale_log2;
+  int window;            // keys a query sees (0x7fffffff: all before it)
+  const float* sink;     // per query head, or null
 };
 
 struct Bars {
@@ -113,6 +118,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
   pdl_wait();
   pdl_trigger();
   const int seq = p.tile_seq[blockIdx.x];
+  if (seq < 0) return;                 // an unused tile of a plan made on the device
   const int tq0 = p.tile_q0[blockIdx.x];
   if (tq0 % tok_per_cta != 0) return;  // the plan lists 64-row tiles; every second one is covered by its predecessor
   const int qs = p.q_start[seq], ql = p.q_len[seq], kl = p.kv_len[seq];
@@ -120,7 +126,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
   int last_tq = tq0 + tok_per_cta;
   if (last_tq > ql) last_tq = ql;
   const int kv_hi = kl - ql + last_tq;
-  const int ntiles = (kv_hi + 63) / 64;
+  const int kv_lo = kl - ql + tq0 - p.window + 1;        // first key the CTA's first row sees
+  const int t_first = kv_lo > 0 ? kv_lo / 64 : 0;
+  const int ntiles = (kv_hi + 63) / 64 - t_first;
 
   if (tid == 0) {
     for (int s = 0; s < kStages; ++s) {
@@ -168,8 +176,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
       tma_prefetch_desc(&tmKV);
       // pages are walked (no division) and the next block-table entry is loaded ahead of the wait for a free
       // stage: this loop is on the latency path of the KV ring
-      int page_i = 0, page_off = 0;
-      int32_t page_next = ntiles > 0 ? bt[0] : 0;
+      int page_i = t_first * 64 / p.page_size, page_off = t_first * 64 % p.page_size;
+      int32_t page_next = ntiles > 0 ? bt[page_i] : 0;
       const long long head_row = static_cast<long long>(kvh) * p.page_size;
       for (int t = 0; t < ntiles; ++t) {
         const int s = t % kStages;
@@ -242,7 +250,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
     const uint32_t o_addr = lane_addr + 128 + grp * 128;
     uint8_t* myP = sP + grp * kPBytes;
     float m_ref = 0.f, l = 0.f;       // P and l are relative to m_ref (a lagging running maximum)
-    bool ok = true;
+    bool ok = true, unset = true;     // unset: no key of this group has been visible to the row yet
     const int n_mine = (ntiles - grp + 1) / 2;
     for (int u = 0; u < n_mine && ok; ++u) {
       const int t = 2 * u + grp;
@@ -256,17 +264,17 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&bars->s_free[grp]);
-      const int kv0 = t * 64;
+      const int kv0 = (t_first + t) * 64;
       // row maximum of the raw scores (four independent chains); only tiles that touch the causal
-      // diagonal or the end of the sequence need the mask
+      // diagonal, the end of the sequence or the edge of the window need the mask
       float mxa[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-      if (kv0 + 63 <= limit) {
+      if (kv0 + 63 <= limit && limit - kv0 < p.window) {
 #pragma unroll
         for (int c = 0; c < 64; ++c) mxa[c & 3] = fmaxf(mxa[c & 3], __uint_as_float(sr[c >> 5][c & 31]));
       } else {
 #pragma unroll
         for (int c = 0; c < 64; ++c) {
-          const float v = (kv0 + c) <= limit ? __uint_as_float(sr[c >> 5][c & 31]) : -INFINITY;
+          const float v = static_cast<uint32_t>(limit - (kv0 + c)) < static_cast<uint32_t>(p.window) ? __uint_as_float(sr[c >> 5][c & 31]) : -INFINITY;
           sr[c >> 5][c & 31] = __float_as_uint(v);
           mxa[c & 3] = fmaxf(mxa[c & 3], v);
         }
@@ -279,8 +287,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
         tc_fence_after();
       }
       bool grow = false;
-      if (u == 0) {
-        m_ref = mx == -INFINITY ? 0.f : mx;
+      if (unset) {                     // everything so far was masked: the sum and the accumulator are zero
+        unset = mx == -INFINITY;
+        m_ref = unset ? 0.f : mx;
       } else {
         grow = mx - m_ref > 8.0f;      // probabilities would exceed 2^8: move the reference
       }
@@ -332,12 +341,15 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
     tc_fence_after();
     if (grp == 0 && ok && n_mine > 0 && *abort_word == 0) {
       float wa = 1.f, wb = 0.f;
-      if (has_b) {
-        const float mb_ = bars->merge_m[r], lb = bars->merge_l[r];
-        const float mm = fmaxf(m_ref, mb_);
-        wa = exp2f(m_ref - mm);
-        wb = lb > 0.f ? exp2f(mb_ - mm) : 0.f;
-        l = l * wa + lb * wb;
+      const float sink2 = p.sink ? p.sink[head] * 1.4426950408889634f : -INFINITY;
+      if (has_b || p.sink) {
+        const float lb = has_b ? bars->merge_l[r] : 0.f;
+        const float ma = l > 0.f ? m_ref : -INFINITY, mb_ = lb > 0.f ? bars->merge_m[r] : -INFINITY;
+        float mm = fmaxf(fmaxf(ma, mb_), sink2);
+        if (mm == -INFINITY) mm = 0.f;           // a row that sees nothing
+        wa = exp2f(ma - mm);
+        wb = exp2f(mb_ - mm);
+        l = l * wa + lb * wb + exp2f(sink2 - mm);
       }
       const float inv = l > 0.f ? 1.f / l : 0.f;
       wa *= inv;
@@ -385,14 +397,16 @@ using namespace mb;
 
 // Prefill tiles of a ragged batch on the tcgen05 kernel. Same KV addressing as mb_paged_attention_tma
 // (kv_base viewed as [total_rows, 128]); head_dim 128, G = n_q / n_kv in {1, 2, 4, 8, 16}, page_size % 64 == 0.
-// tile_seq / tile_q0 is the plan of 64-row tiles; CTAs take pairs of them.
+// tile_seq / tile_q0 is the plan of 64-row tiles (CTAs take pairs of them) or of 128-row tiles; a negative sequence is
+// an unused tile. window: keys a query sees, itself included (0: all); sink: a score per query head that only takes part
+// in the softmax denominator (null: none).
 extern "C" int mb_paged_attention_prefill_tc(const void* q, int ldq, void* out, int ldo, const void* kv_base,
                                              long long total_rows, long long k_off_rows, long long v_off_rows,
                                              long long page_rows, const int32_t* block_table, int bt_stride,
                                              const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
                                              const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, int n_q,
-                                             int n_kv, int head_dim, int page_size, float scale, int* err,
-                                             cudaStream_t stream) {
+                                             int n_kv, int head_dim, int page_size, float scale, int window,
+                                             const float* sink, int* err, cudaStream_t stream) {
   using namespace mb::atc;
   if (n_tiles <= 0) return MB_OK;
   if (head_dim != 128 || n_kv <= 0 || n_q % n_kv || page_size % 64 || total_rows >= (1ll << 31)) return MB_ERR_SHAPE;
@@ -409,6 +423,8 @@ extern "C" int mb_paged_attention_prefill_tc(const void* q, int ldq, void* out, 
   p.k_off_rows = k_off_rows; p.v_off_rows = v_off_rows; p.page_rows = page_rows;
   p.ldq = ldq; p.ldo = ldo; p.bt_stride = bt_stride; p.page_size = page_size; p.n_tiles = n_tiles; p.G = G;
   p.scale_log2 = scale * 1.4426950408889634f;
+  p.window = window > 0 ? window : 0x7fffffff;
+  p.sink = sink;
   CUtensorMap tm;
   const int rc = cached_tmap(&tm, kv_base, static_cast<uint64_t>(total_rows), head_dim, head_dim, 64, 2);
   if (rc != MB_OK) return rc;

@@ -15,6 +15,9 @@
 // to -inf before the softmax. The cache is zero-initialised and only ever holds finite
 // values, which keeps 0 * garbage finite in the PV product.
 //
+// A sliding window starts every walk at the first tile a row sees (one unsigned comparison masks both edges); a sink
+// score per head only adds exp(sink) to the softmax denominator.
+//
 // Reference counterpart: flash_attention_ragged over PagedKVCache
 // (max/kernels/src/nn/attention/gpu/nvidia/sm100/attention.mojo:62, load_warp.mojo).
 #include <cuda.h>
@@ -50,7 +53,26 @@ struct Params {
   long long k_off_rows, v_off_rows, page_rows;
   float scale_log2;
   int q_rows_alloc;      // rows of shared memory reserved for Q (64, or 16 in a decode-only launch)
+  int window;            // keys a query sees (0x7fffffff: all before it)
+  const float* sink;     // per query head, or null
 };
+
+// first 64-token tile of a walk whose first query is at position `pos`
+__device__ __forceinline__ int first_tile(int pos, int window) {
+  const int lo = pos - window + 1;
+  return lo > 0 ? lo >> 6 : 0;
+}
+
+// The denominator with the sink of query head `head` added; `f` becomes the factor for sums taken relative to maximum m.
+__device__ __forceinline__ float add_sink(const Params& p, int head, float m, float l, float& f) {
+  f = 1.f;
+  if (!p.sink) return l;
+  const float s = p.sink[head] * 1.4426950408889634f;
+  const float mm = fmaxf(m, s);
+  if (mm == -INFINITY) return l;
+  f = exp2f(m - mm);
+  return l * f + exp2f(s - mm);
+}
 
 struct Bars {
   uint64_t full[kStages];
@@ -97,7 +119,7 @@ template <int HD, int NP>
 __device__ __forceinline__ void process_block(const bf16* tK, const bf16* tV, int tok_in_tile, int kv0,
                                               const uint32_t (&qf)[HD / 16][4], float (&o)[HD / 8][4],
                                               float (&m)[2], float (&l)[2], const int (&limit)[2],
-                                              float scale_log2, int lane) {
+                                              float scale_log2, uint32_t window, int lane) {
   constexpr int KS = HD / 16, DT = HD / 8;
   const int mi = lane >> 3;
   float sc[2 * NP][4];
@@ -120,7 +142,7 @@ __device__ __forceinline__ void process_block(const bf16* tK, const bf16* tV, in
     for (int e = 0; e < 4; ++e) {
       const int col = kv0 + nt * 8 + 2 * (lane & 3) + (e & 1);
       const int h = e >> 1;
-      const float v = col <= limit[h] ? sc[nt][e] * scale_log2 : -INFINITY;
+      const float v = static_cast<uint32_t>(limit[h] - col) < window ? sc[nt][e] * scale_log2 : -INFINITY;
       sc[nt][e] = v;
       mx[h] = fmaxf(mx[h], v);
     }
@@ -187,6 +209,7 @@ attn_tma_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
   pdl_trigger();
   const bool is_prefill = static_cast<int>(blockIdx.x) < p.n_tiles;
   const int seq = is_prefill ? p.tile_seq[blockIdx.x] : p.decode_seq[blockIdx.x - p.n_tiles];
+  if (seq < 0) return;             // an unused tile of a plan made on the device
   const int tq0 = is_prefill ? p.tile_q0[blockIdx.x] : 0;
   const int qs = p.q_start[seq], ql = p.q_len[seq], kl = p.kv_len[seq];
   const int32_t* bt = p.block_table + static_cast<int64_t>(seq) * p.bt_stride;
@@ -196,6 +219,7 @@ attn_tma_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
     if (last_tq > ql) last_tq = ql;
     kv_hi = kl - ql + last_tq;
   }
+  const int t_first = first_tile(kl - ql + tq0, p.window);
   const int ntiles = (kv_hi + 63) / 64;
 
   if (tid == 0) {
@@ -217,10 +241,10 @@ attn_tma_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
       // table entry of the next tile is loaded before the wait for a free stage, so its latency hides there.
       int s = 0;
       uint32_t ph = 0;
-      int page_i = 0, page_off = 0;
-      int32_t page_next = ntiles > 0 ? bt[0] : 0;
+      int page_i = t_first * 64 / p.page_size, page_off = t_first * 64 % p.page_size;
+      int32_t page_next = ntiles > t_first ? bt[page_i] : 0;
       const long long head_row = static_cast<long long>(kvh) * p.page_size;
-      for (int t = 0; t < ntiles; ++t, s = (s + 1 == STAGES ? 0 : s + 1), ph ^= (s == 0)) {
+      for (int t = t_first; t < ntiles; ++t, s = (s + 1 == STAGES ? 0 : s + 1), ph ^= (s == 0)) {
         const long long row = static_cast<long long>(page_next) * p.page_rows + head_row + page_off;
         page_off += 64;
         if (page_off == p.page_size) { page_off = 0; ++page_i; }
@@ -271,16 +295,16 @@ attn_tma_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
   }
   int s = 0;
   uint32_t ph = 0;
-  for (int t = 0; t < ntiles; ++t, s = (s + 1 == STAGES ? 0 : s + 1), ph ^= (s == 0)) {
+  for (int t = t_first; t < ntiles; ++t, s = (s + 1 == STAGES ? 0 : s + 1), ph ^= (s == 0)) {
     if (!mbar_wait(&bars->full[s], ph, abort_word, p.err, 302)) break;
     const bf16* tK = sKV + s * 2 * kTileElems;
     const bf16* tV = tK + kTileElems;
     if (is_prefill) {
       // every warp runs its 16 rows against all 64 tokens of the tile
-      process_block<HD, 4>(tK, tV, 0, t * 64, qf, o, m, l, limit, p.scale_log2, lane);
+      process_block<HD, 4>(tK, tV, 0, t * 64, qf, o, m, l, limit, p.scale_log2, p.window, lane);
     } else if (t * 64 + warp * 16 < kv_hi) {
       // the 16 packed rows are shared; each warp takes 16 tokens of the tile
-      process_block<HD, 1>(tK, tV, warp * 16, t * 64 + warp * 16, qf, o, m, l, limit, p.scale_log2, lane);
+      process_block<HD, 1>(tK, tV, warp * 16, t * 64 + warp * 16, qf, o, m, l, limit, p.scale_log2, p.window, lane);
     }
     __syncwarp();
     if (lane == 0) mbar_arrive(&bars->empty[s]);
@@ -294,9 +318,11 @@ attn_tma_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
   if (is_prefill) {
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
-      const float inv = l[h] > 0.f ? 1.f / l[h] : 0.f;
       const int r = row_base + (lane >> 2) + h * 8;
       const int tq = tq0 + r / G, head = kvh * G + r % G;
+      float f;
+      const float den = add_sink(p, head, m[h], l[h], f);
+      const float inv = den > 0.f ? f / den : 0.f;
       if (tq < ql) {
         bf16* orow = p.out + static_cast<int64_t>(qs + tq) * p.ldo + head * HD + 2 * (lane & 3);
 #pragma unroll
@@ -338,7 +364,9 @@ attn_tma_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
         wgt[w] = mw == -INFINITY ? 0.f : exp2f(mw - mm);
         L += wgt[w] * mL[w * 16 + r];
       }
-      const float inv = L > 0.f ? 1.f / L : 0.f;
+      float f;
+      const float den = add_sink(p, head, mm, L, f);
+      const float inv = den > 0.f ? f / den : 0.f;
       bf16* orow = p.out + static_cast<int64_t>(qs + tq) * p.ldo + head * HD;
       constexpr int PER = HD / 8;
       const int d0 = (tid & 7) * PER;
@@ -431,7 +459,10 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap tmKV, const Params 
   pdl_trigger();
   // tile counts of the decode sequences (one round of loads by all threads), then their prefix sums
   // (warp 0: lanes own consecutive chunks of the shared-memory array)
-  for (int i = tid; i < nd; i += kThreads) prefix[i + 1] = (p.kv_len[p.decode_seq[i]] + 63) >> 6;
+  for (int i = tid; i < nd; i += kThreads) {
+    const int seq = p.decode_seq[i], kl = p.kv_len[seq];
+    prefix[i + 1] = ((kl + 63) >> 6) - first_tile(kl - p.q_len[seq], p.window);
+  }
   __syncthreads();
   if (warp == 0) {
     const int per = (nd + 31) / 32;
@@ -487,8 +518,10 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap tmKV, const Params 
         if (fu + t1 > u1) t1 = u1 - fu;
         u = fu + t1;
         if (t1 <= t0) continue;   // a sequence without tiles
-        const int32_t* bt = p.block_table + static_cast<int64_t>(p.decode_seq[i]) * p.bt_stride;
-        int page_i = (t0 * 64) / p.page_size, page_off = (t0 * 64) % p.page_size;
+        const int seq = p.decode_seq[i];
+        const int32_t* bt = p.block_table + static_cast<int64_t>(seq) * p.bt_stride;
+        const int t_abs = t0 + first_tile(p.kv_len[seq] - p.q_len[seq], p.window);
+        int page_i = (t_abs * 64) / p.page_size, page_off = (t_abs * 64) % p.page_size;
         int32_t page_next = bt[page_i];
         for (int t = t0; t < t1; ++t) {
           const long long row = static_cast<long long>(page_next) * p.page_rows + head_row + page_off;
@@ -524,6 +557,7 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap tmKV, const Params 
     if (t1 <= t0) continue;
     const int seq = p.decode_seq[i];
     const int qs = p.q_start[seq], ql = p.q_len[seq], kl = p.kv_len[seq];
+    const int tf = first_tile(kl - ql, p.window);
     const bool hi = ql * G > 8;   // rows 8..15 of the packed query tile are in use
     consumer_sync();              // the previous segment no longer reads sQ or the merge slots
     for (int idx = tid; idx < 16 * CH; idx += 128) {
@@ -554,8 +588,8 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap tmKV, const Params 
       if (!mbar_wait(&bars->full[s], ph, abort_word, p.err, 312)) { ok = false; break; }
       const bf16* tK = sKV + s * 2 * kTileElems;
       const bf16* tV = tK + kTileElems;
-      if (t * 64 + warp * 16 < kl)
-        process_block<HD, 1>(tK, tV, warp * 16, t * 64 + warp * 16, qf, o, m, l, limit, p.scale_log2, lane);
+      if ((tf + t) * 64 + warp * 16 < kl)
+        process_block<HD, 1>(tK, tV, warp * 16, (tf + t) * 64 + warp * 16, qf, o, m, l, limit, p.scale_log2, p.window, lane);
       __syncwarp();
       if (lane == 0) mbar_arrive(&bars->empty[s]);
       if (++s == STAGES) { s = 0; ph ^= 1; }
@@ -659,9 +693,11 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap tmKV, const Params 
     if (finish) {
 #pragma unroll
       for (int h = 0; h < 2; ++h) {
-        const float inv = l[h] > 0.f ? 1.f / l[h] : 0.f;
         const int r = (lane >> 2) + h * 8;
         const int tq = r / G, head = kvh * G + r % G;
+        float f;
+        const float den = add_sink(p, head, m[h], l[h], f);
+        const float inv = den > 0.f ? f / den : 0.f;
         if (tq < ql) {
           bf16* orow = p.out + static_cast<int64_t>(qs + tq) * p.ldo + head * HD + 2 * (lane & 3);
 #pragma unroll
@@ -773,14 +809,12 @@ extern "C" int mb_get_attn_tc(void) { return g_attn_tc_min_tiles; }
 // kv_base: start of the KV allocation, viewed as [total_rows, head_dim] bf16. A token of page
 // `pg`, KV head `h`, offset `o` lives at row  k_off_rows (or v_off_rows) + pg*page_rows +
 // h*page_size + o. Requires page_size % 64 == 0.
-extern "C" int mb_paged_attention_tma(const void* q, int ldq, void* out, int ldo, const void* kv_base,
-                                      long long total_rows, long long k_off_rows, long long v_off_rows,
-                                      long long page_rows, const int32_t* block_table, int bt_stride,
-                                      const int32_t* q_start, const int32_t* q_len,
-                                      const int32_t* kv_len, const int32_t* tile_seq,
-                                      const int32_t* tile_q0, int n_tiles, int n_decode,
-                                      const int32_t* decode_seq, int n_q, int n_kv, int head_dim,
-                                      int page_size, float scale, int* err, cudaStream_t stream) {
+static int attention_tma(const void* q, int ldq, void* out, int ldo, const void* kv_base, long long total_rows,
+                         long long k_off_rows, long long v_off_rows, long long page_rows, const int32_t* block_table,
+                         int bt_stride, const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
+                         const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, int n_decode,
+                         const int32_t* decode_seq, int n_q, int n_kv, int head_dim, int page_size, float scale,
+                         int window, const float* sink, int* err, cudaStream_t stream) {
   using namespace mb::at2;
   if (n_tiles <= 0 && n_decode <= 0) return MB_OK;
   if (n_kv <= 0 || n_q % n_kv || page_size % 64 || total_rows >= (1ll << 31)) return MB_ERR_SHAPE;
@@ -796,6 +830,8 @@ extern "C" int mb_paged_attention_tma(const void* q, int ldq, void* out, int ldo
   p.n_tiles = n_tiles < 0 ? 0 : n_tiles;
   p.k_off_rows = k_off_rows; p.v_off_rows = v_off_rows; p.page_rows = page_rows;
   p.scale_log2 = scale * 1.4426950408889634f;
+  p.window = window > 0 ? window : 0x7fffffff;
+  p.sink = sink;
   CUtensorMap tm;
   const int rc = cached_tmap(&tm, kv_base, static_cast<uint64_t>(total_rows), head_dim, head_dim, 64, 2);
   if (rc != MB_OK) return rc;
@@ -829,7 +865,7 @@ extern "C" int mb_paged_attention_tma(const void* q, int ldq, void* out, int ldo
     }
     const int rc2 = mb_paged_attention_prefill_tc(q, ldq, out, ldo, kv_base, total_rows, k_off_rows, v_off_rows,
                                                   page_rows, block_table, bt_stride, q_start, q_len, kv_len, tile_seq,
-                                                  tile_q0, p.n_tiles, n_q, n_kv, head_dim, page_size, scale, err,
+                                                  tile_q0, p.n_tiles, n_q, n_kv, head_dim, page_size, scale, window, sink, err,
                                                   stream);
     if (rc2 != MB_OK && !forked) return rc2;
     if (n_decode <= 0) return rc2;
@@ -882,4 +918,39 @@ extern "C" int mb_paged_attention_tma(const void* q, int ldq, void* out, int ldo
       return MB_ERR_LAUNCH;
   }
   return rc3;
+}
+
+extern "C" int mb_paged_attention_tma(const void* q, int ldq, void* out, int ldo, const void* kv_base,
+                                      long long total_rows, long long k_off_rows, long long v_off_rows,
+                                      long long page_rows, const int32_t* block_table, int bt_stride,
+                                      const int32_t* q_start, const int32_t* q_len,
+                                      const int32_t* kv_len, const int32_t* tile_seq,
+                                      const int32_t* tile_q0, int n_tiles, int n_decode,
+                                      const int32_t* decode_seq, int n_q, int n_kv, int head_dim,
+                                      int page_size, float scale, int* err, cudaStream_t stream) {
+  return attention_tma(q, ldq, out, ldo, kv_base, total_rows, k_off_rows, v_off_rows, page_rows, block_table, bt_stride,
+                       q_start, q_len, kv_len, tile_seq, tile_q0, n_tiles, n_decode, decode_seq, n_q, n_kv, head_dim,
+                       page_size, scale, 0, nullptr, err, stream);
+}
+
+// The same attention with a sliding window (keys a query sees, itself included; 0: all) and a sink score per query head
+// (null: none). A step is either a decode step (n_tiles 0: one row per entry of decode_seq) or prompt tiles: 128-row
+// tiles (128 / G tokens each) with head_dim 128, on the tcgen05 kernel; 64-row tiles with head_dim 64.
+extern "C" int mb_paged_attention_window(const void* q, int ldq, void* out, int ldo, const void* kv_base,
+                                         long long total_rows, long long k_off_rows, long long v_off_rows,
+                                         long long page_rows, const int32_t* block_table, int bt_stride,
+                                         const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
+                                         const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, int n_decode,
+                                         const int32_t* decode_seq, int n_q, int n_kv, int head_dim, int page_size,
+                                         float scale, int window, const float* sink, int* err, cudaStream_t stream) {
+  if (n_tiles > 0 && n_decode > 0) return MB_ERR_SHAPE;
+  if (n_tiles > 0 && head_dim == 128)
+    return mb_paged_attention_prefill_tc(q, ldq, out, ldo, kv_base, total_rows, k_off_rows, v_off_rows, page_rows,
+                                         block_table, bt_stride, q_start, q_len, kv_len, tile_seq, tile_q0, n_tiles, n_q,
+                                         n_kv, head_dim, page_size, scale, window, sink, err, stream);
+  if (n_tiles > 0 && head_dim != 64) return MB_ERR_SHAPE;
+  // head_dim 64 never takes the 128-wide tcgen05 path inside
+  return attention_tma(q, ldq, out, ldo, kv_base, total_rows, k_off_rows, v_off_rows, page_rows, block_table, bt_stride,
+                       q_start, q_len, kv_len, tile_seq, tile_q0, n_tiles, n_decode, decode_seq, n_q, n_kv, head_dim,
+                       page_size, scale, window, sink, err, stream);
 }

@@ -10,7 +10,12 @@
 // written straight into expert order (`scatter` [T, k2]: the rows token t occupies), so it needs no permute kernel
 // either. `rows` restricts the kernel to some rows of x (the ones whose logits are wanted).
 //
-// Also here: tanh-GELU in place and the sigmoid output gate of an attention layer.
+// A second kernel serves layers whose two mixer branches have output norms of their own and whose update is scaled:
+//
+//   x[t]  += mult * (ab_scale * (a / rms(a) * norm_a + b / rms(b) * norm_b) + c)
+//            [+ inject_scale * inject[ids[t]]] [+ step]       (what a looped pass adds before its first layer)
+//
+// Also here: tanh-GELU in place, the sigmoid output gate of an attention layer and the soft cap of logits.
 #include <cuda_runtime.h>
 
 #include "../common/api.h"
@@ -133,6 +138,109 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(const Params<T> p) 
 }
 
 template <typename T>
+struct MixParams {
+  const T *norm_a, *norm_b, *c, *inject, *step;
+  int ldc, ld_inject;
+  float ab_scale, mult, inject_scale;
+};
+
+__device__ __forceinline__ float sq4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+
+// sums of `N` values per thread over the CTA
+template <int N>
+__device__ __forceinline__ void block_sums(float (&v)[N], float (*part)[32]) {
+#pragma unroll
+  for (int i = 0; i < N; ++i) v[i] = warp_allsum(v[i]);
+  if ((threadIdx.x & 31) == 0)
+#pragma unroll
+    for (int i = 0; i < N; ++i) part[i][threadIdx.x >> 5] = v[i];
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    v[i] = 0.f;
+    for (int w = 0; w < static_cast<int>(blockDim.x >> 5); ++w) v[i] += part[i][w];
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(1024) branch_norm_kernel(const Params<T> p, const MixParams<T> m) {
+  extern __shared__ float4 row_cache[];   // the updated row
+  __shared__ float part[2][32], part2[1][32];
+  const int out_row = blockIdx.x;
+  const int row = p.rows ? p.rows[out_row] : out_row;
+  float* xr = p.x + static_cast<size_t>(row) * p.ldx;
+  const T *ar = p.a ? p.a + static_cast<size_t>(row) * p.lda : nullptr, *br = p.b ? p.b + static_cast<size_t>(row) * p.ldb : nullptr;
+  const T* cr = m.c ? m.c + static_cast<size_t>(row) * m.ldc : nullptr;
+  const T *er = nullptr, *ir = nullptr;
+  if (p.table || m.inject) {
+    const int64_t id = p.ids[row];
+    if (id >= 0 && id < p.vocab) {
+      if (p.table) er = p.table + static_cast<size_t>(id) * p.ld_table;
+      if (m.inject) ir = m.inject + static_cast<size_t>(id) * m.ld_inject;
+    }
+  }
+  const int nvec = p.cols_pad >> 2;
+  float inv_a = 1.f, inv_b = 1.f;
+  if (m.norm_a || m.norm_b) {
+    float s[2] = {0.f, 0.f};
+    for (int v = threadIdx.x; v < nvec; v += blockDim.x) {
+      if (m.norm_a) s[0] += sq4(ld4(ar + v * 4));
+      if (m.norm_b) s[1] += sq4(ld4(br + v * 4));
+    }
+    block_sums(s, part);
+    inv_a = 1.f / sqrtf(s[0] / static_cast<float>(p.cols) + p.eps);
+    inv_b = 1.f / sqrtf(s[1] / static_cast<float>(p.cols) + p.eps);
+  }
+  float ss[1] = {0.f};
+  for (int v = threadIdx.x; v < nvec; v += blockDim.x) {
+    const int c = v * 4;
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f), u = x;
+    if (p.table) {
+      if (er) { x = ld4(er + c); x.x *= p.scale; x.y *= p.scale; x.z *= p.scale; x.w *= p.scale; }
+    } else {
+      x = *reinterpret_cast<const float4*>(xr + c);
+    }
+    auto branch = [&](const T* src, const T* w, float inv) {
+      float4 y = ld4(src + c);
+      if (w) {
+        const float4 g = ld4(w + c);
+        y.x *= inv * g.x; y.y *= inv * g.y; y.z *= inv * g.z; y.w *= inv * g.w;
+      }
+      u.x = fmaf(m.ab_scale, y.x, u.x); u.y = fmaf(m.ab_scale, y.y, u.y);
+      u.z = fmaf(m.ab_scale, y.z, u.z); u.w = fmaf(m.ab_scale, y.w, u.w);
+    };
+    if (ar) branch(ar, m.norm_a, inv_a);
+    if (br) branch(br, m.norm_b, inv_b);
+    if (cr) { const float4 y = ld4(cr + c); u.x += y.x; u.y += y.y; u.z += y.z; u.w += y.w; }
+    x.x = fmaf(m.mult, u.x, x.x); x.y = fmaf(m.mult, u.y, x.y); x.z = fmaf(m.mult, u.z, x.z); x.w = fmaf(m.mult, u.w, x.w);
+    if (ir) {
+      const float4 y = ld4(ir + c);
+      x.x = fmaf(m.inject_scale, y.x, x.x); x.y = fmaf(m.inject_scale, y.y, x.y);
+      x.z = fmaf(m.inject_scale, y.z, x.z); x.w = fmaf(m.inject_scale, y.w, x.w);
+    }
+    if (m.step) { const float4 y = ld4(m.step + c); x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w; }
+    if (p.store_x) *reinterpret_cast<float4*>(xr + c) = x;
+    ss[0] += sq4(x);
+    row_cache[v] = x;
+  }
+  if (p.w1 == nullptr) return;
+  block_sums(ss, part2);
+  const float inv = 1.f / sqrtf(ss[0] / static_cast<float>(p.cols) + p.eps);
+  T *o1 = p.n1 + static_cast<size_t>(out_row) * p.ld1, *o2 = p.w2 ? p.n2 + static_cast<size_t>(out_row) * p.ld2 : nullptr;
+  for (int v = threadIdx.x; v < nvec; v += blockDim.x) {
+    const int c = v * 4;
+    float4 x = row_cache[v];
+    x.x *= inv; x.y *= inv; x.z *= inv; x.w *= inv;
+    const float4 w = ld4(p.w1 + c);
+    st4(o1 + c, make_float4(x.x * w.x, x.y * w.y, x.z * w.z, x.w * w.w));
+    if (o2) {
+      const float4 g = ld4(p.w2 + c);
+      st4(o2 + c, make_float4(x.x * g.x, x.y * g.y, x.z * g.z, x.w * g.w));
+    }
+  }
+}
+
+template <typename T>
 static int run(const MbResidualNorm& q, cudaStream_t stream) {
   Params<T> p;
   p.x = q.x; p.ldx = q.ldx;
@@ -149,6 +257,14 @@ static int run(const MbResidualNorm& q, cudaStream_t stream) {
   // few rows: one pass per row with as many threads as it has vectors; many rows: small CTAs, several per SM
   const int most = q.n_rows <= 296 ? 1024 : 256;
   const int threads = nvec >= most ? most : (nvec + 31) / 32 * 32;
+  if (q.norm_a || q.norm_b || q.c || q.inject || q.step || q.mult != 1.f || q.ab_scale != 1.f) {
+    if (q.e || q.scatter || (q.norm_a && !q.a) || (q.norm_b && !q.b)) return MB_ERR_SHAPE;
+    MixParams<T> m = {static_cast<const T*>(q.norm_a), static_cast<const T*>(q.norm_b), static_cast<const T*>(q.c),
+                      static_cast<const T*>(q.inject), static_cast<const T*>(q.step), q.ldc, q.ld_inject, q.ab_scale, q.mult,
+                      q.inject_scale};
+    return launch_plain(branch_norm_kernel<T>, dim3(q.n_rows), dim3(threads), static_cast<size_t>(p.cols_pad) * 4, stream, p, m) ==
+                   cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
+  }
   return launch_plain(residual_norm_kernel<T>, dim3(q.n_rows), dim3(threads), static_cast<size_t>(p.cols_pad) * 4, stream, p) ==
                  cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
 }
@@ -160,6 +276,17 @@ __global__ void gelu_tanh_kernel(T* __restrict__ x, size_t n4) {
   const float4 v = ld4(x + i * 4);
   auto f = [](float z) { return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); };
   st4(x + i * 4, make_float4(f(v.x), f(v.y), f(v.z), f(v.w)));
+}
+
+__global__ void softcap_kernel(float* __restrict__ x, size_t n, float cap) {
+  const size_t i = (static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x) * 4;
+  if (i + 4 <= n) {
+    float4 v = *reinterpret_cast<const float4*>(x + i);
+    v.x = cap * tanhf(v.x / cap); v.y = cap * tanhf(v.y / cap); v.z = cap * tanhf(v.z / cap); v.w = cap * tanhf(v.w / cap);
+    *reinterpret_cast<float4*>(x + i) = v;
+  } else {
+    for (size_t j = i; j < n; ++j) x[j] = cap * tanhf(x[j] / cap);
+  }
 }
 
 // o[r, c] *= sigmoid(g[r, c])
@@ -182,7 +309,7 @@ using namespace mb::resnorm;
 extern "C" int mb_residual_norm(const MbResidualNorm* q, int dtype, cudaStream_t stream) {
   if (q->n_rows <= 0) return MB_OK;
   if (q->cols <= 0 || q->cols > q->cols_pad || q->cols_pad % 4 || q->ldx % 4 || q->lda % 4 || q->ldb % 4 || q->lde % 4 ||
-      q->ld1 % 4 || q->ld2 % 4 || q->ld_table % 4)
+      q->ld1 % 4 || q->ld2 % 4 || q->ld_table % 4 || q->ldc % 4 || q->ld_inject % 4)
     return MB_ERR_SHAPE;
   if (q->cols_pad > 12288) return MB_ERR_TOO_LARGE;
   return dtype == kF32 ? run<float>(*q, stream) : run<__nv_bfloat16>(*q, stream);
@@ -197,6 +324,15 @@ extern "C" int mb_gelu_tanh(void* x, long long n, int dtype, cudaStream_t stream
                                 : launch_plain(gelu_tanh_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream,
                                            static_cast<__nv_bfloat16*>(x), n4);
   return e == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
+}
+
+extern "C" int mb_softcap(float* x, long long n, float cap, cudaStream_t stream) {
+  if (n <= 0) return MB_OK;
+  if (!(cap > 0.f)) return MB_ERR_SHAPE;
+  if (reinterpret_cast<uintptr_t>(x) & 15) return MB_ERR_ALIGN;
+  const dim3 grid(static_cast<unsigned>((n + 1023) / 1024));
+  return launch_plain(softcap_kernel, grid, dim3(256), 0, stream, x, static_cast<size_t>(n), cap) == cudaSuccess ? MB_OK
+                                                                                                                 : MB_ERR_LAUNCH;
 }
 
 extern "C" int mb_sigmoid_gate(void* o, int ldo, const void* g, int ldg, int rows, int cols, int dtype,

@@ -114,6 +114,26 @@ def _gotunex_family() -> ModelFamily:
     return ModelFamily("gotunex", GotunexConfig, GotunexWeights, GotunexModel, kv, act)
 
 
+def _vipotar_family() -> ModelFamily:
+    from ..kv_cache import KVCacheParams
+    from .vipotar import VipotarConfig, VipotarModel, VipotarWeights
+
+    def kv(cfg, page, dtype, prefix):
+        # one key/value plane and one recurrent state per layer run; the state rules out prefix sharing
+        return KVCacheParams(len(cfg.runs), cfg.cache_heads, cfg.head_width, page, dtype, False, False, cfg.state_specs())
+
+    def act(cfg, T, B):
+        per_tok = 0
+        for i, l in enumerate(cfg.layers):
+            a, r = cfg.attention(i), cfg.lightning(i)
+            n = (2 * a.heads_pad + 2 * a.kv_heads) * cfg.head_width + r.heads * (2 * r.dim8 + 3 * r.vdim8)
+            per_tok = max(per_tok, n + (l["mlp"]["ff"] if l.get("mlp") else 0) + 6 * cfg.width_pad)
+        state = kv(cfg, 64, torch.bfloat16, False).state_bytes_per_slot
+        return T * per_tok * 4 + B * cfg.vocab_size * 4 + B * state + (256 << 20)
+
+    return ModelFamily("vipotar", VipotarConfig, VipotarWeights, VipotarModel, kv, act)
+
+
 def _bert_family() -> ModelFamily:
     from ..kv_cache import KVCacheParams
     from .bert import BertConfig, BertModel, BertWeights
@@ -130,7 +150,8 @@ def _bert_family() -> ModelFamily:
 
 def family_for(config) -> ModelFamily:
     """The family that serves `config` (matched on the config class)."""
-    for make in (_llama_family, _deepseek_family, _mamba_family, _lfm2_family, _gotunex_family, _bert_family):
+    for make in (_llama_family, _deepseek_family, _mamba_family, _lfm2_family, _gotunex_family, _vipotar_family,
+                 _bert_family):
         fam = make()
         if isinstance(config, fam.config_class):
             return fam

@@ -8,6 +8,10 @@ the next one in a single kernel (``csrc/kernels/residual_norm.cu``); the PyTorch
   token (a mixture-of-experts branch without a combine kernel);
 * ``w1``/``n1`` and ``w2``/``n2``: norm weights and outputs of up to two parallel branches; ``scatter`` [T, k] writes
   the second one to the rows a token occupies in expert order (no permute kernel);
+* ``norm_a`` / ``norm_b``: the branches ``a`` and ``b`` are RMS-normed with these weights before they are added;
+  ``ab_scale`` multiplies them, ``c`` is a third branch (no norm), ``mult`` multiplies the whole update;
+* ``inject``: adds ``inject_scale * inject[ids]`` to the stream, ``step`` one row to every token (what a looped pass adds
+  before its first layer);
 * ``rows``: work on these rows of ``x`` only (the ones whose logits are wanted), outputs compacted.
 
 The norm is computed in fp32 and rounded once.
@@ -21,20 +25,33 @@ from .._native import lib as _lib
 
 
 def residual_norm_reference(x, ids=None, table=None, scale=1.0, a=None, b=None, e=None, inverse=None, pair_w=1.0, rows=None,
-                            w1=None, n1=None, w2=None, n2=None, scatter=None, cols=0, store_x=True, eps=1e-6):
+                            w1=None, n1=None, w2=None, n2=None, scatter=None, cols=0, store_x=True, eps=1e-6,
+                            norm_a=None, norm_b=None, ab_scale=1.0, c=None, mult=1.0, inject=None, inject_scale=1.0, step=None):
     cols = cols or x.shape[1]
     idx = torch.arange(x.shape[0]) if rows is None else rows.long()
     h = x[idx] if table is None else table[ids[idx]].float() * scale
     s = torch.zeros_like(h)
+
+    def branch(t, w):
+        y = t[idx, : x.shape[1]].float()
+        return y if w is None else y * torch.rsqrt((y * y).sum(-1, keepdim=True) / cols + eps) * w.float()
+
     if e is not None:
         inv = inverse.view(x.shape[0], -1)[idx].long()
         got = e[inv.clamp(min=0)].float() * (inv >= 0).unsqueeze(-1)
         s = got.sum(1) * pair_w
     elif b is not None:
-        s = b[idx, : x.shape[1]].float()
+        s = branch(b, norm_b)
     if a is not None:
-        s = s + a[idx, : x.shape[1]].float()
-    h = h + s
+        s = s + branch(a, norm_a)
+    s = s * ab_scale
+    if c is not None:
+        s = s + branch(c, None)
+    h = h + s * mult
+    if inject is not None:
+        h = h + inject[ids[idx]].float() * inject_scale
+    if step is not None:
+        h = h + step.float()
     if store_x:
         x[idx] = h
     if w1 is None:
@@ -52,11 +69,13 @@ def residual_norm_reference(x, ids=None, table=None, scale=1.0, a=None, b=None, 
 
 
 def residual_norm(x, ids=None, table=None, scale=1.0, a=None, b=None, e=None, inverse=None, pair_w=1.0, rows=None, w1=None,
-                  n1=None, w2=None, n2=None, scatter=None, cols=0, store_x=True, eps=1e-6):
+                  n1=None, w2=None, n2=None, scatter=None, cols=0, store_x=True, eps=1e-6, norm_a=None, norm_b=None, ab_scale=1.0, c=None, mult=1.0,
+                  inject=None, inject_scale=1.0, step=None):
     """x: fp32 [T, width], width padded to a multiple of 4 with zeros; ``cols`` is the true width (the norm's divisor)."""
     if not x.is_cuda:
         return residual_norm_reference(x, ids, table, scale, a, b, e, inverse, pair_w, rows, w1, n1, w2, n2, scatter, cols,
-                                       store_x, eps)
+                                       store_x, eps, norm_a, norm_b, ab_scale, c, mult, inject, inject_scale, step)
     _lib().residual_norm(x, ids, table, float(scale), a, b, e, inverse, 0 if inverse is None else inverse.numel() // x.shape[0],
                          float(pair_w), rows, w1, n1, w2, n2, scatter, cols or x.shape[1], store_x, float(eps),
-                         x.shape[0] if rows is None else rows.numel())
+                         x.shape[0] if rows is None else rows.numel(), norm_a, norm_b, float(ab_scale), c, float(mult), inject,
+                         float(inject_scale), step)

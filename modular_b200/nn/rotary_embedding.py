@@ -28,6 +28,7 @@ class RopeScaling:
     beta_slow: float = 1.0
     mscale: float = 1.0
     mscale_all_dim: float = 0.0
+    attention_factor: Optional[float] = None      # yarn: factor on cosines and sines (None: from ``factor``)
     short_factor: Optional[Sequence[float]] = None
     long_factor: Optional[Sequence[float]] = None
 
@@ -86,7 +87,7 @@ def inverse_frequencies(head_dim: int, theta: float, scaling: RopeScaling,
             att = _yarn_mscale(scaling.factor, scaling.mscale) / _yarn_mscale(
                 scaling.factor, scaling.mscale_all_dim)
         else:
-            att = _yarn_mscale(scaling.factor, 1.0)
+            att = _yarn_mscale(scaling.factor, 1.0) if scaling.attention_factor is None else float(scaling.attention_factor)
     elif t == "longrope":
         orig = scaling.original_max_position_embeddings
         use_long = bool(seq_len and seq_len > orig)

@@ -22,7 +22,7 @@ from . import reference as ref
 __all__ = [
     "linear", "linear_swiglu", "rms_norm", "add_rms_norm", "silu_mul", "embedding",
     "rope_kv_store", "paged_attention", "build_attention_plan", "argmax", "sample",
-    "apply_penalties", "gelu_tanh", "sigmoid_gate", "gemm_workspace", "check_device_error", "linear_decode", "decode_gemm_workspace",
+    "apply_penalties", "gelu_tanh", "softcap", "sigmoid_gate", "gemm_workspace", "check_device_error", "linear_decode", "decode_gemm_workspace",
 ]
 
 _WORKSPACES: dict[int, torch.Tensor] = {}
@@ -270,6 +270,14 @@ def gelu_tanh(x):
         return x.copy_(ref.gelu_tanh(x))
     _lib().gelu_tanh(x)
     return x
+
+
+def softcap(logits, cap: float):
+    """``cap * tanh(logits / cap)`` over fp32 logits, in place."""
+    if not logits.is_cuda:
+        return logits.copy_(cap * torch.tanh(logits / cap))
+    _lib().softcap(logits, float(cap))
+    return logits
 
 
 def sigmoid_gate(o, g, cols):

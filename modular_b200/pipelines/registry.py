@@ -355,6 +355,13 @@ def _register_builtin() -> None:
         name="Gotunex", config_class=GotunexConfig, weights_class=GotunexWeights, model_class=GotunexModel,
         default_encoding="bfloat16", supported_encodings=("bfloat16", "float32"), example_repo_ids=(),
         preset_configs={"tiny-gotunex": GotunexConfig.tiny}), allow_override=True)
+    from ..models.vipotar import VipotarConfig, VipotarModel, VipotarWeights
+
+    # windowed softmax attention and lightning attention side by side, looped layers
+    PIPELINE_REGISTRY.register(SupportedArchitecture(
+        name="Vipotar", config_class=VipotarConfig, weights_class=VipotarWeights, model_class=VipotarModel,
+        default_encoding="bfloat16", supported_encodings=("bfloat16", "float32"), example_repo_ids=(),
+        preset_configs={"tiny-vipotar": VipotarConfig.tiny}), allow_override=True)
     from ..models.bert import BertConfig, BertModel, BertWeights
 
     # encoder-only embedding models (bidirectional attention; MPNet adds relative-position biases); embeddings only
