@@ -63,7 +63,7 @@ def bench_engine(cfg, prefill: int, seqs: int, batch: int, context: int, steps: 
 
     from ..entrypoints.llm import LLM
     from ..models import family_for
-    from ..pipelines.context import TextContext
+    from ..pipelines.context import SamplingParams, TextContext
 
     n_tok = max(prefill * seqs, context * 4)
     page = 128
@@ -76,6 +76,7 @@ def bench_engine(cfg, prefill: int, seqs: int, batch: int, context: int, steps: 
     llm = LLM(cfg, weights, device="cuda:0", dtype=torch.bfloat16, max_length=max(prefill, context + steps + 16) + 128,
               max_batch_size=max(batch, seqs), max_batch_input_tokens=n_tok, page_size=page, num_kv_pages=need, enable_prefix_caching=False,
               enable_overlap_scheduler=False, graph_batch_sizes=[batch], seed=seed)
+    native = llm.model.use_executor
     rng = np.random.default_rng(seed)
     ids = lambda n: rng.integers(0, cfg.vocab_size, size=n)
     n_ctx = 0
@@ -83,7 +84,7 @@ def bench_engine(cfg, prefill: int, seqs: int, batch: int, context: int, steps: 
     def admit(n):
         nonlocal n_ctx
         n_ctx += 1
-        c = TextContext.from_prompt(ids(n), llm.max_length, f"r{n_ctx}")
+        c = TextContext.from_prompt(ids(n), llm.max_length, f"r{n_ctx}", SamplingParams(temperature=0.0, ignore_eos=True))
         llm.kv.claim(c)
         llm.kv.alloc(c)
         return c
@@ -91,7 +92,10 @@ def bench_engine(cfg, prefill: int, seqs: int, batch: int, context: int, steps: 
     def timed(ctxs, want):
         a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
         a.record()
-        llm.pipeline.score(ctxs, want)
+        if native:                       # the step runs in the native executor and samples greedily
+            llm.pipeline.execute(ctxs)
+        else:
+            llm.pipeline.score(ctxs, want)
         b.record()
         b.synchronize()
         return a.elapsed_time(b)
@@ -105,12 +109,13 @@ def bench_engine(cfg, prefill: int, seqs: int, batch: int, context: int, steps: 
     ctxs = []
     while len(ctxs) < batch:
         part = [admit(context) for _ in range(min(4, batch - len(ctxs)))]
-        llm.pipeline.score(part, [[]] * len(part))
+        timed(part, [[]] * len(part))
         ctxs += part
     dec = []
     for _ in range(5 + steps):
         for c in ctxs:
-            c.tokens.extend(ids(1))
+            if not native:
+                c.tokens.extend(ids(1))
             llm.kv.alloc(c)
         dec.append(timed(ctxs, [[0]] * batch))
     ops.check_device_error()
@@ -118,7 +123,7 @@ def bench_engine(cfg, prefill: int, seqs: int, batch: int, context: int, steps: 
     p, d = med(pre[3:]), med(dec[5:])
     return {"params": cfg.param_count(), "prefill_tokens": prefill * seqs, "prefill_ms": p, "prefill_tok_s": prefill * seqs / p * 1e3,
             "decode_batch": batch, "context": context, "decode_ms": d, "decode_tok_s": batch / d * 1e3,
-            "graph_replays": llm.model.graph_replays}
+            "graph_replays": getattr(llm.model, "graph_replays", None)}
 
 
 def run_models(sizes=("w2048", "w4096", "w7168"), prefill=2048, seqs=4, batches=(1, 64), context=2048, steps=20):

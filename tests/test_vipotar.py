@@ -379,6 +379,30 @@ def test_lightning_remembers_one_token(gap, device, dtype):
         assert rel(got[place + gap], want[place + gap]) < (1e-5 if dtype == torch.float32 else 4e-3)
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("H,d,dv", [(3, 128, 128), (2, 24, 40), (1, 96, 64), (5, 64, 72), (2, 32, 8)])
+def test_lightning_chunks_agree_with_the_scan(H, d, dv):
+    """The tensor-core kernel on bf16 activations against the fp32 scan of the same values: outputs up to their rounding, the
+    state far closer than 16 bits would allow."""
+    from modular_b200._native import lib
+
+    lens, gone = [1, 2, 63, 64, 65, 200, 129], [0, 5, 0, 70, 1, 0, 64]
+    T, B, dp = sum(lens), len(lens), lib().delta_dim_pad(d)
+    decay = torch.tensor([0.999, 0.6, 0.97, 1.0, 0.05])[:H]
+    powers = (decay.double().unsqueeze(1) ** torch.arange(65)).float().cuda()
+    x = rand(T, H * (2 * d + dv), seed=H).bfloat16().cuda()
+    ql, kl = i32(*lens).cuda(), i32(*[n + g for n, g in zip(lens, gone)]).cuda()
+    qs, idx, init = (torch.cumsum(ql, 0) - ql).int(), i32(3, 0, 6, 2, -1, 1, 5).cuda(), rand(8, H, dv, dp, seed=1).cuda()
+    init[..., d:] = 0
+    got = []
+    for dtype in (torch.bfloat16, torch.float32):
+        st, o = init.clone(), torch.zeros(T, H * dv, dtype=dtype, device="cuda")
+        lib().lightning(x.to(dtype), 0, H * d, 2 * H * d, decay.cuda(), powers, o, st, idx, qs, ql, kl, H, d, dv, False)
+        got.append((o, st))
+    assert rel(got[0][1], got[1][1].cpu()) < 2e-5 and rel(got[0][0], got[1][0].cpu()) < 3e-3
+    assert torch.equal(got[0][1][[4, 7]], init[[4, 7]])
+
+
 @pytest.mark.parametrize("device,dtype", RUNS)
 def test_lightning_without_a_slot(device, dtype):
     """Sequences with slot -1 start from zero and keep nothing (the dummies of a padded decode batch)."""
