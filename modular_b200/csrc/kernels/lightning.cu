@@ -114,7 +114,7 @@ __device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], const void* p) {
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)) : "memory");
 }
 __device__ __forceinline__ void mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
@@ -125,6 +125,39 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
   const __nv_bfloat162 l = __floats2bfloat162_rn(x - f.x, y - f.y);
   hi = *reinterpret_cast<const uint32_t*>(&h);
   lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+
+// Products of 16 queries (rows 16 W ..) with the keys at or before them, decayed, into sP as hi and lo parts.
+template <int W, int DK>
+__device__ __forceinline__ void chunk_products(const __nv_bfloat16* sQ, const __nv_bfloat16* sK, __nv_bfloat16* sP, const float* pw, int lane) {
+  constexpr int LDK = DK + 8;
+  const int mi = lane >> 3, r8 = lane & 7, row4 = lane >> 2, col2 = 2 * (lane & 3);
+  float sc[2 * (W + 1)][4];
+#pragma unroll
+  for (int i = 0; i < 2 * (W + 1); ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.f;
+#pragma unroll
+  for (int kb = 0; kb < DK / 16; ++kb) {
+    uint32_t a[4];
+    ldsm4(a, sQ + (W * 16 + (lane & 15)) * LDK + kb * 16 + (lane >> 4) * 8);
+#pragma unroll
+    for (int np = 0; np <= W; ++np) {
+      uint32_t b[4];
+      ldsm4(b, sK + (np * 16 + (mi >> 1) * 8 + r8) * LDK + kb * 16 + (mi & 1) * 8);
+      mma(sc[2 * np], a, b[0], b[1]);
+      mma(sc[2 * np + 1], a, b[2], b[3]);
+    }
+  }
+#pragma unroll
+  for (int nt = 0; nt < 2 * (W + 1); ++nt)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int i = W * 16 + row4 + 8 * e, d = i - (nt * 8 + col2);            // distance to the first of two keys
+      const float a0 = d >= 0 ? sc[nt][2 * e] * pw[d] : 0.f, a1 = d >= 1 ? sc[nt][2 * e + 1] * pw[d - 1] : 0.f;
+      uint32_t hi, lo;
+      split2(a0, a1, hi, lo);
+      *reinterpret_cast<uint32_t*>(sP + i * kLdP + nt * 8 + col2) = hi;
+      *reinterpret_cast<uint32_t*>(sP + (kChunk + i) * kLdP + nt * 8 + col2) = lo;
+    }
 }
 
 // One CTA walks the chunks of one (sequence, head, 64 value columns). DK: key width padded to a multiple of 32.
@@ -175,42 +208,17 @@ __global__ void __launch_bounds__(kThreads, 2) lightning_chunk_kernel(const MbLi
     }
   bool have_state = resume;
   for (int c0 = 0, it = 0; c0 < n; c0 += kChunk, ++it) {
-    const int m = min(kChunk, n - c0), blocks = (m + 15) / 16;
+    const int m = min(kChunk, n - c0);
     const bf16 *sQ = stages + (it & 1) * kStage, *sK = sQ + kChunk * LDK, *sV = sK + kChunk * LDK;
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                 // this chunk is in; the last one is done with its stage and with sP
     if (c0 + kChunk < n) fetch(c0 + kChunk, stages + ((it + 1) & 1) * kStage);
-    // products of this warp's 16 queries with the keys at or before them
-    if (warp < blocks) {
-      float sc[8][4];
-#pragma unroll
-      for (int i = 0; i < 8; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.f;
-#pragma unroll
-      for (int kb = 0; kb < KB; ++kb) {
-        uint32_t a[4];
-        ldsm4(a, sQ + (warp * 16 + (lane & 15)) * LDK + kb * 16 + (lane >> 4) * 8);
-#pragma unroll
-        for (int np = 0; np < 4; ++np) {
-          if (np > warp) break;
-          uint32_t b[4];
-          ldsm4(b, sK + (np * 16 + (mi >> 1) * 8 + r8) * LDK + kb * 16 + (mi & 1) * 8);
-          mma(sc[2 * np], a, b[0], b[1]);
-          mma(sc[2 * np + 1], a, b[2], b[3]);
-        }
-      }
-#pragma unroll
-      for (int nt = 0; nt < 8; ++nt) {
-        if (nt > 2 * warp + 1) break;
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int i = warp * 16 + row4 + 8 * e, d = i - (nt * 8 + col2);     // distance to the first of two keys
-          const float a0 = d >= 0 ? sc[nt][2 * e] * pw[d] : 0.f, a1 = d >= 1 ? sc[nt][2 * e + 1] * pw[d - 1] : 0.f;
-          uint32_t hi, lo;
-          split2(a0, a1, hi, lo);
-          *reinterpret_cast<uint32_t*>(sP + i * kLdP + nt * 8 + col2) = hi;
-          *reinterpret_cast<uint32_t*>(sP + (kChunk + i) * kLdP + nt * 8 + col2) = lo;
-        }
-      }
+    // straight-line code from here on: rows beyond the end of the sequence are zeros and cost what full ones cost
+    switch (warp) {
+      case 0: chunk_products<0, DK>(sQ, sK, sP, pw, lane); break;
+      case 1: chunk_products<1, DK>(sQ, sK, sP, pw, lane); break;
+      case 2: chunk_products<2, DK>(sQ, sK, sP, pw, lane); break;
+      default: chunk_products<3, DK>(sQ, sK, sP, pw, lane); break;
     }
     // what the state before the chunk contributes, for all queries and this warp's 16 value columns
     float o[4][2][4];
@@ -226,17 +234,13 @@ __global__ void __launch_bounds__(kThreads, 2) lightning_chunk_kernel(const MbLi
         for (int j = 0; j < 2; ++j)
 #pragma unroll
           for (int e = 0; e < 2; ++e) split2(S[2 * kb + e][2 * j], S[2 * kb + e][2 * j + 1], hi[j][e], lo[j][e]);
+        uint32_t a[4][4];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          if (i >= blocks) break;
-          uint32_t a[4];
-          ldsm4(a, sQ + (i * 16 + (lane & 15)) * LDK + kb * 16 + (lane >> 4) * 8);
+        for (int i = 0; i < 4; ++i) ldsm4(a[i], sQ + (i * 16 + (lane & 15)) * LDK + kb * 16 + (lane >> 4) * 8);
 #pragma unroll
-          for (int j = 0; j < 2; ++j) {
-            mma(o[i][j], a, hi[j][0], hi[j][1]);
-            mma(o[i][j], a, lo[j][0], lo[j][1]);
-          }
-        }
+        for (int i = 0; i < 4; ++i) { mma(o[i][0], a[i], hi[0][0], hi[0][1]); mma(o[i][1], a[i], hi[1][0], hi[1][1]); }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { mma(o[i][0], a[i], lo[0][0], lo[0][1]); mma(o[i][1], a[i], lo[1][0], lo[1][1]); }
       }
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
@@ -248,14 +252,12 @@ __global__ void __launch_bounds__(kThreads, 2) lightning_chunk_kernel(const MbLi
     __syncthreads();                                 // the products of every warp are in sP
 #pragma unroll
     for (int kb = 0; kb < 4; ++kb) {
-      if (kb >= blocks) break;
       uint32_t b[4];
       ldsm4_t(b, sV + (kb * 16 + (mi & 1) * 8 + r8) * kLdV + warp * 16 + (mi >> 1) * 8);
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        if (i < kb || i >= blocks) continue;
+      for (int half = 0; half < 2; ++half) {
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
+        for (int i = kb; i < 4; ++i) {
           uint32_t a[4];
           ldsm4(a, sP + (half * kChunk + i * 16 + (lane & 15)) * kLdP + kb * 16 + (lane >> 4) * 8);
           mma(o[i][0], a, b[0], b[1]);
@@ -285,7 +287,6 @@ __global__ void __launch_bounds__(kThreads, 2) lightning_chunk_kernel(const MbLi
     have_state = true;
 #pragma unroll
     for (int kb = 0; kb < 4; ++kb) {
-      if (kb >= blocks) break;
       uint32_t a[4], hi[4], lo[4];                   // value columns as rows: transposed fragments of V, decayed
       ldsm4_t(a, sV + (kb * 16 + (mi >> 1) * 8 + r8) * kLdV + warp * 16 + (mi & 1) * 8);
 #pragma unroll
@@ -295,13 +296,18 @@ __global__ void __launch_bounds__(kThreads, 2) lightning_chunk_kernel(const MbLi
         split2(f.x * pw[d > 0 ? d : 0], f.y * pw[d > 1 ? d - 1 : 0], hi[q], lo[q]);
       }
 #pragma unroll
-      for (int t = 0; t < KB; ++t) {
-        uint32_t b[4];
+      for (int t = 0; t < KB; t += 2) {
+        uint32_t b[4], c[4];
         ldsm4_t(b, sK + (kb * 16 + (mi & 1) * 8 + r8) * LDK + t * 16 + (mi >> 1) * 8);
+        ldsm4_t(c, sK + (kb * 16 + (mi & 1) * 8 + r8) * LDK + t * 16 + 16 + (mi >> 1) * 8);
         mma(S[2 * t], hi, b[0], b[1]);
         mma(S[2 * t + 1], hi, b[2], b[3]);
+        mma(S[2 * t + 2], hi, c[0], c[1]);
+        mma(S[2 * t + 3], hi, c[2], c[3]);
         mma(S[2 * t], lo, b[0], b[1]);
         mma(S[2 * t + 1], lo, b[2], b[3]);
+        mma(S[2 * t + 2], lo, c[0], c[1]);
+        mma(S[2 * t + 3], lo, c[2], c[3]);
       }
     }
   }
@@ -329,18 +335,34 @@ static int launch_chunk(const MbLightning& p, cudaStream_t stream) {
                       col_blocks) == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
 }
 
+// sigmoid of an output gate: fp32 runs take the accurate exponential, 16-bit runs (the result is rounded) the fast one
+template <typename T>
+__device__ __forceinline__ float gate_of(float z) {
+  if constexpr (sizeof(T) == 4) return sigmoidf(z);
+  return __fdividef(1.f, 1.f + __expf(-z));
+}
+
 // o[t, :] = o / rms(o over the `n` true columns) * w * sigmoid(gate), in place; padding columns hold zeros
 template <typename T>
 __global__ void __launch_bounds__(1024) lightning_norm_kernel(T* __restrict__ o, int ldo, const T* __restrict__ gate, int ldg,
                                                               const T* __restrict__ w, int cols, int n, float eps) {
+  constexpr int kHeld = 4;                           // 4-wide pieces a thread keeps in registers; more are read again
   __shared__ float part[32];
   const size_t t = blockIdx.x;
   T* row = o + t * ldo;
   const T* g = gate + t * ldg;
+  float4 v[kHeld], b[kHeld];
   float ss = 0.f;
-  for (int c = threadIdx.x * 4; c < cols; c += blockDim.x * 4) {
-    const float4 v = ld4(row + c);
-    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+#pragma unroll
+  for (int i = 0; i < kHeld; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 4;
+    v[i] = c < cols ? ld4(row + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    b[i] = c < cols ? ld4(g + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+  }
+  for (int c = (threadIdx.x + kHeld * blockDim.x) * 4; c < cols; c += blockDim.x * 4) {
+    const float4 e = ld4(row + c);
+    ss += e.x * e.x + e.y * e.y + e.z * e.z + e.w * e.w;
   }
   ss = warp_allsum(ss);
   if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = ss;
@@ -348,11 +370,17 @@ __global__ void __launch_bounds__(1024) lightning_norm_kernel(T* __restrict__ o,
   float tot = 0.f;
   for (int i = 0; i < static_cast<int>(blockDim.x >> 5); ++i) tot += part[i];
   const float inv = 1.f / sqrtf(tot / static_cast<float>(n) + eps);
-  for (int c = threadIdx.x * 4; c < cols; c += blockDim.x * 4) {
-    const float4 v = ld4(row + c), a = ld4(w + c), b = ld4(g + c);
-    st4(row + c, make_float4(v.x * inv * a.x * sigmoidf(b.x), v.y * inv * a.y * sigmoidf(b.y), v.z * inv * a.z * sigmoidf(b.z),
-                             v.w * inv * a.w * sigmoidf(b.w)));
+  auto put = [&](int c, float4 e, float4 gt) {
+    const float4 a = ld4(w + c);
+    st4(row + c, make_float4(e.x * inv * a.x * gate_of<T>(gt.x), e.y * inv * a.y * gate_of<T>(gt.y), e.z * inv * a.z * gate_of<T>(gt.z),
+                             e.w * inv * a.w * gate_of<T>(gt.w)));
+  };
+#pragma unroll
+  for (int i = 0; i < kHeld; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 4;
+    if (c < cols) put(c, v[i], b[i]);
   }
+  for (int c = (threadIdx.x + kHeld * blockDim.x) * 4; c < cols; c += blockDim.x * 4) put(c, ld4(row + c), ld4(g + c));
 }
 
 template <typename T, int RL4>
