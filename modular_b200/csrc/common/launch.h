@@ -55,4 +55,11 @@ inline cudaError_t launch_plain(void (*kern)(KArgs...), dim3 grid, dim3 block, s
   return cudaGetLastError();
 }
 
+// One or the other: a kernel whose neighbours on the stream are ordinary launches goes without the attribute.
+template <typename... KArgs, typename... Args>
+inline cudaError_t launch_either(bool dependent, void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
+                                 Args&&... args) {
+  return dependent ? launch_k(kern, grid, block, smem, stream, args...) : launch_plain(kern, grid, block, smem, stream, args...);
+}
+
 }  // namespace mb

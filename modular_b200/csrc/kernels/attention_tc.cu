@@ -436,7 +436,8 @@ extern "C" int mb_paged_attention_prefill_tc(const void* q, int ldq, void* out, 
       return MB_ERR_LAUNCH;
     configured.done();
   }
-  return launch_k(attn_tc_kernel, dim3(n_tiles, n_kv), dim3(kThreads), smem, stream, tm, p) == cudaSuccess
+  // windows and sinks belong to families whose layer kernels are ordinary launches
+  return launch_either(window <= 0 && sink == nullptr, attn_tc_kernel, dim3(n_tiles, n_kv), dim3(kThreads), smem, stream, tm, p) == cudaSuccess
              ? MB_OK
              : MB_ERR_LAUNCH;
 }

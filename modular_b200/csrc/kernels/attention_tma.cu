@@ -55,6 +55,7 @@ struct Params {
   int q_rows_alloc;      // rows of shared memory reserved for Q (64, or 16 in a decode-only launch)
   int window;            // keys a query sees (0x7fffffff: all before it)
   const float* sink;     // per query head, or null
+  bool dependent;        // programmatic dependent launch
 };
 
 // first 64-token tile of a walk whose first query is at position `pos`
@@ -736,7 +737,7 @@ static int launch_split(const CUtensorMap& tm, const Params& p, int n_decode, in
       return MB_ERR_LAUNCH;
     configured.done();
   }
-  if (launch_k(kern, dim3(GX, n_kv), dim3(kThreads), smem, stream, tm, p, sp) != cudaSuccess) return MB_ERR_LAUNCH;
+  if (launch_either(p.dependent, kern, dim3(GX, n_kv), dim3(kThreads), smem, stream, tm, p, sp) != cudaSuccess) return MB_ERR_LAUNCH;
   return MB_OK;
 }
 
@@ -754,7 +755,7 @@ static int launch_one(const CUtensorMap& tm, Params p, int n_ctas, int n_kv, int
     configured.done();
   }
   p.q_rows_alloc = q_rows;
-  if (launch_k(kern, dim3(n_ctas, n_kv), dim3(kThreads), smem, stream, tm, p) != cudaSuccess) return MB_ERR_LAUNCH;
+  if (launch_either(p.dependent, kern, dim3(n_ctas, n_kv), dim3(kThreads), smem, stream, tm, p) != cudaSuccess) return MB_ERR_LAUNCH;
   return MB_OK;
 }
 
@@ -832,6 +833,7 @@ static int attention_tma(const void* q, int ldq, void* out, int ldo, const void*
   p.scale_log2 = scale * 1.4426950408889634f;
   p.window = window > 0 ? window : 0x7fffffff;
   p.sink = sink;
+  p.dependent = window <= 0 && sink == nullptr;
   CUtensorMap tm;
   const int rc = cached_tmap(&tm, kv_base, static_cast<uint64_t>(total_rows), head_dim, head_dim, 64, 2);
   if (rc != MB_OK) return rc;
