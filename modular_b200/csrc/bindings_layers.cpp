@@ -99,6 +99,67 @@ void residual_norm(Tensor& x, const Opt& ids, const Opt& table, double scale, co
   check_rc(mb_residual_norm(&p, dt == at::kFloat ? 1 : 0, cur_stream()), "residual_norm");
 }
 
+// seam with norms on both sides of a branch, see MbSandwichNorm
+void sandwich_norm(Tensor& x, const Opt& ids, const Opt& table, double scale, const Opt& inject_ids, const Opt& inject, const Opt& a,
+                   const Opt& e, const Opt& inverse, const Opt& pair_w, const Opt& rows, const Opt& w_u, const Opt& b_u, double mult,
+                   const Opt& w1, const Opt& b1, const Opt& n1, int cols, bool store_x, double eps, int n_rows) {
+  MbSandwichNorm p = {};
+  p.ldx = ld_of(x, at::kFloat, "x"); p.x = x.data_ptr<float>();
+  p.cols = cols; p.cols_pad = static_cast<int>(x.size(1)); p.store_x = store_x; p.eps = static_cast<float>(eps); p.n_rows = n_rows;
+  p.scale = static_cast<float>(scale); p.mult = static_cast<float>(mult);
+  const int64_t T = x.size(0);
+  const at::ScalarType dt = given(w1) ? w1->scalar_type() : given(a) ? a->scalar_type() : given(e) ? e->scalar_type() : at::kBFloat16;
+  auto matrix = [&](const Opt& t, const char* what, int64_t min_rows) {
+    const int ld = ld_of(*t, dt, what);
+    TORCH_CHECK(t->size(1) >= p.cols_pad && t->size(0) >= min_rows, "sandwich_norm: ", what, " shape");
+    return ld;
+  };
+  auto index = [&](const Opt& t, const char* what) {
+    TORCH_CHECK(given(t) && t->is_cuda() && t->is_contiguous() && t->scalar_type() == at::kLong && t->numel() >= T, "sandwich_norm: ", what);
+    return t->data_ptr<int64_t>();
+  };
+  auto weight = [&](const Opt& t, const char* what) -> const void* {
+    if (!given(t)) return nullptr;
+    TORCH_CHECK(t->is_cuda() && t->is_contiguous() && t->scalar_type() == dt && t->numel() >= p.cols_pad, "sandwich_norm: ", what);
+    return t->data_ptr();
+  };
+  if (given(table)) {
+    p.ld_table = matrix(table, "table", 0); p.table = table->data_ptr(); p.ids = index(ids, "ids"); p.vocab = static_cast<int>(table->size(0));
+  }
+  if (given(inject)) {
+    p.ld_inject = matrix(inject, "inject", 0); p.inject = inject->data_ptr(); p.inject_ids = index(inject_ids, "inject_ids");
+    p.inject_rows = static_cast<int>(inject->size(0));
+  }
+  if (given(a)) { p.lda = matrix(a, "a", T); p.a = a->data_ptr(); }
+  if (given(e)) {
+    TORCH_CHECK(given(inverse) && inverse->dim() == 2 && given(pair_w), "sandwich_norm: inverse [T, k] and pair_w");
+    p.top_k = static_cast<int>(inverse->size(1));
+    p.lde = matrix(e, "e", T * p.top_k); p.e = e->data_ptr();
+    p.inverse = i32(*inverse, T * p.top_k, "inverse"); p.pair_w = f32(*pair_w, T * p.top_k, "pair_w");
+  }
+  if (given(rows)) p.rows = i32(*rows, n_rows, "rows");
+  else TORCH_CHECK(n_rows <= T, "sandwich_norm: rows");
+  p.w_u = weight(w_u, "w_u"); p.b_u = weight(b_u, "b_u"); p.w1 = weight(w1, "w1"); p.b1 = weight(b1, "b1");
+  if (given(w1)) { TORCH_CHECK(given(n1), "sandwich_norm: n1"); p.ld1 = matrix(n1, "n1", n_rows); p.n1 = n1->data_ptr(); }
+  check_rc(mb_sandwich_norm(&p, dt == at::kFloat ? 1 : 0, cur_stream()), "sandwich_norm");
+}
+
+// window, sink and output gate of an attention call; `use` is what the C interface takes (null: none of them)
+struct AttnOptions {
+  MbAttnOptions o = {};
+  const MbAttnOptions* use = nullptr;
+  AttnOptions(int window, const Opt& sink, const Opt& gate, double gate_mult, int64_t T, int64_t heads, at::ScalarType dt, const char* what) {
+    o.window = window;
+    o.gate_mult = static_cast<float>(gate_mult);
+    if (given(sink)) o.sink = f32(*sink, heads, "sink");
+    if (given(gate)) {
+      o.ld_gate = ld_of(*gate, dt, "gate"); o.gate = gate->data_ptr();
+      TORCH_CHECK(gate->size(0) >= T && gate->size(1) >= heads, what, ": gate [T, heads]");
+    }
+    if (window > 0 || o.sink || o.gate) use = &o;
+  }
+};
+
 void latent_post_down(const Tensor& x, int q_rank, const Opt& gamma_q, const Opt& q_out, int kv_off, int R, int Rp,
                       const Opt& gamma_kv, int rot_dim, int Dp, int dims, bool interleaved, double eps,
                       const Tensor& positions, const Tensor& cos_sin, const Tensor& slots, const Opt& cache) {
@@ -132,7 +193,7 @@ void latent_post_down(const Tensor& x, int q_rank, const Opt& gamma_q, const Opt
 // q_lat [T, h, Rp], q_rope [T, h, Dp] (any token stride, heads contiguous blocks), cache [pages, page, >= Rp + Dp]
 void latent_attention(const Tensor& q_lat, const Tensor& q_rope, const Tensor& cache, const Tensor& block_table,
                       const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, Tensor& out, double scale,
-                      const Opt& sink, bool one_token, const Opt& ws, bool allow_tc) {
+                      const Opt& sink, bool one_token, const Opt& ws, bool allow_tc, int window, const Opt& gate, double gate_mult) {
   const int dt = dtype_of(q_lat, "q_lat");
   TORCH_CHECK(q_lat.is_cuda() && q_lat.dim() == 3 && q_lat.stride(2) == 1 && q_rope.dim() == 3 && q_rope.stride(2) == 1 &&
                   out.is_contiguous() && out.sizes() == q_lat.sizes() && q_rope.size(0) == q_lat.size(0) &&
@@ -142,7 +203,7 @@ void latent_attention(const Tensor& q_lat, const Tensor& q_rope, const Tensor& c
                   block_table.scalar_type() == at::kInt,
               "latent_attention layout");
   const int T = q_lat.size(0), h = q_lat.size(1), R = q_lat.size(2), D = q_rope.size(2), B = q_len.numel();
-  const float* sk = given(sink) ? f32(*sink, h, "sink") : nullptr;
+  const AttnOptions opt(window, sink, gate, gate_mult, T, h, q_lat.scalar_type(), "latent_attention");
   const int32_t *qs = i32(q_start, B, "q_start"), *ql = i32(q_len, B, "q_len"), *kl = i32(kv_len, B, "kv_len");
   const int32_t* bt = block_table.data_ptr<int32_t>();
   const int page = cache.size(1), bts = block_table.stride(0), ldc = cache.stride(1);
@@ -154,13 +215,13 @@ void latent_attention(const Tensor& q_lat, const Tensor& q_rope, const Tensor& c
       mb_mla_tc_usable(T, T, h, R, page)) {
     if (one_token) {
       check_rc(mb_mla_decode_tc(q_lat.data_ptr(), q_rope.data_ptr(), out.data_ptr(), cache.data_ptr(), cache.stride(0),
-                                cache.size(0), bt, bts, qs, ql, kl, T, B, h, page, scale, sk,
+                                cache.size(0), bt, bts, qs, ql, kl, T, B, h, page, scale, opt.use,
                                 static_cast<int>(q_rope.stride(1)), error_flag(), cur_stream()),
                "mla_decode_tc");
     } else {
       auto scratch = at::empty({2 * static_cast<int64_t>(T)}, q_start.options());
       check_rc(mb_mla_prefill_tc(q_lat.data_ptr(), q_rope.data_ptr(), out.data_ptr(), cache.data_ptr(), cache.stride(0),
-                                 cache.size(0), bt, bts, qs, ql, kl, T, B, h, page, scale, sk,
+                                 cache.size(0), bt, bts, qs, ql, kl, T, B, h, page, scale, opt.use,
                                  static_cast<int>(q_rope.stride(1)), scratch.data_ptr<int32_t>(),
                                  error_flag(), cur_stream()),
                "mla_prefill_tc");
@@ -169,7 +230,7 @@ void latent_attention(const Tensor& q_lat, const Tensor& q_rope, const Tensor& c
   }
   if (mma) {
     check_rc(mb_mla_paged_attention_ex(q_lat.data_ptr(), q_lat.stride(0), q_rope.data_ptr(), q_rope.stride(0), q_rope.stride(1),
-                                       out.data_ptr(), cache.data_ptr(), cache.stride(0), ldc, bt, bts, qs, ql, kl, T, B, h, R, page, scale, sk,
+                                       out.data_ptr(), cache.data_ptr(), cache.stride(0), ldc, bt, bts, qs, ql, kl, T, B, h, R, page, scale, opt.use,
                                        given(ws) ? ws->data_ptr() : nullptr, given(ws) ? ws->nbytes() : 0, num_sms(),
                                        cur_stream()),
              "mla_paged_attention");
@@ -177,16 +238,16 @@ void latent_attention(const Tensor& q_lat, const Tensor& q_rope, const Tensor& c
   }
   check_rc(mb_latent_attention(q_lat.data_ptr(), q_lat.stride(0), q_lat.stride(1), q_rope.data_ptr(), q_rope.stride(0),
                                q_rope.stride(1), out.data_ptr(), out.stride(0), out.stride(1), cache.data_ptr(),
-                               cache.stride(0), ldc, page, bt, bts, qs, ql, kl, T, B, h, R, D, scale, sk, dt, cur_stream()),
+                               cache.stride(0), ldc, page, bt, bts, qs, ql, kl, T, B, h, R, D, scale, opt.use, dt, cur_stream()),
            "latent_attention");
 }
 
 // x: projection rows with the column blocks of q, k, v and beta at the given offsets; see MbDelta for the rest
-void delta_rule(const Tensor& x, int q_off, int k_off, int v_off, int b_off, const Tensor& conv_w, const Tensor& z,
+void delta_rule(const Tensor& x, int q_off, int k_off, int v_off, int b_off, const Tensor& conv_w, const Opt& z,
                 const Tensor& A_log, const Tensor& dt_bias, const Tensor& gate, const Tensor& norm_w, double eps,
                 std::vector<Tensor>& scratch, Tensor& out, Tensor& state, Tensor& conv_state, const Tensor& state_idx,
                 const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, int heads, int kv_heads, int dim, int vdim,
-                bool one_token) {
+                bool one_token, int a_off, bool gate_silu, double out_mult) {
   MbDelta p = {};
   const int dt = dtype_of(x, "x");
   const at::ScalarType st = x.scalar_type();
@@ -201,15 +262,21 @@ void delta_rule(const Tensor& x, int q_off, int k_off, int v_off, int b_off, con
                   v_off + heads * vdim <= x.size(1) && b_off + heads <= x.size(1), "delta_rule: columns");
   TORCH_CHECK(conv_w.is_contiguous() && conv_w.scalar_type() == st && conv_w.dim() == 2 && conv_w.size(0) == C, "delta_rule: conv_w");
   p.conv_w = conv_w.data_ptr(); p.taps = conv_w.size(1);
-  p.ldz = ld_of(z, at::kFloat, "z"); p.z = z.data_ptr<float>();
-  TORCH_CHECK(z.size(0) >= T && z.size(1) >= heads * dim, "delta_rule: z");
-  p.A_log = f32(A_log, heads, "A_log"); p.dt_bias = f32(dt_bias, static_cast<int64_t>(heads) * dim, "dt_bias");
+  if (given(z)) {
+    p.ldz = ld_of(*z, at::kFloat, "z"); p.z = z->data_ptr<float>();
+    TORCH_CHECK(z->size(0) >= T && z->size(1) >= heads * dim, "delta_rule: z");
+  } else {                                       // one decay per head, from columns of x
+    TORCH_CHECK(a_off >= 0 && a_off + heads <= x.size(1), "delta_rule: a_off");
+    p.a_off = a_off;
+  }
+  p.gate_silu = gate_silu; p.out_mult = static_cast<float>(out_mult);
+  p.A_log = f32(A_log, heads, "A_log"); p.dt_bias = f32(dt_bias, static_cast<int64_t>(heads) * (given(z) ? dim : 1), "dt_bias");
   p.ld_gate = ld_of(gate, st, "gate"); p.gate = gate.data_ptr();
   TORCH_CHECK(gate.size(0) >= T && gate.size(1) >= heads * vdim, "delta_rule: gate");
   TORCH_CHECK(norm_w.is_contiguous() && norm_w.scalar_type() == st && norm_w.numel() >= vdim, "delta_rule: norm_w");
   p.norm_w = norm_w.data_ptr(); p.eps = static_cast<float>(eps);
   TORCH_CHECK(scratch.size() == 7, "delta_rule: scratch is {q, k, g, v, beta, kq, o}");
-  const int64_t need[7] = {T * kv_heads * p.dim_pad, T * kv_heads * p.dim_pad, T * heads * p.dim_pad, T * heads * vdim,
+  const int64_t need[7] = {T * kv_heads * p.dim_pad, T * kv_heads * p.dim_pad, T * heads * (given(z) ? p.dim_pad : 1), T * heads * vdim,
                            T * heads, T * kv_heads, T * heads * vdim};
   float** dst[7] = {&p.q, &p.k, &p.g, &p.v, &p.beta, &p.kq, &p.o};
   for (int i = 0; i < 7; ++i) *dst[i] = const_cast<float*>(f32(scratch[i], need[i], "delta_rule scratch"));
@@ -223,6 +290,38 @@ void delta_rule(const Tensor& x, int q_off, int k_off, int v_off, int b_off, con
   p.state_idx = i32(state_idx, p.B, "state_idx"); p.q_start = i32(q_start, p.B, "q_start");
   p.q_len = i32(q_len, p.B, "q_len"); p.kv_len = i32(kv_len, p.B, "kv_len");
   check_rc(mb_delta_rule(&p, dt, num_sms(), cur_stream()), "delta_rule");
+}
+
+// x: projection rows with the column blocks of q, k and v at the given offsets; see MbGla
+void gla(const Tensor& x, int q_off, int k_off, int v_off, const Tensor& z, const Tensor& z_bias, double q_scale, double inv_tau,
+         const Tensor& gate, bool gate_silu, double out_mult, const Tensor& norm_w, double eps, int norm_dim, Tensor& o, Tensor& out,
+         Tensor& state, const Tensor& state_idx, const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, int heads, int dim,
+         int vdim, bool one_token) {
+  MbGla p = {};
+  const at::ScalarType st = x.scalar_type();
+  p.T = x.size(0); p.B = q_len.numel(); p.heads = heads; p.dim = dim; p.vdim = vdim; p.one_token = one_token;
+  p.dim_pad = mb_delta_dim_pad(dim);
+  TORCH_CHECK(p.dim_pad > 0, "gla: key width ", dim, " is beyond the supported maximum");
+  const int64_t T = p.T;
+  p.x = x.data_ptr(); p.ldx = ld_of(x, st, "x"); p.q_off = q_off; p.k_off = k_off; p.v_off = v_off;
+  TORCH_CHECK(q_off + heads * dim <= x.size(1) && k_off + heads * dim <= x.size(1) && v_off + heads * vdim <= x.size(1), "gla: columns");
+  p.ldz = ld_of(z, at::kFloat, "z"); p.z = z.data_ptr<float>();
+  TORCH_CHECK(z.size(0) >= T && z.size(1) >= heads * dim, "gla: z");
+  p.z_bias = f32(z_bias, static_cast<int64_t>(heads) * dim, "z_bias");
+  p.q_scale = static_cast<float>(q_scale); p.inv_tau = static_cast<float>(inv_tau);
+  p.ld_gate = ld_of(gate, st, "gate"); p.gate = gate.data_ptr(); p.gate_silu = gate_silu; p.out_mult = static_cast<float>(out_mult);
+  TORCH_CHECK(gate.size(0) >= T && gate.size(1) >= heads * vdim, "gla: gate");
+  TORCH_CHECK(norm_w.is_contiguous() && norm_w.scalar_type() == st && norm_w.numel() >= vdim, "gla: norm_w");
+  p.norm_w = norm_w.data_ptr(); p.eps = static_cast<float>(eps); p.norm_dim = norm_dim;
+  p.o = const_cast<float*>(f32(o, one_token ? 0 : T * heads * vdim, "gla: o"));
+  p.ld_out = ld_of(out, st, "out"); p.out = out.data_ptr();
+  TORCH_CHECK(out.size(0) >= T && out.size(1) >= heads * vdim, "gla: out");
+  TORCH_CHECK(state.is_contiguous() && state.scalar_type() == at::kFloat && state.dim() == 4 && state.size(1) == heads &&
+                  state.size(2) == vdim && state.size(3) == p.dim_pad, "gla: state [slots, heads, vdim, dim_pad]");
+  p.state = state.data_ptr<float>();
+  p.state_idx = i32(state_idx, p.B, "state_idx"); p.q_start = i32(q_start, p.B, "q_start");
+  p.q_len = i32(q_len, p.B, "q_len"); p.kv_len = i32(kv_len, p.B, "kv_len");
+  check_rc(mb_gla(&p, dtype_of(x, "x"), num_sms(), cur_stream()), "gla");
 }
 
 // the cache [pages, 2, planes, kv heads, page, head width] at one plane
@@ -241,7 +340,8 @@ struct CacheView {
 
 // x: projection rows; queries at column 0 .., see MbBlockPrep
 void block_prep(Tensor& x, int q_off, int heads, int k_off, int v_off, int kv_heads, int dims, const Tensor& positions,
-                const Opt& cos_sin, const Tensor& slots, Tensor& kv, int plane, int silu_off, int silu_n, int relu2_off, int relu2_n) {
+                const Opt& cos_sin, const Tensor& slots, Tensor& kv, int plane, int silu_off, int silu_n, int relu2_off, int relu2_n,
+                const Opt& q_norm, const Opt& k_norm, int norm_dim, double eps, bool halves) {
   MbBlockPrep p = {};
   p.x = x.data_ptr(); p.ldx = ld_of(x, x.scalar_type(), "x"); p.T = x.size(0);
   const CacheView c(kv, plane, kv_heads, "block_prep");
@@ -259,6 +359,13 @@ void block_prep(Tensor& x, int q_off, int heads, int k_off, int v_off, int kv_he
   p.positions = i32(positions, p.T, "positions"); p.slots = slots.data_ptr<int64_t>();
   p.k_cache = c.k; p.v_cache = c.v; p.page_size = c.page; p.page_stride = c.page_stride; p.head_stride = c.head_stride;
   p.silu_off = silu_off; p.silu_n = silu_n; p.relu2_off = relu2_off; p.relu2_n = relu2_n;
+  auto weight = [&](const Opt& t) -> const void* {
+    if (!given(t)) return nullptr;
+    TORCH_CHECK(t->is_cuda() && t->is_contiguous() && t->scalar_type() == x.scalar_type() && t->numel() >= c.hd, "block_prep: norm weight");
+    return t->data_ptr();
+  };
+  p.q_norm = weight(q_norm); p.k_norm = weight(k_norm); p.norm_dim = norm_dim > 0 ? norm_dim : c.hd; p.eps = static_cast<float>(eps);
+  p.halves = halves;
   check_rc(mb_block_prep(&p, dtype_of(x, "x"), cur_stream()), "block_prep");
 }
 
@@ -266,20 +373,20 @@ void block_prep(Tensor& x, int q_off, int heads, int k_off, int v_off, int kv_he
 // none of them given: the kernel on the CUDA cores.
 void window_attention(const Tensor& q, Tensor& out, const Tensor& kv, int plane, const Tensor& block_table, const Tensor& q_start,
                       const Tensor& q_len, const Tensor& kv_len, const Opt& tile_seq, const Opt& tile_q0, const Opt& decode_seq,
-                      int n_q, int n_kv, double scale, int window, const Opt& sink) {
+                      int n_q, int n_kv, double scale, int window, const Opt& sink, const Opt& gate, double gate_mult) {
   const CacheView c(kv, plane, n_kv, "window_attention");
   const int dt = dtype_of(q, "q"), ldq = ld_of(q, q.scalar_type(), "q"), ldo = ld_of(out, q.scalar_type(), "out");
   const int B = q_len.numel(), T = q.size(0);
   TORCH_CHECK(kv.scalar_type() == q.scalar_type() && q.size(1) >= static_cast<int64_t>(n_q) * c.hd && out.size(0) >= T &&
                   out.size(1) >= static_cast<int64_t>(n_q) * c.hd && block_table.scalar_type() == at::kInt &&
                   block_table.dim() == 2 && block_table.stride(1) == 1 && block_table.size(0) >= B, "window_attention layout");
-  const float* sk = given(sink) ? f32(*sink, n_q, "sink") : nullptr;
+  const AttnOptions opt(window, sink, gate, gate_mult, T, n_q, q.scalar_type(), "window_attention");
   const int32_t *qs = i32(q_start, B, "q_start"), *ql = i32(q_len, B, "q_len"), *kl = i32(kv_len, B, "kv_len");
   const int32_t* bt = block_table.data_ptr<int32_t>();
   const int bts = block_table.stride(0);
   if (!given(tile_seq) && !given(decode_seq)) {
     check_rc(mb_window_attention(q.data_ptr(), ldq, out.data_ptr(), ldo, c.k, c.v, c.page_stride, c.head_stride, c.page, bt, bts, qs,
-                                 ql, kl, T, B, n_q, n_kv, c.hd, static_cast<float>(scale), window, sk, dt, cur_stream()),
+                                 ql, kl, T, B, n_q, n_kv, c.hd, static_cast<float>(scale), opt.use, dt, cur_stream()),
              "window_attention");
     return;
   }
@@ -291,7 +398,7 @@ void window_attention(const Tensor& q, Tensor& out, const Tensor& kv, int plane,
                                      n_tiles ? i32(*tile_seq, n_tiles, "tile_seq") : nullptr,
                                      n_tiles ? i32(*tile_q0, n_tiles, "tile_q0") : nullptr, n_tiles, n_dec,
                                      n_dec ? i32(*decode_seq, n_dec, "decode_seq") : nullptr, n_q, n_kv, c.hd, c.page,
-                                     static_cast<float>(scale), window, sk, error_flag(), cur_stream()),
+                                     static_cast<float>(scale), opt.use, error_flag(), cur_stream()),
            "paged_attention_window");
 }
 
@@ -352,9 +459,16 @@ void mb::bind_layers(py::module_& m) {
   });
   m.def("latent_attention", &latent_attention, py::arg("q_lat"), py::arg("q_rope"), py::arg("cache"), py::arg("block_table"),
         py::arg("q_start"), py::arg("q_len"), py::arg("kv_len"), py::arg("out"), py::arg("scale"), py::arg("sink") = none,
-        py::arg("one_token") = false, py::arg("ws") = none, py::arg("allow_tc") = true);
-  m.def("block_prep", &block_prep);
-  m.def("window_attention", &window_attention);
+        py::arg("one_token") = false, py::arg("ws") = none, py::arg("allow_tc") = true, py::arg("window") = 0,
+        py::arg("gate") = none, py::arg("gate_mult") = 1.0);
+  m.def("block_prep", &block_prep, py::arg("x"), py::arg("q_off"), py::arg("heads"), py::arg("k_off"), py::arg("v_off"),
+        py::arg("kv_heads"), py::arg("dims"), py::arg("positions"), py::arg("cos_sin"), py::arg("slots"), py::arg("kv"), py::arg("plane"),
+        py::arg("silu_off") = 0, py::arg("silu_n") = 0, py::arg("relu2_off") = 0, py::arg("relu2_n") = 0, py::arg("q_norm") = none,
+        py::arg("k_norm") = none, py::arg("norm_dim") = 0, py::arg("eps") = 1e-6, py::arg("halves") = false);
+  m.def("window_attention", &window_attention, py::arg("q"), py::arg("out"), py::arg("kv"), py::arg("plane"), py::arg("block_table"),
+        py::arg("q_start"), py::arg("q_len"), py::arg("kv_len"), py::arg("tile_seq"), py::arg("tile_q0"), py::arg("decode_seq"),
+        py::arg("n_q"), py::arg("n_kv"), py::arg("scale"), py::arg("window") = 0, py::arg("sink") = none, py::arg("gate") = none,
+        py::arg("gate_mult") = 1.0);
   m.def("attention_plan", [](const Tensor& q_len, int tok_per_tile, Tensor& tile_seq, Tensor& tile_q0) {
     const int n = tile_seq.numel();
     check_rc(mb_attention_plan(i32(q_len, 1, "q_len"), q_len.numel(), tok_per_tile, n,
@@ -370,7 +484,45 @@ void mb::bind_layers(py::module_& m) {
                                dtype_of(o, "o"), cur_stream()), "lightning_norm");
   });
   m.def("delta_dim_pad", [](int dim) { return mb_delta_dim_pad(dim); });
-  m.def("delta_rule", &delta_rule);
+  m.def("delta_rule", &delta_rule, py::arg("x"), py::arg("q_off"), py::arg("k_off"), py::arg("v_off"), py::arg("b_off"), py::arg("conv_w"),
+        py::arg("z"), py::arg("A_log"), py::arg("dt_bias"), py::arg("gate"), py::arg("norm_w"), py::arg("eps"), py::arg("scratch"),
+        py::arg("out"), py::arg("state"), py::arg("conv_state"), py::arg("state_idx"), py::arg("q_start"), py::arg("q_len"),
+        py::arg("kv_len"), py::arg("heads"), py::arg("kv_heads"), py::arg("dim"), py::arg("vdim"), py::arg("one_token"),
+        py::arg("a_off") = -1, py::arg("gate_silu") = false, py::arg("out_mult") = 1.0);
+  m.def("gla", &gla);
+  m.def("sandwich_norm", &sandwich_norm);
+  m.def("bigram_rows", [](const Tensor& tokens, const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, const Tensor& state_idx,
+                          Tensor& last, Tensor& out, int64_t mul_prev, int64_t mul_cur, int64_t buckets) {
+    const int T = tokens.numel(), B = q_len.numel();
+    TORCH_CHECK(tokens.is_cuda() && tokens.is_contiguous() && tokens.scalar_type() == at::kLong && last.is_cuda() && last.is_contiguous() &&
+                    last.scalar_type() == at::kLong && out.is_cuda() && out.is_contiguous() && out.scalar_type() == at::kLong &&
+                    out.numel() >= T, "bigram_rows: int64 CUDA tensors");
+    check_rc(mb_bigram_rows(tokens.data_ptr<int64_t>(), i32(q_start, B, "q_start"), i32(q_len, B, "q_len"), i32(kv_len, B, "kv_len"),
+                            i32(state_idx, B, "state_idx"), last.data_ptr<int64_t>(), out.data_ptr<int64_t>(), T, B, mul_prev, mul_cur,
+                            buckets, cur_stream()), "bigram_rows");
+  });
+  m.def("moe_score_route", [](const Tensor& logits, const Opt& bias, Tensor& ids, Tensor& w, Tensor& rank, Tensor& counts, int n_group,
+                              int keep, bool norm_topk, double scaling) {
+    const int T = ids.size(0), k = ids.size(1), E = counts.numel(), ld = ld_of(logits, at::kFloat, "logits");
+    TORCH_CHECK(ids.dim() == 2 && logits.size(0) >= T && logits.size(1) >= E, "moe_score_route shapes");
+    check_rc(mb_moe_score_route(logits.data_ptr<float>(), ld, given(bias) ? f32(*bias, E, "bias") : nullptr,
+                                const_cast<int32_t*>(i32(ids, 0, "ids")), const_cast<float*>(f32(w, static_cast<int64_t>(T) * k, "w")),
+                                const_cast<int32_t*>(i32(rank, static_cast<int64_t>(T) * k, "rank")),
+                                const_cast<int32_t*>(i32(counts, E, "counts")), T, E, n_group, keep, k, norm_topk ? 1 : 0,
+                                static_cast<float>(scaling), cur_stream()), "moe_score_route");
+  });
+  m.def("moe_place_rows", [](const Tensor& x, const Tensor& ids, const Tensor& rank, const Tensor& counts, Tensor& offsets, Tensor& inverse,
+                             Tensor& dst) {
+    const int T = ids.size(0), k = ids.size(1), E = counts.numel(), es = x.element_size();
+    const int ld = ld_of(x, x.scalar_type(), "x");
+    TORCH_CHECK(dst.is_cuda() && dst.is_contiguous() && dst.dim() == 2 && dst.size(1) == x.size(1) && dst.scalar_type() == x.scalar_type() &&
+                    dst.size(0) >= static_cast<int64_t>(T) * k && x.size(0) >= T, "moe_place_rows shapes");
+    check_rc(mb_moe_place_rows(x.data_ptr(), static_cast<long long>(ld) * es, i32(ids, static_cast<int64_t>(T) * k, "ids"),
+                               i32(rank, static_cast<int64_t>(T) * k, "rank"), i32(counts, E, "counts"),
+                               const_cast<int32_t*>(i32(offsets, E + 1, "offsets")),
+                               const_cast<int32_t*>(i32(inverse, static_cast<int64_t>(T) * k, "inverse")), dst.data_ptr(), T, E, k,
+                               static_cast<int>(x.size(1)) * es, cur_stream()), "moe_place_rows");
+  });
   m.def("moe_table_route", [](const Tensor& ids, const Tensor& tables, const Tensor& desc, int max_experts, Tensor& inverse,
                               Tensor& offsets) {
     TORCH_CHECK(ids.is_cuda() && ids.is_contiguous() && ids.scalar_type() == at::kLong && desc.is_cuda() && desc.is_contiguous() &&

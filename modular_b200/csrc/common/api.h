@@ -105,10 +105,17 @@ int mb_silu_mul_quant_fp8(const void* gate_up, void* q_fp8, float* scales, int M
 void mb_set_mla_split_workspace(void* ws, size_t ws_bytes, int* counters, int n_counters);
 void mb_set_mla_split(int mode);
 size_t mb_mla_split_workspace_bytes(int num_sms);
+// What attention variants add to causal softmax attention; a null pointer instead of the struct means none of it.
+typedef struct {
+  int window;                          // keys a query sees, itself included (0: all before it)
+  const float* sink;                   // per query head: a score without key or value in the softmax denominator (null: none)
+  const void* gate; int ld_gate;       // outputs of head h of token t are multiplied by gate_mult * sigmoid(gate[t, h]);
+  float gate_mult;                     // same element type as the queries (null: no gate)
+} MbAttnOptions;
 int mb_mla_prefill_tc(const void* q_lat, const void* q_rope, void* out, const void* cache, long long page_stride,
                       long long n_pages, const int32_t* block_table, int bt_stride, const int32_t* q_start,
                       const int32_t* q_len, const int32_t* kv_len, int T, int B, int n_heads, int page_size, float scale,
-                      const float* sink, int ld_rope, int32_t* tok_scratch, int* err, cudaStream_t stream);
+                      const MbAttnOptions* opt, int ld_rope, int32_t* tok_scratch, int* err, cudaStream_t stream);
 int mb_mla_post_down(const void* qkv_a, int ld, int q_lora, int R, const void* gamma_q, const void* gamma_kv, float eps,
                      const int32_t* positions, const float* cos_sin, const int64_t* slots, void* q_a_out, void* cache,
                      int T, int page_size, long long page_stride, cudaStream_t stream);
@@ -175,7 +182,7 @@ int mb_paged_attention_window(const void* q, int ldq, void* out, int ldo, const 
                               int bt_stride, const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
                               const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, int n_decode,
                               const int32_t* decode_seq, int n_q, int n_kv, int head_dim, int page_size, float scale,
-                              int window, const float* sink, int* err, cudaStream_t stream);
+                              const MbAttnOptions* opt, int* err, cudaStream_t stream);
 
 // Split-KV decode (attention_tma.cu): decode-only steps cut the KV tiles of all sequences into equal shares per
 // CTA once this process-wide workspace is set (partials + zeroed counters, one per KV head and sequence).
@@ -189,8 +196,8 @@ int mb_paged_attention_prefill_tc(const void* q, int ldq, void* out, int ldo, co
                                   long long page_rows, const int32_t* block_table, int bt_stride,
                                   const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
                                   const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, int n_q,
-                                  int n_kv, int head_dim, int page_size, float scale, int window,
-                                  const float* sink, int* err, cudaStream_t stream);
+                                  int n_kv, int head_dim, int page_size, float scale,
+                                  const MbAttnOptions* opt, int* err, cudaStream_t stream);
 // Route the prefill tiles of mb_paged_attention_tma through the tcgen05 kernel when a step has at least
 // `min_tiles` 64-row tiles (process-wide; 0 = never).
 void mb_set_attn_tc(int min_tiles);
@@ -203,12 +210,12 @@ int mb_mla_tc_usable(int T, int B, int n_heads, int R, int page_size);
 int mb_mla_decode_tc(const void* q_lat, const void* q_rope, void* out, const void* cache, long long page_stride,
                      long long n_pages, const int32_t* block_table, int bt_stride, const int32_t* q_start,
                      const int32_t* q_len, const int32_t* kv_len, int T, int B, int n_heads, int page_size,
-                     float scale, const float* sink, int ld_rope, int* err, cudaStream_t stream);
-// any latent width of {64, 128, 192, 256, 384, 512}, row strides, an optional softmax sink per head and a KV split
+                     float scale, const MbAttnOptions* opt, int ld_rope, int* err, cudaStream_t stream);
+// any latent width of {64, 128, 192, 256, 384, 512}, row strides, the options of MbAttnOptions and a KV split
 int mb_mla_paged_attention_ex(const void* q_lat, long long ld_ql, const void* q_rope, long long ld_qr, int hs_qr, void* out,
                               const void* cache, long long page_stride, int ld_cache, const int32_t* block_table,
                               int bt_stride, const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len, int T,
-                              int B, int n_heads, int R, int page_size, float scale, const float* sink, void* ws,
+                              int B, int n_heads, int R, int page_size, float scale, const MbAttnOptions* opt, void* ws,
                               size_t ws_bytes, int num_sms, cudaStream_t stream);
 int mb_mla_paged_attention(const void* q_lat, const void* q_rope, void* out, const void* cache,
                            long long page_stride, const int32_t* block_table, int bt_stride,
@@ -227,8 +234,8 @@ int mb_rotate_heads(void* x, int ld, int T, int heads, int head_stride, int dims
 int mb_latent_attention(const void* q_lat, int ld_ql, int hs_ql, const void* q_rope, int ld_qr, int hs_qr, void* out,
                         int ld_out, int hs_out, const void* cache, long long page_stride, int ld_cache, int page_size,
                         const int32_t* block_table, int bt_stride, const int32_t* q_start, const int32_t* q_len,
-                        const int32_t* kv_len, int T, int B, int n_heads, int Rp, int Dp, float scale, const float* sink,
-                        int dtype, cudaStream_t stream);
+                        const int32_t* kv_len, int T, int B, int n_heads, int Rp, int Dp, float scale,
+                        const MbAttnOptions* opt, int dtype, cudaStream_t stream);
 
 // ---- seams of an fp32 residual stream (residual_norm.cu); null pointers switch parts off -----
 typedef struct {
@@ -249,18 +256,42 @@ typedef struct {
   const void* step;                                                      // x += step, one row for every token
 } MbResidualNorm;
 int mb_residual_norm(const MbResidualNorm* p, int dtype, cudaStream_t stream);
+// Seam of layers that norm every branch before and after it; one branch at a time, null pointers switch parts off:
+//   x  = table[ids] * scale (or x);   x += inject[inject_ids];   u = a, or sum_k pair_w[., k] e[inverse[., k]]
+//   x += mult * norm(u; w_u, b_u) (or mult * u);   n1 = norm(x; w1, b1)
+// norm: layer norm with weight and bias, or an RMS norm where the biases are null.
+typedef struct {
+  float* x; int ldx;
+  const int64_t* ids; const void* table; float scale; int vocab, ld_table;
+  const int64_t* inject_ids; const void* inject; int inject_rows, ld_inject;
+  const void* a; int lda;
+  const void* e; int lde; const int32_t* inverse; const float* pair_w; int top_k;
+  const int32_t* rows;
+  const void *w_u, *b_u; float mult;
+  const void *w1, *b1; void* n1; int ld1;
+  int n_rows, cols, cols_pad, store_x;
+  float eps;
+} MbSandwichNorm;
+int mb_sandwich_norm(const MbSandwichNorm* p, int dtype, cudaStream_t stream);
+// Rows of a bigram table: (previous token * mul_prev + token * mul_cur) mod buckets, `buckets` for a sequence's first token.
+// The token before a step comes from `last` [slots] where the step continues a sequence; the step's last token goes there.
+int mb_bigram_rows(const int64_t* tokens, const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
+                   const int32_t* state_idx, int64_t* last, int64_t* out, int T, int B, long long mul_prev, long long mul_cur,
+                   long long buckets, cudaStream_t stream);
 int mb_gelu_tanh(void* x, long long n, int dtype, cudaStream_t stream);
 // x[i] = cap * tanh(x[i] / cap) over fp32 logits
 int mb_softcap(float* x, long long n, float cap, cudaStream_t stream);
 int mb_sigmoid_gate(void* o, int ldo, const void* g, int ldg, int rows, int cols, int dtype, cudaStream_t stream);
 
-// ---- gated delta rule with per-channel decay (delta_rule.cu) ---------------------------------
+// ---- gated delta rule with a decay per channel or per head (delta_rule.cu) ---------------------------------
 typedef struct {
   const void* x; int ldx, q_off, k_off, v_off, b_off;    // projection rows [T, ldx]: column blocks of q, k, v, beta
   const void* conv_w; int taps;                          // [q | k | v channels, taps]
-  const float* z; int ldz;                               // decay projection [T, heads * dim]
-  const float *A_log, *dt_bias;                          // [heads], [heads * dim]
+  const float* z; int ldz;                               // decay projection [T, heads * dim] (null: one decay per head)
+  int a_off;                                             // z null: column of the decay projection in x, one per head
+  const float *A_log, *dt_bias;                          // [heads], [heads * dim] or [heads]
   const void* gate; int ld_gate;                         // output gate projection [T, heads * vdim]
+  int gate_silu; float out_mult;                         // output: norm(o) * out_mult * (sigmoid or silu)(gate)
   const void* norm_w; float eps;                         // [vdim]
   float *q, *k, *g, *v, *beta, *kq, *o;                  // fp32 scratch (q, k, g rows are dim_pad wide)
   void* out; int ld_out;                                 // [T, heads * vdim]
@@ -271,6 +302,15 @@ typedef struct {
 } MbDelta;
 int mb_delta_dim_pad(int dim);
 int mb_delta_rule(const MbDelta* p, int dtype, int num_sms, cudaStream_t stream);
+// out[t, h * vdim ..] = rms_norm(o[t, h]) * w * mult * (sigmoid or silu)(gate[t, h * vdim ..]); o fp32 [T, heads, vdim]; the
+// norm divides by n <= vdim (columns beyond n hold zeros)
+typedef struct {
+  const float* o; void* out; int ld_out;
+  const void* gate; int ld_gate; const void* norm_w;
+  int T, heads, vdim, n, gate_silu;
+  float eps, mult;
+} MbHeadOut;
+int mb_head_norm_gate(const MbHeadOut* p, int dtype, cudaStream_t stream);
 
 // ---- sliding-window attention of any size, and what surrounds it (attention_window.cu) -------
 typedef struct {
@@ -280,6 +320,9 @@ typedef struct {
   const int64_t* slots;                                  // cache slot per token (negative: not stored)
   void *k_cache, *v_cache; int page_size; long long page_stride, head_stride;
   int silu_off, silu_n, relu2_off, relu2_n;              // columns that become silu(x), relu(x)^2 (0: none)
+  // RMS norm of every query / key head over its first norm_dim columns (the rest are zeros), before the rotation; null: none
+  const void *q_norm, *k_norm; int norm_dim; float eps;  // weights [hd]
+  int halves;                                            // pairs (i, i + dims / 2) instead of neighbours
 } MbBlockPrep;
 int mb_block_prep(const MbBlockPrep* p, int dtype, cudaStream_t stream);
 int mb_attention_plan(const int32_t* q_len, int B, int tok_per_tile, int n_tiles, int32_t* tile_seq, int32_t* tile_q0,
@@ -287,7 +330,7 @@ int mb_attention_plan(const int32_t* q_len, int B, int tok_per_tile, int n_tiles
 int mb_window_attention(const void* q, int ldq, void* out, int ldo, const void* k_cache, const void* v_cache,
                         long long page_stride, long long head_stride, int page_size, const int32_t* block_table, int bt_stride,
                         const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len, int T, int B, int n_q, int n_kv,
-                        int hd, float scale, int window, const float* sink, int dtype, cudaStream_t stream);
+                        int hd, float scale, const MbAttnOptions* opt, int dtype, cudaStream_t stream);
 
 // ---- lightning attention: a constant decay per head (lightning.cu) ---------------------------
 typedef struct {
@@ -302,6 +345,20 @@ typedef struct {
 int mb_lightning(const MbLightning* p, int dtype, int num_sms, cudaStream_t stream);
 int mb_lightning_norm(void* o, int ldo, const void* gate, int ldg, const void* w, int T, int cols, int n, float eps, int dtype,
                       cudaStream_t stream);
+
+// ---- gated linear attention: a decay per key channel (gla.cu) ---------------------------------
+typedef struct {
+  const void* x; int ldx, q_off, k_off, v_off;           // projection rows; heads of dim / vdim columns (multiples of 8)
+  const float* z; int ldz; const float* z_bias;          // decay projection [T, heads * dim], its bias; decay = sigmoid(z + bias)^(1 / tau)
+  float q_scale, inv_tau;
+  const void* gate; int ld_gate, gate_silu; float out_mult; const void* norm_w; float eps; int norm_dim;   // as in MbHeadOut
+  float* o;                                              // fp32 scratch [T, heads, vdim]
+  void* out; int ld_out;                                 // [T, heads * vdim]
+  float* state;                                          // [slots, heads, vdim, dim_pad]
+  const int32_t *state_idx, *q_start, *q_len, *kv_len;
+  int T, B, heads, dim, dim_pad, vdim, one_token;
+} MbGla;
+int mb_gla(const MbGla* p, int dtype, int num_sms, cudaStream_t stream);
 
 // ---- fp32 products (gemm_simt.cu) ------------------------------------------------------------
 int mb_gemm_f32(const float* x, const float* w, float* y, const float* r, int M, int N, int K, int ldx, int ldw, int ldy,
@@ -318,6 +375,13 @@ int mb_moe_table_route(const int64_t* ids, int T, const int32_t* tables, const i
 int mb_moe_router_group_limited(const float* logits, const float* bias, int32_t* topk_ids, float* topk_w,
                                 int T, int E, int n_group, int topk_group, int top_k, int norm_topk,
                                 float scaling, int ld, cudaStream_t stream);
+// The same choice with one warp per token, and the first half of the sort by expert: rank[t, k] is the pair's place among its
+// expert's pairs, counts [E] (zero on entry) their number. mb_moe_place_rows does the rest: offsets [E + 1], inverse [T, top_k]
+// and the token rows copied into expert order.
+int mb_moe_score_route(const float* logits, int ld, const float* bias, int32_t* ids, float* w, int32_t* rank, int32_t* counts, int T,
+                       int E, int n_group, int keep, int top_k, int norm_topk, float scaling, cudaStream_t stream);
+int mb_moe_place_rows(const void* x, long long ldx_bytes, const int32_t* ids, const int32_t* rank, const int32_t* counts,
+                      int32_t* offsets, int32_t* inverse, void* dst, int T, int E, int top_k, int row_bytes, cudaStream_t stream);
 int mb_moe_router_softmax_topk(const float* logits, int32_t* topk_ids, float* topk_w, int T, int E,
                                int top_k, int norm_topk, int ld, cudaStream_t stream);
 int mb_moe_create_indices(const int32_t* topk_ids, int n_pairs, int e_begin, int e_end, int32_t* counts,

@@ -34,6 +34,7 @@
 #include <stdint.h>
 
 #include "../common/api.h"
+#include "../common/head_gate.cuh"
 #include "../common/launch.h"
 #include "../common/ptx.cuh"
 #include "gemm_common.h"
@@ -66,6 +67,7 @@ struct Params {
   float scale_log2;
   int window;            // keys a query sees (0x7fffffff: all before it)
   const float* sink;     // per query head, or null
+  HeadGate gate;
 };
 
 struct Bars {
@@ -352,8 +354,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
         l = l * wa + lb * wb + exp2f(sink2 - mm);
       }
       const float inv = l > 0.f ? 1.f / l : 0.f;
-      wa *= inv;
-      wb *= inv;
+      const float inv_g = tq < ql ? inv * p.gate(qs + tq, head) : inv;
+      wa *= inv_g;
+      wb *= inv_g;
       bf16* orow = p.out + static_cast<int64_t>(qs + (tq < ql ? tq : 0)) * p.ldo + head * HD;
 #pragma unroll
       for (int q4 = 0; q4 < 4; ++q4) {
@@ -398,15 +401,14 @@ using namespace mb;
 // Prefill tiles of a ragged batch on the tcgen05 kernel. Same KV addressing as mb_paged_attention_tma
 // (kv_base viewed as [total_rows, 128]); head_dim 128, G = n_q / n_kv in {1, 2, 4, 8, 16}, page_size % 64 == 0.
 // tile_seq / tile_q0 is the plan of 64-row tiles (CTAs take pairs of them) or of 128-row tiles; a negative sequence is
-// an unused tile. window: keys a query sees, itself included (0: all); sink: a score per query head that only takes part
-// in the softmax denominator (null: none).
+// an unused tile.
 extern "C" int mb_paged_attention_prefill_tc(const void* q, int ldq, void* out, int ldo, const void* kv_base,
                                              long long total_rows, long long k_off_rows, long long v_off_rows,
                                              long long page_rows, const int32_t* block_table, int bt_stride,
                                              const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
                                              const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, int n_q,
-                                             int n_kv, int head_dim, int page_size, float scale, int window,
-                                             const float* sink, int* err, cudaStream_t stream) {
+                                             int n_kv, int head_dim, int page_size, float scale,
+                                             const MbAttnOptions* opt, int* err, cudaStream_t stream) {
   using namespace mb::atc;
   if (n_tiles <= 0) return MB_OK;
   if (head_dim != 128 || n_kv <= 0 || n_q % n_kv || page_size % 64 || total_rows >= (1ll << 31)) return MB_ERR_SHAPE;
@@ -423,8 +425,9 @@ extern "C" int mb_paged_attention_prefill_tc(const void* q, int ldq, void* out, 
   p.k_off_rows = k_off_rows; p.v_off_rows = v_off_rows; p.page_rows = page_rows;
   p.ldq = ldq; p.ldo = ldo; p.bt_stride = bt_stride; p.page_size = page_size; p.n_tiles = n_tiles; p.G = G;
   p.scale_log2 = scale * 1.4426950408889634f;
-  p.window = window > 0 ? window : 0x7fffffff;
-  p.sink = sink;
+  p.window = opt && opt->window > 0 ? opt->window : 0x7fffffff;
+  p.sink = opt ? opt->sink : nullptr;
+  p.gate = HeadGate(opt);
   CUtensorMap tm;
   const int rc = cached_tmap(&tm, kv_base, static_cast<uint64_t>(total_rows), head_dim, head_dim, 64, 2);
   if (rc != MB_OK) return rc;
@@ -436,8 +439,8 @@ extern "C" int mb_paged_attention_prefill_tc(const void* q, int ldq, void* out, 
       return MB_ERR_LAUNCH;
     configured.done();
   }
-  // windows and sinks belong to families whose layer kernels are ordinary launches
-  return launch_either(window <= 0 && sink == nullptr, attn_tc_kernel, dim3(n_tiles, n_kv), dim3(kThreads), smem, stream, tm, p) == cudaSuccess
+  // these options belong to families whose layer kernels are ordinary launches
+  return launch_either(opt == nullptr, attn_tc_kernel, dim3(n_tiles, n_kv), dim3(kThreads), smem, stream, tm, p) == cudaSuccess
              ? MB_OK
              : MB_ERR_LAUNCH;
 }

@@ -26,6 +26,7 @@
 #include <stdint.h>
 
 #include "../common/api.h"
+#include "../common/head_gate.cuh"
 #include "../common/launch.h"
 #include "../common/ptx.cuh"
 #include "gemm_common.h"
@@ -55,6 +56,7 @@ struct Params {
   int q_rows_alloc;      // rows of shared memory reserved for Q (64, or 16 in a decode-only launch)
   int window;            // keys a query sees (0x7fffffff: all before it)
   const float* sink;     // per query head, or null
+  HeadGate gate;
   bool dependent;        // programmatic dependent launch
 };
 
@@ -323,8 +325,8 @@ attn_tma_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
       const int tq = tq0 + r / G, head = kvh * G + r % G;
       float f;
       const float den = add_sink(p, head, m[h], l[h], f);
-      const float inv = den > 0.f ? f / den : 0.f;
       if (tq < ql) {
+        const float inv = den > 0.f ? f / den * p.gate(qs + tq, head) : 0.f;
         bf16* orow = p.out + static_cast<int64_t>(qs + tq) * p.ldo + head * HD + 2 * (lane & 3);
 #pragma unroll
         for (int dt = 0; dt < DT; ++dt)
@@ -367,7 +369,7 @@ attn_tma_kernel(const __grid_constant__ CUtensorMap tmKV, const Params p) {
       }
       float f;
       const float den = add_sink(p, head, mm, L, f);
-      const float inv = den > 0.f ? f / den : 0.f;
+      const float inv = den > 0.f ? f / den * p.gate(qs + tq, head) : 0.f;
       bf16* orow = p.out + static_cast<int64_t>(qs + tq) * p.ldo + head * HD;
       constexpr int PER = HD / 8;
       const int d0 = (tid & 7) * PER;
@@ -698,8 +700,8 @@ attn_decode_split_kernel(const __grid_constant__ CUtensorMap tmKV, const Params 
         const int tq = r / G, head = kvh * G + r % G;
         float f;
         const float den = add_sink(p, head, m[h], l[h], f);
-        const float inv = den > 0.f ? f / den : 0.f;
         if (tq < ql) {
+          const float inv = den > 0.f ? f / den * p.gate(qs + tq, head) : 0.f;
           bf16* orow = p.out + static_cast<int64_t>(qs + tq) * p.ldo + head * HD + 2 * (lane & 3);
 #pragma unroll
           for (int dt = 0; dt < DT; ++dt)
@@ -815,7 +817,7 @@ static int attention_tma(const void* q, int ldq, void* out, int ldo, const void*
                          int bt_stride, const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
                          const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, int n_decode,
                          const int32_t* decode_seq, int n_q, int n_kv, int head_dim, int page_size, float scale,
-                         int window, const float* sink, int* err, cudaStream_t stream) {
+                         const MbAttnOptions* opt, int* err, cudaStream_t stream) {
   using namespace mb::at2;
   if (n_tiles <= 0 && n_decode <= 0) return MB_OK;
   if (n_kv <= 0 || n_q % n_kv || page_size % 64 || total_rows >= (1ll << 31)) return MB_ERR_SHAPE;
@@ -831,9 +833,10 @@ static int attention_tma(const void* q, int ldq, void* out, int ldo, const void*
   p.n_tiles = n_tiles < 0 ? 0 : n_tiles;
   p.k_off_rows = k_off_rows; p.v_off_rows = v_off_rows; p.page_rows = page_rows;
   p.scale_log2 = scale * 1.4426950408889634f;
-  p.window = window > 0 ? window : 0x7fffffff;
-  p.sink = sink;
-  p.dependent = window <= 0 && sink == nullptr;
+  p.window = opt && opt->window > 0 ? opt->window : 0x7fffffff;
+  p.sink = opt ? opt->sink : nullptr;
+  p.gate = HeadGate(opt);
+  p.dependent = opt == nullptr;
   CUtensorMap tm;
   const int rc = cached_tmap(&tm, kv_base, static_cast<uint64_t>(total_rows), head_dim, head_dim, 64, 2);
   if (rc != MB_OK) return rc;
@@ -867,7 +870,7 @@ static int attention_tma(const void* q, int ldq, void* out, int ldo, const void*
     }
     const int rc2 = mb_paged_attention_prefill_tc(q, ldq, out, ldo, kv_base, total_rows, k_off_rows, v_off_rows,
                                                   page_rows, block_table, bt_stride, q_start, q_len, kv_len, tile_seq,
-                                                  tile_q0, p.n_tiles, n_q, n_kv, head_dim, page_size, scale, window, sink, err,
+                                                  tile_q0, p.n_tiles, n_q, n_kv, head_dim, page_size, scale, opt, err,
                                                   stream);
     if (rc2 != MB_OK && !forked) return rc2;
     if (n_decode <= 0) return rc2;
@@ -932,11 +935,10 @@ extern "C" int mb_paged_attention_tma(const void* q, int ldq, void* out, int ldo
                                       int page_size, float scale, int* err, cudaStream_t stream) {
   return attention_tma(q, ldq, out, ldo, kv_base, total_rows, k_off_rows, v_off_rows, page_rows, block_table, bt_stride,
                        q_start, q_len, kv_len, tile_seq, tile_q0, n_tiles, n_decode, decode_seq, n_q, n_kv, head_dim,
-                       page_size, scale, 0, nullptr, err, stream);
+                       page_size, scale, nullptr, err, stream);
 }
 
-// The same attention with a sliding window (keys a query sees, itself included; 0: all) and a sink score per query head
-// (null: none). A step is either a decode step (n_tiles 0: one row per entry of decode_seq) or prompt tiles: 128-row
+// The same attention with a sliding window, a sink score per query head and an output gate. A step is either a decode step (n_tiles 0: one row per entry of decode_seq) or prompt tiles: 128-row
 // tiles (128 / G tokens each) with head_dim 128, on the tcgen05 kernel; 64-row tiles with head_dim 64.
 extern "C" int mb_paged_attention_window(const void* q, int ldq, void* out, int ldo, const void* kv_base,
                                          long long total_rows, long long k_off_rows, long long v_off_rows,
@@ -944,15 +946,15 @@ extern "C" int mb_paged_attention_window(const void* q, int ldq, void* out, int 
                                          const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
                                          const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, int n_decode,
                                          const int32_t* decode_seq, int n_q, int n_kv, int head_dim, int page_size,
-                                         float scale, int window, const float* sink, int* err, cudaStream_t stream) {
+                                         float scale, const MbAttnOptions* opt, int* err, cudaStream_t stream) {
   if (n_tiles > 0 && n_decode > 0) return MB_ERR_SHAPE;
   if (n_tiles > 0 && head_dim == 128)
     return mb_paged_attention_prefill_tc(q, ldq, out, ldo, kv_base, total_rows, k_off_rows, v_off_rows, page_rows,
                                          block_table, bt_stride, q_start, q_len, kv_len, tile_seq, tile_q0, n_tiles, n_q,
-                                         n_kv, head_dim, page_size, scale, window, sink, err, stream);
+                                         n_kv, head_dim, page_size, scale, opt, err, stream);
   if (n_tiles > 0 && head_dim != 64) return MB_ERR_SHAPE;
   // head_dim 64 never takes the 128-wide tcgen05 path inside
   return attention_tma(q, ldq, out, ldo, kv_base, total_rows, k_off_rows, v_off_rows, page_rows, block_table, bt_stride,
                        q_start, q_len, kv_len, tile_seq, tile_q0, n_tiles, n_decode, decode_seq, n_q, n_kv, head_dim,
-                       page_size, scale, window, sink, err, stream);
+                       page_size, scale, opt, err, stream);
 }

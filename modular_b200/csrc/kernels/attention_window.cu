@@ -4,7 +4,7 @@
 //
 //   mb_block_prep         everything between the stacked input projection of a parallel block and its branches, in one
 //                         launch: queries rotated in place, keys rotated and stored in the cache with the values, silu on
-//                         one column range and squared relu on another
+//                         one column range and squared relu on another; or, with per-head norms, norms and rotation
 //   mb_attention_plan     prompt tiles of a ragged step (sequence and first token of each), made on the device
 //   mb_window_attention   causal attention of any head width, window and group size, optional sink score per head
 //
@@ -12,6 +12,7 @@
 #include <cuda_runtime.h>
 
 #include "../common/api.h"
+#include "../common/head_gate.cuh"
 #include "../common/launch.h"
 #include "../common/scalar.cuh"
 
@@ -118,6 +119,56 @@ __global__ void __launch_bounds__(256) block_prep_kernel(const MbBlockPrep p) {
   }
 }
 
+// The same for heads that are normed first, or whose pairs lie half the rotated width apart: a warp owns a head of a token.
+template <typename T>
+__global__ void __launch_bounds__(256) head_prep_kernel(const MbBlockPrep p) {
+  extern __shared__ __align__(16) float rows[];            // one head per warp
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  int u = blockIdx.y * (blockDim.x >> 5) + warp;
+  if (u >= p.heads + 2 * p.kv_heads) return;
+  T* row = static_cast<T*>(p.x) + static_cast<size_t>(t) * p.ldx;
+  const bool is_q = u < p.heads, is_v = u >= p.heads + p.kv_heads;
+  T *src = row + (is_q ? p.q_off + u * p.hd : (is_v ? p.v_off + (u - p.heads - p.kv_heads) * p.hd : p.k_off + (u - p.heads) * p.hd)),
+    *dst = src;
+  if (!is_q) {
+    const int64_t slot = p.slots[t];
+    if (slot < 0) return;
+    const int h = is_v ? u - p.heads - p.kv_heads : u - p.heads;
+    dst = static_cast<T*>(is_v ? p.v_cache : p.k_cache) + (slot / p.page_size) * p.page_stride + h * p.head_stride +
+          static_cast<long long>(slot % p.page_size) * p.hd;
+  }
+  if (is_v) {
+    for (int c = lane * 4; c < p.hd; c += 128) st4(dst + c, ld4(src + c));
+    return;
+  }
+  float* s = rows + warp * p.hd;
+  float ss = 0.f;
+  for (int c = lane * 4; c < p.hd; c += 128) {
+    const float4 x = ld4(src + c);
+    ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
+    *reinterpret_cast<float4*>(s + c) = x;
+  }
+  const T* w = static_cast<const T*>(is_q ? p.q_norm : p.k_norm);
+  if (w != nullptr) {
+    const float inv = 1.f / sqrtf(warp_allsum(ss) / static_cast<float>(p.norm_dim) + p.eps);
+    for (int c = lane * 4; c < p.hd; c += 128) {           // the columns this lane wrote
+      const float4 x = *reinterpret_cast<const float4*>(s + c), g = ld4(w + c);
+      *reinterpret_cast<float4*>(s + c) = make_float4(x.x * inv * g.x, x.y * inv * g.y, x.z * inv * g.z, x.w * inv * g.w);
+    }
+  }
+  __syncwarp();
+  const float* cs = p.dims > 0 ? p.cos_sin + static_cast<size_t>(p.positions[t]) * p.dims : nullptr;
+  const int half = p.dims / 2;
+  auto turned = [&](int c) {
+    if (c >= p.dims) return s[c];
+    const bool second = p.halves ? c >= half : (c & 1);
+    const int pr = p.halves ? (second ? c - half : c) : c / 2;
+    const int iu = p.halves ? pr : 2 * pr, iv = p.halves ? pr + half : 2 * pr + 1;
+    return second ? s[iv] * cs[pr] + s[iu] * cs[half + pr] : s[iu] * cs[pr] - s[iv] * cs[half + pr];
+  };
+  for (int c = lane * 4; c < p.hd; c += 128) st4(dst + c, make_float4(turned(c), turned(c + 1), turned(c + 2), turned(c + 3)));
+}
+
 constexpr int kPlanSeqs = 4096;
 
 __global__ void __launch_bounds__(1024)
@@ -167,6 +218,7 @@ struct Attn {
   long long page_stride, head_stride;
   const int32_t *block_table, *q_start, *q_len, *kv_len;
   const float* sink;
+  HeadGate gate;
   float scale;
 };
 
@@ -219,7 +271,7 @@ attention_kernel(const Attn p, const T* __restrict__ q, const T* __restrict__ k_
   float den = p.sink ? expf(p.sink[head] - M) : 0.f, f[kWarps];
 #pragma unroll
   for (int i = 0; i < kWarps; ++i) { f[i] = expf(sml[i] - M); den = fmaf(sml[kWarps + i], f[i], den); }
-  const float inv = 1.f / den;
+  const float inv = p.gate.of<T>(t, head) / den;
   T* dst = out + static_cast<size_t>(t) * p.ldo + static_cast<size_t>(head) * p.hd;
   for (int c = tid; c < p.hd; c += blockDim.x) {
     float v = 0.f;
@@ -257,6 +309,14 @@ extern "C" int mb_block_prep(const MbBlockPrep* p, int dtype, cudaStream_t strea
     return MB_ERR_SHAPE;
   if ((reinterpret_cast<uintptr_t>(p->x) | reinterpret_cast<uintptr_t>(p->k_cache) | reinterpret_cast<uintptr_t>(p->v_cache)) & 15)
     return MB_ERR_ALIGN;
+  if (p->q_norm || p->k_norm || p->halves) {
+    if (p->silu_n || p->relu2_n || p->norm_dim <= 0 || p->norm_dim > p->hd || p->hd > 1024) return MB_ERR_SHAPE;
+    const dim3 g(p->T, (p->heads + 2 * p->kv_heads + 7) / 8);
+    const size_t smem = static_cast<size_t>(8) * p->hd * sizeof(float);      // at most 32 KiB
+    const cudaError_t e = dtype == kF32 ? launch_plain(winattn::head_prep_kernel<float>, g, dim3(256), smem, stream, *p)
+                                        : launch_plain(winattn::head_prep_kernel<__nv_bfloat16>, g, dim3(256), smem, stream, *p);
+    return e == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
+  }
   const long long work = static_cast<long long>(p->heads) * ((p->dims + 7) / 8) + 2ll * p->kv_heads * (p->hd / 8) + p->silu_n / 8 +
                          p->relu2_n / 8;
   const long long blocks = (work + 255) / 256;
@@ -280,12 +340,12 @@ extern "C" int mb_attention_plan(const int32_t* q_len, int B, int tok_per_tile, 
 extern "C" int mb_window_attention(const void* q, int ldq, void* out, int ldo, const void* k_cache, const void* v_cache,
                                    long long page_stride, long long head_stride, int page_size, const int32_t* block_table,
                                    int bt_stride, const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len, int T, int B,
-                                   int n_q, int n_kv, int hd, float scale, int window, const float* sink, int dtype,
+                                   int n_q, int n_kv, int hd, float scale, const MbAttnOptions* opt, int dtype,
                                    cudaStream_t stream) {
   if (T <= 0 || B <= 0) return MB_OK;
   if (n_kv <= 0 || n_q % n_kv || n_q > 65535 || hd <= 0) return MB_ERR_SHAPE;
-  winattn::Attn p = {ldq, ldo, B, bt_stride, page_size, hd, n_q / n_kv, window > 0 ? window : 0x7fffffff, page_stride, head_stride,
-                     block_table, q_start, q_len, kv_len, sink, scale};
+  winattn::Attn p = {ldq, ldo, B, bt_stride, page_size, hd, n_q / n_kv, opt && opt->window > 0 ? opt->window : 0x7fffffff, page_stride, head_stride,
+                     block_table, q_start, q_len, kv_len, opt ? opt->sink : nullptr, HeadGate(opt), scale};
   return dtype == kF32 ? winattn::dispatch<float>(p, q, k_cache, v_cache, out, T, n_q, stream)
                        : winattn::dispatch<__nv_bfloat16>(p, q, k_cache, v_cache, out, T, n_q, stream);
 }

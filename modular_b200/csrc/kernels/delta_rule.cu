@@ -1,4 +1,5 @@
-// Gated delta rule with a decay per key channel, for ragged batches. Per head, with a state S [dim, vdim] in fp32:
+// Gated delta rule with a decay per key channel or per head, for ragged batches. Per head, with a state S [dim, vdim] in
+// fp32:
 //   S <- diag(g) S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
 // q, k and v pass a short causal convolution and silu first, q and k are unit vectors per head, and o is RMS-normed over
 // vdim, scaled by a weight and gated.
@@ -14,7 +15,7 @@
 //                       [slot, head, column, row]; sequences of one token are a decode step, for which one CTA owns a
 //                       whole head and also applies the output norm and gate. The convolution state is advanced at the
 //                       end of this kernel, after every read of it by the first one.
-//   delta_out_kernel    output norm and gate for longer sequences, one warp per (token, head)
+//   head_out_kernel     output norm and gate for longer sequences, one warp per (token, head)
 //
 // A chunked formulation on the tensor cores would round what enters the recurrence to 16 bits; this one keeps it in fp32.
 #include <cuda_runtime.h>
@@ -72,14 +73,27 @@ __device__ __forceinline__ float conv_act(float z) {
 
 __device__ __forceinline__ float softplusf(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
+// factor of the output gate
+__device__ __forceinline__ float gate_of(float z, int silu, float mult) { return mult * (silu ? siluf(z) : sigmoidf(z)); }
+
+// units of the preparation that make decays and step sizes: one per head, or 32 heads together with one decay per head
+__device__ __host__ __forceinline__ int decay_units(const MbDelta& p) { return p.z ? p.heads : (p.heads + 31) / 32; }
+template <typename T>
+__device__ __forceinline__ void head_decay(const MbDelta& p, const T* row, int t, int h) {
+  if (h >= p.heads) return;
+  const size_t i = static_cast<size_t>(t) * p.heads + h;
+  p.g[i] = expf(-expf(p.A_log[h]) * softplusf(ldf(row + p.a_off + h) + p.dt_bias[h]));
+  p.beta[i] = sigmoidf(ldf(row + p.b_off + h));
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) delta_prep_kernel(const MbDelta p) {
   const int t = blockIdx.x, lane = threadIdx.x & 31;
   const int unit = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int KH = p.kv_heads, H = p.heads, D = p.dim, V = p.vdim, DP = p.dim_pad;
   const int qkC = KH * D, vC = H * V, C = 2 * qkC + vC, W = p.taps;
-  const int v_units = (vC + 127) / 128;
-  if (unit >= KH + H + v_units) return;
+  const int v_units = (vC + 127) / 128, G = decay_units(p);
+  if (unit >= KH + G + v_units) return;
   int s = t;
   if (!p.one_token) {
     int lo = 0, hi = p.B - 1;
@@ -125,7 +139,9 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const MbDelta p) {
       ko[c] = c < D ? ko[c] * ik : 0.f;
     }
     if (lane == 0) p.kq[static_cast<size_t>(t) * KH + unit] = kq * iq * ik;
-  } else if (unit < KH + H) {
+  } else if (unit < KH + G && !p.z) {
+    head_decay(p, row, t, (unit - KH) * 32 + lane);
+  } else if (unit < KH + G) {
     const int h = unit - KH;
     const float a = expf(p.A_log[h]);
     const float* z = p.z + static_cast<size_t>(t) * p.ldz + h * D;
@@ -133,7 +149,7 @@ __global__ void __launch_bounds__(256) delta_prep_kernel(const MbDelta p) {
     for (int c = lane; c < DP; c += 32) go[c] = c < D ? expf(-a * softplusf(z[c] + p.dt_bias[h * D + c])) : 0.f;
     if (lane == 0) p.beta[static_cast<size_t>(t) * H + h] = sigmoidf(ldf(row + p.b_off + h));
   } else {
-    const int c0 = (unit - KH - H) * 128;
+    const int c0 = (unit - KH - G) * 128;
     for (int c = c0 + lane; c < min(c0 + 128, vC); c += 32)
       p.v[static_cast<size_t>(t) * vC + c] = conv_silu(2 * qkC + c, p.v_off + c);
   }
@@ -189,7 +205,8 @@ __global__ void __launch_bounds__(256) delta_prep_fast_kernel(const MbDelta p, i
   const int unit = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int KH = p.kv_heads, H = p.heads, D = p.dim, V = p.vdim, DP = p.dim_pad;
   const int qkC = KH * D, vC = H * V, C = 2 * qkC + vC;
-  if (unit >= KH + H + (vC + 127) / 128) return;
+  const int G = decay_units(p);
+  if (unit >= KH + G + (vC + 127) / 128) return;
   const int tb = blockIdx.x * tile, te = min(tb + tile, p.T);
   int s = tb;
   if (!p.one_token) {
@@ -200,9 +217,9 @@ __global__ void __launch_bounds__(256) delta_prep_fast_kernel(const MbDelta p, i
     }
     s = lo;
   }
-  const bool is_qk = unit < KH, is_g = !is_qk && unit < KH + H;
+  const bool is_qk = unit < KH, is_g = !is_qk && unit < KH + G;
   const int c = lane * 4;
-  const int v0 = is_qk || is_g ? 0 : (unit - KH - H) * 128;
+  const int v0 = is_qk || is_g ? 0 : (unit - KH - G) * 128;
   const bool on = is_qk || is_g ? c < D : v0 + c < vC;
   const T* w = static_cast<const T*>(p.conv_w);
   const T* xq = static_cast<const T*>(p.x) + (is_qk ? p.q_off + unit * D + c : p.v_off + v0 + c);
@@ -211,9 +228,10 @@ __global__ void __launch_bounds__(256) delta_prep_fast_kernel(const MbDelta p, i
   ConvLane<W> ca, cb;
   if (on && !is_g) ca.taps(w + static_cast<size_t>(ch_a) * W);
   if (on && is_qk) cb.taps(w + static_cast<size_t>(ch_b) * W);
-  const float a_log = is_g ? expf(p.A_log[unit - KH]) : 0.f;
+  const bool chan_g = is_g && p.z;
+  const float a_log = chan_g ? expf(p.A_log[unit - KH]) : 0.f;
   float4 bias = make_float4(0.f, 0.f, 0.f, 0.f);
-  if (is_g && on) bias = *reinterpret_cast<const float4*>(p.dt_bias + (unit - KH) * D + c);
+  if (chan_g && on) bias = *reinterpret_cast<const float4*>(p.dt_bias + (unit - KH) * D + c);
   const float scale = 1.f / sqrtf(static_cast<float>(D));
   float4 fut_a = make_float4(0.f, 0.f, 0.f, 0.f), fut_b = fut_a;
   if (on && !is_g) fut_a = ld4(xq + static_cast<size_t>(tb) * p.ldx);
@@ -253,6 +271,8 @@ __global__ void __launch_bounds__(256) delta_prep_fast_kernel(const MbDelta p, i
         *reinterpret_cast<float4*>(p.k + o) = make_float4(k.x * ik, k.y * ik, k.z * ik, k.w * ik);
       }
       if (lane == 0) p.kq[static_cast<size_t>(t) * KH + unit] = kq * iq * ik;
+    } else if (is_g && !chan_g) {
+      head_decay(p, static_cast<const T*>(p.x) + row, t, (unit - KH) * 32 + lane);
     } else if (is_g) {
       const int h = unit - KH;
       float4 g = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -269,9 +289,9 @@ __global__ void __launch_bounds__(256) delta_prep_fast_kernel(const MbDelta p, i
   }
 }
 
-template <typename T, int RL4, int NC, int MAXT, bool FUSE>
+template <typename T, int RL4, int NC, int MAXT, bool FUSE, bool HEADG>
 __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int col_blocks, int chunk) {
-  constexpr int DP = 32 * RL4;
+  constexpr int DP = 32 * RL4, NP = HEADG ? 2 : 3, NS = HEADG ? 4 : 2;     // fp32 vectors and scalars per token
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[32];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -282,13 +302,13 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
   const int t0 = p.q_start[s], n = p.q_len[s], slot = p.state_idx[s];
   const bool resume = slot >= 0 && p.kv_len[s] > n;
   if (n > 0) {
-    const int row_floats = 3 * DP + cols;          // q | k | g | v columns, then beta and k . q per token
-    const int stage_floats = chunk * (row_floats + 2);
+    const int row_floats = NP * DP + cols;         // q | k | (g) | v columns, then beta, k . q (and g) per token
+    const int stage_floats = chunk * (row_floats + NS);
     float* so = sm + 2 * stage_floats;             // FUSE: outputs of one token
     auto fetch = [&](int c0, float* dst) {         // every thread walks the tokens of its piece of the row
       const int m = min(chunk, n - c0);
       const size_t t = static_cast<size_t>(t0 + c0);
-      for (int pc = tid; pc < 3 * DP / 4; pc += blockDim.x) {
+      for (int pc = tid; pc < NP * DP / 4; pc += blockDim.x) {
         const int which = pc / (DP / 4), c = (pc % (DP / 4)) * 4;
         const float* src = which == 0 ? p.q + (t * KH + kh) * DP : which == 1 ? p.k + (t * KH + kh) * DP : p.g + (t * H + h) * DP;
         src += c;
@@ -298,12 +318,14 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
       }
       if (tid < cols && cbase + tid < V) {
         const float* src = p.v + (t * H + h) * V + cbase + tid;
-        float* d = dst + 3 * DP + tid;
+        float* d = dst + NP * DP + tid;
         for (int j = 0; j < m; ++j, src += H * V, d += row_floats) cp_async4(d, src);
       }
       float* sc = dst + chunk * row_floats;
-      for (int i = tid; i < 2 * m; i += blockDim.x)
-        cp_async4(sc + i, (i & 1) ? p.kq + (t + (i >> 1)) * KH + kh : p.beta + (t + (i >> 1)) * H + h);
+      for (int i = tid; i < NS * m; i += blockDim.x) {
+        const int k = i % NS;
+        if (k < 3) cp_async4(sc + i, k == 1 ? p.kq + (t + i / NS) * KH + kh : (k == 0 ? p.beta : p.g) + (t + i / NS) * H + h);
+      }
       cp_async_commit();
     };
     fetch(0, sm);
@@ -333,7 +355,8 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
       for (int j = 0; j < m; ++j) {
         const float* rowp = buf + j * row_floats;
         u64x2 kr[RL4];
-        uint64_t a[NC][2], b[NC][2];
+        uint64_t a[NC][2], b[NC][2], gh = 0ull;
+        if (HEADG) gh = pack2(sc[NS * j + 2], sc[NS * j + 2]);
 #pragma unroll
         for (int c = 0; c < NC; ++c) a[c][0] = a[c][1] = b[c][0] = b[c][1] = 0ull;
 #pragma unroll
@@ -341,7 +364,7 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
           const int r = (i * 8 + rg) * 4;
           const u64x2 q4 = *reinterpret_cast<const u64x2*>(rowp + r);
           const u64x2 k4 = *reinterpret_cast<const u64x2*>(rowp + DP + r);
-          const u64x2 g4 = *reinterpret_cast<const u64x2*>(rowp + 2 * DP + r);
+          const u64x2 g4 = HEADG ? u64x2{gh, gh} : *reinterpret_cast<const u64x2*>(rowp + 2 * DP + r);
           kr[i] = k4;
 #pragma unroll
           for (int c = 0; c < NC; ++c) {
@@ -371,8 +394,8 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
           r = (b2 ? q1 : a1) + __shfl_xor_sync(0xffffffffu, b2 ? a1 : q1, 2);
           r += __shfl_xor_sync(0xffffffffu, r, 1);
         }
-        const float beta = sc[2 * j], kq = sc[2 * j + 1];
-        const float vv = rowp[3 * DP + my_col];
+        const float beta = sc[NS * j], kq = sc[NS * j + 1];
+        const float vv = rowp[NP * DP + my_col];
         const float u = beta * (vv - r);           // meaningful in the lanes that hold a key product
         float uc[NC], u_mine = 0.f;
 #pragma unroll
@@ -405,7 +428,7 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
           const float inv = 1.f / sqrtf(tot / static_cast<float>(V) + p.eps);
           const size_t t = static_cast<size_t>(t0 + c0 + j);
           for (int c = tid; c < V; c += blockDim.x) {
-            const float gate = sigmoidf(ldf(static_cast<const T*>(p.gate) + t * p.ld_gate + h * V + c));
+            const float gate = gate_of(ldf(static_cast<const T*>(p.gate) + t * p.ld_gate + h * V + c), p.gate_silu, p.out_mult);
             stf(static_cast<T*>(p.out) + t * p.ld_out + h * V + c, so[c] * inv * ldf(static_cast<const T*>(p.norm_w) + c) * gate);
           }
           __syncthreads();
@@ -441,48 +464,75 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
 }
 
 template <typename T>
-__global__ void __launch_bounds__(256) delta_out_kernel(const MbDelta p) {
+__global__ void __launch_bounds__(256) head_out_kernel(const MbHeadOut p) {
   const int V = p.vdim, lane = threadIdx.x & 31;
   const long long unit = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (unit >= static_cast<long long>(p.T) * p.heads) return;
   const size_t t = static_cast<size_t>(unit / p.heads);
   const int h = static_cast<int>(unit % p.heads);
   const float* o = p.o + unit * V;
+  const T *gate = static_cast<const T*>(p.gate) + t * p.ld_gate + h * V, *w = static_cast<const T*>(p.norm_w);
+  T* out = static_cast<T*>(p.out) + t * p.ld_out + h * V;
   float ss = 0.f;
-  for (int c = lane; c < V; c += 32) ss = fmaf(o[c], o[c], ss);
-  const float inv = 1.f / sqrtf(warp_allsum(ss) / static_cast<float>(V) + p.eps);
-  for (int c = lane; c < V; c += 32) {
-    const float gate = sigmoidf(ldf(static_cast<const T*>(p.gate) + t * p.ld_gate + h * V + c));
-    stf(static_cast<T*>(p.out) + t * p.ld_out + h * V + c, o[c] * inv * ldf(static_cast<const T*>(p.norm_w) + c) * gate);
+  if (V <= 256 && V % 4 == 0 && p.ld_gate % 4 == 0 && p.ld_out % 4 == 0 &&
+      ((reinterpret_cast<uintptr_t>(p.o) | reinterpret_cast<uintptr_t>(p.gate) | reinterpret_cast<uintptr_t>(p.norm_w) |
+        reinterpret_cast<uintptr_t>(p.out)) & 15) == 0) {     // the head stays in registers
+    float4 x[2], g[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int c = (lane + 32 * i) * 4;
+      x[i] = c < V ? *reinterpret_cast<const float4*>(o + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      g[i] = c < V ? ld4(gate + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
+    }
+    const float inv = 1.f / sqrtf(warp_allsum(ss) / static_cast<float>(p.n) + p.eps);
+    auto f = [&](float z) { return gate_of(z, p.gate_silu, p.mult) * inv; };
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int c = (lane + 32 * i) * 4;
+      if (c >= V) continue;
+      const float4 a = ld4(w + c);
+      st4(out + c, make_float4(x[i].x * a.x * f(g[i].x), x[i].y * a.y * f(g[i].y), x[i].z * a.z * f(g[i].z), x[i].w * a.w * f(g[i].w)));
+    }
+    return;
   }
+  for (int c = lane; c < V; c += 32) ss = fmaf(o[c], o[c], ss);
+  const float inv = 1.f / sqrtf(warp_allsum(ss) / static_cast<float>(p.n) + p.eps);
+  for (int c = lane; c < V; c += 32) stf(out + c, o[c] * inv * ldf(w + c) * gate_of(ldf(gate + c), p.gate_silu, p.mult));
 }
 
-template <typename T, int RL4, int NC>
+template <typename T>
+static int head_out(const MbHeadOut& p, cudaStream_t stream) {
+  const long long units = static_cast<long long>(p.T) * p.heads;
+  return launch_plain(head_out_kernel<T>, dim3(static_cast<unsigned>((units + 7) / 8)), dim3(256), 0, stream, p) == cudaSuccess
+             ? MB_OK : MB_ERR_LAUNCH;
+}
+
+template <typename T, int RL4, int NC, bool HEADG>
 static int scan_launch(const MbDelta& p, int warps, bool fuse, cudaStream_t stream) {
   constexpr int MAXT = RL4 <= 8 ? 512 : 256;
   const int cols = warps * 4 * NC, col_blocks = (p.vdim + cols - 1) / cols;
-  const int per_token = (3 * 32 * RL4 + cols + 2) * 4;
+  const int per_token = ((HEADG ? 2 : 3) * 32 * RL4 + cols + (HEADG ? 4 : 2)) * 4;
   // tokens per stage: even, so that the second stage stays 16-byte aligned (a one-token step has no second stage)
   int chunk = p.one_token ? 1 : 40 * 1024 / (2 * per_token);
   if (!p.one_token) chunk = chunk > 16 ? 16 : chunk < 2 ? 2 : chunk & ~1;
   const size_t smem = static_cast<size_t>(2) * chunk * per_token + (fuse ? cols * 4 : 0) + 16;
   const dim3 grid(p.heads * col_blocks, p.B);
   if (fuse)
-    return launch_plain(delta_scan_kernel<T, RL4, NC, MAXT, true>, grid, dim3(warps * 32), smem, stream, p, col_blocks, chunk) ==
+    return launch_plain(delta_scan_kernel<T, RL4, NC, MAXT, true, HEADG>, grid, dim3(warps * 32), smem, stream, p, col_blocks, chunk) ==
                    cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
-  if (launch_plain(delta_scan_kernel<T, RL4, NC, MAXT, false>, grid, dim3(warps * 32), smem, stream, p, col_blocks, chunk) !=
+  if (launch_plain(delta_scan_kernel<T, RL4, NC, MAXT, false, HEADG>, grid, dim3(warps * 32), smem, stream, p, col_blocks, chunk) !=
       cudaSuccess)
     return MB_ERR_LAUNCH;
-  const long long units = static_cast<long long>(p.T) * p.heads;
-  return launch_plain(delta_out_kernel<T>, dim3(static_cast<unsigned>((units + 7) / 8)), dim3(256), 0, stream, p) == cudaSuccess
-             ? MB_OK : MB_ERR_LAUNCH;
+  const MbHeadOut o = {p.o, p.out, p.ld_out, p.gate, p.ld_gate, p.norm_w, p.T, p.heads, p.vdim, p.vdim, p.gate_silu, p.eps, p.out_mult};
+  return head_out<T>(o, stream);
 }
 
-template <typename T, int RL4>
-static int scan(const MbDelta& p, int num_sms, cudaStream_t stream) {
+template <typename T, int RL4, bool HEADG>
+static int scan_by_width(const MbDelta& p, int num_sms, cudaStream_t stream) {
   constexpr int max_warps = (RL4 <= 8 ? 512 : 256) / 32;
   const int head_warps = (p.vdim + 7) / 8;
-  if (p.one_token && head_warps <= max_warps) return scan_launch<T, RL4, 2>(p, head_warps, true, stream);
+  if (p.one_token && head_warps <= max_warps) return scan_launch<T, RL4, 2, HEADG>(p, head_warps, true, stream);
   // longer sequences: four columns per lane where the registers allow it (the rows are read once for all of them), and
   // CTAs of up to four warps as long as the grid has one per SM
   auto fit = [&](int per_warp) {
@@ -492,18 +542,23 @@ static int scan(const MbDelta& p, int num_sms, cudaStream_t stream) {
     return w;
   };
   if constexpr (RL4 <= 4) {
-    if (p.vdim >= 16) return scan_launch<T, RL4, 4>(p, fit(16), false, stream);
+    if (p.vdim >= 16) return scan_launch<T, RL4, 4, HEADG>(p, fit(16), false, stream);
   }
-  return scan_launch<T, RL4, 2>(p, fit(8), false, stream);
+  return scan_launch<T, RL4, 2, HEADG>(p, fit(8), false, stream);
+}
+
+template <typename T, int RL4>
+static int scan(const MbDelta& p, int num_sms, cudaStream_t stream) {
+  return p.z ? scan_by_width<T, RL4, false>(p, num_sms, stream) : scan_by_width<T, RL4, true>(p, num_sms, stream);
 }
 
 template <typename T>
 static int run(const MbDelta& p, int num_sms, cudaStream_t stream) {
   const int vC = p.heads * p.vdim;
-  const int units = p.kv_heads + p.heads + (vC + 127) / 128;
+  const int units = p.kv_heads + decay_units(p) + (vC + 127) / 128;
   // vector loads: four channels per lane, every row and block start aligned to them
   const bool fast = p.dim <= 128 && p.dim % 4 == 0 && vC % 4 == 0 && p.taps >= 2 && p.taps <= 4 && p.ldx % 8 == 0 &&
-                    p.q_off % 8 == 0 && p.k_off % 8 == 0 && p.v_off % 8 == 0 && p.ldz % 4 == 0 &&
+                    p.q_off % 8 == 0 && p.k_off % 8 == 0 && p.v_off % 8 == 0 && (!p.z || p.ldz % 4 == 0) &&
                     ((reinterpret_cast<uintptr_t>(p.x) | reinterpret_cast<uintptr_t>(p.z) | reinterpret_cast<uintptr_t>(p.v) |
                       reinterpret_cast<uintptr_t>(p.dt_bias)) & 15) == 0;
   const int tile = p.T <= 4 * p.B ? 1 : 16;
@@ -537,6 +592,12 @@ extern "C" int mb_delta_dim_pad(int dim) {
   for (int s : sizes)
     if (dim <= s) return s;
   return 0;
+}
+
+extern "C" int mb_head_norm_gate(const MbHeadOut* p, int dtype, cudaStream_t stream) {
+  if (p->T <= 0) return MB_OK;
+  if (p->heads <= 0 || p->vdim <= 0 || p->n <= 0 || p->n > p->vdim) return MB_ERR_SHAPE;
+  return dtype == kF32 ? delta::head_out<float>(*p, stream) : delta::head_out<__nv_bfloat16>(*p, stream);
 }
 
 extern "C" int mb_delta_rule(const MbDelta* p, int dtype, int num_sms, cudaStream_t stream) {

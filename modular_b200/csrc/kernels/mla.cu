@@ -22,6 +22,7 @@
 #include <stdint.h>
 
 #include "../common/api.h"
+#include "../common/head_gate.cuh"
 #include "../common/launch.h"
 
 namespace mb {
@@ -37,6 +38,8 @@ struct Params {
   bf16* out;           // [T, h, R]
   const bf16* cache;   // page p, slot s at cache + p * page_stride + s * ld_cache
   const float* sink;   // per head: a score without key or value that joins the softmax denominator (nullptr: none)
+  HeadGate gate;
+  int window;          // keys a query sees (0x7fffffff: all before it)
   // KV split: grid z parts walk equal shares of the 64-token tiles and leave (O, m, l) of their valid rows in `ws`,
   // [part][T * h][R] then [part][T * h][2]; a second kernel combines them
   float* ws;
@@ -146,9 +149,10 @@ __global__ void __launch_bounds__(256, 1) mla_kernel(const Params p) {
   int last_tq = tq0 + tokens_per_tile;
   if (last_tq > ql) last_tq = ql;
   const int kv_hi = kl - ql + last_tq;  // exclusive bound of the KV positions any row here may see
-  const int tiles_all = (kv_hi + 63) / 64;
-  const int tiles_per = (tiles_all + p.nsplit - 1) / p.nsplit;
-  const int t_begin = static_cast<int>(blockIdx.z) * tiles_per;
+  const int kv_lo = kl - ql + tq0 - p.window + 1;  // the first one the tile's first row sees
+  const int t_first = kv_lo > 0 ? kv_lo / 64 : 0, tiles_all = (kv_hi + 63) / 64;
+  const int tiles_per = (tiles_all - t_first + p.nsplit - 1) / p.nsplit;
+  const int t_begin = t_first + static_cast<int>(blockIdx.z) * tiles_per;
   const int t_end = min(tiles_all, t_begin + tiles_per);     // trailing parts may be empty
   load_kv_tile<R>(sK, p, bt, t_begin * 64, kv_hi, tid);
   cp_async_commit();
@@ -202,7 +206,7 @@ __global__ void __launch_bounds__(256, 1) mla_kernel(const Params p) {
       for (int e = 0; e < 4; ++e) {
         const int col = kv0 + nt * 8 + 2 * (lane & 3) + (e & 1);
         const int h = e >> 1;
-        const float v = col <= limit[h] ? s[nt][e] * p.scale_log2 : -INFINITY;
+        const float v = static_cast<uint32_t>(limit[h] - col) < static_cast<uint32_t>(p.window) ? s[nt][e] * p.scale_log2 : -INFINITY;
         s[nt][e] = v;
         mx[h] = fmaxf(mx[h], v);
       }
@@ -276,6 +280,7 @@ __global__ void __launch_bounds__(256, 1) mla_kernel(const Params p) {
       const float f = exp2f(m[h] - mm);
       inv = f / (l[h] * f + exp2f(sk - mm));
     }
+    inv *= p.gate(qs + tq, head);
     {
       bf16* orow = p.out + (static_cast<int64_t>(qs + tq) * p.n_heads + head) * R + chalf * HALF + 2 * (lane & 3);
 #pragma unroll
@@ -287,7 +292,7 @@ __global__ void __launch_bounds__(256, 1) mla_kernel(const Params p) {
 
 // Combines the parts of a KV-split launch: one warp per (token, head), part weights exp2(m - max).
 __global__ void __launch_bounds__(256)
-mla_combine_kernel(const float* __restrict__ ws, bf16* __restrict__ out, const float* __restrict__ sink, int n_rows,
+mla_combine_kernel(const float* __restrict__ ws, bf16* __restrict__ out, const float* __restrict__ sink, const HeadGate gate, int n_rows,
                    int n_heads, int R, int nsplit) {
   const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (row >= n_rows) return;
@@ -302,7 +307,7 @@ mla_combine_kernel(const float* __restrict__ ws, bf16* __restrict__ out, const f
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
   if (sink) den += exp2f(sk - M);
-  const float inv = den > 0.f ? 1.f / den : 0.f;
+  const float inv = den > 0.f ? gate(row / n_heads, row % n_heads) / den : 0.f;
   for (int c = lane * 2; c < R; c += 64) {
     float2 acc = make_float2(0.f, 0.f);
     for (int q = 0; q < nsplit; ++q) {
@@ -443,7 +448,7 @@ static int launch(const Params& p, int grid_x, cudaStream_t stream) {
   if (p.nsplit > 1) {
     const int n_rows = p.T * p.n_heads;
     if (launch_plain(mla_combine_kernel, dim3((n_rows + 7) / 8), dim3(256), 0, stream, static_cast<const float*>(p.ws), p.out,
-                 p.sink, n_rows, p.n_heads, R, p.nsplit) != cudaSuccess)
+                 p.sink, p.gate, n_rows, p.n_heads, R, p.nsplit) != cudaSuccess)
       return MB_ERR_LAUNCH;
   }
   return MB_OK;
@@ -494,7 +499,7 @@ extern "C" int mb_mla_paged_attention_ex(const void* q_lat, long long ld_ql, con
                                          void* out, const void* cache, long long page_stride, int ld_cache,
                                          const int32_t* block_table, int bt_stride, const int32_t* q_start,
                                          const int32_t* q_len, const int32_t* kv_len, int T, int B, int n_heads, int R,
-                                         int page_size, float scale, const float* sink, void* ws, size_t ws_bytes,
+                                         int page_size, float scale, const MbAttnOptions* opt, void* ws, size_t ws_bytes,
                                          int num_sms, cudaStream_t stream) {
   if (T <= 0 || B <= 0) return MB_OK;
   if (ld_cache < R + mla::DR || ld_cache % 8 || page_stride % 8 || ld_ql % 8 || ld_qr % 8 || hs_qr % 8) return MB_ERR_SHAPE;
@@ -510,14 +515,16 @@ extern "C" int mb_mla_paged_attention_ex(const void* q_lat, long long ld_ql, con
   p.page_stride = page_stride; p.B = B; p.bt_stride = bt_stride; p.n_heads = n_heads; p.HB = heads_per_tile(n_heads);
   p.page_size = page_size;
   p.scale_log2 = scale * 1.4426950408889634f;
-  p.sink = sink; p.ld_cache = ld_cache; p.T = T; p.ld_ql = ld_ql; p.ld_qr = ld_qr; p.hs_qr = hs_qr;
+  p.sink = opt ? opt->sink : nullptr; p.gate = HeadGate(opt);
+  p.window = opt && opt->window > 0 ? opt->window : 0x7fffffff; p.ld_cache = ld_cache; p.T = T; p.ld_ql = ld_ql; p.ld_qr = ld_qr; p.hs_qr = hs_qr;
   p.ws = static_cast<float*>(ws); p.nsplit = 1;
   const int tpt = 64 / p.HB;
   const int grid_x = (T + tpt - 1) / tpt + B;  // >= sum over sequences of ceil(q_len / tpt)
   if (ws != nullptr) {
     // decode-sized steps: tiles of the batch that really exist are at most T, so count those
     const long long ctas = static_cast<long long>(T < grid_x ? T : grid_x) * (n_heads / p.HB);
-    const long long max_tiles = static_cast<long long>(bt_stride) * page_size / 64;
+    long long max_tiles = static_cast<long long>(bt_stride) * page_size / 64;
+    if (p.window / 64 + 2 < max_tiles) max_tiles = p.window / 64 + 2;
     long long ns = ctas > 0 ? num_sms / ctas : 1;
     if (ns > max_tiles / 2) ns = max_tiles / 2;      // at least two tiles per part
     if (ns > 32) ns = 32;

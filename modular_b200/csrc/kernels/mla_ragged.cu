@@ -6,13 +6,14 @@
 //                         latent is RMS-normed and stored, with the rotated key part behind it, in the token's cache
 //                         row. A layer that reads another layer's cache has no key/value columns and stores nothing.
 //   mb_rotate_heads       rotates the first `dims` values of every head of a column block, in place
-//   mb_latent_attention   absorbed attention over the paged rows [latent | rotated part], causal, with an optional
-//                         learned sink per head that only takes part in the softmax denominator
+//   mb_latent_attention   absorbed attention over the paged rows [latent | rotated part], causal, with the options of
+//                         MbAttnOptions (window, sink, output gate)
 //
 // Rows are padded: a cache row holds Rp >= R latent values and Dp >= rotated values, the rest is zero.
 #include <cuda_runtime.h>
 
 #include "../common/api.h"
+#include "../common/head_gate.cuh"
 #include "../common/launch.h"
 #include "../common/scalar.cuh"
 
@@ -129,6 +130,8 @@ struct Attn {
   long long page_stride;
   const int32_t *block_table, *q_start, *q_len, *kv_len;
   const float* sink;
+  HeadGate gate;
+  int window;
   float scale;
 };
 
@@ -151,6 +154,7 @@ attention_kernel(const Attn p, const T* __restrict__ q_lat, const T* __restrict_
   const int off = t - p.q_start[lo];
   if (off >= p.q_len[lo]) return;               // a row of no sequence
   const int keys = p.kv_len[lo] - p.q_len[lo] + off + 1;
+  const int first = keys > p.window ? keys - p.window : 0;
   const int32_t* bt = p.block_table + static_cast<size_t>(lo) * p.bt_stride;
   float* sq = sm;
   float* so = sm + LD;
@@ -163,7 +167,7 @@ attention_kernel(const Attn p, const T* __restrict__ q_lat, const T* __restrict_
 #pragma unroll
   for (int i = 0; i < VPL; ++i) o[i] = 0.f;
   float m = -INFINITY, l = 0.f;
-  for (int j = warp; j < keys; j += kWarps) {
+  for (int j = first + warp; j < keys; j += kWarps) {
     const T* row = cache + static_cast<size_t>(bt[j / p.page_size]) * p.page_stride +
                    static_cast<size_t>(j % p.page_size) * p.ld_cache;
     float k[VPL], s = 0.f;
@@ -196,7 +200,7 @@ attention_kernel(const Attn p, const T* __restrict__ q_lat, const T* __restrict_
   float f[kWarps];
 #pragma unroll
   for (int i = 0; i < kWarps; ++i) { f[i] = expf(sml[i] - M); den = fmaf(sml[kWarps + i], f[i], den); }
-  const float inv = 1.f / den;
+  const float inv = p.gate.of<T>(t, head) / den;
   T* dst = out + static_cast<size_t>(t) * p.ld_out + static_cast<size_t>(head) * p.hs_out;
   for (int c = tid; c < p.Rp; c += blockDim.x) {
     float v = 0.f;
@@ -281,12 +285,13 @@ extern "C" int mb_latent_attention(const void* q_lat, int ld_ql, int hs_ql, cons
                                    void* out, int ld_out, int hs_out, const void* cache, long long page_stride,
                                    int ld_cache, int page_size, const int32_t* block_table, int bt_stride,
                                    const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len, int T, int B,
-                                   int n_heads, int Rp, int Dp, float scale, const float* sink, int dtype,
+                                   int n_heads, int Rp, int Dp, float scale, const MbAttnOptions* opt, int dtype,
                                    cudaStream_t stream) {
   if (T <= 0 || B <= 0) return MB_OK;
   if (ld_cache < Rp + Dp || n_heads <= 0) return MB_ERR_SHAPE;
   latent::Attn p = {ld_ql, ld_qr, hs_ql, hs_qr, ld_out, hs_out, B, bt_stride, page_size, ld_cache, Rp, Dp, n_heads,
-                    page_stride, block_table, q_start, q_len, kv_len, sink, scale};
+                    page_stride, block_table, q_start, q_len, kv_len, opt ? opt->sink : nullptr, HeadGate(opt),
+                    opt && opt->window > 0 ? opt->window : 0x7fffffff, scale};
   return dtype == kF32 ? latent::dispatch_attn<float>(p, q_lat, q_rope, cache, out, T, stream)
                        : latent::dispatch_attn<__nv_bfloat16>(p, q_lat, q_rope, cache, out, T, stream);
 }

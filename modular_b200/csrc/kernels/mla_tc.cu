@@ -31,6 +31,7 @@
 #include <stdint.h>
 
 #include "../common/api.h"
+#include "../common/head_gate.cuh"
 #include "../common/launch.h"
 #include "../common/ptx.cuh"
 #include "gemm_common.h"
@@ -71,6 +72,8 @@ struct Params {
   int bt_stride, n_heads, page_size;
   float scale_log2;
   const float* sink;               // per head: a score without key or value in the softmax denominator (nullptr: none)
+  HeadGate gate;
+  int window;                      // keys a query sees (0x7fffffff: all before it)
 };
 
 struct Bars {
@@ -129,11 +132,12 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap tmQl, const __grid_constant__ 
   }
   if (ql <= 0) return;   // whole CTA, before any barrier or TMEM allocation
   const int32_t* bt = p.block_table + static_cast<int64_t>(seq) * p.bt_stride;
-  const int tiles_all = (kl + 63) / 64;
+  const int kv_lo = kl > p.window ? kl - p.window : 0;                // the first key this query sees
+  const int t_first = kv_lo / 64, tiles_all = (kl + 63) / 64 - t_first;
   // this part's tiles [t_begin, t_begin + ntiles); parts are as even as possible and the trailing ones may be empty
   const int tiles_per = p.nsplit > 1 ? (tiles_all + p.nsplit - 1) / p.nsplit : tiles_all;
-  const int t_begin = part * tiles_per;
-  const int ntiles = max(0, min(tiles_all, t_begin + tiles_per) - t_begin);
+  const int t_begin = t_first + part * tiles_per;
+  const int ntiles = max(0, min(tiles_all, (part + 1) * tiles_per) - part * tiles_per);
   const int n_parts = tiles_per > 0 ? (tiles_all + tiles_per - 1) / tiles_per : 1;   // parts that have tiles
   if (part > 0 && ntiles == 0) return;            // whole CTA, before any barrier or TMEM allocation
   const int q_row = qs * p.n_heads + hb * 128;   // row of the [T*h, .] views of q_lat / q_rope / out
@@ -270,13 +274,13 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap tmQl, const __grid_constant__ 
       if (lane == 0) mbar_arrive(&bars->s_free[b]);
       const int kv0 = (t_begin + t) * 64;
       float mxa[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-      if (kv0 + 64 <= kl) {
+      if (kv0 + 64 <= kl && kv0 >= kv_lo) {
 #pragma unroll
         for (int c = 0; c < 64; ++c) mxa[c & 3] = fmaxf(mxa[c & 3], __uint_as_float(sr[c >> 5][c & 31]));
       } else {
 #pragma unroll
         for (int c = 0; c < 64; ++c) {
-          const float v = (kv0 + c) < kl ? __uint_as_float(sr[c >> 5][c & 31]) : -INFINITY;
+          const float v = (kv0 + c) < kl && (kv0 + c) >= kv_lo ? __uint_as_float(sr[c >> 5][c & 31]) : -INFINITY;
           sr[c >> 5][c & 31] = __float_as_uint(v);
           mxa[c & 3] = fmaxf(mxa[c & 3], v);
         }
@@ -340,6 +344,7 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap tmQl, const __grid_constant__ 
         const float f = exp2f(m_ref - M);
         inv = f / (l * f + exp2f(sk - M));
       }
+      inv *= p.gate(qs, hb * 128 + r);
       if (ntiles > 0 && ok) {
 #pragma unroll 1
         for (int q8 = 0; q8 < 8; ++q8) {
@@ -396,7 +401,7 @@ mla_tc_kernel(const __grid_constant__ CUtensorMap tmQl, const __grid_constant__ 
           wq[q] = lq > 0.f ? exp2f(__ldcg(pp + 256 * 128 + r) - M) : 0.f;
           L += lq * wq[q];
         }
-        const float inv = L > 0.f ? 1.f / L : 0.f;
+        const float inv = L > 0.f ? p.gate(qs, hb * 128 + r) / L : 0.f;
 #pragma unroll 1
         for (int c8 = 0; c8 < 32; ++c8) {
           float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
@@ -480,16 +485,16 @@ extern "C" int mb_mla_tc_usable(int T, int B, int n_heads, int R, int page_size)
 static int mla_tc_launch(const void* q_lat, const void* q_rope, void* out, const void* cache, long long page_stride,
                          long long n_pages, const int32_t* block_table, int bt_stride, const int32_t* q_start,
                          const int32_t* q_len, const int32_t* kv_len, int T, int B, int n_heads, int page_size,
-                         float scale, const float* sink, int ld_rope, int32_t* tok_scratch, int* err,
+                         float scale, const MbAttnOptions* opt, int ld_rope, int32_t* tok_scratch, int* err,
                          cudaStream_t stream);
 
 extern "C" int mb_mla_decode_tc(const void* q_lat, const void* q_rope, void* out, const void* cache,
                                 long long page_stride, long long n_pages, const int32_t* block_table, int bt_stride,
                                 const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len, int T, int B,
-                                int n_heads, int page_size, float scale, const float* sink, int ld_rope, int* err,
+                                int n_heads, int page_size, float scale, const MbAttnOptions* opt, int ld_rope, int* err,
                                 cudaStream_t stream) {
   return mla_tc_launch(q_lat, q_rope, out, cache, page_stride, n_pages, block_table, bt_stride, q_start, q_len, kv_len,
-                       T, B, n_heads, page_size, scale, sink, ld_rope, nullptr, err, stream);
+                       T, B, n_heads, page_size, scale, opt, ld_rope, nullptr, err, stream);
 }
 
 // Any ragged batch (prefill, chunks, mixed steps) on the same tensor-core kernel: every query token is one CTA
@@ -498,17 +503,17 @@ extern "C" int mb_mla_decode_tc(const void* q_lat, const void* q_rope, void* out
 extern "C" int mb_mla_prefill_tc(const void* q_lat, const void* q_rope, void* out, const void* cache,
                                  long long page_stride, long long n_pages, const int32_t* block_table, int bt_stride,
                                  const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len, int T, int B,
-                                 int n_heads, int page_size, float scale, const float* sink, int ld_rope,
+                                 int n_heads, int page_size, float scale, const MbAttnOptions* opt, int ld_rope,
                                  int32_t* tok_scratch, int* err, cudaStream_t stream) {
   if (tok_scratch == nullptr) return MB_ERR_SHAPE;
   return mla_tc_launch(q_lat, q_rope, out, cache, page_stride, n_pages, block_table, bt_stride, q_start, q_len, kv_len,
-                       T, B, n_heads, page_size, scale, sink, ld_rope, tok_scratch, err, stream);
+                       T, B, n_heads, page_size, scale, opt, ld_rope, tok_scratch, err, stream);
 }
 
 static int mla_tc_launch(const void* q_lat, const void* q_rope, void* out, const void* cache, long long page_stride,
                          long long n_pages, const int32_t* block_table, int bt_stride, const int32_t* q_start,
                          const int32_t* q_len, const int32_t* kv_len, int T, int B, int n_heads, int page_size,
-                         float scale, const float* sink, int ld_rope, int32_t* tok_scratch, int* err,
+                         float scale, const MbAttnOptions* opt, int ld_rope, int32_t* tok_scratch, int* err,
                          cudaStream_t stream) {
   using namespace mb::mlatc;
   if (T <= 0 || B <= 0) return MB_OK;
@@ -534,7 +539,8 @@ static int mla_tc_launch(const void* q_lat, const void* q_rope, void* out, const
       if (cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || sms <= 0) sms = 148;
     }
     // as many parts as fill the SMs once, at least four tiles each (the block table bounds the tiles of a sequence)
-    const long long max_tiles = static_cast<long long>(bt_stride) * page_size / 64;
+    long long max_tiles = static_cast<long long>(bt_stride) * page_size / 64;
+    if (opt && opt->window > 0 && opt->window / 64 + 2 < max_tiles) max_tiles = opt->window / 64 + 2;
     long long ns = sms / units;
     if (ns > max_tiles / 4) ns = max_tiles / 4;
     if (ns > 16) ns = 16;
@@ -548,7 +554,9 @@ static int mla_tc_launch(const void* q_lat, const void* q_rope, void* out, const
   p.err = err;
   p.page_rows = page_rows; p.bt_stride = bt_stride; p.n_heads = n_heads; p.page_size = page_size;
   p.scale_log2 = scale * 1.4426950408889634f;
-  p.sink = sink;
+  p.sink = opt ? opt->sink : nullptr;
+  p.gate = HeadGate(opt);
+  p.window = opt && opt->window > 0 ? opt->window : 0x7fffffff;
   CUtensorMap tql, tqr, tkv;
   int rc = cached_tmap(&tql, q_lat, static_cast<uint64_t>(T) * n_heads, R, R, 128, 2);
   if (rc != MB_OK) return rc;

@@ -5,6 +5,9 @@
 //                             best `topk_group` groups, top-k experts inside them, weights from
 //                             the un-biased scores, optional normalisation, times a scaling factor.
 //   moe_router_softmax_topk   plain softmax top-k routing (Mixtral / Qwen style).
+//   moe_score_route           the group-limited choice with one warp per token, which also counts the pairs of every
+//   moe_place_rows            expert; the second kernel scans the counts and copies token rows into expert order, so a
+//                             routed layer costs two launches between its router product and its experts.
 //   moe_table_route           routing by token id: a table names every id's experts, so the expert order of
 //                             all layers of a step is known before the first layer runs (one launch).
 //   moe_create_indices        counting sort of (token, slot) pairs by expert: CSR offsets per
@@ -181,6 +184,133 @@ __global__ void moe_scatter_kernel(const int32_t* __restrict__ ids, int n, int32
   }
 }
 
+// Keys that order like the floats they are made from (all finite or infinite values).
+__device__ __forceinline__ uint32_t order_key(float v) {
+  const uint32_t b = __float_as_uint(v);
+  return (b & 0x80000000u) ? ~b : (b | 0x80000000u);
+}
+
+constexpr int kRouteWarps = 8;
+
+// One warp per token; a lane holds the experts lane, lane + 32, ... (EPL of them at most).
+template <int EPL>
+__global__ void __launch_bounds__(kRouteWarps * 32)
+score_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int32_t* __restrict__ ids,
+                   float* __restrict__ w, int32_t* __restrict__ rank, int32_t* __restrict__ counts, int T, int E, int n_group, int keep,
+                   int top_k, int norm_topk, float scaling) {
+  extern __shared__ float sh[];                  // per warp: choice scores [E] | group scores [n_group]
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * kRouteWarps + warp;
+  if (t >= T) return;
+  float *choice = sh + warp * (E + n_group), *gscore = choice + E;
+  const int gsize = E / n_group;
+  float score[EPL], mine[EPL];
+#pragma unroll
+  for (int i = 0; i < EPL; ++i) {
+    const int e = lane + 32 * i;
+    score[i] = 0.f; mine[i] = -INFINITY;
+    if (e < E) {
+      score[i] = 1.f / (1.f + expf(-logits[static_cast<size_t>(t) * ld + e]));
+      mine[i] = score[i] + (bias ? bias[e] : 0.f);
+      choice[e] = mine[i];
+    }
+  }
+  __syncwarp();
+  if (keep < n_group) {
+    for (int g = lane; g < n_group; g += 32) {   // sum of the two largest choice scores of a group
+      float m1 = -INFINITY, m2 = -INFINITY;
+      for (int j = 0; j < gsize; ++j) {
+        const float v = choice[g * gsize + j];
+        if (v > m1) { m2 = m1; m1 = v; } else if (v > m2) { m2 = v; }
+      }
+      gscore[g] = gsize > 1 ? m1 + m2 : m1;
+    }
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) {
+      const int e = lane + 32 * i;
+      if (e >= E) continue;
+      const int g = e / gsize;
+      const float v = gscore[g];
+      int better = 0;
+      for (int o = 0; o < n_group; ++o) better += gscore[o] > v || (gscore[o] == v && o < g);
+      if (better >= keep) mine[i] = -INFINITY;
+    }
+  }
+  int my_id = 0;
+  float my_w = 0.f;
+  for (int k = 0; k < top_k; ++k) {
+    uint32_t best = 0;
+    int bi = 0;
+    float bs = 0.f;
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) {
+      const uint32_t key = order_key(mine[i]);
+      if (key > best) { best = key; bi = i; bs = score[i]; }
+    }
+    const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+    const int e = static_cast<int>(__reduce_min_sync(0xffffffffu, best == top ? static_cast<uint32_t>(lane + 32 * bi) : 0xffffffffu));
+    const float ws = __shfl_sync(0xffffffffu, bs, e & 31);
+    if ((e & 31) == lane)
+#pragma unroll
+      for (int i = 0; i < EPL; ++i)
+        if (i == (e >> 5)) mine[i] = -INFINITY;
+    if (lane == k) { my_id = e; my_w = ws; }
+  }
+  float sum = lane < top_k ? my_w : 0.f;
+  if (norm_topk) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    my_w /= sum + 1e-20f;
+  }
+  if (lane < top_k) {
+    const size_t i = static_cast<size_t>(t) * top_k + lane;
+    ids[i] = my_id;
+    w[i] = my_w * scaling;
+    rank[i] = my_id < E ? atomicAdd(&counts[my_id], 1) : -1;
+  }
+}
+
+__global__ void __launch_bounds__(256)
+place_rows_kernel(const uint8_t* __restrict__ x, long long ldx, const int32_t* __restrict__ ids, const int32_t* __restrict__ rank,
+                  const int32_t* __restrict__ counts, int32_t* __restrict__ offsets, int32_t* __restrict__ inverse,
+                  uint8_t* __restrict__ dst, int E, int top_k, int row_bytes) {
+  extern __shared__ int32_t first[];             // exclusive scan of the counts
+  __shared__ int32_t pos[32];
+  const int t = blockIdx.x, lane = threadIdx.x;
+  if (threadIdx.x < 32) {
+    int base = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + lane, c = e < E ? counts[e] : 0;
+      int s = c;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int u = __shfl_up_sync(0xffffffffu, s, o);
+        if (lane >= o) s += u;
+      }
+      if (e < E) {
+        first[e] = base + s - c;
+        if (t == 0) offsets[e] = base + s - c;
+      }
+      base += __shfl_sync(0xffffffffu, s, 31);
+    }
+    if (t == 0 && lane == 0) offsets[E] = base;
+    __syncwarp();
+    if (lane < top_k) {
+      const size_t i = static_cast<size_t>(t) * top_k + lane;
+      const int r = rank[i];
+      pos[lane] = r < 0 ? -1 : first[ids[i]] + r;
+      inverse[i] = pos[lane];
+    }
+  }
+  __syncthreads();
+  const uint8_t* src = x + t * ldx;
+  for (int c = threadIdx.x * 16; c < row_bytes; c += blockDim.x * 16) {
+    const uint4 v = *reinterpret_cast<const uint4*>(src + c);
+    for (int k = 0; k < top_k; ++k)
+      if (pos[k] >= 0) *reinterpret_cast<uint4*>(dst + static_cast<size_t>(pos[k]) * row_bytes + c) = v;
+  }
+}
+
 // Routing by token id for all mixture-of-experts layers of a step. One CTA per layer sorts the layer's (token, slot)
 // pairs by expert: desc[l] = {first element of the layer's table in `tables`, experts per token, experts, sum of the
 // earlier layers' experts per token, sum of the earlier layers' (experts + 1), vocabulary rows of the table}.
@@ -300,6 +430,38 @@ extern "C" int mb_moe_router_group_limited(const float* logits, const float* bia
   router_group_limited_kernel<<<T, threads, (E + 2 * n_group) * sizeof(float), stream>>>(
       logits, bias, topk_ids, topk_w, E, n_group, topk_group, top_k, norm_topk, scaling, ld);
   return MB_OK_OR_LAUNCH();
+}
+
+extern "C" int mb_moe_score_route(const float* logits, int ld, const float* bias, int32_t* ids, float* w, int32_t* rank, int32_t* counts,
+                                  int T, int E, int n_group, int keep, int top_k, int norm_topk, float scaling, cudaStream_t stream) {
+  if (T <= 0) return MB_OK;
+  if (E <= 0 || E > 1024 || n_group < 1 || E % n_group || keep < 1 || keep > n_group || top_k < 1 || top_k > 32 ||
+      top_k > keep * (E / n_group))
+    return MB_ERR_SHAPE;
+  const dim3 grid((T + kRouteWarps - 1) / kRouteWarps), block(kRouteWarps * 32);
+  const size_t smem = static_cast<size_t>(kRouteWarps) * (E + n_group) * sizeof(float);
+  if (smem > 48 * 1024) return MB_ERR_TOO_LARGE;
+  auto go = [&](auto kern) {
+    return launch_plain(kern, grid, block, smem, stream, logits, ld, bias, ids, w, rank, counts, T, E, n_group, keep, top_k, norm_topk,
+                        scaling) == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
+  };
+  if (E <= 32) return go(score_route_kernel<1>);
+  if (E <= 64) return go(score_route_kernel<2>);
+  if (E <= 128) return go(score_route_kernel<4>);
+  if (E <= 256) return go(score_route_kernel<8>);
+  return go(score_route_kernel<32>);
+}
+
+extern "C" int mb_moe_place_rows(const void* x, long long ldx_bytes, const int32_t* ids, const int32_t* rank, const int32_t* counts,
+                                 int32_t* offsets, int32_t* inverse, void* dst, int T, int E, int top_k, int row_bytes,
+                                 cudaStream_t stream) {
+  if (T <= 0) return MB_OK;
+  if (E <= 0 || E > 1024 || top_k < 1 || top_k > 32 || row_bytes % 16 || ldx_bytes % 16) return MB_ERR_SHAPE;
+  if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(dst)) & 15) return MB_ERR_ALIGN;
+  const int threads = row_bytes >= 4096 ? 256 : row_bytes >= 2048 ? 128 : row_bytes >= 1024 ? 64 : 32;
+  return launch_plain(place_rows_kernel, dim3(T), dim3(threads), static_cast<size_t>(E) * 4, stream, static_cast<const uint8_t*>(x),
+                      ldx_bytes, ids, rank, counts, offsets, inverse, static_cast<uint8_t*>(dst), E, top_k, row_bytes) == cudaSuccess
+             ? MB_OK : MB_ERR_LAUNCH;
 }
 
 extern "C" int mb_moe_router_softmax_topk(const float* logits, int32_t* topk_ids, float* topk_w, int T,

@@ -15,6 +15,13 @@
 //   x[t]  += mult * (ab_scale * (a / rms(a) * norm_a + b / rms(b) * norm_b) + c)
 //            [+ inject_scale * inject[ids[t]]] [+ step]       (what a looped pass adds before its first layer)
 //
+// A third one serves layers that norm a branch before and after it (sandwich norms), with layer norms or RMS norms:
+//
+//   x[t]  += mult * norm(u[t]; w_u, b_u),   n1[t] = norm(x[t]; w1, b1),   u = a[t] or sum_k pair_w[t, k] e[inverse[t, k]]
+//
+// with the embedding (and rows of a second table, chosen by ids of their own) ahead of the first layer. A row lives in
+// registers from its first read to its last write; means and squared deviations are two sums, as the norm is defined.
+//
 // Also here: tanh-GELU in place, the sigmoid output gate of an attention layer and the soft cap of logits.
 #include <cuda_runtime.h>
 
@@ -269,6 +276,152 @@ static int run(const MbResidualNorm& q, cudaStream_t stream) {
                  cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
 }
 
+// ---- sandwich norms
+template <typename T, int NV, bool CENTER>
+__global__ void __launch_bounds__(1024) sandwich_norm_kernel(const MbSandwichNorm p) {
+  __shared__ float part[4][1][32];
+  __shared__ int32_t pos[32];
+  __shared__ float pw[32];
+  const int out_row = blockIdx.x, nvec = p.cols_pad >> 2;
+  const int row = p.rows ? p.rows[out_row] : out_row;
+  float* xr = p.x + static_cast<size_t>(row) * p.ldx;
+  const T *ar = p.a ? static_cast<const T*>(p.a) + static_cast<size_t>(row) * p.lda : nullptr, *er = nullptr, *ir = nullptr;
+  const T* ee = static_cast<const T*>(p.e);
+  if (p.table) {
+    const int64_t id = p.ids[row];
+    if (id >= 0 && id < p.vocab) er = static_cast<const T*>(p.table) + static_cast<size_t>(id) * p.ld_table;
+  }
+  if (p.inject) {
+    const int64_t id = p.inject_ids[row];
+    if (id >= 0 && id < p.inject_rows) ir = static_cast<const T*>(p.inject) + static_cast<size_t>(id) * p.ld_inject;
+  }
+  if (ee) {
+    if (threadIdx.x < p.top_k) {
+      pos[threadIdx.x] = p.inverse[static_cast<size_t>(row) * p.top_k + threadIdx.x];
+      pw[threadIdx.x] = p.pair_w[static_cast<size_t>(row) * p.top_k + threadIdx.x];
+    }
+    __syncthreads();
+  }
+  float4 x[NV], u[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int v = threadIdx.x + i * blockDim.x, c = v * 4;
+    x[i] = u[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (v >= nvec) continue;
+    if (!p.table) x[i] = *reinterpret_cast<const float4*>(xr + c);
+    else if (er) { const float4 y = ld4(er + c); x[i] = make_float4(y.x * p.scale, y.y * p.scale, y.z * p.scale, y.w * p.scale); }
+    if (ir) { const float4 y = ld4(ir + c); x[i].x += y.x; x[i].y += y.y; x[i].z += y.z; x[i].w += y.w; }
+    if (ar) u[i] = ld4(ar + c);
+    if (ee) {
+#pragma unroll 4
+      for (int k = 0; k < p.top_k; ++k) {
+        if (pos[k] < 0) continue;
+        const float4 y = ld4(ee + static_cast<size_t>(pos[k]) * p.lde + c);
+        u[i].x = fmaf(pw[k], y.x, u[i].x); u[i].y = fmaf(pw[k], y.y, u[i].y);
+        u[i].z = fmaf(pw[k], y.z, u[i].z); u[i].w = fmaf(pw[k], y.w, u[i].w);
+      }
+    }
+  }
+  // r becomes the deviations from its mean (CENTER; zero beyond the true width); the result is 1 / sqrt(mean of squares + eps)
+  auto scale_of = [&](float4 (&r)[NV], int stage) {
+    const float n = static_cast<float>(p.cols);
+    if (CENTER) {
+      float s[1] = {0.f};
+#pragma unroll
+      for (int i = 0; i < NV; ++i) s[0] += (r[i].x + r[i].y) + (r[i].z + r[i].w);     // padding holds zeros
+      block_sums(s, part[stage]);
+      const float mean = s[0] / n;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = (threadIdx.x + i * blockDim.x) * 4;
+        r[i].x = c < p.cols ? r[i].x - mean : 0.f; r[i].y = c + 1 < p.cols ? r[i].y - mean : 0.f;
+        r[i].z = c + 2 < p.cols ? r[i].z - mean : 0.f; r[i].w = c + 3 < p.cols ? r[i].w - mean : 0.f;
+      }
+    }
+    float q[1] = {0.f};
+#pragma unroll
+    for (int i = 0; i < NV; ++i) q[0] += sq4(r[i]);
+    block_sums(q, part[stage + 1]);
+    return 1.f / sqrtf(q[0] / n + p.eps);
+  };
+  auto affine = [&](float4 r, float inv, const void* w, const void* b, int c) {
+    const float4 g = ld4(static_cast<const T*>(w) + c);
+    float4 y = make_float4(r.x * inv * g.x, r.y * inv * g.y, r.z * inv * g.z, r.w * inv * g.w);
+    if (CENTER) { const float4 o = ld4(static_cast<const T*>(b) + c); y.x += o.x; y.y += o.y; y.z += o.z; y.w += o.w; }
+    return y;
+  };
+  if (ar || ee) {
+    const float inv = p.w_u ? scale_of(u, 0) : 1.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int v = threadIdx.x + i * blockDim.x;
+      if (v >= nvec) continue;
+      const float4 y = p.w_u ? affine(u[i], inv, p.w_u, p.b_u, v * 4) : u[i];
+      x[i].x = fmaf(p.mult, y.x, x[i].x); x[i].y = fmaf(p.mult, y.y, x[i].y);
+      x[i].z = fmaf(p.mult, y.z, x[i].z); x[i].w = fmaf(p.mult, y.w, x[i].w);
+    }
+  }
+  if (p.store_x) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int v = threadIdx.x + i * blockDim.x;
+      if (v < nvec) *reinterpret_cast<float4*>(xr + v * 4) = x[i];
+    }
+  }
+  if (!p.w1) return;
+  const float inv = scale_of(x, 2);
+  T* o1 = static_cast<T*>(p.n1) + static_cast<size_t>(out_row) * p.ld1;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int v = threadIdx.x + i * blockDim.x;
+    if (v < nvec) st4(o1 + v * 4, affine(x[i], inv, p.w1, p.b1, v * 4));
+  }
+}
+
+template <typename T, bool CENTER>
+static int run_sandwich(const MbSandwichNorm& p, cudaStream_t stream) {
+  const int nvec = p.cols_pad / 4;
+  // few rows: as many threads as a row has vectors; many rows: CTAs of 256, several per SM
+  const int most = p.n_rows <= 296 ? 1024 : 256, warps = (nvec + 31) / 32;
+  int nv = (nvec + most - 1) / most;
+  nv = nv <= 1 ? 1 : nv <= 2 ? 2 : 4;
+  const int threads = (warps + nv - 1) / nv * 32;
+  if (threads > 1024) return MB_ERR_TOO_LARGE;
+  cudaError_t e;
+  if (nv == 1) e = launch_plain(sandwich_norm_kernel<T, 1, CENTER>, dim3(p.n_rows), dim3(threads), 0, stream, p);
+  else if (nv == 2) e = launch_plain(sandwich_norm_kernel<T, 2, CENTER>, dim3(p.n_rows), dim3(threads), 0, stream, p);
+  else e = launch_plain(sandwich_norm_kernel<T, 4, CENTER>, dim3(p.n_rows), dim3(threads), 0, stream, p);
+  return e == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
+}
+
+__global__ void bigram_rows_kernel(const int64_t* __restrict__ tokens, const int32_t* __restrict__ q_start,
+                                   const int32_t* __restrict__ q_len, const int32_t* __restrict__ kv_len,
+                                   const int32_t* __restrict__ state_idx, int64_t* __restrict__ last, int64_t* __restrict__ out, int T,
+                                   int B, long long mul_prev, long long mul_cur, long long buckets) {
+  const int t = blockIdx.x * blockDim.x + threadIdx.x;
+  if (t >= T) return;
+  int lo = 0, hi = B - 1;                       // the last sequence that starts at or before t
+  while (lo < hi) {
+    const int mid = (lo + hi + 1) >> 1;
+    if (q_start[mid] <= t) lo = mid; else hi = mid - 1;
+  }
+  const int off = t - q_start[lo], n = q_len[lo];
+  if (off < 0 || off >= n) { out[t] = buckets; return; }   // a row of no sequence
+  const long long cur = tokens[t];
+  long long prev = -1;
+  if (off > 0) {
+    prev = tokens[t - 1];
+  } else {                                      // one thread per sequence reads its slot and then advances it
+    const int slot = state_idx[lo];
+    if (slot >= 0) {
+      if (kv_len[lo] > n) prev = last[slot];
+      last[slot] = tokens[t + n - 1];
+    }
+  }
+  long long r = prev < 0 ? buckets : (prev * mul_prev + cur * mul_cur) % buckets;
+  out[t] = r < 0 ? r + buckets : r;
+}
+
 template <typename T>
 __global__ void gelu_tanh_kernel(T* __restrict__ x, size_t n4) {
   const size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
@@ -313,6 +466,26 @@ extern "C" int mb_residual_norm(const MbResidualNorm* q, int dtype, cudaStream_t
     return MB_ERR_SHAPE;
   if (q->cols_pad > 12288) return MB_ERR_TOO_LARGE;
   return dtype == kF32 ? run<float>(*q, stream) : run<__nv_bfloat16>(*q, stream);
+}
+
+extern "C" int mb_sandwich_norm(const MbSandwichNorm* q, int dtype, cudaStream_t stream) {
+  if (q->n_rows <= 0) return MB_OK;
+  if (q->cols <= 0 || q->cols > q->cols_pad || q->cols_pad % 4 || q->ldx % 4 || q->lda % 4 || q->lde % 4 || q->ld1 % 4 ||
+      q->ld_table % 4 || q->ld_inject % 4 || (q->a && q->e) || (q->e && (q->top_k <= 0 || q->top_k > 32)) ||
+      (q->w_u && q->w1 && (q->b_u == nullptr) != (q->b1 == nullptr)))
+    return MB_ERR_SHAPE;
+  const bool center = q->b_u != nullptr || q->b1 != nullptr;
+  if (dtype == kF32) return center ? run_sandwich<float, true>(*q, stream) : run_sandwich<float, false>(*q, stream);
+  return center ? run_sandwich<__nv_bfloat16, true>(*q, stream) : run_sandwich<__nv_bfloat16, false>(*q, stream);
+}
+
+extern "C" int mb_bigram_rows(const int64_t* tokens, const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
+                              const int32_t* state_idx, int64_t* last, int64_t* out, int T, int B, long long mul_prev,
+                              long long mul_cur, long long buckets, cudaStream_t stream) {
+  if (T <= 0 || B <= 0) return MB_OK;
+  if (buckets <= 0) return MB_ERR_SHAPE;
+  return launch_plain(bigram_rows_kernel, dim3((T + 255) / 256), dim3(256), 0, stream, tokens, q_start, q_len, kv_len, state_idx, last,
+                      out, T, B, mul_prev, mul_cur, buckets) == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
 }
 
 extern "C" int mb_gelu_tanh(void* x, long long n, int dtype, cudaStream_t stream) {

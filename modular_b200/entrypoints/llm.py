@@ -160,6 +160,8 @@ class LLM:
             dkvp = dfam.kv_params(draft_model_config, page_size, dtype, False)   # no prefix cache: drafts get rewritten
             if dfam.name in ("mamba", "lfm2") or dkvp.state_specs:
                 raise ValueError("a draft model with recurrent state cannot take back rejected tokens")
+            if dkvp.paged_specs:
+                raise ValueError("a draft model keeps all its cache rows in one paged tensor")
             if on_gpu:
                 free, total = torch.cuda.mem_get_info(self.device)
                 d_budget = int(0.1 * (free - (1.0 - device_memory_utilization) * total))
@@ -189,6 +191,8 @@ class LLM:
         extra = {"tp": self.tp} if fam.supports_tp else {}
         if kvp.state_specs:
             extra["state"] = self.kv.state
+        if kvp.paged_specs:
+            extra["paged"] = self.kv.paged
         if ep_size > 1:
             from ..parallel.ep import EPContext
 

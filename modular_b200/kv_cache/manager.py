@@ -22,6 +22,9 @@ Families with recurrent layers add *state slots*: fixed-size tensors per request
 slot per live request, taken with its first pages and given back when it is released. A state cannot be shared or
 restored by prefix, so such caches run without prefix caching.
 
+Families whose layers keep different kinds of rows add *paged tensors* (``KVCacheParams.paged_specs``): further rows per
+token in the same pages, ``[num_pages, planes, page_size, width]``, addressed with the same block table and slots.
+
 Block hashes are chained: ``h_i = H(h_{i-1} || tokens of page i)`` with the request's salt
 folded into the seed; the final token of a prompt is never hashed, so a full-prompt hit
 still leaves one token to run (reference: block_manager.py:62, :91-98).
@@ -76,6 +79,8 @@ class KVCacheParams:
     enable_prefix_caching: bool = True
     # recurrent state per request: (name, shape of one slot, dtype)
     state_specs: tuple = ()
+    # further rows per token in the same pages, of the cache's dtype: (name, planes, width)
+    paged_specs: tuple = ()
 
     def __post_init__(self):
         if self.state_specs and self.enable_prefix_caching:
@@ -93,7 +98,8 @@ class KVCacheParams:
     @property
     def bytes_per_page(self) -> int:
         el = torch.empty(0, dtype=self.dtype).element_size()
-        return self.kv_dim * self.n_layers * self.n_kv_heads * self.page_size * self.head_dim * el
+        extra = sum(planes * width for _, planes, width in self.paged_specs)
+        return (self.kv_dim * self.n_layers * self.n_kv_heads * self.head_dim + extra) * self.page_size * el
 
     def shape(self, num_pages: int) -> tuple:
         return (num_pages, self.kv_dim, self.n_layers, self.n_kv_heads, self.page_size, self.head_dim)
@@ -131,6 +137,10 @@ class PagedKVCacheManager:
                                   if max_seq_len else num_pages)
         self.kv = (torch.zeros(params.shape(num_pages), dtype=params.dtype, device=self.device)
                    if allocate else None)
+        self.paged = ({name: torch.zeros((num_pages, planes, params.page_size, width), dtype=params.dtype, device=self.device)
+                       for name, planes, width in params.paged_specs} if allocate else {})
+        if params.paged_specs and host_pages > 0:
+            raise ValueError("the host and disk tiers of the cache hold keys and values only: not available with paged tensors")
         self._req: dict[str, _ReqState] = {}
         # recurrent state, one slot per live request: name -> [slots, *shape]
         if params.state_specs and state_slots < 1:

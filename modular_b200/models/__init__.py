@@ -134,6 +134,38 @@ def _vipotar_family() -> ModelFamily:
     return ModelFamily("vipotar", VipotarConfig, VipotarWeights, VipotarModel, kv, act)
 
 
+def _mavidra_family() -> ModelFamily:
+    from ..kv_cache import KVCacheParams
+    from .mavidra import GLA, LATENT, MavidraConfig, MavidraModel, MavidraWeights
+
+    def kv(cfg, page, dtype, prefix):
+        # keys and values of the parallel layers, latent rows as a further paged tensor; recurrent state (and the last token)
+        # in slots, which rule out prefix sharing
+        state, planes = cfg.state_specs(), len(cfg.of_type("parallel"))
+        return KVCacheParams(max(planes, 1), cfg.cache_heads, cfg.head_width if planes else 8, page, dtype, False, prefix and not state,
+                             state, cfg.paged_specs())
+
+    def act(cfg, T, B):
+        per_tok = 0
+        for i, l in enumerate(cfg.layers):
+            if l["type"] == LATENT:
+                a = cfg.latent(i)
+                n = a.heads * (a.head_width + 2 * a.cache_width + 2 * a.vdim_pad) + a.q_rank
+            elif l["type"] == GLA:
+                g = cfg.gla(i)
+                n = g.heads * (4 * g.dim8 + 6 * g.vdim8)
+            else:
+                a, d = cfg.attention(i), cfg.delta(i)
+                n = 2 * (a.heads_pad + a.kv_heads) * cfg.head_width + 8 * d.heads * (d.dim + d.vdim)
+            if l.get("mlp") is not None:
+                n = max(n, l["mlp"]["router"]["top"] * (2 * cfg.width_pad + l["mlp"]["expert"]["ff"]))
+            per_tok = max(per_tok, 6 * cfg.width_pad + n)
+        state = kv(cfg, 64, torch.bfloat16, False).state_bytes_per_slot
+        return T * per_tok * 4 + B * cfg.vocab_size * 4 + B * state + (256 << 20)
+
+    return ModelFamily("mavidra", MavidraConfig, MavidraWeights, MavidraModel, kv, act)
+
+
 def _bert_family() -> ModelFamily:
     from ..kv_cache import KVCacheParams
     from .bert import BertConfig, BertModel, BertWeights
@@ -151,7 +183,7 @@ def _bert_family() -> ModelFamily:
 def family_for(config) -> ModelFamily:
     """The family that serves `config` (matched on the config class)."""
     for make in (_llama_family, _deepseek_family, _mamba_family, _lfm2_family, _gotunex_family, _vipotar_family,
-                 _bert_family):
+                 _mavidra_family, _bert_family):
         fam = make()
         if isinstance(config, fam.config_class):
             return fam

@@ -1,12 +1,12 @@
-"""Gated delta rule with one decay per key channel, behind short convolutions (a linear-attention mixer).
+"""Gated delta rule with a decay per key channel or per head, behind short convolutions (a linear-attention mixer).
 
 Per head, with a state ``S`` [dim, vdim] kept in fp32:
 
     S <- diag(g) S;    u = beta (v - S^T k);    S <- S + k u^T;    o = S^T q
 
 q, k, v are projections that pass a causal depthwise convolution and silu, q and k are unit vectors, the decay is
-``g = exp(-exp(A_log) softplus(W_a2 W_a1 h + dt_bias))``, and the output is RMS-normed per head, scaled and gated by
-``sigmoid(W_g2 W_g1 h)``. What a sequence carries between steps is ``S`` of every head and the last ``taps - 1`` inputs
+``g = exp(-exp(A_log) softplus(a + dt_bias))`` with ``a = W_a2 W_a1 h`` per channel or ``a = W_a h`` per head, and the output is
+RMS-normed per head, scaled and gated by ``sigmoid(W_g2 W_g1 h)`` or ``silu(W_g h)``. What a sequence carries between steps is ``S`` of every head and the last ``taps - 1`` inputs
 of the convolutions: two tensors of the engine's state slots (``state_specs``), indexed by ``state_idx[s]`` (-1: start
 from zero and keep nothing), read when the step continues a sequence (``kv_len > q_len``).
 
@@ -56,9 +56,11 @@ class DeltaRuleConfig:
     dim: int
     vdim: int
     taps: int
-    decay_rank: int
-    gate_rank: int
+    decay_rank: int              # low-rank decays per channel and gates behind a sigmoid, or, with head_decay,
+    gate_rank: int               # one decay per head and a full-rank gate behind silu (both ranks unused)
     eps: float
+    head_decay: bool = False
+    out_mult: float = 1.0        # factor on the output
 
     @property
     def channels(self) -> int:
@@ -69,8 +71,10 @@ class DeltaRuleConfig:
         """(name, rows, first row) of the stacked input projection; every block starts at a multiple of 8 (the
         low-rank ones, which are GEMM inputs, are at least 64 wide)."""
         out, at = [], 0
+        tail = ((("g", self.heads * self.vdim), ("a", self.heads)) if self.head_decay else
+                (("a1", self.decay_rank), ("g1", self.gate_rank)))
         for name, n in (("q", self.kv_heads * self.dim), ("k", self.kv_heads * self.dim), ("v", self.heads * self.vdim),
-                        ("a1", self.decay_rank), ("g1", self.gate_rank), ("b", self.heads)):
+                        *tail, ("b", self.heads)):
             out.append((name, n, at))
             at += self.block_rows(name, n)
         return tuple(out)
@@ -92,8 +96,8 @@ def delta_step_reference(q, k, v, g, beta, S):
 
 
 class DeltaRule:
-    """Weights of one mixer. ``w_in``: the projections that read the layer input, stacked ``[q | k | v | a1 | g1 | b]``
-    (one GEMM); ``w_a2`` / ``w_g2``: the second halves of the low-rank decay and gate projections; ``w_o``."""
+    """Weights of one mixer. ``w_in``: the projections that read the layer input, stacked ``[q | k | v | a1 | g1 | b]`` or
+    ``[q | k | v | g | a | b]`` (one GEMM); ``w_a2`` / ``w_g2``: the second halves of low-rank decay and gate projections; ``w_o``."""
 
     def __init__(self, cfg: DeltaRuleConfig, tensors: dict, width_pad: int, device, dtype):
         """``tensors``: the mixer's tensors by their short names (``q``, ``q.conv``, ``a1``, ...)."""
@@ -101,9 +105,11 @@ class DeltaRule:
         put = lambda t, dt=dtype: t.to(device=device, dtype=dt).contiguous()
         self.w_in = put(torch.cat([pad_to(tensors[n], c.block_rows(n, rows), width_pad) for n, rows, _ in c.blocks]))
         self.off = {n: at for n, _, at in c.blocks}
+        self.in_rows = self.w_in.shape[0]
         self.conv_w = put(torch.cat([tensors[n + ".conv"] for n in "qkv"]))
-        self.w_a2 = put(pad_to(tensors["a2"], up8(c.heads * c.dim), c.block_rows("a1", c.decay_rank)))
-        self.w_g2 = put(pad_to(tensors["g2"], up8(c.heads * c.vdim), c.block_rows("g1", c.gate_rank)))
+        if not c.head_decay:
+            self.w_a2 = put(pad_to(tensors["a2"], up8(c.heads * c.dim), c.block_rows("a1", c.decay_rank)))
+            self.w_g2 = put(pad_to(tensors["g2"], up8(c.heads * c.vdim), c.block_rows("g1", c.gate_rank)))
         self.A_log = put(tensors["A_log"], torch.float32)
         self.dt_bias = put(tensors["dt_bias"], torch.float32)
         self.norm = put(tensors["norm"])
@@ -113,22 +119,30 @@ class DeltaRule:
         """x [T, width] -> [T, width]; ``lin`` is the GEMM for this step's size."""
         c, T, dev = self.cfg, x.shape[0], x.device
         px = lin(x, self.w_in)
-        a0, g0 = self.off["a1"], self.off["g1"]
-        z = ops.linear(px[:, a0: a0 + self.w_a2.shape[1]], self.w_a2, out_dtype=torch.float32)
-        gate = ops.linear(px[:, g0: g0 + self.w_g2.shape[1]], self.w_g2)
         width = self.w_o.shape[1]
         out = torch.empty(T, width, dtype=x.dtype, device=dev)
         if width != c.heads * c.vdim:
             out[:, c.heads * c.vdim:].zero_()
-        core = delta_rule_cuda if x.is_cuda else delta_rule_reference
-        core(self, px, z, gate, out, state, conv_state, state_idx, q_start, q_len, kv_len, one_token)
+        self.mix(px, out, state, conv_state, state_idx, q_start, q_len, kv_len, one_token)
         return lin(out, self.w_o)
+
+    def mix(self, px, out, state, conv_state, state_idx, q_start, q_len, kv_len, one_token: bool):
+        """From the stacked projection ``px`` to the gated heads, in the first heads * vdim columns of ``out``."""
+        c = self.cfg
+        if c.head_decay:
+            z, gate = None, px[:, self.off["g"]: self.off["g"] + c.heads * c.vdim]
+        else:
+            a0, g0 = self.off["a1"], self.off["g1"]
+            z = ops.linear(px[:, a0: a0 + self.w_a2.shape[1]], self.w_a2, out_dtype=torch.float32)
+            gate = ops.linear(px[:, g0: g0 + self.w_g2.shape[1]], self.w_g2)
+        core = delta_rule_cuda if px.is_cuda else delta_rule_reference
+        core(self, px, z, gate, out, state, conv_state, state_idx, q_start, q_len, kv_len, one_token)
 
 
 def delta_rule_cuda(m: DeltaRule, px, z, gate, out, state, conv_state, state_idx, q_start, q_len, kv_len, one_token):
     c, T = m.cfg, px.shape[0]
     dp = dim_pad(c.dim)
-    sizes = (T * c.kv_heads * dp, T * c.kv_heads * dp, T * c.heads * dp, T * c.heads * c.vdim, T * c.heads, T * c.kv_heads,
+    sizes = (T * c.kv_heads * dp, T * c.kv_heads * dp, T * c.heads * (1 if c.head_decay else dp), T * c.heads * c.vdim, T * c.heads, T * c.kv_heads,
              T * c.heads * c.vdim)
     ends, at = [], 0
     for n in sizes:                       # one allocation, every part 16-byte aligned
@@ -137,7 +151,7 @@ def delta_rule_cuda(m: DeltaRule, px, z, gate, out, state, conv_state, state_idx
     buf = torch.empty(at, dtype=torch.float32, device=px.device)
     _lib().delta_rule(px, m.off["q"], m.off["k"], m.off["v"], m.off["b"], m.conv_w, z, m.A_log, m.dt_bias, gate, m.norm, c.eps,
                       [buf[s: s + n] for s, n in ends], out, state, conv_state, state_idx, q_start, q_len, kv_len, c.heads,
-                      c.kv_heads, c.dim, c.vdim, one_token)
+                      c.kv_heads, c.dim, c.vdim, one_token, a_off=m.off.get("a", -1), gate_silu=c.head_decay, out_mult=c.out_mult)
 
 
 def delta_rule_reference(m: DeltaRule, px, z, gate, out, state, conv_state, state_idx, q_start, q_len, kv_len, one_token=False):
@@ -145,7 +159,8 @@ def delta_rule_reference(m: DeltaRule, px, z, gate, out, state, conv_state, stat
     H, KH, d, dv, W = c.heads, c.kv_heads, c.dim, c.vdim, c.taps
     raw = torch.cat([px[:, m.off[n]: m.off[n] + r].float() for n, r, _ in c.blocks[:3]], 1)
     beta = torch.sigmoid(px[:, m.off["b"]: m.off["b"] + H].float())
-    g = torch.exp(-torch.exp(m.A_log).view(1, H, 1) * F.softplus(z[:, : H * d].float() + m.dt_bias).view(-1, H, d))
+    a = px[:, m.off["a"]: m.off["a"] + H] if c.head_decay else z[:, : H * d]
+    g = torch.exp(-torch.exp(m.A_log).view(1, H, 1) * F.softplus(a.float() + m.dt_bias).view(a.shape[0], H, -1))
     rep = H // KH
     unit = lambda t: t / torch.sqrt((t * t).sum(-1, keepdim=True) + 1e-6)
     for s in range(q_len.numel()):
@@ -165,5 +180,6 @@ def delta_rule_reference(m: DeltaRule, px, z, gate, out, state, conv_state, stat
         if slot >= 0:
             state[slot, :, :, :d] = S
         o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + c.eps) * m.norm.float()
-        o = o.reshape(n, H * dv) * torch.sigmoid(gate[t0: t0 + n, : H * dv].float())
+        act = F.silu if c.head_decay else torch.sigmoid
+        o = o.reshape(n, H * dv) * act(gate[t0: t0 + n, : H * dv].float()) * c.out_mult
         out[t0: t0 + n, : H * dv] = o.to(out.dtype)

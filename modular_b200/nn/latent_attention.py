@@ -2,9 +2,9 @@
 (the normed key/value latent and a rotated key part that all heads share).
 
 Runs in the absorbed form for prefill and decode alike: ``q_lat = W_uk^T q`` per head, attention over the cached rows,
-``o = W_uv o_lat`` per head. Options: rotate-half or interleaved rotary pairs, a learned sink per head (a score without
-key or value in the softmax denominator), a sigmoid output gate, and reading another layer's cache rows (a layer
-without a key/value projection of its own).
+``o = W_uv o_lat`` per head. Options: rotate-half or interleaved rotary pairs, a sliding window, a learned sink per head (a
+score without key or value in the softmax denominator), a sigmoid output gate per value column or per head, and reading
+another layer's cache rows (a layer without a key/value projection of its own).
 
 Column layouts are padded for the kernels, with zeros: per head ``[dim -> multiple of 64 | rot_dim -> 64]`` for queries,
 ``[kv_rank -> a kernel size | rot_dim -> 64]`` for cache rows, vdim -> multiple of 8.
@@ -55,6 +55,9 @@ class LatentAttentionConfig:
     eps: float
     own_cache: bool = True   # False: the layer reads another layer's cache rows
     interleaved: bool = False
+    window: int = 0          # keys a query sees, itself included (0: all before it)
+    sink: bool = True
+    head_gate: bool = False  # the output gate is one number per head, applied inside the attention kernels
 
     @property
     def head_width(self) -> int:
@@ -102,7 +105,7 @@ class LatentAttention:
             parts.append(pad_to(t["dkv"], up8(n), width_pad))
             self.kv_off, at = at, at + up8(n)
         self.g_off = at
-        parts.append(pad_to(pad_heads(t["g"], H, c.vdim, vp), H * vp, width_pad))
+        parts.append(pad_to(t["g"], up8(H), width_pad) if c.head_gate else pad_to(pad_heads(t["g"], H, c.vdim, vp), H * vp, width_pad))
         self.w_in = put(torch.cat(parts))
         self.q_norm = put(t["dq.norm"])
         self.kv_norm = put(t["dkv.norm"]) if c.own_cache else None
@@ -118,7 +121,7 @@ class LatentAttention:
         uv = new(H, vp, Rp)
         uv[:, : c.vdim, : c.kv_rank] = t["uv"].view(H, c.vdim, c.kv_rank)
         self.w_uv = put(uv)                                          # [h, vdim, latent]: latent outputs to values
-        self.sink = put(t["sink"], torch.float32)
+        self.sink = put(t["sink"], torch.float32) if c.sink else None
         self.w_o = put(pad_to(pad_heads(t["o"].t().contiguous(), H, c.vdim, vp).t(), width_pad, gemm_k(H * vp)))
 
     def __call__(self, x, lin, cache, cos_sin, positions, slots, block_table, q_start, q_len, kv_len, one_token: bool):
@@ -134,13 +137,14 @@ class LatentAttention:
         ops.batched_linear_heads(q, self.w_uk, q_lat, c.head_width, Rp)
         q_rope = q.view(T, H, c.head_width)[:, :, dp:]
         o_lat = latent_attention(q_lat.view(T, H, Rp), q_rope, cache, block_table, q_start, q_len, kv_len, c.scale, self.sink,
-                                 one_token)
+                                 one_token, c.window, px[:, self.g_off: self.g_off + H] if c.head_gate else None)
         width = H * c.vdim_pad
         o = torch.empty(T, self.w_o.shape[1], dtype=x.dtype, device=x.device)
         if o.shape[1] != width:
             o[:, width:].zero_()
         ops.batched_linear_heads(o_lat.view(T, H * Rp), self.w_uv, o, Rp, c.vdim_pad)
-        ops.sigmoid_gate(o, px[:, self.g_off:], width)
+        if not c.head_gate:
+            ops.sigmoid_gate(o, px[:, self.g_off:], width)
         return lin(o, self.w_o)
 
 
@@ -179,14 +183,14 @@ def rotate_heads(x, heads, head_stride, dims, interleaved, positions, cos_sin):
         part.copy_(ops.reference.apply_rope(part.unsqueeze(1), cos, sin, interleaved).squeeze(1))
 
 
-def latent_attention(q_lat, q_rope, cache, block_table, q_start, q_len, kv_len, scale, sink=None, one_token=False):
-    """Absorbed attention over paged latent rows; returns [T, h, latent]."""
+def latent_attention(q_lat, q_rope, cache, block_table, q_start, q_len, kv_len, scale, sink=None, one_token=False, window=0, gate=None):
+    """Absorbed attention over paged latent rows; returns [T, h, latent]. ``gate`` [T, h]: heads are multiplied by its sigmoid."""
     if q_lat.is_cuda:
         out = torch.empty_like(q_lat)
         if q_lat.dtype == torch.bfloat16:
             ops.ensure_mla_split_workspace(q_lat.device)
         _lib().latent_attention(q_lat, q_rope, cache, block_table, q_start, q_len, kv_len, out, scale, sink, one_token,
-                                _split_ws(q_lat.device))
+                                _split_ws(q_lat.device), window=window, gate=gate)
         return out
     T, H, Rp = q_lat.shape
     LD, page = Rp + q_rope.shape[2], cache.shape[1]
@@ -196,10 +200,13 @@ def latent_attention(q_lat, q_rope, cache, block_table, q_start, q_len, kv_len, 
         t0, n, kl = int(q_start[s]), int(q_len[s]), int(kv_len[s])
         k = cache[block_table[s, : (kl + page - 1) // page].long()].reshape(-1, cache.shape[2])[:kl, :LD].float()
         sc = torch.einsum("qhd,kd->hqk", q[t0: t0 + n], k) * scale
-        late = torch.arange(kl).unsqueeze(0) > torch.arange(n).unsqueeze(1) + (kl - n)
-        sc = sc.masked_fill(late, float("-inf"))
+        dist = torch.arange(n).unsqueeze(1) + (kl - n) - torch.arange(kl).unsqueeze(0)
+        sc = sc.masked_fill((dist < 0) | (dist >= (window or kl)), float("-inf"))
         if sink is not None:
             sc = torch.cat([sc, sink.view(H, 1, 1).expand(H, n, 1)], -1)
         p = torch.softmax(sc, -1)[..., :kl]
-        out[t0: t0 + n] = torch.einsum("hqk,kd->qhd", p, k[:, :Rp]).to(out.dtype)
+        o = torch.einsum("hqk,kd->qhd", p, k[:, :Rp])
+        if gate is not None:
+            o = o * torch.sigmoid(gate[t0: t0 + n].float()).unsqueeze(2)
+        out[t0: t0 + n] = o.to(out.dtype)
     return out

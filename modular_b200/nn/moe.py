@@ -304,6 +304,62 @@ class TableRouter:
         return inverse.view(-1, table.shape[1]).int(), offsets
 
 
+@dataclass
+class ScoreRouterConfig:
+    """Sigmoid scores, a choice among the ``keep`` best of ``groups`` groups of neighbouring experts (a group counts its two
+    best choice scores), weights from the scores without the correction."""
+    experts: int
+    top: int
+    groups: int = 1
+    keep: int = 1
+    renormalize: bool = False
+    scaling: float = 1.0
+
+    def __post_init__(self):
+        if self.experts < 1 or self.groups < 1 or self.experts % self.groups:
+            raise ValueError(f"{self.experts} experts cannot form {self.groups} equal groups")
+        if not 1 <= self.keep <= self.groups or not 1 <= self.top <= self.keep * (self.experts // self.groups):
+            raise ValueError(f"{self.top} experts out of {self.keep} groups of {self.experts // self.groups}")
+        if self.top > 32 or self.experts > 1024:
+            raise ValueError("at most 32 of at most 1024 experts per token")
+
+
+class ScoreRouter:
+    """Router of one layer for experts whose rows are kept in expert order: ``route`` goes from the router's input to the rows
+    of every expert; the layer's seam weighs and adds what comes back."""
+
+    def __init__(self, cfg: ScoreRouterConfig, gate, correction, width_pad: int, device, dtype):
+        self.cfg = cfg
+        E8 = (cfg.experts + 7) // 8 * 8
+        self.gate = F.pad(gate, (0, width_pad - gate.shape[1], 0, E8 - gate.shape[0])).to(device=device, dtype=dtype).contiguous()
+        self.correction = None if correction is None else correction.to(device=device, dtype=torch.float32).contiguous()
+
+    def route(self, x, counts):
+        """x [T, width]; ``counts`` int32 [experts], zero. Returns (rows [T * top, width] in expert order, offsets int32
+        [experts + 1], inverse int32 [T, top]: row of every pair, weights fp32 [T, top])."""
+        c, T, dev = self.cfg, x.shape[0], x.device
+        logits = ops.linear(x, self.gate, out_dtype=torch.float32)
+        if not x.is_cuda:
+            m = MoEConfig(0, 0, c.experts, c.top, n_group=c.groups, topk_group=c.keep, norm_topk_prob=c.renormalize,
+                          routed_scaling_factor=c.scaling)
+            ids, w = route_group_limited_ref(logits[:, : c.experts], self.correction, m)
+            flat = ids.reshape(-1).long()
+            order = torch.argsort(flat, stable=True)
+            inverse = torch.empty_like(order)
+            inverse[order] = torch.arange(order.numel())
+            offsets = torch.zeros(c.experts + 1, dtype=torch.int32)
+            offsets[1:] = torch.cumsum(torch.bincount(flat, minlength=c.experts), 0)
+            return x[order // c.top], offsets, inverse.view(T, c.top).int(), w
+        i32 = lambda *s: torch.empty(*s, dtype=torch.int32, device=dev)
+        ids, rank, inverse, offsets = i32(T, c.top), i32(T, c.top), i32(T, c.top), i32(c.experts + 1)
+        w = torch.empty(T, c.top, dtype=torch.float32, device=dev)
+        L = _lib()
+        L.moe_score_route(logits, self.correction, ids, w, rank, counts, c.groups, c.keep, c.renormalize, c.scaling)
+        rows = torch.empty(T * c.top, x.shape[1], dtype=x.dtype, device=dev)
+        L.moe_place_rows(x, ids, rank, counts, offsets, inverse, rows)
+        return rows, offsets, inverse, w
+
+
 def expert_mlp(xp, offsets, w_gate_up, w_down, max_rows: int):
     """SwiGLU experts on rows already in expert order: xp [rows, H] -> [rows, H]; w_gate_up [E, 2I, H], w_down [E, H, I].
     ``max_rows`` bounds the rows of one expert (the step's tokens when a token's experts differ)."""

@@ -14,6 +14,11 @@ the next one in a single kernel (``csrc/kernels/residual_norm.cu``); the PyTorch
   before its first layer);
 * ``rows``: work on these rows of ``x`` only (the ones whose logits are wanted), outputs compacted.
 
+``sandwich_norm`` is the seam of layers that norm every branch before *and* after it, one branch at a time:
+``x += mult * norm(u; w_u, b_u)`` with ``u`` a branch output or the weighted sum of expert outputs in expert order, then
+``n1 = norm(x; w1, b1)``; layer norms with biases, RMS norms without. ``inject`` adds rows of a second table, chosen by ids of
+their own, to the embedding.
+
 The norm is computed in fp32 and rounded once.
 """
 
@@ -79,3 +84,45 @@ def residual_norm(x, ids=None, table=None, scale=1.0, a=None, b=None, e=None, in
                          float(pair_w), rows, w1, n1, w2, n2, scatter, cols or x.shape[1], store_x, float(eps),
                          x.shape[0] if rows is None else rows.numel(), norm_a, norm_b, float(ab_scale), c, float(mult), inject,
                          float(inject_scale), step)
+
+
+def sandwich_norm_reference(x, ids=None, table=None, scale=1.0, inject_ids=None, inject=None, a=None, e=None, inverse=None, pair_w=None,
+                            rows=None, w_u=None, b_u=None, mult=1.0, w1=None, b1=None, n1=None, cols=0, store_x=True, eps=1e-6):
+    cols = cols or x.shape[1]
+    idx = torch.arange(x.shape[0]) if rows is None else rows.long()
+
+    def norm(t, w, b):
+        d = t[:, :cols]
+        if b is not None:
+            d = d - d.mean(-1, keepdim=True)
+        y = torch.zeros_like(t)
+        y[:, :cols] = d * torch.rsqrt((d * d).mean(-1, keepdim=True) + eps) * w.float()[:cols]
+        if b is not None:
+            y[:, :cols] += b.float()[:cols]
+        return y
+
+    h = x[idx] if table is None else table[ids[idx]].float() * scale
+    if inject is not None:
+        h = h + inject[inject_ids[idx]].float()
+    u = None
+    if a is not None:
+        u = a[idx, : x.shape[1]].float()
+    elif e is not None:
+        inv = inverse[idx].long()
+        u = (e[inv.clamp(min=0)].float() * (pair_w[idx] * (inv >= 0)).unsqueeze(-1)).sum(1)
+    if u is not None:
+        h = h + mult * (u if w_u is None else norm(u, w_u, b_u))
+    if store_x:
+        x[idx] = h
+    if w1 is not None:
+        n1[: idx.numel()] = norm(h, w1, b1).to(n1.dtype)
+
+
+def sandwich_norm(x, ids=None, table=None, scale=1.0, inject_ids=None, inject=None, a=None, e=None, inverse=None, pair_w=None, rows=None,
+                  w_u=None, b_u=None, mult=1.0, w1=None, b1=None, n1=None, cols=0, store_x=True, eps=1e-6):
+    """x: fp32 [T, width], width padded to a multiple of 4 with zeros; ``cols`` is the true width."""
+    if not x.is_cuda:
+        return sandwich_norm_reference(x, ids, table, scale, inject_ids, inject, a, e, inverse, pair_w, rows, w_u, b_u, mult, w1, b1, n1,
+                                       cols, store_x, eps)
+    _lib().sandwich_norm(x, ids, table, float(scale), inject_ids, inject, a, e, inverse, pair_w, rows, w_u, b_u, float(mult), w1, b1, n1,
+                         cols or x.shape[1], store_x, float(eps), x.shape[0] if rows is None else rows.numel())

@@ -1,8 +1,11 @@
-"""Softmax attention over the keys of a sliding window, with grouped heads, partial rotation and a sink.
+"""Softmax attention over the keys of a sliding window, with grouped heads, partial rotation, a sink, and optionally normed
+queries and keys and an output gate per head.
 
 A query at position i sees the keys j with ``0 <= i - j < window`` (0: all before it). Queries and keys rotate in
-neighbouring pairs over their first ``rot_dims`` dimensions. ``sink`` is one score per query head that takes part in the
-softmax denominator only: ``p_j = exp(s_j) / (exp(sink) + sum_j exp(s_j))``.
+neighbouring pairs (or pairs half the rotated width apart, ``halves``) over their first ``rot_dims`` dimensions; ``qk_norm``
+RMS-norms every head of both before that. ``sink`` is one score per query head that takes part in the softmax denominator
+only: ``p_j = exp(s_j) / (exp(sink) + sum_j exp(s_j))``. ``head_gate`` multiplies a head's output by ``sigmoid(W_g h)``, inside
+the attention kernels; ``out_mult`` is a further factor on it.
 
 The cache is the paged key/value cache of the grouped-query families ``[pages, 2, planes, kv heads, page, head width]``.
 Keys and values share one head width, zero-padded: 64 or 128 where the tensor-core kernels fit (``head_width``), and the
@@ -45,12 +48,20 @@ class WindowAttentionConfig:
     rope_scaling: Optional[RopeScaling] = None
     window: int = 0                  # 0: every key before the query
     zero_sink: bool = False          # a sink of score 0 for every head
+    sink: bool = False               # a learned sink
+    halves: bool = False             # pairs (i, i + rot_dims / 2)
+    qk_norm: bool = False
+    eps: float = 1e-6                # of those norms
+    head_gate: bool = False
+    out_mult: float = 1.0            # needs head_gate
 
     def __post_init__(self):
         if self.heads % self.kv_heads:
             raise ValueError(f"{self.heads} heads are no multiple of {self.kv_heads} key/value heads")
         if self.rot_dims % 2 or self.rot_dims > self.dim:
             raise ValueError(f"{self.rot_dims} rotated dimensions of {self.dim}")
+        if self.out_mult != 1.0 and not self.head_gate:
+            raise ValueError("a factor on the output is part of the head gate")
         if self.window < 0:
             raise ValueError("a window holds at least the token itself")
 
@@ -88,8 +99,8 @@ def tensor_core_plan(group: int, hd: int, dtype, page: int, q_start, q_len, T: i
 
 
 class WindowAttention:
-    """Weights of one attention mixer. ``w_in``: rows ``[q | k | v]`` of a stacked input projection, every head ``hd`` wide;
-    ``w_o`` [width, heads_pad * hd]."""
+    """Weights of one attention mixer. ``w_in``: rows ``[q | k | v | gate]`` of a stacked input projection, every head ``hd``
+    wide (the gate has one row per padded head); ``w_o`` [width, heads_pad * hd]."""
 
     def __init__(self, cfg: WindowAttentionConfig, tensors: dict, hd: int, width_pad: int, device, dtype):
         c = self.cfg = cfg
@@ -100,29 +111,48 @@ class WindowAttention:
             t = t.view(KH, group, d, t.shape[1])
             return F.pad(t, (0, width_pad - t.shape[3], 0, hd - d, 0, group_pad - group)).reshape(-1, width_pad)
 
-        self.w_in = torch.cat([rows(tensors["q"], G, Gp, c.dim), rows(tensors["k"], 1, 1, c.dim), rows(tensors["v"], 1, 1, c.vdim)])
+        per_head = lambda t: F.pad(t.view(KH, G), (0, Gp - G)).reshape(-1)
+        parts = [rows(tensors["q"], G, Gp, c.dim), rows(tensors["k"], 1, 1, c.dim), rows(tensors["v"], 1, 1, c.vdim)]
+        self.g_off = (c.heads_pad + 2 * KH) * hd
+        if c.head_gate:
+            g = F.pad(tensors["g"].view(KH, G, -1), (0, width_pad - tensors["g"].shape[1], 0, Gp - G)).reshape(-1, width_pad)
+            parts.append(F.pad(g, (0, 0, 0, up8(c.heads_pad) - c.heads_pad)))
+        self.w_in = torch.cat(parts)
         o = tensors["o"]
         o = F.pad(o.view(o.shape[0], KH, G, c.vdim), (0, hd - c.vdim, 0, Gp - G)).reshape(o.shape[0], -1)
         self.w_o = F.pad(o, (0, 0, 0, width_pad - o.shape[0])).to(device=device, dtype=dtype).contiguous()
         self.k_off, self.v_off = c.heads_pad * hd, (c.heads_pad + KH) * hd
-        self.in_rows = (c.heads_pad + 2 * KH) * hd
+        self.in_rows = self.w_in.shape[0]
         self.sink = torch.zeros(c.heads_pad, dtype=torch.float32, device=device) if c.zero_sink else None
+        if c.sink:
+            self.sink = per_head(tensors["sink"].float()).to(device=device).contiguous()
+        norm = lambda t: F.pad(t, (0, hd - c.dim)).to(device=device, dtype=dtype).contiguous()
+        self.q_norm, self.k_norm = (norm(tensors["q.norm"]), norm(tensors["k.norm"])) if c.qk_norm else (None, None)
 
-    def __call__(self, q, kv, plane: int, block_table, q_start, q_len, kv_len, plan: Optional[AttentionPlan]):
+    def prep(self, px, positions, cos_sin, slots, kv, plane: int):
+        """Norms and rotation of the queries in place, and of the keys on their way into the cache with the values."""
+        c = self.cfg
+        block_prep(px, c.heads_pad, self.k_off, self.v_off, c.kv_heads, c.rot_dims, positions, cos_sin, slots, kv, plane,
+                   q_norm=self.q_norm, k_norm=self.k_norm, norm_dim=c.dim, eps=c.eps, halves=c.halves)
+
+    def __call__(self, q, kv, plane: int, block_table, q_start, q_len, kv_len, plan: Optional[AttentionPlan], out=None, gate=None):
         """q [T, heads_pad * hd]: rotated queries; the step's keys and values are in the cache. Returns [T, heads_pad * hd]."""
-        c, out = self.cfg, torch.empty(q.shape[0], self.w_o.shape[1], dtype=q.dtype, device=q.device)
+        c = self.cfg
+        if out is None:
+            out = torch.empty(q.shape[0], self.w_o.shape[1], dtype=q.dtype, device=q.device)
         return window_attention(q, kv, plane, block_table, q_start, q_len, kv_len, c.heads_pad, c.kv_heads, c.scale, c.window,
-                                self.sink, plan, out)
+                                self.sink, plan, out, gate, c.out_mult)
 
 
-def window_attention(q, kv, plane, block_table, q_start, q_len, kv_len, heads, kv_heads, scale, window=0, sink=None, plan=None, out=None):
+def window_attention(q, kv, plane, block_table, q_start, q_len, kv_len, heads, kv_heads, scale, window=0, sink=None, plan=None, out=None,
+                     gate=None, gate_mult=1.0):
     hd = kv.shape[5]
     if out is None:
         out = torch.empty(q.shape[0], heads * hd, dtype=q.dtype, device=q.device)
     if q.is_cuda:
         p = plan or AttentionPlan()
         _lib().window_attention(q, out, kv, plane, block_table, q_start, q_len, kv_len, p.tile_seq, p.tile_q0, p.decode_seq, heads,
-                                kv_heads, scale, window, sink)
+                                kv_heads, scale, window, sink, gate, gate_mult)
         return out
     page = kv.shape[4]
     for s in range(q_len.numel()):
@@ -136,30 +166,43 @@ def window_attention(q, kv, plane, block_table, q_start, q_len, kv_len, heads, k
         if sink is not None:
             score = torch.cat([score, sink.view(-1, 1, 1).expand(-1, n, 1)], 2)
         w = torch.softmax(score, -1)[..., :total]
-        out[t0: t0 + n] = torch.einsum("htj,jhd->thd", w, v).reshape(n, -1).to(out.dtype)
+        o = torch.einsum("htj,jhd->thd", w, v)
+        if gate is not None:
+            o = o * (gate_mult * torch.sigmoid(gate[t0: t0 + n].float())).unsqueeze(2)
+        out[t0: t0 + n] = o.reshape(n, -1).to(out.dtype)
     return out
 
 
-def block_prep(x, heads, k_off, v_off, kv_heads, dims, positions, cos_sin, slots, kv, plane, silu=(0, 0), relu2=(0, 0)):
+def block_prep(x, heads, k_off, v_off, kv_heads, dims, positions, cos_sin, slots, kv, plane, silu=(0, 0), relu2=(0, 0), q_norm=None,
+               k_norm=None, norm_dim=0, eps=1e-6, halves=False):
     """What lies between the stacked input projection ``x`` of a parallel block and its branches, in one launch: queries
     (columns from 0) rotate in place, keys rotate and go into the cache with the values, ``silu`` and ``relu2`` (squared
-    relu) name column ranges (first, count) that are activated in place."""
+    relu) name column ranges (first, count) that are activated in place. ``q_norm`` / ``k_norm`` [head width]: heads are RMS-normed
+    over their first ``norm_dim`` columns first. ``halves``: pairs lie ``dims / 2`` apart. These two exclude the activations."""
     if x.is_cuda:
-        _lib().block_prep(x, 0, heads, k_off, v_off, kv_heads, dims, positions, cos_sin, slots, kv, plane, *silu, *relu2)
+        _lib().block_prep(x, 0, heads, k_off, v_off, kv_heads, dims, positions, cos_sin, slots, kv, plane, *silu, *relu2, q_norm=q_norm,
+                          k_norm=k_norm, norm_dim=norm_dim, eps=eps, halves=halves)
         return
     T, hd, page = x.shape[0], kv.shape[5], kv.shape[4]
 
-    def rotated(t):
+    def rotated(t, w):
         t = t.float().clone()
-        if dims:
+        if w is not None:
+            t *= torch.rsqrt(t.pow(2).sum(-1, keepdim=True) / (norm_dim or hd) + eps) * w.float()
+        if dims and halves:
+            cs = cos_sin[positions.long()].unsqueeze(1)
+            c, s = cs[..., : dims // 2], cs[..., dims // 2:]
+            u, v = t[..., : dims // 2].clone(), t[..., dims // 2: dims].clone()
+            t[..., : dims // 2], t[..., dims // 2: dims] = u * c - v * s, v * c + u * s
+        elif dims:
             cs = cos_sin[positions.long()].unsqueeze(1)
             c, s = cs[..., : dims // 2], cs[..., dims // 2:]
             u, v = t[..., 0:dims:2].clone(), t[..., 1:dims:2].clone()
             t[..., 0:dims:2], t[..., 1:dims:2] = u * c - v * s, v * c + u * s
         return t
 
-    x[:, : heads * hd] = rotated(x[:, : heads * hd].reshape(T, heads, hd)).reshape(T, -1).to(x.dtype)
-    k = rotated(x[:, k_off: k_off + kv_heads * hd].reshape(T, kv_heads, hd)).to(kv.dtype)
+    x[:, : heads * hd] = rotated(x[:, : heads * hd].reshape(T, heads, hd), q_norm).reshape(T, -1).to(x.dtype)
+    k = rotated(x[:, k_off: k_off + kv_heads * hd].reshape(T, kv_heads, hd), k_norm).to(kv.dtype)
     v = x[:, v_off: v_off + kv_heads * hd].reshape(T, kv_heads, hd)
     ok = slots >= 0
     pg, off = slots[ok] // page, slots[ok] % page

@@ -362,6 +362,13 @@ def _register_builtin() -> None:
         name="Vipotar", config_class=VipotarConfig, weights_class=VipotarWeights, model_class=VipotarModel,
         default_encoding="bfloat16", supported_encodings=("bfloat16", "float32"), example_repo_ids=(),
         preset_configs={"tiny-vipotar": VipotarConfig.tiny}), allow_override=True)
+    from ..models.mavidra import MavidraConfig, MavidraModel, MavidraWeights
+
+    # gated linear attention, windowed latent attention, and softmax attention beside a delta rule, with routed experts
+    PIPELINE_REGISTRY.register(SupportedArchitecture(
+        name="Mavidra", config_class=MavidraConfig, weights_class=MavidraWeights, model_class=MavidraModel,
+        default_encoding="bfloat16", supported_encodings=("bfloat16", "float32"), example_repo_ids=(),
+        preset_configs={"tiny-mavidra": MavidraConfig.tiny}), allow_override=True)
     from ..models.bert import BertConfig, BertModel, BertWeights
 
     # encoder-only embedding models (bidirectional attention; MPNet adds relative-position biases); embeddings only

@@ -89,6 +89,8 @@ def export_pages(kv_manager, request_id: str, n_tokens: int) -> torch.Tensor:
     """Copy of the pages holding the first ``n_tokens`` tokens of a request."""
     if kv_manager.params.state_specs:
         raise ValueError("a request with recurrent state cannot be moved by its cache pages alone")
+    if kv_manager.params.paged_specs:
+        raise ValueError("pages with further paged tensors are not moved")
     n = (n_tokens + kv_manager.page_size - 1) // kv_manager.page_size
     idx = torch.as_tensor(kv_manager.blocks_of(request_id)[:n], device=kv_manager.kv.device)
     return kv_manager.kv.index_select(0, idx)
