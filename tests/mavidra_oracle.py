@@ -7,6 +7,11 @@ import math
 import torch
 
 DT = torch.float64
+ROUND = lambda x: x              # applied to the inputs and outputs of matrix products: tests set it to see what rounding does
+
+
+def linear(x, w):
+    return ROUND(ROUND(x) @ w.T)
 
 
 def sigmoid(z):
@@ -52,14 +57,12 @@ def embedding(tokens, w, spec):
 def rotate(x, rot, first_position=0, halves=True):
     """x [T, heads, d]: pairs (i, i + dims / 2) of the first ``dims`` values turn (neighbours when not ``halves``)."""
     n = rot["dims"]
-    out = x.clone()
-    for p in range(x.shape[0]):
-        for i in range(n // 2):
-            a = (first_position + p) * rot["base"] ** (-2.0 * i / n)
-            iu, iv = (i, i + n // 2) if halves else (2 * i, 2 * i + 1)
-            u, v = x[p, :, iu], x[p, :, iv]
-            out[p, :, iu] = u * math.cos(a) - v * math.sin(a)
-            out[p, :, iv] = v * math.cos(a) + u * math.sin(a)
+    i = torch.arange(n // 2)
+    a = (first_position + torch.arange(x.shape[0], dtype=DT)).view(-1, 1) * float(rot["base"]) ** (-2.0 * i.to(DT) / max(n, 1))
+    cos, sin = torch.cos(a).to(x.dtype).unsqueeze(1), torch.sin(a).to(x.dtype).unsqueeze(1)
+    iu, iv = (i, i + n // 2) if halves else (2 * i, 2 * i + 1)
+    u, v, out = x[..., iu], x[..., iv], x.clone()
+    out[..., iu], out[..., iv] = u * cos - v * sin, v * cos + u * sin
     return out
 
 
@@ -92,12 +95,12 @@ def grouped_attention(q, k, v, scale, sink=None, window=None):
 
 def left_mixer(h, w, p, m, eps):
     T, H, G, d, dv = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    q = rotate(rms((h @ w[p + "q"].T).view(T, H, d), w[p + "q.norm"], eps), m["rot"])
-    k = rotate(rms((h @ w[p + "k"].T).view(T, G, d), w[p + "k.norm"], eps), m["rot"])
-    v = (h @ w[p + "v"].T).view(T, G, dv)
+    q = rotate(rms(linear(h, w[p + "q"]).view(T, H, d), w[p + "q.norm"], eps), m["rot"])
+    k = rotate(rms(linear(h, w[p + "k"]).view(T, G, d), w[p + "k.norm"], eps), m["rot"])
+    v = linear(h, w[p + "v"]).view(T, G, dv)
     o = grouped_attention(q, k, v, m["scale"], w[p + "sink"])
-    o = o * sigmoid(h @ w[p + "g"].T).unsqueeze(2)
-    return o.reshape(T, H * dv) @ w[p + "o"].T
+    o = o * sigmoid(linear(h, w[p + "g"])).unsqueeze(2)
+    return linear(o.reshape(T, H * dv), w[p + "o"])
 
 
 def short_conv(x, taps):
@@ -127,16 +130,16 @@ def delta_scan(q, k, v, g, beta, state=None):
 
 def right_mixer(h, w, p, m, eps):
     T, H, G, d, dv = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
-    conv = lambda n: silu(short_conv(h @ w[p + n].T, w[p + n + ".conv"]))
+    conv = lambda n: silu(short_conv(linear(h, w[p + n]), w[p + n + ".conv"]))
     group = torch.arange(H) // (H // G)
     q = unit(conv("q").view(T, G, d))[:, group] * d ** -0.5
     k = unit(conv("k").view(T, G, d))[:, group]
     v = conv("v").view(T, H, dv)
-    beta = sigmoid(h @ w[p + "b"].T)
-    g = torch.exp(-torch.exp(w[p + "A_log"]) * softplus(h @ w[p + "a"].T + w[p + "dt_bias"]))
+    beta = sigmoid(linear(h, w[p + "b"]))
+    g = torch.exp(-torch.exp(w[p + "A_log"]) * softplus(linear(h, w[p + "a"]) + w[p + "dt_bias"]))
     o, _ = delta_scan(q, k, v, g, beta)
-    o = rms(o, w[p + "norm"], eps) * silu(h @ w[p + "g"].T).view(T, H, dv)
-    return o.reshape(T, H * dv) @ w[p + "o"].T
+    o = rms(o, w[p + "norm"], eps) * silu(linear(h, w[p + "g"])).view(T, H, dv)
+    return linear(o.reshape(T, H * dv), w[p + "o"])
 
 
 def parallel_mixer(h, w, p, m, eps):
@@ -156,19 +159,19 @@ def gla_scan(q, k, v, alpha, state=None):
 
 def gla_mixer(h, w, p, m, eps):
     T, H, d, dv = h.shape[0], m["heads"], m["dim"], m["vdim"]
-    q = (h @ w[p + "q"].T).view(T, H, d) * d ** -0.5
-    k = (h @ w[p + "k"].T).view(T, H, d)
-    v = (h @ w[p + "v"].T).view(T, H, dv)
-    z = h @ w[p + "a1"].T @ w[p + "a2"].T + w[p + "a2.b"]
+    q = linear(h, w[p + "q"]).view(T, H, d) * d ** -0.5
+    k = linear(h, w[p + "k"]).view(T, H, d)
+    v = linear(h, w[p + "v"]).view(T, H, dv)
+    z = linear(linear(h, w[p + "a1"]), w[p + "a2"]) + w[p + "a2.b"]
     alpha = torch.exp(-softplus(-z) / m["tau"]).view(T, H, d)            # sigmoid(z) ** (1 / tau)
     o, _ = gla_scan(q, k, v, alpha)
-    o = rms(o, w[p + "norm"], eps).reshape(T, H * dv) * silu(h @ w[p + "g"].T)
-    return o @ w[p + "o"].T
+    o = rms(o, w[p + "norm"], eps).reshape(T, H * dv) * silu(linear(h, w[p + "g"]))
+    return linear(o, w[p + "o"])
 
 
 def latent_rows(h, w, p, m, eps):
     """What the cache keeps of a layer: the normed latent [T, kv_rank] and the rotated key part [T, rot_dim]."""
-    kv = h @ w[p + "dkv"].T
+    kv = linear(h, w[p + "dkv"])
     c = rms(kv[:, : m["kv_rank"]], w[p + "dkv.norm"], eps)
     return c, rotate(kv[:, m["kv_rank"]:].unsqueeze(1), m["rot"], halves=False).squeeze(1)
 
@@ -177,13 +180,13 @@ def latent_mixer(h, w, p, m, eps, rows):
     """``rows``: the layer's own latent rows, or those of the layer it shares with."""
     T, H, d, r, dv = h.shape[0], m["heads"], m["dim"], m["rot_dim"], m["vdim"]
     c, kr = rows
-    q = (rms(h @ w[p + "dq"].T, w[p + "dq.norm"], eps) @ w[p + "uq"].T).view(T, H, d + r)
+    q = linear(rms(linear(h, w[p + "dq"]), w[p + "dq.norm"], eps), w[p + "uq"]).view(T, H, d + r)
     q = torch.cat([q[..., :d], rotate(q[..., d:], m["rot"], halves=False)], 2)
-    k = torch.cat([(c @ w[p + "uk"].T).view(T, H, d), kr.unsqueeze(1).expand(T, H, r)], 2)
-    v = (c @ w[p + "uv"].T).view(T, H, dv)
+    k = torch.cat([linear(c, w[p + "uk"]).view(T, H, d), kr.unsqueeze(1).expand(T, H, r)], 2)
+    v = linear(c, w[p + "uv"]).view(T, H, dv)
     o = grouped_attention(q, k, v, m["scale"], window=m["mask"]["size"])
-    o = o * sigmoid(h @ w[p + "g"].T).unsqueeze(2)
-    return o.reshape(T, H * dv) @ w[p + "o"].T
+    o = o * sigmoid(linear(h, w[p + "g"])).unsqueeze(2)
+    return linear(o.reshape(T, H * dv), w[p + "o"])
 
 
 def choose(scores, correction, router):
@@ -200,14 +203,26 @@ def choose(scores, correction, router):
     return sorted(open_, key=lambda e: (-float(choice[e]), e))[: router["top"]]
 
 
+def choice_margin(scores, correction, router):
+    """How far the nearest other choice of experts is, in choice scores: what an implementation that rounds may get wrong."""
+    choice, n = scores + correction, router["groups"]["count"]
+    size, keep, top = choice.shape[0] // n, router["groups"]["keep"], router["top"]
+    best = torch.stack([choice[g * size: (g + 1) * size].sort(descending=True).values[:2].sum() for g in range(n)])
+    order = best.argsort(descending=True)
+    gap = best[order[keep - 1]] - best[order[keep]] if keep < n else torch.tensor(math.inf)
+    open_ = torch.cat([choice[g * size: (g + 1) * size] for g in order[:keep]]).sort(descending=True).values
+    return min(float(gap), float(open_[top - 1] - open_[top]) if top < len(open_) else math.inf)
+
+
 def moe(h, w, p, ff):
+    h = ROUND(h)
     s = sigmoid(h @ w[p + "router"].T)
     rows = []
     for t in range(h.shape[0]):
         y = torch.zeros(h.shape[1], dtype=h.dtype)
         for e in choose(s[t], w[p + "correction"], ff["router"]):
-            a = silu(w[f"{p}e{e}.gate"] @ h[t]) * (w[f"{p}e{e}.up"] @ h[t])
-            y = y + s[t, e] * (w[f"{p}e{e}.down"] @ a)
+            a = silu(linear(h[t], w[f"{p}e{e}.gate"])) * linear(h[t], w[f"{p}e{e}.up"])
+            y = y + s[t, e] * linear(a, w[f"{p}e{e}.down"])
         rows.append(y)
     return torch.stack(rows)
 
@@ -234,4 +249,4 @@ def forward(cfg, w, tokens):
         if l.get("mlp") is not None:
             x = x + mult * norm(moe(norm(x, p + "norm2"), w, p + "mlp.", l["mlp"]), p + "norm2b")
         stream.append(x)
-    return norm(x, "final.norm") @ w["embed"].T, torch.stack(stream)
+    return linear(norm(x, "final.norm"), w["embed"]), torch.stack(stream)
