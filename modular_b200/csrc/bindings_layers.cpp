@@ -296,7 +296,7 @@ void delta_rule(const Tensor& x, int q_off, int k_off, int v_off, int b_off, con
 void gla(const Tensor& x, int q_off, int k_off, int v_off, const Tensor& z, const Tensor& z_bias, double q_scale, double inv_tau,
          const Tensor& gate, bool gate_silu, double out_mult, const Tensor& norm_w, double eps, int norm_dim, Tensor& o, Tensor& out,
          Tensor& state, const Tensor& state_idx, const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, int heads, int dim,
-         int vdim, bool one_token) {
+         int vdim, bool one_token, bool allow_chunks) {
   MbGla p = {};
   const at::ScalarType st = x.scalar_type();
   p.T = x.size(0); p.B = q_len.numel(); p.heads = heads; p.dim = dim; p.vdim = vdim; p.one_token = one_token;
@@ -321,7 +321,17 @@ void gla(const Tensor& x, int q_off, int k_off, int v_off, const Tensor& z, cons
   p.state = state.data_ptr<float>();
   p.state_idx = i32(state_idx, p.B, "state_idx"); p.q_start = i32(q_start, p.B, "q_start");
   p.q_len = i32(q_len, p.B, "q_len"); p.kv_len = i32(kv_len, p.B, "kv_len");
-  check_rc(mb_gla(&p, dtype_of(x, "x"), num_sms(), cur_stream()), "gla");
+  const int dt = dtype_of(x, "x"), chunks = allow_chunks ? mb_gla_chunks(&p, dt) : 0;
+  Tensor plan, qk, ends;
+  if (chunks > 0) {
+    plan = at::empty({2, chunks}, q_start.options());
+    qk = at::empty({chunks, heads, 4, 64, p.dim_pad}, x.options());
+    ends = at::empty({chunks, heads, p.dim_pad}, z.options());
+    int32_t* t = plan.data_ptr<int32_t>();
+    check_rc(mb_attention_plan(p.q_len, p.B, 64, chunks, t, t + chunks, cur_stream()), "gla plan");
+    p.tile_seq = t; p.tile_q0 = t + chunks; p.n_tiles = chunks; p.qk = qk.data_ptr(); p.ends = ends.data_ptr<float>();
+  }
+  check_rc(mb_gla(&p, dt, num_sms(), cur_stream()), "gla");
 }
 
 // the cache [pages, 2, planes, kv heads, page, head width] at one plane
@@ -489,7 +499,10 @@ void mb::bind_layers(py::module_& m) {
         py::arg("out"), py::arg("state"), py::arg("conv_state"), py::arg("state_idx"), py::arg("q_start"), py::arg("q_len"),
         py::arg("kv_len"), py::arg("heads"), py::arg("kv_heads"), py::arg("dim"), py::arg("vdim"), py::arg("one_token"),
         py::arg("a_off") = -1, py::arg("gate_silu") = false, py::arg("out_mult") = 1.0);
-  m.def("gla", &gla);
+  m.def("gla", &gla, py::arg("x"), py::arg("q_off"), py::arg("k_off"), py::arg("v_off"), py::arg("z"), py::arg("z_bias"), py::arg("q_scale"),
+        py::arg("inv_tau"), py::arg("gate"), py::arg("gate_silu"), py::arg("out_mult"), py::arg("norm_w"), py::arg("eps"), py::arg("norm_dim"),
+        py::arg("o"), py::arg("out"), py::arg("state"), py::arg("state_idx"), py::arg("q_start"), py::arg("q_len"), py::arg("kv_len"),
+        py::arg("heads"), py::arg("dim"), py::arg("vdim"), py::arg("one_token"), py::arg("allow_chunks") = true);
   m.def("sandwich_norm", &sandwich_norm);
   m.def("bigram_rows", [](const Tensor& tokens, const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, const Tensor& state_idx,
                           Tensor& last, Tensor& out, int64_t mul_prev, int64_t mul_cur, int64_t buckets) {

@@ -357,7 +357,11 @@ typedef struct {
   float* state;                                          // [slots, heads, vdim, dim_pad]
   const int32_t *state_idx, *q_start, *q_len, *kv_len;
   int T, B, heads, dim, dim_pad, vdim, one_token;
+  // long steps in bf16 run in chunks of 64 tokens (mb_gla_chunks says how many at most; 0: token by token): a plan of the chunks
+  // made by mb_attention_plan, [chunks, heads, 4, 64, dim_pad] bf16 and [chunks, heads, dim_pad] fp32 of scratch
+  const int32_t *tile_seq, *tile_q0; int n_tiles; void* qk; float* ends;
 } MbGla;
+int mb_gla_chunks(const MbGla* p, int dtype);
 int mb_gla(const MbGla* p, int dtype, int num_sms, cudaStream_t stream);
 
 // ---- fp32 products (gemm_simt.cu) ------------------------------------------------------------

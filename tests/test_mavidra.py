@@ -383,6 +383,36 @@ def test_gated_linear_attention_remembers_one_token(gap, device, dtype):
                want[20 + gap]) > 0.2                                                            # without that token: something else
 
 
+@pytest.mark.gpu
+@pytest.mark.parametrize("H,d,dv", [(2, 8, 8), (3, 64, 64), (5, 96, 72), (2, 128, 128), (1, 40, 200), (4, 32, 256)])
+@pytest.mark.parametrize("pace", [0.02, 1.0, 6.0, 40.0])
+def test_gated_linear_chunks_agree_with_the_scan(H, d, dv, pace):
+    """Chunks on the tensor cores against the fp32 token loop on the same values: sequences that begin, go on, end inside a chunk or
+    have one token, decays from none to all within a token (some channels fast beside slow ones)."""
+    from modular_b200._native import lib
+
+    lens, old, slots = [150, 1, 64, 2, 200, 63], [0, 5, 64, 7, 130, 1], [3, 0, 5, -1, 1, 6]
+    T = sum(lens)
+    r = lambda *s, seed: rand(*s, seed=seed).cuda()
+    cols = H * (2 * d + 2 * dv)
+    x, w = r(T, cols, seed=d).bfloat16(), (1.0 + 0.1 * r(dv, seed=1)).bfloat16()
+    z = pace * torch.where(torch.arange(H * d).cuda() % 3 > 0, -1.0, 0.3) * r(T, H * d, seed=2).abs()
+    bias, pad = r(H * d, seed=3), next(n for n in (32, 64, 96, 128) if d <= n)
+    idx, ql = i32(*slots).cuda(), i32(*lens).cuda()
+    kl, qs = (ql + i32(*old).cuda()).int(), (torch.cumsum(ql, 0) - ql).int()
+    init = r(8, H, dv, pad, seed=4)
+    init[..., d:] = 0
+    got = []
+    for dtype in (torch.bfloat16, torch.float32):
+        xx, st = x.to(dtype), init.clone()
+        o, out = torch.empty(T, H * dv, device="cuda"), torch.empty(T, H * dv, dtype=dtype, device="cuda")
+        lib().gla(xx, 0, H * d, 2 * H * d, z, bias, d ** -0.5, 1.0, xx[:, H * (2 * d + dv):], True, 0.9, w.to(dtype), 1e-5, dv, o, out, st, idx, qs,
+                  ql, kl, H, d, dv, False)
+        got.append((o, out, st))
+    assert rel(got[0][2], got[1][2].cpu()) < 2e-5 and rel(got[0][0], got[1][0].cpu()) < 3e-5 and rel(got[0][1], got[1][1].cpu()) < 5e-3
+    assert torch.equal(got[0][2][[2, 4, 7]], init[[2, 4, 7]]) and got[0][2].isfinite().all()
+
+
 @pytest.mark.parametrize("device,dtype", RUNS)
 def test_recurrences_without_a_slot(device, dtype):
     """Sequences with slot -1 start from zero and keep nothing (the dummies of a padded decode batch)."""
