@@ -75,6 +75,7 @@ def run_kernels(s: dict, name: str, prefill: int = 2048, seqs: int = 4, batch: i
     from ..nn.delta_rule import DeltaRule, DeltaRuleConfig, delta_rule_cuda
     from ..nn.gated_linear_attention import GatedLinearAttention, GatedLinearConfig
     from ..nn.latent_attention import latent_attention
+    from ..nn.moe import TableRouter
     from ..nn.residual import residual_norm, sandwich_norm
     from ..nn.rotary_embedding import cos_sin_table
     from ..nn.window_attention import block_prep, tensor_core_plan, window_attention
@@ -193,11 +194,11 @@ def run_kernels(s: dict, name: str, prefill: int = 2048, seqs: int = 4, batch: i
         gm.a_bias, gm.norm, gx = torch.zeros(h * e, device="cuda"), bf(e), bf(T, 4 * h * e)
         add("gated linear attention", "delta rule", phase, lambda: gm.mix(gx, z, out, st, idx, qs, ql, kl_new, one), like,
             T * h * e * (8.0 + 4.0 + 2.0) + state, 5.0 * T * h * e * e, FP32_TFLOPS, lby, lfl)
-        # --- bigram rows, beside the other kernel that looks a row up by token id
-        toks, last, table = torch.randint(0, 1000, (T,), device="cuda"), torch.zeros(B, 1, dtype=torch.int64, device="cuda"), bf(1000, W)
-        bc = BigramConfig(1009, 31, 7)
-        add("bigram_rows", "embedding", phase, lambda: bigram_rows(bc, toks, qs, ql, kl_new, idx, last), lambda: ops.embedding(toks, table),
-            16.0 * T, like_bytes=4.0 * T * W)
+        # --- bigram rows, beside the other kernel that turns token ids into row numbers (one layer's experts)
+        toks, last = torch.randint(0, 1000, (T,), device="cuda"), torch.zeros(B, 1, dtype=torch.int64, device="cuda")
+        bc, table = BigramConfig(1009, 31, 7), TableRouter([torch.rand(1000, E).topk(1, -1).indices.int()], [E], "cuda")
+        add("bigram_rows", "moe_table_route (1 layer, top 1)", phase, lambda: bigram_rows(bc, toks, qs, ql, kl_new, idx, last),
+            lambda: table.route(toks), 16.0 * T)
         del lx, nx, gx, st, cv, z, g, out
         torch.cuda.empty_cache()
     return rows

@@ -73,8 +73,12 @@ __device__ __forceinline__ float conv_act(float z) {
 
 __device__ __forceinline__ float softplusf(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
-// factor of the output gate
-__device__ __forceinline__ float gate_of(float z, int silu, float mult) { return mult * (silu ? siluf(z) : sigmoidf(z)); }
+// factor of the output gate: fp32 runs take the accurate exponential, 16-bit runs (the result is rounded) the fast one
+template <typename T>
+__device__ __forceinline__ float gate_of(float z, int silu, float mult) {
+  if constexpr (sizeof(T) == 4) return mult * (silu ? siluf(z) : sigmoidf(z));
+  return __fdividef(silu ? mult * z : mult, 1.f + __expf(-z));
+}
 
 // units of the preparation that make decays and step sizes: one per head, or 32 heads together with one decay per head
 __device__ __host__ __forceinline__ int decay_units(const MbDelta& p) { return p.z ? p.heads : (p.heads + 31) / 32; }
@@ -428,7 +432,7 @@ __global__ void __launch_bounds__(MAXT) delta_scan_kernel(const MbDelta p, int c
           const float inv = 1.f / sqrtf(tot / static_cast<float>(V) + p.eps);
           const size_t t = static_cast<size_t>(t0 + c0 + j);
           for (int c = tid; c < V; c += blockDim.x) {
-            const float gate = gate_of(ldf(static_cast<const T*>(p.gate) + t * p.ld_gate + h * V + c), p.gate_silu, p.out_mult);
+            const float gate = gate_of<T>(ldf(static_cast<const T*>(p.gate) + t * p.ld_gate + h * V + c), p.gate_silu, p.out_mult);
             stf(static_cast<T*>(p.out) + t * p.ld_out + h * V + c, so[c] * inv * ldf(static_cast<const T*>(p.norm_w) + c) * gate);
           }
           __syncthreads();
@@ -486,7 +490,7 @@ __global__ void __launch_bounds__(256) head_out_kernel(const MbHeadOut p) {
       ss += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
     }
     const float inv = 1.f / sqrtf(warp_allsum(ss) / static_cast<float>(p.n) + p.eps);
-    auto f = [&](float z) { return gate_of(z, p.gate_silu, p.mult) * inv; };
+    auto f = [&](float z) { return gate_of<T>(z, p.gate_silu, p.mult) * inv; };
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       const int c = (lane + 32 * i) * 4;
@@ -498,7 +502,7 @@ __global__ void __launch_bounds__(256) head_out_kernel(const MbHeadOut p) {
   }
   for (int c = lane; c < V; c += 32) ss = fmaf(o[c], o[c], ss);
   const float inv = 1.f / sqrtf(warp_allsum(ss) / static_cast<float>(p.n) + p.eps);
-  for (int c = lane; c < V; c += 32) stf(out + c, o[c] * inv * ldf(w + c) * gate_of(ldf(gate + c), p.gate_silu, p.mult));
+  for (int c = lane; c < V; c += 32) stf(out + c, o[c] * inv * ldf(w + c) * gate_of<T>(ldf(gate + c), p.gate_silu, p.mult));
 }
 
 template <typename T>

@@ -65,6 +65,9 @@ __device__ __forceinline__ float sum4(uint64_t a, uint64_t b) {
 // logarithm of the decay: log sigmoid(y) / tau
 __device__ __forceinline__ float log_decay(float y, float inv_tau) { return (fminf(y, 0.f) - log1pf(expf(-fabsf(y)))) * inv_tau; }
 
+// The same for the chunk kernels, whose operands keep 16 to 17 bits: relative error of a few 1e-7 plus 1e-7 per unit of |y|
+__device__ __forceinline__ float log_decay_fast(float y, float inv_tau) { return (fminf(y, 0.f) - log1pf(__expf(-fabsf(y)))) * inv_tau; }
+
 template <typename T, int RL4, int NC, int MAXT, bool FUSE>
 __global__ void __launch_bounds__(MAXT) gla_scan_kernel(const MbGla p, int col_blocks, int chunk) {
   constexpr int DP = 32 * RL4, E = 16 / static_cast<int>(sizeof(T));       // elements per 16-byte copy
@@ -426,8 +429,8 @@ __global__ void __launch_bounds__(kThreads, 2) gla_intra_kernel(const MbGla p) {
 #pragma unroll
     for (int i = 0; i < kSub; ++i) {
       if (on && I * kSub + i < m) {
-        run.x += log_decay(b[i].x + bias.x, p.inv_tau);
-        run.y += log_decay(b[i].y + bias.y, p.inv_tau);
+        run.x += log_decay_fast(b[i].x + bias.x, p.inv_tau);
+        run.y += log_decay_fast(b[i].y + bias.y, p.inv_tau);
       }
       b[i] = run;
     }
@@ -436,9 +439,9 @@ __global__ void __launch_bounds__(kThreads, 2) gla_intra_kernel(const MbGla p) {
     for (int i = 0; i < kSub; ++i) {
       const float2 qv = unpack2(q[i]), kv = unpack2(k[i]);
       const int r = I * kSub + i;
-      *reinterpret_cast<float2*>(sm.q + r * LDQ + c) = make_float2(qv.x * p.q_scale * expf(b[i].x), qv.y * p.q_scale * expf(b[i].y));
+      *reinterpret_cast<float2*>(sm.q + r * LDQ + c) = make_float2(qv.x * p.q_scale * __expf(b[i].x), qv.y * p.q_scale * __expf(b[i].y));
       uint32_t hi, lo;
-      split2(kv.x * expf(run.x - b[i].x), kv.y * expf(run.y - b[i].y), hi, lo);
+      split2(kv.x * __expf(run.x - b[i].x), kv.y * __expf(run.y - b[i].y), hi, lo);
       *reinterpret_cast<uint32_t*>(sm.kh + r * LDK + c) = hi;
       *reinterpret_cast<uint32_t*>(sm.kl + r * LDK + c) = lo;
     }
@@ -601,10 +604,18 @@ __global__ void __launch_bounds__(kThreads, 1) gla_state_kernel(const MbGla p, i
     if (c0 + kC < n) fetch(it + 1, stages[(it + 1) & 1]);
     if (have_state) {                                // S^T q for all queries and this warp's 16 value columns
       float o[4][2][4];
+      float2 was[4][2][2];                           // what the other kernel left; read while the products run
+      float* out = p.o + (t0 + c0 + row4) * H * V + h * V + v0 + warp * 16 + col2;
 #pragma unroll
       for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int j = 0; j < 2; ++j) o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f;
+        for (int j = 0; j < 2; ++j) {
+          o[i][j][0] = o[i][j][1] = o[i][j][2] = o[i][j][3] = 0.f;
+#pragma unroll
+          for (int e = 0; e < 2; ++e)
+            if (i * 16 + row4 + 8 * e < m && v0 + warp * 16 + j * 8 + col2 < V)
+              was[i][j][e] = *reinterpret_cast<const float2*>(out + static_cast<size_t>(i * 16 + 8 * e) * H * V + j * 8);
+        }
 #pragma unroll
       for (int kb = 0; kb < KB; ++kb) {
         uint32_t hi[2][2], lo[2][2];
@@ -623,22 +634,15 @@ __global__ void __launch_bounds__(kThreads, 1) gla_state_kernel(const MbGla p, i
           mma(o[i][0], a, lo[0][0], lo[0][1]); mma(o[i][1], a, lo[1][0], lo[1][1]);
         }
       }
-      float* out = p.o + (t0 + c0) * H * V + h * V;
 #pragma unroll
       for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int r = i * 16 + row4 + 8 * e;
-          if (r >= m) continue;
+        for (int j = 0; j < 2; ++j)
 #pragma unroll
-          for (int j = 0; j < 2; ++j) {
-            const int c = v0 + warp * 16 + j * 8 + col2;
-            if (c >= V) continue;
-            float2* d = reinterpret_cast<float2*>(out + static_cast<size_t>(r) * H * V + c);
-            const float2 was = *d;
-            *d = make_float2(was.x + o[i][j][2 * e], was.y + o[i][j][2 * e + 1]);
-          }
-        }
+          for (int e = 0; e < 2; ++e)
+            if (i * 16 + row4 + 8 * e < m && v0 + warp * 16 + j * 8 + col2 < V)
+              *reinterpret_cast<float2*>(out + static_cast<size_t>(i * 16 + 8 * e) * H * V + j * 8) =
+                  make_float2(was[i][j][e].x + o[i][j][2 * e], was[i][j][e].y + o[i][j][2 * e + 1]);
 #pragma unroll
       for (int t = 0; t < 2 * KB; ++t) {
         const float2 f = *reinterpret_cast<const float2*>(sg.end + 8 * t + col2);

@@ -290,11 +290,12 @@ __global__ void __launch_bounds__(256, 1) mla_kernel(const Params p) {
   }
 }
 
-// Combines the parts of a KV-split launch: one warp per (token, head), part weights exp2(m - max).
+// Combines the parts of a KV-split launch: one warp per (token, head) and 64 columns, part weights exp2(m - max).
 __global__ void __launch_bounds__(256)
 mla_combine_kernel(const float* __restrict__ ws, bf16* __restrict__ out, const float* __restrict__ sink, const HeadGate gate, int n_rows,
                    int n_heads, int R, int nsplit) {
-  const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int unit = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  const int row = unit / (R / 64), c = unit % (R / 64) * 64 + lane * 2;
   if (row >= n_rows) return;
   const float2* ml = reinterpret_cast<const float2*>(ws + static_cast<int64_t>(nsplit) * n_rows * R);
   float2 mine = lane < nsplit ? ml[static_cast<int64_t>(lane) * n_rows + row] : make_float2(-INFINITY, 0.f);
@@ -308,17 +309,15 @@ mla_combine_kernel(const float* __restrict__ ws, bf16* __restrict__ out, const f
   for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
   if (sink) den += exp2f(sk - M);
   const float inv = den > 0.f ? gate(row / n_heads, row % n_heads) / den : 0.f;
-  for (int c = lane * 2; c < R; c += 64) {
-    float2 acc = make_float2(0.f, 0.f);
-    for (int q = 0; q < nsplit; ++q) {
-      const float fq = __shfl_sync(0xffffffffu, f, q);
-      if (fq == 0.f) continue;         // also a part without tiles, whose rows hold zeros
-      const float2 v = *reinterpret_cast<const float2*>(ws + (static_cast<int64_t>(q) * n_rows + row) * R + c);
-      acc.x = fmaf(fq, v.x, acc.x);
-      acc.y = fmaf(fq, v.y, acc.y);
-    }
-    *reinterpret_cast<uint32_t*>(out + static_cast<int64_t>(row) * R + c) = pack_bf16(acc.x * inv, acc.y * inv);
+  float2 acc = make_float2(0.f, 0.f);
+#pragma unroll 4
+  for (int q = 0; q < nsplit; ++q) {
+    const float fq = __shfl_sync(0xffffffffu, f, q);       // 0 also for a part without tiles, whose rows hold zeros
+    const float2 v = *reinterpret_cast<const float2*>(ws + (static_cast<int64_t>(q) * n_rows + row) * R + c);
+    acc.x = fmaf(fq, v.x, acc.x);
+    acc.y = fmaf(fq, v.y, acc.y);
   }
+  *reinterpret_cast<uint32_t*>(out + static_cast<int64_t>(row) * R + c) = pack_bf16(acc.x * inv, acc.y * inv);
 }
 
 // cache[slot] = [c_kv | k_rope]; one warp per token, 16-byte copies
@@ -446,8 +445,8 @@ static int launch(const Params& p, int grid_x, cudaStream_t stream) {
   dim3 grid(grid_x, p.n_heads / p.HB, p.nsplit);
   if (launch_plain(kern, grid, dim3(256), smem, stream, p) != cudaSuccess) return MB_ERR_LAUNCH;
   if (p.nsplit > 1) {
-    const int n_rows = p.T * p.n_heads;
-    if (launch_plain(mla_combine_kernel, dim3((n_rows + 7) / 8), dim3(256), 0, stream, static_cast<const float*>(p.ws), p.out,
+    const int n_rows = p.T * p.n_heads, units = n_rows * (R / 64);
+    if (launch_plain(mla_combine_kernel, dim3((units + 7) / 8), dim3(256), 0, stream, static_cast<const float*>(p.ws), p.out,
                  p.sink, p.gate, n_rows, p.n_heads, R, p.nsplit) != cudaSuccess)
       return MB_ERR_LAUNCH;
   }

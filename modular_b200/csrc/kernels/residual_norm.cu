@@ -20,7 +20,8 @@
 //   x[t]  += mult * norm(u[t]; w_u, b_u),   n1[t] = norm(x[t]; w1, b1),   u = a[t] or sum_k pair_w[t, k] e[inverse[t, k]]
 //
 // with the embedding (and rows of a second table, chosen by ids of their own) ahead of the first layer. A row lives in
-// registers from its first read to its last write; means and squared deviations are two sums, as the norm is defined.
+// registers from its first read to its last write. Every warp takes the mean and the squared deviations of its own values, and
+// the parts of the warps are put together (counts, means, deviations), so a norm costs one barrier.
 //
 // Also here: tanh-GELU in place, the sigmoid output gate of an attention layer and the soft cap of logits.
 #include <cuda_runtime.h>
@@ -277,9 +278,15 @@ static int run(const MbResidualNorm& q, cudaStream_t stream) {
 }
 
 // ---- sandwich norms
+// count, mean and sum of squared deviations of some values
+struct Part {
+  float n, mean, m2;
+};
+
 template <typename T, int NV, bool CENTER>
 __global__ void __launch_bounds__(1024) sandwich_norm_kernel(const MbSandwichNorm p) {
-  __shared__ float part[4][1][32];
+  __shared__ float sums[2][32];
+  __shared__ Part parts[2][32];
   __shared__ int32_t pos[32];
   __shared__ float pw[32];
   const int out_row = blockIdx.x, nvec = p.cols_pad >> 2;
@@ -325,24 +332,52 @@ __global__ void __launch_bounds__(1024) sandwich_norm_kernel(const MbSandwichNor
   // r becomes the deviations from its mean (CENTER; zero beyond the true width); the result is 1 / sqrt(mean of squares + eps)
   auto scale_of = [&](float4 (&r)[NV], int stage) {
     const float n = static_cast<float>(p.cols);
-    if (CENTER) {
-      float s[1] = {0.f};
+    if (!CENTER) {
+      float q[1] = {0.f};
 #pragma unroll
-      for (int i = 0; i < NV; ++i) s[0] += (r[i].x + r[i].y) + (r[i].z + r[i].w);     // padding holds zeros
-      block_sums(s, part[stage]);
-      const float mean = s[0] / n;
+      for (int i = 0; i < NV; ++i) q[0] += sq4(r[i]);
+      block_sums(q, &sums[stage]);
+      return 1.f / sqrtf(q[0] / n + p.eps);
+    }
+    // deviations from the mean of this warp's values first
+    float sum = 0.f, count = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      sum += (r[i].x + r[i].y) + (r[i].z + r[i].w);                          // padding holds zeros
+      const int c = ((threadIdx.x & ~31) + i * blockDim.x) * 4;              // the warp's 128 columns
+      count += static_cast<float>(min(max(p.cols - c, 0), 128));
+    }
+    sum = warp_allsum(sum);
+    float mean = count > 0.f ? sum / count : 0.f, m2 = 0.f;
+    auto shift = [&](float by) {
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         const int c = (threadIdx.x + i * blockDim.x) * 4;
-        r[i].x = c < p.cols ? r[i].x - mean : 0.f; r[i].y = c + 1 < p.cols ? r[i].y - mean : 0.f;
-        r[i].z = c + 2 < p.cols ? r[i].z - mean : 0.f; r[i].w = c + 3 < p.cols ? r[i].w - mean : 0.f;
+        if (c + 3 < p.cols) {
+          r[i].x -= by; r[i].y -= by; r[i].z -= by; r[i].w -= by;
+        } else if (c < p.cols) {
+          r[i].x -= by;
+          if (c + 1 < p.cols) r[i].y -= by;
+          if (c + 2 < p.cols) r[i].z -= by;
+        }
       }
-    }
-    float q[1] = {0.f};
+    };
+    shift(mean);
 #pragma unroll
-    for (int i = 0; i < NV; ++i) q[0] += sq4(r[i]);
-    block_sums(q, part[stage + 1]);
-    return 1.f / sqrtf(q[0] / n + p.eps);
+    for (int i = 0; i < NV; ++i) m2 += sq4(r[i]);
+    m2 = warp_allsum(m2);
+    const int warps = blockDim.x >> 5;
+    if (warps > 1) {                                                         // then the warps' parts together
+      if ((threadIdx.x & 31) == 0) parts[stage][threadIdx.x >> 5] = Part{count, mean, m2};
+      __syncthreads();
+      const int lane = threadIdx.x & 31;
+      Part a = {0.f, 0.f, 0.f};
+      if (lane < warps) a = parts[stage][lane];
+      const float all = warp_allsum(a.n * a.mean) / n;
+      m2 = warp_allsum(fmaf(a.n * (a.mean - all), a.mean - all, a.m2));
+      shift(all - mean);
+    }
+    return 1.f / sqrtf(m2 / n + p.eps);
   };
   auto affine = [&](float4 r, float inv, const void* w, const void* b, int c) {
     const float4 g = ld4(static_cast<const T*>(w) + c);
@@ -369,7 +404,7 @@ __global__ void __launch_bounds__(1024) sandwich_norm_kernel(const MbSandwichNor
     }
   }
   if (!p.w1) return;
-  const float inv = scale_of(x, 2);
+  const float inv = scale_of(x, 1);
   T* o1 = static_cast<T*>(p.n1) + static_cast<size_t>(out_row) * p.ld1;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
@@ -381,8 +416,8 @@ __global__ void __launch_bounds__(1024) sandwich_norm_kernel(const MbSandwichNor
 template <typename T, bool CENTER>
 static int run_sandwich(const MbSandwichNorm& p, cudaStream_t stream) {
   const int nvec = p.cols_pad / 4;
-  // few rows: as many threads as a row has vectors; many rows: CTAs of 256, several per SM
-  const int most = p.n_rows <= 296 ? 1024 : 256, warps = (nvec + 31) / 32;
+  // few rows: as many threads as a row has vectors; many rows: small CTAs, several per SM
+  const int most = p.n_rows <= 296 ? 512 : 256, warps = (nvec + 31) / 32;
   int nv = (nvec + most - 1) / most;
   nv = nv <= 1 ? 1 : nv <= 2 ? 2 : 4;
   const int threads = (warps + nv - 1) / nv * 32;
