@@ -305,60 +305,39 @@ def _deepseek_arm(args, defaults) -> int:
     return 0
 
 
-def _gotunex_arm(args) -> int:
-    """Gotunex (latent attention and delta-rule layers, experts by token id) at sizes that resemble a real model's layers,
-    beside DeepSeek-V3 layers of the same width, heads, latents and experts: prefill and decode throughput of whole models
-    on one GPU, and every kernel beside the like kernel of an existing family. One JSON line; ``value`` is the decode
-    throughput of the first size at the largest batch."""
+# designs with a benchmark module of their own: (module, name, what their layers are called, which of its models is the design's)
+DESIGNS = {
+    "gotunex": ("gotunex_bench", "Gotunex", "layers", lambda model: model.startswith("gotunex (delta")),
+    "vipotar": ("vipotar_bench", "Vipotar", "layer runs", lambda model: model == "vipotar"),
+    "mavidra": ("mavidra_bench", "Mavidra", "layers", lambda model: model == "mavidra"),
+}
+
+
+def _design_arm(args) -> int:
+    """One of ``DESIGNS`` at sizes that resemble a real model's layers, beside existing families of equal size: prefill and decode
+    throughput of whole models on one GPU, and every kernel beside the like kernel of an existing family. One JSON line;
+    ``value`` is the decode throughput of the first size at the largest batch."""
+    import importlib
+
     import torch
 
+    module, name, unit, is_mine = DESIGNS[args.model]
     if int(os.environ.get("WORLD_SIZE", "1")) > 1:
-        raise SystemExit("--model gotunex runs on one GPU")
+        raise SystemExit(f"--model {args.model} runs on one GPU")
     torch.cuda.set_device(0)
-    from modular_b200.benchmark import gotunex_bench
-
+    bench = importlib.import_module(f"modular_b200.benchmark.{module}")
     sampler = ClockSampler(0)
     sampler.start()
-    res = gotunex_bench.main(steps=max(args.steps, 5))
+    res = bench.main(steps=max(args.steps, 5))
     clocks = sampler.stop()
-    mine = [r for r in res["models"] if r["model"].startswith("gotunex (delta")]
+    mine = [r for r in res["models"] if is_mine(r["model"])]
     best = max((r for r in mine if r["size"] == mine[0]["size"]), key=lambda r: r["decode_batch"])
     print(json.dumps({
         "metric": "decode_tokens_per_s", "value": best["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": max(args.steps, 5),
         "warmup": 5, "ms_per_step": best["decode_ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
         "dtype": "bf16 (fp32 residual stream, recurrent state, norms and softmax)",
         "data": "synthetic uniform-random token ids; random-init weights", "impl": "ours",
-        "config": {"model": f"Gotunex, size {best['size']}, {best['layers']} layers", "global_batch": best["decode_batch"],
-                   "seq_len": best["context"], "parallelism": "one GPU",
-                   "l2_policy": "models: inputs larger than L2; kernels: L2 flushed before every call"},
-        "clocks": clocks, **res}), flush=True)
-    return 0
-
-
-def _vipotar_arm(args) -> int:
-    """Vipotar (windowed softmax attention beside lightning attention, looped layers) at sizes that resemble a real model's
-    layers, beside Gotunex and Llama layers of equal size: prefill and decode throughput of whole models on one GPU, and every
-    kernel beside the like kernel of an existing family. One JSON line; ``value`` is the decode throughput of the first size
-    at the largest batch."""
-    import torch
-
-    if int(os.environ.get("WORLD_SIZE", "1")) > 1:
-        raise SystemExit("--model vipotar runs on one GPU")
-    torch.cuda.set_device(0)
-    from modular_b200.benchmark import vipotar_bench
-
-    sampler = ClockSampler(0)
-    sampler.start()
-    res = vipotar_bench.main(steps=max(args.steps, 5))
-    clocks = sampler.stop()
-    mine = [r for r in res["models"] if r["model"] == "vipotar"]
-    best = max((r for r in mine if r["size"] == mine[0]["size"]), key=lambda r: r["decode_batch"])
-    print(json.dumps({
-        "metric": "decode_tokens_per_s", "value": best["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": max(args.steps, 5),
-        "warmup": 5, "ms_per_step": best["decode_ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
-        "dtype": "bf16 (fp32 residual stream, recurrent state, norms and softmax)",
-        "data": "synthetic uniform-random token ids; random-init weights", "impl": "ours",
-        "config": {"model": f"Vipotar, size {best['size']}, {best['layers']} layer runs", "global_batch": best["decode_batch"],
+        "config": {"model": f"{name}, size {best['size']}, {best['layers']} {unit}", "global_batch": best["decode_batch"],
                    "seq_len": best["context"], "parallelism": "one GPU",
                    "l2_policy": "models: inputs larger than L2; kernels: L2 flushed before every call"},
         "clocks": clocks, **res}), flush=True)
@@ -381,26 +360,22 @@ def main() -> int:
     ap.add_argument("--server", action="store_true",
                     help="measure through the HTTP serving endpoint on more than one GPU too (by default only "
                          "one-GPU runs do: on N GPUs the endpoint needs a second bring-up of all ranks)")
-    ap.add_argument("--model", default="llama8b", choices=["llama8b", "llama70b-fp8", "deepseek-v3", "gotunex", "vipotar"],
+    ap.add_argument("--model", default="llama8b", choices=["llama8b", "llama70b-fp8", "deepseek-v3", *DESIGNS],
                     help="llama8b: the headline config (bf16, any --gpus); llama70b-fp8: Llama-3.3-70B shapes with "
                          "block-scaled fp8 weights, tensor parallel over --gpus (input 2048 / output 512 / "
                          "concurrency 128 unless given); deepseek-v3: DeepSeek-V3 shapes, fp8 routed experts, "
                          "expert parallel over --gpus with data-parallel attention (concurrency 256 over all ranks); gotunex: "
                          "prefill / decode throughput and kernels of that design beside DeepSeek-V3 layers of equal size; vipotar: "
-                         "the same beside Gotunex and Llama layers of equal size")
+                         "the same beside Gotunex and Llama layers of equal size; mavidra: the same beside Gotunex layers")
     args = ap.parse_args()
     if args.model == "deepseek-v3":
         if args.impl == "reference":
             return _reference_arm(args)
         return _deepseek_arm(args, ap.parse_args([]))
-    if args.model == "gotunex":
+    if args.model in DESIGNS:
         if args.impl == "reference":
             return _reference_arm(args)
-        return _gotunex_arm(args)
-    if args.model == "vipotar":
-        if args.impl == "reference":
-            return _reference_arm(args)
-        return _vipotar_arm(args)
+        return _design_arm(args)
     if args.model == "llama70b-fp8":
         defaults = ap.parse_args([])
         if args.input_len == defaults.input_len:
