@@ -302,12 +302,9 @@ __global__ void __launch_bounds__(1024) sandwich_norm_kernel(const MbSandwichNor
     const int64_t id = p.inject_ids[row];
     if (id >= 0 && id < p.inject_rows) ir = static_cast<const T*>(p.inject) + static_cast<size_t>(id) * p.ld_inject;
   }
-  if (ee) {
-    if (threadIdx.x < p.top_k) {
-      pos[threadIdx.x] = p.inverse[static_cast<size_t>(row) * p.top_k + threadIdx.x];
-      pw[threadIdx.x] = p.pair_w[static_cast<size_t>(row) * p.top_k + threadIdx.x];
-    }
-    __syncthreads();
+  if (ee && threadIdx.x < p.top_k) {
+    pos[threadIdx.x] = p.inverse[static_cast<size_t>(row) * p.top_k + threadIdx.x];
+    pw[threadIdx.x] = p.pair_w[static_cast<size_t>(row) * p.top_k + threadIdx.x];
   }
   float4 x[NV], u[NV];
 #pragma unroll
@@ -319,13 +316,22 @@ __global__ void __launch_bounds__(1024) sandwich_norm_kernel(const MbSandwichNor
     else if (er) { const float4 y = ld4(er + c); x[i] = make_float4(y.x * p.scale, y.y * p.scale, y.z * p.scale, y.w * p.scale); }
     if (ir) { const float4 y = ld4(ir + c); x[i].x += y.x; x[i].y += y.y; x[i].z += y.z; x[i].w += y.w; }
     if (ar) u[i] = ld4(ar + c);
-    if (ee) {
+  }
+  if (ee) {
+    __syncthreads();
 #pragma unroll 4
-      for (int k = 0; k < p.top_k; ++k) {
-        if (pos[k] < 0) continue;
-        const float4 y = ld4(ee + static_cast<size_t>(pos[k]) * p.lde + c);
-        u[i].x = fmaf(pw[k], y.x, u[i].x); u[i].y = fmaf(pw[k], y.y, u[i].y);
-        u[i].z = fmaf(pw[k], y.z, u[i].z); u[i].w = fmaf(pw[k], y.w, u[i].w);
+    for (int k = 0; k < p.top_k; ++k) {
+      const int at = pos[k];
+      if (at < 0) continue;
+      const float w = pw[k];
+      const T* src = ee + static_cast<size_t>(at) * p.lde;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int v = threadIdx.x + i * blockDim.x;
+        if (v >= nvec) continue;
+        const float4 y = ld4(src + v * 4);
+        u[i].x = fmaf(w, y.x, u[i].x); u[i].y = fmaf(w, y.y, u[i].y);
+        u[i].z = fmaf(w, y.z, u[i].z); u[i].w = fmaf(w, y.w, u[i].w);
       }
     }
   }
@@ -417,7 +423,7 @@ template <typename T, bool CENTER>
 static int run_sandwich(const MbSandwichNorm& p, cudaStream_t stream) {
   const int nvec = p.cols_pad / 4;
   // few rows: as many threads as a row has vectors; many rows: small CTAs, several per SM
-  const int most = p.n_rows <= 296 ? 512 : 256, warps = (nvec + 31) / 32;
+  const int most = p.n_rows <= 296 ? 1024 : 256, warps = (nvec + 31) / 32;
   int nv = (nvec + most - 1) / most;
   nv = nv <= 1 ? 1 : nv <= 2 ? 2 : 4;
   const int threads = (warps + nv - 1) / nv * 32;

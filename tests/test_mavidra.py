@@ -706,11 +706,11 @@ def test_schedules(mixed_model, name, device, dtype):
 @pytest.mark.parametrize("cfg", [
     config(gla()), config(latent()), config(parallel()),
     config((parallel(heads=1, kv_heads=1, dim=4, vdim=4, dims=2, rheads=1, rkv=1, rdim=4, rvdim=4, conv=1), moe(1, 1, 1, 1, 4)),
-           (gla(1, 4, 4, 1.0), None), (latent(1, 4, 2, 4, 4, 4, 1), moe(2, 1, 2, 1, 4)), width=40, vocab=33, bigram=(1, 0, 0)),
+           (gla(1, 4, 4, 1.0), None), (latent(1, 4, 2, 4, 4, 4, 1), moe(2, 1, 2, 1, 4)), width=42, vocab=33, bigram=(1, 0, 0)),
     config(latent(), (latent(heads=6, dim=100, vdim=8, kv_from=0, window=70), None), latent(kv_rank=200, rot_dim=64, window=2), eps=1e-3, width=136, vocab=258,
            mult=1.0, scale=2.0),
     config((parallel(heads=10, kv_heads=2, dim=104, vdim=80, dims=60, rheads=7, rkv=7, rdim=104, rvdim=48), moe(12, 5, 4, 3, 136)), gla(7, 104, 48, 9.0),
-           width=200, vocab=98, bigram=(500, 499, 3)),
+           width=202, vocab=98, bigram=(500, 499, 3)),
     config(parallel(dim=200, vdim=144, dims=66, rheads=2, rdim=144, rvdim=8), parallel(heads=3, kv_heads=1, dim=32, vdim=32, dims=32), width=88)],
     ids=["gla only", "latent only", "parallel only", "tiny", "latent", "wide", "wide heads"])
 def test_other_sizes(cfg, device, dtype):
