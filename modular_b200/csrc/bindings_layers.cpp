@@ -144,6 +144,68 @@ void sandwich_norm(Tensor& x, const Opt& ids, const Opt& table, double scale, co
   check_rc(mb_sandwich_norm(&p, dt == at::kFloat ? 1 : 0, cur_stream()), "sandwich_norm");
 }
 
+// seam with elementwise norms and an optional token shift, see MbTanhSeam; `x_out` may be `x` where there is no shift
+void tanh_seam(const Opt& x, const Opt& x_out, const Opt& ids, const Opt& table, double scale, const Opt& a, const Opt& e,
+               const Opt& inverse, const Opt& pair_w, const Opt& self, const Opt& rows, const Opt& w_u, const Opt& b_u, double alpha_u,
+               const Opt& w1, const Opt& b1, double alpha_1, const Opt& n1, const Opt& shift, const Opt& prev, const Opt& state_idx,
+               const Opt& q_start, const Opt& q_len, const Opt& kv_len, bool one_token, int cols_pad, int n_rows) {
+  MbTanhSeam p = {};
+  p.cols_pad = cols_pad; p.n_rows = n_rows; p.scale = static_cast<float>(scale);
+  p.alpha_u = static_cast<float>(alpha_u); p.alpha_1 = static_cast<float>(alpha_1);
+  const at::ScalarType dt = given(w1) ? w1->scalar_type() : given(w_u) ? w_u->scalar_type() : given(table) ? table->scalar_type() : at::kBFloat16;
+  int64_t T = n_rows;
+  auto stream_rows = [&](const Opt& t, const char* what) {
+    const int ld = ld_of(*t, at::kFloat, what);
+    TORCH_CHECK(t->size(1) >= cols_pad && (p.ldx == 0 || ld == p.ldx), "tanh_seam: ", what, " shape");
+    p.ldx = ld;
+    T = t->size(0);
+    return t->data_ptr<float>();
+  };
+  TORCH_CHECK(given(x) || given(table), "tanh_seam: x or table");
+  if (given(x)) p.x = stream_rows(x, "x");
+  if (given(x_out)) {
+    const int64_t before = T;
+    p.x_out = stream_rows(x_out, "x_out");
+    TORCH_CHECK(!given(x) || T == before, "tanh_seam: x_out rows");
+  }
+  auto matrix = [&](const Opt& t, const char* what, int64_t min_rows) {
+    const int ld = ld_of(*t, dt, what);
+    TORCH_CHECK(t->size(1) >= cols_pad && t->size(0) >= min_rows, "tanh_seam: ", what, " shape");
+    return ld;
+  };
+  auto weight = [&](const Opt& t, const char* what) -> const void* {
+    if (!given(t)) return nullptr;
+    TORCH_CHECK(t->is_cuda() && t->is_contiguous() && t->scalar_type() == dt && t->numel() >= cols_pad, "tanh_seam: ", what);
+    return t->data_ptr();
+  };
+  if (given(table)) {
+    TORCH_CHECK(given(ids) && ids->is_cuda() && ids->is_contiguous() && ids->scalar_type() == at::kLong && ids->numel() >= T, "tanh_seam: ids");
+    p.ld_table = matrix(table, "table", 0); p.table = table->data_ptr(); p.ids = ids->data_ptr<int64_t>();
+    p.vocab = static_cast<int>(table->size(0));
+  }
+  if (given(a)) { p.lda = matrix(a, "a", T); p.a = a->data_ptr(); }
+  if (given(e)) {
+    TORCH_CHECK(given(inverse) && inverse->dim() == 2 && given(pair_w), "tanh_seam: inverse [T, k] and pair_w");
+    p.top_k = static_cast<int>(inverse->size(1));
+    p.lde = matrix(e, "e", T * p.top_k); p.e = e->data_ptr();
+    p.inverse = i32(*inverse, T * p.top_k, "inverse"); p.pair_w = f32(*pair_w, T * p.top_k, "pair_w");
+    if (given(self)) { p.ld_self = matrix(self, "self", T); p.self = self->data_ptr(); }
+  }
+  if (given(rows)) p.rows = i32(*rows, n_rows, "rows");
+  else TORCH_CHECK(n_rows <= T, "tanh_seam: rows");
+  p.w_u = weight(w_u, "w_u"); p.b_u = weight(b_u, "b_u"); p.w1 = weight(w1, "w1"); p.b1 = weight(b1, "b1");
+  if (given(w1)) { TORCH_CHECK(given(n1), "tanh_seam: n1"); p.ld1 = matrix(n1, "n1", n_rows); p.n1 = n1->data_ptr(); }
+  if (given(shift)) {
+    TORCH_CHECK(given(prev) && prev->is_cuda() && prev->is_contiguous() && prev->scalar_type() == at::kFloat && prev->dim() == 2 &&
+                    prev->size(1) == cols_pad && given(state_idx) && given(q_start) && given(q_len) && given(kv_len), "tanh_seam: shift state");
+    p.shift = weight(shift, "shift"); p.prev = prev->data_ptr<float>();
+    p.B = q_len->numel(); p.one_token = one_token;
+    p.state_idx = i32(*state_idx, p.B, "state_idx"); p.q_start = i32(*q_start, p.B, "q_start");
+    p.q_len = i32(*q_len, p.B, "q_len"); p.kv_len = i32(*kv_len, p.B, "kv_len");
+  }
+  check_rc(mb_tanh_seam(&p, dt == at::kFloat ? 1 : 0, cur_stream()), "tanh_seam");
+}
+
 // window, sink and output gate of an attention call; `use` is what the C interface takes (null: none of them)
 struct AttnOptions {
   MbAttnOptions o = {};
@@ -334,6 +396,40 @@ void gla(const Tensor& x, int q_off, int k_off, int v_off, const Tensor& z, cons
   check_rc(mb_gla(&p, dt, num_sms(), cur_stream()), "gla");
 }
 
+// x: projection rows with the column blocks of r, k, v and the removal rates at the given offsets; see MbGeneralDelta
+void general_delta(const Tensor& x, int r_off, int k_off, int v_off, int a_off, const Tensor& a_bias, const Tensor& z, const Tensor& z_bias,
+                   const Tensor& gate, const Tensor& norm_w, double eps, int norm_dim, Tensor& rows, Tensor& o, Tensor& out, Tensor& state,
+                   const Tensor& state_idx, const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, int heads, int dim, int vdim,
+                   bool one_token) {
+  MbGeneralDelta p = {};
+  const at::ScalarType st = x.scalar_type();
+  p.T = x.size(0); p.B = q_len.numel(); p.heads = heads; p.dim = dim; p.vdim = vdim; p.one_token = one_token;
+  p.dim_pad = mb_delta_dim_pad(dim);
+  TORCH_CHECK(p.dim_pad > 0, "general_delta: key width ", dim, " is beyond the supported maximum");
+  const int64_t T = p.T, HD = static_cast<int64_t>(heads) * dim, HV = static_cast<int64_t>(heads) * vdim;
+  p.x = x.data_ptr(); p.ldx = ld_of(x, st, "x"); p.r_off = r_off; p.k_off = k_off; p.v_off = v_off; p.a_off = a_off;
+  TORCH_CHECK(r_off + HD <= x.size(1) && k_off + HD <= x.size(1) && v_off + HV <= x.size(1) && a_off + HD <= x.size(1),
+              "general_delta: columns");
+  p.a_bias = f32(a_bias, HD, "a_bias"); p.z_bias = f32(z_bias, HD, "z_bias");
+  p.ldz = ld_of(z, at::kFloat, "z"); p.z = z.data_ptr<float>();
+  TORCH_CHECK(z.size(0) >= T && z.size(1) >= HD, "general_delta: z");
+  p.ld_gate = ld_of(gate, st, "gate"); p.gate = gate.data_ptr();
+  TORCH_CHECK(gate.size(0) >= T && gate.size(1) >= HV, "general_delta: gate");
+  TORCH_CHECK(norm_w.is_cuda() && norm_w.is_contiguous() && norm_w.scalar_type() == st && norm_w.numel() >= HV, "general_delta: norm_w");
+  p.norm_w = norm_w.data_ptr(); p.eps = static_cast<float>(eps); p.norm_dim = norm_dim;
+  const bool fused = one_token && vdim <= (p.dim_pad <= 256 ? 128 : 64);       // no scratch where one launch does it all
+  p.rows = const_cast<float*>(f32(rows, fused ? 0 : T * heads * (4 * p.dim_pad + 4), "general_delta: rows"));
+  p.o = const_cast<float*>(f32(o, fused ? 0 : T * HV, "general_delta: o"));
+  p.ld_out = ld_of(out, st, "out"); p.out = out.data_ptr();
+  TORCH_CHECK(out.size(0) >= T && out.size(1) >= HV, "general_delta: out");
+  TORCH_CHECK(state.is_contiguous() && state.scalar_type() == at::kFloat && state.dim() == 4 && state.size(1) == heads &&
+                  state.size(2) == vdim && state.size(3) == p.dim_pad, "general_delta: state [slots, heads, vdim, dim_pad]");
+  p.state = state.data_ptr<float>();
+  p.state_idx = i32(state_idx, p.B, "state_idx"); p.q_start = i32(q_start, p.B, "q_start");
+  p.q_len = i32(q_len, p.B, "q_len"); p.kv_len = i32(kv_len, p.B, "kv_len");
+  check_rc(mb_general_delta(&p, dtype_of(x, "x"), num_sms(), cur_stream()), "general_delta");
+}
+
 // the cache [pages, 2, planes, kv heads, page, head width] at one plane
 struct CacheView {
   char *k, *v;
@@ -351,7 +447,7 @@ struct CacheView {
 // x: projection rows; queries at column 0 .., see MbBlockPrep
 void block_prep(Tensor& x, int q_off, int heads, int k_off, int v_off, int kv_heads, int dims, const Tensor& positions,
                 const Opt& cos_sin, const Tensor& slots, Tensor& kv, int plane, int silu_off, int silu_n, int relu2_off, int relu2_n,
-                const Opt& q_norm, const Opt& k_norm, int norm_dim, double eps, bool halves) {
+                const Opt& q_norm, const Opt& k_norm, int norm_dim, double eps, bool halves, const Opt& bias) {
   MbBlockPrep p = {};
   p.x = x.data_ptr(); p.ldx = ld_of(x, x.scalar_type(), "x"); p.T = x.size(0);
   const CacheView c(kv, plane, kv_heads, "block_prep");
@@ -376,6 +472,8 @@ void block_prep(Tensor& x, int q_off, int heads, int k_off, int v_off, int kv_he
   };
   p.q_norm = weight(q_norm); p.k_norm = weight(k_norm); p.norm_dim = norm_dim > 0 ? norm_dim : c.hd; p.eps = static_cast<float>(eps);
   p.halves = halves;
+  if (given(bias)) p.bias = f32(*bias, std::max<int64_t>(q_off + static_cast<int64_t>(heads) * c.hd,
+                                                        std::max(k_off, v_off) + static_cast<int64_t>(kv_heads) * c.hd), "bias");
   check_rc(mb_block_prep(&p, dtype_of(x, "x"), cur_stream()), "block_prep");
 }
 
@@ -474,7 +572,8 @@ void mb::bind_layers(py::module_& m) {
   m.def("block_prep", &block_prep, py::arg("x"), py::arg("q_off"), py::arg("heads"), py::arg("k_off"), py::arg("v_off"),
         py::arg("kv_heads"), py::arg("dims"), py::arg("positions"), py::arg("cos_sin"), py::arg("slots"), py::arg("kv"), py::arg("plane"),
         py::arg("silu_off") = 0, py::arg("silu_n") = 0, py::arg("relu2_off") = 0, py::arg("relu2_n") = 0, py::arg("q_norm") = none,
-        py::arg("k_norm") = none, py::arg("norm_dim") = 0, py::arg("eps") = 1e-6, py::arg("halves") = false);
+        py::arg("k_norm") = none, py::arg("norm_dim") = 0, py::arg("eps") = 1e-6, py::arg("halves") = false,
+        py::arg("bias") = none);
   m.def("window_attention", &window_attention, py::arg("q"), py::arg("out"), py::arg("kv"), py::arg("plane"), py::arg("block_table"),
         py::arg("q_start"), py::arg("q_len"), py::arg("kv_len"), py::arg("tile_seq"), py::arg("tile_q0"), py::arg("decode_seq"),
         py::arg("n_q"), py::arg("n_kv"), py::arg("scale"), py::arg("window") = 0, py::arg("sink") = none, py::arg("gate") = none,
@@ -504,6 +603,17 @@ void mb::bind_layers(py::module_& m) {
         py::arg("o"), py::arg("out"), py::arg("state"), py::arg("state_idx"), py::arg("q_start"), py::arg("q_len"), py::arg("kv_len"),
         py::arg("heads"), py::arg("dim"), py::arg("vdim"), py::arg("one_token"), py::arg("allow_chunks") = true);
   m.def("sandwich_norm", &sandwich_norm);
+  m.def("tanh_seam", &tanh_seam);
+  m.def("general_delta", &general_delta);
+  m.def("tanh_cols", [](Tensor& x) {
+    const int ld = ld_of(x, x.scalar_type(), "x");
+    check_rc(mb_tanh_cols(x.data_ptr(), ld, x.size(0), x.size(1), dtype_of(x, "x"), cur_stream()), "tanh_cols");
+  });
+  m.def("xielu", [](Tensor& x, double up, double down) {
+    const int ld = ld_of(x, x.scalar_type(), "x");
+    check_rc(mb_xielu(x.data_ptr(), ld, x.size(0), x.size(1), static_cast<float>(up), static_cast<float>(down), dtype_of(x, "x"),
+                      cur_stream()), "xielu");
+  });
   m.def("bigram_rows", [](const Tensor& tokens, const Tensor& q_start, const Tensor& q_len, const Tensor& kv_len, const Tensor& state_idx,
                           Tensor& last, Tensor& out, int64_t mul_prev, int64_t mul_cur, int64_t buckets) {
     const int T = tokens.numel(), B = q_len.numel();
@@ -515,15 +625,18 @@ void mb::bind_layers(py::module_& m) {
                             buckets, cur_stream()), "bigram_rows");
   });
   m.def("moe_score_route", [](const Tensor& logits, const Opt& bias, Tensor& ids, Tensor& w, Tensor& rank, Tensor& counts, int n_group,
-                              int keep, bool norm_topk, double scaling) {
-    const int T = ids.size(0), k = ids.size(1), E = counts.numel(), ld = ld_of(logits, at::kFloat, "logits");
+                              int keep, bool norm_topk, double scaling, bool softmax, bool group_max, int identity) {
+    const int T = ids.size(0), k = ids.size(1), E = counts.numel() + identity, ld = ld_of(logits, at::kFloat, "logits");
     TORCH_CHECK(ids.dim() == 2 && logits.size(0) >= T && logits.size(1) >= E, "moe_score_route shapes");
     check_rc(mb_moe_score_route(logits.data_ptr<float>(), ld, given(bias) ? f32(*bias, E, "bias") : nullptr,
                                 const_cast<int32_t*>(i32(ids, 0, "ids")), const_cast<float*>(f32(w, static_cast<int64_t>(T) * k, "w")),
                                 const_cast<int32_t*>(i32(rank, static_cast<int64_t>(T) * k, "rank")),
-                                const_cast<int32_t*>(i32(counts, E, "counts")), T, E, n_group, keep, k, norm_topk ? 1 : 0,
-                                static_cast<float>(scaling), cur_stream()), "moe_score_route");
-  });
+                                const_cast<int32_t*>(i32(counts, E - identity, "counts")), T, E, n_group, keep, k, norm_topk ? 1 : 0,
+                                static_cast<float>(scaling), softmax ? 1 : 0, group_max ? 1 : 0, identity, cur_stream()),
+             "moe_score_route");
+  }, py::arg("logits"), py::arg("bias"), py::arg("ids"), py::arg("w"), py::arg("rank"), py::arg("counts"), py::arg("n_group"),
+     py::arg("keep"), py::arg("norm_topk"), py::arg("scaling"), py::arg("softmax") = false, py::arg("group_max") = false,
+     py::arg("identity") = 0);
   m.def("moe_place_rows", [](const Tensor& x, const Tensor& ids, const Tensor& rank, const Tensor& counts, Tensor& offsets, Tensor& inverse,
                              Tensor& dst) {
     const int T = ids.size(0), k = ids.size(1), E = counts.numel(), es = x.element_size();

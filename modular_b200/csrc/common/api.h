@@ -278,7 +278,32 @@ int mb_sandwich_norm(const MbSandwichNorm* p, int dtype, cudaStream_t stream);
 int mb_bigram_rows(const int64_t* tokens, const int32_t* q_start, const int32_t* q_len, const int32_t* kv_len,
                    const int32_t* state_idx, int64_t* last, int64_t* out, int T, int B, long long mul_prev, long long mul_cur,
                    long long buckets, cudaStream_t stream);
+// Seam of layers whose norms are elementwise (dynamic tanh), before and after every branch, one branch at a time; null pointers
+// switch parts off:
+//   x_out = (table[ids] * scale or x) + T(u; alpha_u, w_u, b_u),   T(y; alpha, w, b) = tanh(alpha * y) * w + b
+//   u     = [a] + [sum_k pair_w[., k] (inverse[., k] >= 0 ? e[inverse[., k]] : self)]
+//   n1    = h = T(x_out; alpha_1, w1, b1), or with a token shift  n1[t] = h[t] + (h[t - 1] - h[t]) * shift
+// With a shift, x_out is another buffer than x, and the row ahead of a step comes from prev [slots, cols_pad] where the step
+// continues a sequence (zeros otherwise); the step's last h goes there.
+typedef struct {
+  const float* x; float* x_out; int ldx;                 // one row stride for both; x_out may be null (nothing is stored)
+  const int64_t* ids; const void* table; float scale; int vocab, ld_table;
+  const void* a; int lda;
+  const void* e; int lde; const int32_t* inverse; const float* pair_w; int top_k;
+  const void* self; int ld_self;
+  const int32_t* rows;
+  const void *w_u, *b_u; float alpha_u;
+  const void *w1, *b1; float alpha_1; void* n1; int ld1;
+  const void* shift; float* prev;
+  const int32_t *state_idx, *q_start, *q_len, *kv_len; int B, one_token;
+  int n_rows, cols_pad;
+} MbTanhSeam;
+int mb_tanh_seam(const MbTanhSeam* p, int dtype, cudaStream_t stream);
 int mb_gelu_tanh(void* x, long long n, int dtype, cudaStream_t stream);
+// In place over cols columns (a multiple of 8) of every row: tanh, or xIELU(z) = up z^2 + z / 2 for z > 0 and
+// down (exp(z) - 1 - z) + z / 2 otherwise
+int mb_tanh_cols(void* x, int ldx, int rows, int cols, int dtype, cudaStream_t stream);
+int mb_xielu(void* x, int ldx, int rows, int cols, float up, float down, int dtype, cudaStream_t stream);
 // x[i] = cap * tanh(x[i] / cap) over fp32 logits
 int mb_softcap(float* x, long long n, float cap, cudaStream_t stream);
 int mb_sigmoid_gate(void* o, int ldo, const void* g, int ldg, int rows, int cols, int dtype, cudaStream_t stream);
@@ -309,6 +334,7 @@ typedef struct {
   const void* gate; int ld_gate; const void* norm_w;
   int T, heads, vdim, n, gate_silu;
   float eps, mult;
+  int w_stride;                                          // norm weights of head h start at h * w_stride (0: shared by the heads)
 } MbHeadOut;
 int mb_head_norm_gate(const MbHeadOut* p, int dtype, cudaStream_t stream);
 
@@ -323,6 +349,7 @@ typedef struct {
   // RMS norm of every query / key head over its first norm_dim columns (the rest are zeros), before the rotation; null: none
   const void *q_norm, *k_norm; int norm_dim; float eps;  // weights [hd]
   int halves;                                            // pairs (i, i + dims / 2) instead of neighbours
+  const float* bias;                                     // added to the columns of q, k and v first, indexed like a row of x (halves only)
 } MbBlockPrep;
 int mb_block_prep(const MbBlockPrep* p, int dtype, cudaStream_t stream);
 int mb_attention_plan(const int32_t* q_len, int B, int tok_per_tile, int n_tiles, int32_t* tile_seq, int32_t* tile_q0,
@@ -364,6 +391,20 @@ typedef struct {
 int mb_gla_chunks(const MbGla* p, int dtype);
 int mb_gla(const MbGla* p, int dtype, int num_sms, cudaStream_t stream);
 
+// ---- generalized delta rule: a decay and a removal rate per key channel (general_delta.cu) -----
+typedef struct {
+  const void* x; int ldx, r_off, k_off, v_off, a_off;    // projection rows; heads of dim / vdim columns (multiples of 8)
+  const float* a_bias;                                   // [heads * dim]; removal rate = sigmoid(a + a_bias)
+  const float* z; int ldz; const float* z_bias;          // [T, heads * dim], [heads * dim]; decay = exp(-exp(-1/2) sigmoid(z + z_bias))
+  const void* gate; int ld_gate; const void* norm_w; float eps; int norm_dim;   // as in MbHeadOut, norm weights [heads * vdim]
+  float *rows, *o;                                       // fp32 scratch [T, heads, 4 dim_pad + 4] and [T, heads, vdim]
+  void* out; int ld_out;                                 // [T, heads * vdim]
+  float* state;                                          // [slots, heads, vdim, dim_pad]
+  const int32_t *state_idx, *q_start, *q_len, *kv_len;
+  int T, B, heads, dim, dim_pad, vdim, one_token;
+} MbGeneralDelta;
+int mb_general_delta(const MbGeneralDelta* p, int dtype, int num_sms, cudaStream_t stream);
+
 // ---- fp32 products (gemm_simt.cu) ------------------------------------------------------------
 int mb_gemm_f32(const float* x, const float* w, float* y, const float* r, int M, int N, int K, int ldx, int ldw, int ldy,
                 int ldr, cudaStream_t stream);
@@ -382,8 +423,11 @@ int mb_moe_router_group_limited(const float* logits, const float* bias, int32_t*
 // The same choice with one warp per token, and the first half of the sort by expert: rank[t, k] is the pair's place among its
 // expert's pairs, counts [E] (zero on entry) their number. mb_moe_place_rows does the rest: offsets [E + 1], inverse [T, top_k]
 // and the token rows copied into expert order.
+// Scores are sigmoids or (softmax) a softmax over all E; a group counts its two best choice scores or (group_max) its best one.
+// The last `identity` of the E are no experts: they are chosen like the others and have rank -1.
 int mb_moe_score_route(const float* logits, int ld, const float* bias, int32_t* ids, float* w, int32_t* rank, int32_t* counts, int T,
-                       int E, int n_group, int keep, int top_k, int norm_topk, float scaling, cudaStream_t stream);
+                       int E, int n_group, int keep, int top_k, int norm_topk, float scaling, int softmax, int group_max, int identity,
+                       cudaStream_t stream);
 int mb_moe_place_rows(const void* x, long long ldx_bytes, const int32_t* ids, const int32_t* rank, const int32_t* counts,
                       int32_t* offsets, int32_t* inverse, void* dst, int T, int E, int top_k, int row_bytes, cudaStream_t stream);
 int mb_moe_router_softmax_topk(const float* logits, int32_t* topk_ids, float* topk_w, int T, int E,

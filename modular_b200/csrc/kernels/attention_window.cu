@@ -4,7 +4,8 @@
 //
 //   mb_block_prep         everything between the stacked input projection of a parallel block and its branches, in one
 //                         launch: queries rotated in place, keys rotated and stored in the cache with the values, silu on
-//                         one column range and squared relu on another; or, with per-head norms, norms and rotation
+//                         one column range and squared relu on another; or, with per-head norms, norms and rotation; or, with
+//                         pairs half the rotated width apart, biases, rotation and store
 //   mb_attention_plan     prompt tiles of a ragged step (sequence and first token of each), made on the device
 //   mb_window_attention   causal attention of any head width, window and group size, optional sink score per head
 //
@@ -137,14 +138,20 @@ __global__ void __launch_bounds__(256) head_prep_kernel(const MbBlockPrep p) {
     dst = static_cast<T*>(is_v ? p.v_cache : p.k_cache) + (slot / p.page_size) * p.page_stride + h * p.head_stride +
           static_cast<long long>(slot % p.page_size) * p.hd;
   }
+  const float* bias = p.bias ? p.bias + (src - row) : nullptr;
+  auto biased = [&](int c) {
+    float4 x = ld4(src + c);
+    if (bias) { const float4 b = *reinterpret_cast<const float4*>(bias + c); x.x += b.x; x.y += b.y; x.z += b.z; x.w += b.w; }
+    return x;
+  };
   if (is_v) {
-    for (int c = lane * 4; c < p.hd; c += 128) st4(dst + c, ld4(src + c));
+    for (int c = lane * 4; c < p.hd; c += 128) st4(dst + c, biased(c));
     return;
   }
   float* s = rows + warp * p.hd;
   float ss = 0.f;
   for (int c = lane * 4; c < p.hd; c += 128) {
-    const float4 x = ld4(src + c);
+    const float4 x = biased(c);
     ss += x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w;
     *reinterpret_cast<float4*>(s + c) = x;
   }
@@ -167,6 +174,66 @@ __global__ void __launch_bounds__(256) head_prep_kernel(const MbBlockPrep p) {
     return second ? s[iv] * cs[pr] + s[iu] * cs[half + pr] : s[iu] * cs[pr] - s[iv] * cs[half + pr];
   };
   for (int c = lane * 4; c < p.hd; c += 128) st4(dst + c, make_float4(turned(c), turned(c + 1), turned(c + 2), turned(c + 3)));
+}
+
+// Biases, rotation (pairs half the rotated width apart, that half a multiple of 8) and store, without norms: a thread owns eight
+// pairs of a head, or eight columns that pass.
+template <typename T>
+__global__ void __launch_bounds__(256) pair_prep_kernel(const MbBlockPrep p, int q_items, int k_items, int v_items) {
+  const int per = p.heads * q_items + p.kv_heads * (k_items + v_items);
+  const long long id = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (id >= static_cast<long long>(p.T) * per) return;
+  const int t = static_cast<int>(id / per), half = p.dims / 2, h8 = half / 8;
+  int i = static_cast<int>(id % per), off, part;           // first column of the head in x, piece of the head
+  T* row = static_cast<T*>(p.x) + static_cast<size_t>(t) * p.ldx;
+  T* dst;
+  bool turns = true;
+  if (i < p.heads * q_items) {
+    off = p.q_off + (i / q_items) * p.hd;
+    part = i % q_items;
+    dst = row + off;
+  } else {
+    i -= p.heads * q_items;
+    const bool is_v = i >= p.kv_heads * k_items;
+    if (is_v) i -= p.kv_heads * k_items;
+    const int items = is_v ? v_items : k_items, h = i / items;
+    const int64_t slot = p.slots[t];
+    if (slot < 0) return;
+    part = i % items;
+    off = (is_v ? p.v_off : p.k_off) + h * p.hd;
+    dst = static_cast<T*>(is_v ? p.v_cache : p.k_cache) + (slot / p.page_size) * p.page_stride + h * p.head_stride +
+          static_cast<long long>(slot % p.page_size) * p.hd;
+    turns = !is_v;
+  }
+  auto take = [&](Vec8<T>& x, int c) {
+    x.load(row + off + c);
+    if (!p.bias) return;
+    const float4 a = *reinterpret_cast<const float4*>(p.bias + off + c), b = *reinterpret_cast<const float4*>(p.bias + off + c + 4);
+    x.v[0] += a.x; x.v[1] += a.y; x.v[2] += a.z; x.v[3] += a.w; x.v[4] += b.x; x.v[5] += b.y; x.v[6] += b.z; x.v[7] += b.w;
+  };
+  Vec8<T> u;
+  if (!turns || part >= h8) {
+    const int c = turns ? p.dims + (part - h8) * 8 : part * 8;
+    take(u, c);
+    u.store(dst + c);
+    return;
+  }
+  const int c = part * 8;
+  Vec8<T> v;
+  take(u, c);
+  take(v, half + c);
+  const float* cs = p.cos_sin + static_cast<size_t>(p.positions[t]) * p.dims + c;
+  float co[8], si[8];
+  *reinterpret_cast<float4*>(co) = *reinterpret_cast<const float4*>(cs); *reinterpret_cast<float4*>(co + 4) = *reinterpret_cast<const float4*>(cs + 4);
+  *reinterpret_cast<float4*>(si) = *reinterpret_cast<const float4*>(cs + half); *reinterpret_cast<float4*>(si + 4) = *reinterpret_cast<const float4*>(cs + half + 4);
+#pragma unroll
+  for (int k = 0; k < 8; ++k) {
+    const float a = u.v[k], b = v.v[k];
+    u.v[k] = a * co[k] - b * si[k];
+    v.v[k] = b * co[k] + a * si[k];
+  }
+  u.store(dst + c);
+  v.store(dst + half + c);
 }
 
 constexpr int kPlanSeqs = 4096;
@@ -309,6 +376,17 @@ extern "C" int mb_block_prep(const MbBlockPrep* p, int dtype, cudaStream_t strea
     return MB_ERR_SHAPE;
   if ((reinterpret_cast<uintptr_t>(p->x) | reinterpret_cast<uintptr_t>(p->k_cache) | reinterpret_cast<uintptr_t>(p->v_cache)) & 15)
     return MB_ERR_ALIGN;
+  if (p->bias && (!p->halves || (reinterpret_cast<uintptr_t>(p->bias) & 15))) return MB_ERR_SHAPE;
+  if (!p->q_norm && !p->k_norm && p->halves && p->dims % 16 == 0 && !p->silu_n && !p->relu2_n &&
+      (reinterpret_cast<uintptr_t>(p->cos_sin) & 15) == 0) {
+    const int rot = p->dims / 16, rest = (p->hd - p->dims) / 8, q = rot + (p->bias ? rest : 0);
+    const long long n = static_cast<long long>(p->T) * (p->heads * q + p->kv_heads * (rot + rest + p->hd / 8));
+    if (n == 0) return MB_OK;
+    const dim3 g(static_cast<unsigned>((n + 255) / 256));
+    const cudaError_t e = dtype == kF32 ? launch_plain(winattn::pair_prep_kernel<float>, g, dim3(256), 0, stream, *p, q, rot + rest, p->hd / 8)
+                                        : launch_plain(winattn::pair_prep_kernel<__nv_bfloat16>, g, dim3(256), 0, stream, *p, q, rot + rest, p->hd / 8);
+    return e == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
+  }
   if (p->q_norm || p->k_norm || p->halves) {
     if (p->silu_n || p->relu2_n || p->norm_dim <= 0 || p->norm_dim > p->hd || p->hd > 1024) return MB_ERR_SHAPE;
     const dim3 g(p->T, (p->heads + 2 * p->kv_heads + 7) / 8);

@@ -475,7 +475,7 @@ __global__ void __launch_bounds__(256) head_out_kernel(const MbHeadOut p) {
   const size_t t = static_cast<size_t>(unit / p.heads);
   const int h = static_cast<int>(unit % p.heads);
   const float* o = p.o + unit * V;
-  const T *gate = static_cast<const T*>(p.gate) + t * p.ld_gate + h * V, *w = static_cast<const T*>(p.norm_w);
+  const T *gate = static_cast<const T*>(p.gate) + t * p.ld_gate + h * V, *w = static_cast<const T*>(p.norm_w) + h * p.w_stride;
   T* out = static_cast<T*>(p.out) + t * p.ld_out + h * V;
   float ss = 0.f;
   if (V <= 256 && V % 4 == 0 && p.ld_gate % 4 == 0 && p.ld_out % 4 == 0 &&

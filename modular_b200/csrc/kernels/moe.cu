@@ -5,7 +5,8 @@
 //                             best `topk_group` groups, top-k experts inside them, weights from
 //                             the un-biased scores, optional normalisation, times a scaling factor.
 //   moe_router_softmax_topk   plain softmax top-k routing (Mixtral / Qwen style).
-//   moe_score_route           the group-limited choice with one warp per token, which also counts the pairs of every
+//   moe_score_route           the group-limited choice (sigmoid or softmax scores, groups by their best or two best, identity
+//                             experts without weights among the candidates) with one warp per token, which also counts the pairs of every
 //   moe_place_rows            expert; the second kernel scans the counts and copies token rows into expert order, so a
 //                             routed layer costs two launches between its router product and its experts.
 //   moe_table_route           routing by token id: a table names every id's experts, so the expert order of
@@ -197,32 +198,49 @@ template <int EPL>
 __global__ void __launch_bounds__(kRouteWarps * 32)
 score_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int32_t* __restrict__ ids,
                    float* __restrict__ w, int32_t* __restrict__ rank, int32_t* __restrict__ counts, int T, int E, int n_group, int keep,
-                   int top_k, int norm_topk, float scaling) {
+                   int top_k, int norm_topk, float scaling, int softmax, int group_max, int real) {
   extern __shared__ float sh[];                  // per warp: choice scores [E] | group scores [n_group]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, t = blockIdx.x * kRouteWarps + warp;
   if (t >= T) return;
   float *choice = sh + warp * (E + n_group), *gscore = choice + E;
   const int gsize = E / n_group;
   float score[EPL], mine[EPL];
+  if (softmax) {
+    float top = -INFINITY, sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) {
+      const int e = lane + 32 * i;
+      score[i] = e < E ? logits[static_cast<size_t>(t) * ld + e] : -INFINITY;
+      top = fmaxf(top, score[i]);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) { score[i] = expf(score[i] - top); sum += score[i]; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+#pragma unroll
+    for (int i = 0; i < EPL; ++i) score[i] /= sum;
+  }
 #pragma unroll
   for (int i = 0; i < EPL; ++i) {
     const int e = lane + 32 * i;
-    score[i] = 0.f; mine[i] = -INFINITY;
+    mine[i] = -INFINITY;
     if (e < E) {
-      score[i] = 1.f / (1.f + expf(-logits[static_cast<size_t>(t) * ld + e]));
+      if (!softmax) score[i] = 1.f / (1.f + expf(-logits[static_cast<size_t>(t) * ld + e]));
       mine[i] = score[i] + (bias ? bias[e] : 0.f);
       choice[e] = mine[i];
     }
   }
   __syncwarp();
   if (keep < n_group) {
-    for (int g = lane; g < n_group; g += 32) {   // sum of the two largest choice scores of a group
+    for (int g = lane; g < n_group; g += 32) {   // the largest choice score of a group, or the sum of its two largest
       float m1 = -INFINITY, m2 = -INFINITY;
       for (int j = 0; j < gsize; ++j) {
         const float v = choice[g * gsize + j];
         if (v > m1) { m2 = m1; m1 = v; } else if (v > m2) { m2 = v; }
       }
-      gscore[g] = gsize > 1 ? m1 + m2 : m1;
+      gscore[g] = gsize > 1 && !group_max ? m1 + m2 : m1;
     }
     __syncwarp();
 #pragma unroll
@@ -266,7 +284,7 @@ score_route_kernel(const float* __restrict__ logits, int ld, const float* __rest
     const size_t i = static_cast<size_t>(t) * top_k + lane;
     ids[i] = my_id;
     w[i] = my_w * scaling;
-    rank[i] = my_id < E ? atomicAdd(&counts[my_id], 1) : -1;
+    rank[i] = my_id < real ? atomicAdd(&counts[my_id], 1) : -1;
   }
 }
 
@@ -433,9 +451,10 @@ extern "C" int mb_moe_router_group_limited(const float* logits, const float* bia
 }
 
 extern "C" int mb_moe_score_route(const float* logits, int ld, const float* bias, int32_t* ids, float* w, int32_t* rank, int32_t* counts,
-                                  int T, int E, int n_group, int keep, int top_k, int norm_topk, float scaling, cudaStream_t stream) {
+                                  int T, int E, int n_group, int keep, int top_k, int norm_topk, float scaling, int softmax, int group_max,
+                                  int identity, cudaStream_t stream) {
   if (T <= 0) return MB_OK;
-  if (E <= 0 || E > 1024 || n_group < 1 || E % n_group || keep < 1 || keep > n_group || top_k < 1 || top_k > 32 ||
+  if (E <= 0 || E > 1024 || identity < 0 || identity >= E || n_group < 1 || E % n_group || keep < 1 || keep > n_group || top_k < 1 || top_k > 32 ||
       top_k > keep * (E / n_group))
     return MB_ERR_SHAPE;
   const dim3 grid((T + kRouteWarps - 1) / kRouteWarps), block(kRouteWarps * 32);
@@ -443,7 +462,7 @@ extern "C" int mb_moe_score_route(const float* logits, int ld, const float* bias
   if (smem > 48 * 1024) return MB_ERR_TOO_LARGE;
   auto go = [&](auto kern) {
     return launch_plain(kern, grid, block, smem, stream, logits, ld, bias, ids, w, rank, counts, T, E, n_group, keep, top_k, norm_topk,
-                        scaling) == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
+                        scaling, softmax, group_max, E - identity) == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
   };
   if (E <= 32) return go(score_route_kernel<1>);
   if (E <= 64) return go(score_route_kernel<2>);

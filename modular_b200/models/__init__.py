@@ -166,6 +166,35 @@ def _mavidra_family() -> ModelFamily:
     return ModelFamily("mavidra", MavidraConfig, MavidraWeights, MavidraModel, kv, act)
 
 
+def _vobosun_family() -> ModelFamily:
+    from ..kv_cache import KVCacheParams
+    from .vobosun import ATTENTION, VobosunConfig, VobosunModel, VobosunWeights
+
+    def kv(cfg, page, dtype, prefix):
+        # one key/value plane per attention layer; recurrent states and the last normed rows in slots, which rule out prefix sharing
+        planes = len(cfg.of_type(ATTENTION))
+        return KVCacheParams(max(planes, 1), cfg.cache_heads, cfg.head_width if planes else 8, page, dtype, False, False, cfg.state_specs())
+
+    def act(cfg, T, B):
+        per_tok = 0
+        for i, l in enumerate(cfg.layers):
+            if l["type"] == ATTENTION:
+                a = cfg.attention(i)
+                n = (2 * a.heads_pad + 2 * a.kv_heads) * cfg.head_width
+            else:
+                n = 12 * l["mixer"]["heads"] * cfg.delta(i).dim8
+            ff = l.get("mlp")
+            if ff is not None and ff["kind"] == "dense":
+                n = max(n, ff["ff"])
+            elif ff is not None:
+                n = max(n, ff["router"]["top"] * (2 * cfg.width_pad + ff["expert"]["ff"]) + 2 * (ff.get("shared") or {"ff": 0})["ff"])
+            per_tok = max(per_tok, 8 * cfg.width_pad + n)
+        state = kv(cfg, 64, torch.bfloat16, False).state_bytes_per_slot
+        return T * per_tok * 4 + B * cfg.vocab_size * 4 + B * state + (256 << 20)
+
+    return ModelFamily("vobosun", VobosunConfig, VobosunWeights, VobosunModel, kv, act)
+
+
 def _bert_family() -> ModelFamily:
     from ..kv_cache import KVCacheParams
     from .bert import BertConfig, BertModel, BertWeights
@@ -183,7 +212,7 @@ def _bert_family() -> ModelFamily:
 def family_for(config) -> ModelFamily:
     """The family that serves `config` (matched on the config class)."""
     for make in (_llama_family, _deepseek_family, _mamba_family, _lfm2_family, _gotunex_family, _vipotar_family,
-                 _mavidra_family, _bert_family):
+                 _mavidra_family, _vobosun_family, _bert_family):
         fam = make()
         if isinstance(config, fam.config_class):
             return fam

@@ -306,22 +306,32 @@ class TableRouter:
 
 @dataclass
 class ScoreRouterConfig:
-    """Sigmoid scores, a choice among the ``keep`` best of ``groups`` groups of neighbouring experts (a group counts its two
-    best choice scores), weights from the scores without the correction."""
+    """Sigmoid scores (``softmax``: a softmax over all candidates), a choice among the ``keep`` best of ``groups`` groups of
+    neighbouring candidates (a group counts its two best choice scores, or with ``group_max`` its best one), weights from the scores
+    without the correction. The candidates are the experts and, behind them, ``identity`` identity experts, which give the input back
+    and have no weights."""
     experts: int
     top: int
     groups: int = 1
     keep: int = 1
     renormalize: bool = False
     scaling: float = 1.0
+    softmax: bool = False
+    group_max: bool = False
+    identity: int = 0
 
     def __post_init__(self):
-        if self.experts < 1 or self.groups < 1 or self.experts % self.groups:
-            raise ValueError(f"{self.experts} experts cannot form {self.groups} equal groups")
-        if not 1 <= self.keep <= self.groups or not 1 <= self.top <= self.keep * (self.experts // self.groups):
-            raise ValueError(f"{self.top} experts out of {self.keep} groups of {self.experts // self.groups}")
-        if self.top > 32 or self.experts > 1024:
+        n = self.candidates
+        if self.experts < 1 or self.identity < 0 or self.groups < 1 or n % self.groups:
+            raise ValueError(f"{n} experts cannot form {self.groups} equal groups")
+        if not 1 <= self.keep <= self.groups or not 1 <= self.top <= self.keep * (n // self.groups):
+            raise ValueError(f"{self.top} experts out of {self.keep} groups of {n // self.groups}")
+        if self.top > 32 or n > 1024:
             raise ValueError("at most 32 of at most 1024 experts per token")
+
+    @property
+    def candidates(self) -> int:
+        return self.experts + self.identity
 
 
 class ScoreRouter:
@@ -330,31 +340,45 @@ class ScoreRouter:
 
     def __init__(self, cfg: ScoreRouterConfig, gate, correction, width_pad: int, device, dtype):
         self.cfg = cfg
-        E8 = (cfg.experts + 7) // 8 * 8
+        E8 = (cfg.candidates + 7) // 8 * 8
         self.gate = F.pad(gate, (0, width_pad - gate.shape[1], 0, E8 - gate.shape[0])).to(device=device, dtype=dtype).contiguous()
         self.correction = None if correction is None else correction.to(device=device, dtype=torch.float32).contiguous()
 
+    def choose_reference(self, logits):
+        """logits [T, candidates] -> (candidates chosen [T, top], weights fp32 [T, top])."""
+        c, z = self.cfg, logits.float()
+        scores = torch.softmax(z, -1) if c.softmax else torch.sigmoid(z)
+        choice = scores if self.correction is None else scores + self.correction
+        g = choice.view(z.shape[0], c.groups, -1)
+        best = g.topk(1 if c.group_max else min(2, g.shape[2]), dim=-1).values.sum(-1)
+        kept = torch.zeros_like(best, dtype=torch.bool).scatter_(1, best.topk(c.keep, dim=-1).indices, True)
+        ids = g.masked_fill(~kept.unsqueeze(-1), float("-inf")).reshape(z.shape).topk(c.top, dim=-1).indices
+        w = scores.gather(1, ids)
+        if c.renormalize:
+            w = w / (w.sum(-1, keepdim=True) + 1e-20)
+        return ids, w * c.scaling
+
     def route(self, x, counts):
         """x [T, width]; ``counts`` int32 [experts], zero. Returns (rows [T * top, width] in expert order, offsets int32
-        [experts + 1], inverse int32 [T, top]: row of every pair, weights fp32 [T, top])."""
+        [experts + 1], inverse int32 [T, top]: row of every pair (-1: an identity expert), weights fp32 [T, top])."""
         c, T, dev = self.cfg, x.shape[0], x.device
         logits = ops.linear(x, self.gate, out_dtype=torch.float32)
         if not x.is_cuda:
-            m = MoEConfig(0, 0, c.experts, c.top, n_group=c.groups, topk_group=c.keep, norm_topk_prob=c.renormalize,
-                          routed_scaling_factor=c.scaling)
-            ids, w = route_group_limited_ref(logits[:, : c.experts], self.correction, m)
-            flat = ids.reshape(-1).long()
-            order = torch.argsort(flat, stable=True)
+            ids, w = self.choose_reference(logits[:, : c.candidates])
+            flat = ids.reshape(-1)
+            order = torch.argsort(flat, stable=True)             # identity experts come last
             inverse = torch.empty_like(order)
             inverse[order] = torch.arange(order.numel())
+            inverse[flat >= c.experts] = -1
             offsets = torch.zeros(c.experts + 1, dtype=torch.int32)
-            offsets[1:] = torch.cumsum(torch.bincount(flat, minlength=c.experts), 0)
+            offsets[1:] = torch.cumsum(torch.bincount(flat, minlength=c.candidates)[: c.experts], 0)
             return x[order // c.top], offsets, inverse.view(T, c.top).int(), w
         i32 = lambda *s: torch.empty(*s, dtype=torch.int32, device=dev)
         ids, rank, inverse, offsets = i32(T, c.top), i32(T, c.top), i32(T, c.top), i32(c.experts + 1)
         w = torch.empty(T, c.top, dtype=torch.float32, device=dev)
         L = _lib()
-        L.moe_score_route(logits, self.correction, ids, w, rank, counts, c.groups, c.keep, c.renormalize, c.scaling)
+        L.moe_score_route(logits, self.correction, ids, w, rank, counts, c.groups, c.keep, c.renormalize, c.scaling, c.softmax,
+                          c.group_max, c.identity)
         rows = torch.empty(T * c.top, x.shape[1], dtype=x.dtype, device=dev)
         L.moe_place_rows(x, ids, rank, counts, offsets, inverse, rows)
         return rows, offsets, inverse, w
@@ -384,3 +408,10 @@ def expert_mlp(xp, offsets, w_gate_up, w_down, max_rows: int):
         L.grouped_gemm_bf16(xp, w_gate_up, act, offsets, max_rows, True, 0)
         L.grouped_gemm_bf16(act, w_down, out, offsets, max_rows, False, 0)
     return out
+
+
+def gated_mlp(x, w_gate_up, w_down):
+    """One SwiGLU feed-forward: x [T, H], w_gate_up [2I, H], w_down [H, I]."""
+    if x.is_cuda and x.dtype == torch.float32:
+        return ops.linear(ops.silu_mul(ops.linear(x, w_gate_up)), w_down)
+    return ops.linear(ops.linear_swiglu(x, w_gate_up), w_down)

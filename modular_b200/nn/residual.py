@@ -19,6 +19,12 @@ the next one in a single kernel (``csrc/kernels/residual_norm.cu``); the PyTorch
 ``n1 = norm(x; w1, b1)``; layer norms with biases, RMS norms without. ``inject`` adds rows of a second table, chosen by ids of
 their own, to the embedding.
 
+``tanh_seam`` (``csrc/kernels/tanh_seam.cu``) is the same seam for elementwise norms, dynamic tanh ``T(y) = tanh(alpha * y) * w + b``,
+each given as a triple ``(alpha, w, b)``: ``x_out = x + T(u)``, ``n1 = T(x_out)``. The branch ``u`` is ``a``, the weighted expert
+outputs ``e``, or their sum; a pair whose ``inverse`` is negative belongs to an identity expert and gives the token's row of
+``self_rows``. With a ``shift`` vector, ``n1[t]`` moves by it towards the normed row of the token before. That needs a second buffer
+``x_out`` and the sequences of the step; ``prev`` [slots, width] keeps every sequence's last normed row.
+
 The norm is computed in fp32 and rounded once.
 """
 
@@ -126,3 +132,52 @@ def sandwich_norm(x, ids=None, table=None, scale=1.0, inject_ids=None, inject=No
                                        cols, store_x, eps)
     _lib().sandwich_norm(x, ids, table, float(scale), inject_ids, inject, a, e, inverse, pair_w, rows, w_u, b_u, float(mult), w1, b1, n1,
                          cols or x.shape[1], store_x, float(eps), x.shape[0] if rows is None else rows.numel())
+
+
+def tanh_seam_reference(x=None, x_out=None, ids=None, table=None, scale=1.0, a=None, e=None, inverse=None, pair_w=None, self_rows=None,
+                        rows=None, norm_u=None, norm1=None, n1=None, shift=None, prev=None, state_idx=None, q_start=None, q_len=None,
+                        kv_len=None):
+    T = lambda y, n: torch.tanh(n[0] * y) * n[1].float() + n[2].float()
+    idx = torch.arange(x.shape[0] if x is not None else ids.numel()) if rows is None else rows.long()
+    h = x[idx] if table is None else table[ids[idx]].float() * scale
+    u = None if a is None else a[idx, : h.shape[1]].float()
+    if e is not None:
+        inv, w = inverse[idx].long(), pair_w[idx].unsqueeze(-1)
+        y = torch.where((inv >= 0).unsqueeze(-1), e[inv.clamp(min=0)].float(), 0.0)
+        if self_rows is not None:
+            y = torch.where((inv >= 0).unsqueeze(-1), y, self_rows[idx, : h.shape[1]].float().unsqueeze(1))
+        u = (y * w).sum(1) if u is None else u + (y * w).sum(1)
+    if u is not None:
+        h = h + T(u, norm_u)
+    if x_out is not None:
+        x_out[idx] = h
+    if norm1 is None:
+        return
+    y = T(h, norm1)
+    if shift is not None:
+        before = torch.zeros_like(y)
+        before[1:] = y[:-1]
+        for s in range(q_len.numel()):
+            t0, n, slot = int(q_start[s]), int(q_len[s]), int(state_idx[s])
+            if n == 0:
+                continue
+            before[t0] = prev[slot] if slot >= 0 and int(kv_len[s]) > n else 0.0
+            if slot >= 0:
+                prev[slot] = y[t0 + n - 1]
+        y = y + (before - y) * shift.float()
+    n1[: idx.numel()] = y.to(n1.dtype)
+
+
+def tanh_seam(x=None, x_out=None, ids=None, table=None, scale=1.0, a=None, e=None, inverse=None, pair_w=None, self_rows=None, rows=None,
+              norm_u=None, norm1=None, n1=None, shift=None, prev=None, state_idx=None, q_start=None, q_len=None, kv_len=None):
+    """``x`` (or ``table`` rows) fp32 [T, width] -> ``x_out`` (may be ``x`` without a shift; None: not stored) and ``n1``."""
+    some = x if x is not None else table
+    if not some.is_cuda:
+        return tanh_seam_reference(x, x_out, ids, table, scale, a, e, inverse, pair_w, self_rows, rows, norm_u, norm1, n1, shift, prev,
+                                   state_idx, q_start, q_len, kv_len)
+    if e is None:
+        self_rows = None
+    n_rows = rows.numel() if rows is not None else x.shape[0] if x is not None else ids.numel()
+    (au, wu, bu), (a1, w1, b1) = norm_u or (0.0, None, None), norm1 or (0.0, None, None)
+    _lib().tanh_seam(x, x_out, ids, table, float(scale), a, e, inverse, pair_w, self_rows, rows, wu, bu, au, w1, b1, a1, n1, shift, prev,
+                     state_idx, q_start, q_len, kv_len, shift is not None and n_rows == q_len.numel(), some.shape[1], n_rows)

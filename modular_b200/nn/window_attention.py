@@ -1,9 +1,9 @@
-"""Softmax attention over the keys of a sliding window, with grouped heads, partial rotation, a sink, and optionally normed
+"""Softmax attention over the keys of a sliding window, with grouped heads, partial rotation, a sink, and optionally biases, normed
 queries and keys and an output gate per head.
 
 A query at position i sees the keys j with ``0 <= i - j < window`` (0: all before it). Queries and keys rotate in
 neighbouring pairs (or pairs half the rotated width apart, ``halves``) over their first ``rot_dims`` dimensions; ``qk_norm``
-RMS-norms every head of both before that. ``sink`` is one score per query head that takes part in the softmax denominator
+RMS-norms every head of both before that. ``bias`` adds a vector to q, k and v (in fp32, on the way through the rotation). ``sink`` is one score per query head that takes part in the softmax denominator
 only: ``p_j = exp(s_j) / (exp(sink) + sum_j exp(s_j))``. ``head_gate`` multiplies a head's output by ``sigmoid(W_g h)``, inside
 the attention kernels; ``out_mult`` is a further factor on it.
 
@@ -50,6 +50,7 @@ class WindowAttentionConfig:
     zero_sink: bool = False          # a sink of score 0 for every head
     sink: bool = False               # a learned sink
     halves: bool = False             # pairs (i, i + rot_dims / 2)
+    bias: bool = False               # on q, k and v; needs halves
     qk_norm: bool = False
     eps: float = 1e-6                # of those norms
     head_gate: bool = False
@@ -60,6 +61,8 @@ class WindowAttentionConfig:
             raise ValueError(f"{self.heads} heads are no multiple of {self.kv_heads} key/value heads")
         if self.rot_dims % 2 or self.rot_dims > self.dim:
             raise ValueError(f"{self.rot_dims} rotated dimensions of {self.dim}")
+        if self.bias and not self.halves:
+            raise ValueError("biases are added by the kernel for pairs half the rotated width apart")
         if self.out_mult != 1.0 and not self.head_gate:
             raise ValueError("a factor on the output is part of the head gate")
         if self.window < 0:
@@ -126,6 +129,11 @@ class WindowAttention:
         self.sink = torch.zeros(c.heads_pad, dtype=torch.float32, device=device) if c.zero_sink else None
         if c.sink:
             self.sink = per_head(tensors["sink"].float()).to(device=device).contiguous()
+        self.bias = None
+        if c.bias:
+            column = lambda n, *a: rows(tensors[n + ".b"].float().view(-1, 1), *a)[:, 0]
+            parts = [column("q", G, Gp, c.dim), column("k", 1, 1, c.dim), column("v", 1, 1, c.vdim)]
+            self.bias = torch.cat(parts).to(device=device, dtype=torch.float32).contiguous()
         norm = lambda t: F.pad(t, (0, hd - c.dim)).to(device=device, dtype=dtype).contiguous()
         self.q_norm, self.k_norm = (norm(tensors["q.norm"]), norm(tensors["k.norm"])) if c.qk_norm else (None, None)
 
@@ -133,7 +141,8 @@ class WindowAttention:
         """Norms and rotation of the queries in place, and of the keys on their way into the cache with the values."""
         c = self.cfg
         block_prep(px, c.heads_pad, self.k_off, self.v_off, c.kv_heads, c.rot_dims, positions, cos_sin, slots, kv, plane,
-                   q_norm=self.q_norm, k_norm=self.k_norm, norm_dim=c.dim, eps=c.eps, halves=c.halves)
+                   q_norm=self.q_norm, k_norm=self.k_norm, norm_dim=c.dim, eps=c.eps, halves=c.halves,
+                   bias=self.bias)
 
     def __call__(self, q, kv, plane: int, block_table, q_start, q_len, kv_len, plan: Optional[AttentionPlan], out=None, gate=None):
         """q [T, heads_pad * hd]: rotated queries; the step's keys and values are in the cache. Returns [T, heads_pad * hd]."""
@@ -174,19 +183,21 @@ def window_attention(q, kv, plane, block_table, q_start, q_len, kv_len, heads, k
 
 
 def block_prep(x, heads, k_off, v_off, kv_heads, dims, positions, cos_sin, slots, kv, plane, silu=(0, 0), relu2=(0, 0), q_norm=None,
-               k_norm=None, norm_dim=0, eps=1e-6, halves=False):
+               k_norm=None, norm_dim=0, eps=1e-6, halves=False, bias=None):
     """What lies between the stacked input projection ``x`` of a parallel block and its branches, in one launch: queries
     (columns from 0) rotate in place, keys rotate and go into the cache with the values, ``silu`` and ``relu2`` (squared
     relu) name column ranges (first, count) that are activated in place. ``q_norm`` / ``k_norm`` [head width]: heads are RMS-normed
-    over their first ``norm_dim`` columns first. ``halves``: pairs lie ``dims / 2`` apart. These two exclude the activations."""
+    over their first ``norm_dim`` columns first. ``halves``: pairs lie ``dims / 2`` apart. These two exclude the activations.
+    ``bias`` (fp32, one value per column, with ``halves``) is added to q, k and v first."""
     if x.is_cuda:
         _lib().block_prep(x, 0, heads, k_off, v_off, kv_heads, dims, positions, cos_sin, slots, kv, plane, *silu, *relu2, q_norm=q_norm,
-                          k_norm=k_norm, norm_dim=norm_dim, eps=eps, halves=halves)
+                          k_norm=k_norm, norm_dim=norm_dim, eps=eps, halves=halves, bias=bias)
         return
     T, hd, page = x.shape[0], kv.shape[5], kv.shape[4]
+    take = lambda off, n: x[:, off: off + n * hd].float().add(0.0 if bias is None else bias[off: off + n * hd]).reshape(T, n, hd)
 
     def rotated(t, w):
-        t = t.float().clone()
+        t = t.clone()
         if w is not None:
             t *= torch.rsqrt(t.pow(2).sum(-1, keepdim=True) / (norm_dim or hd) + eps) * w.float()
         if dims and halves:
@@ -201,9 +212,9 @@ def block_prep(x, heads, k_off, v_off, kv_heads, dims, positions, cos_sin, slots
             t[..., 0:dims:2], t[..., 1:dims:2] = u * c - v * s, v * c + u * s
         return t
 
-    x[:, : heads * hd] = rotated(x[:, : heads * hd].reshape(T, heads, hd), q_norm).reshape(T, -1).to(x.dtype)
-    k = rotated(x[:, k_off: k_off + kv_heads * hd].reshape(T, kv_heads, hd), k_norm).to(kv.dtype)
-    v = x[:, v_off: v_off + kv_heads * hd].reshape(T, kv_heads, hd)
+    x[:, : heads * hd] = rotated(take(0, heads), q_norm).reshape(T, -1).to(x.dtype)
+    k = rotated(take(k_off, kv_heads), k_norm).to(kv.dtype)
+    v = take(v_off, kv_heads).to(kv.dtype)
     ok = slots >= 0
     pg, off = slots[ok] // page, slots[ok] % page
     kv[pg, 0, plane, :kv_heads, off] = k[ok]

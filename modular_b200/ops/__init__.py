@@ -22,7 +22,7 @@ from . import reference as ref
 __all__ = [
     "linear", "linear_swiglu", "rms_norm", "add_rms_norm", "silu_mul", "embedding",
     "rope_kv_store", "paged_attention", "build_attention_plan", "argmax", "sample",
-    "apply_penalties", "gelu_tanh", "softcap", "sigmoid_gate", "gemm_workspace", "check_device_error", "linear_decode", "decode_gemm_workspace",
+    "apply_penalties", "gelu_tanh", "xielu", "tanh", "softcap", "sigmoid_gate", "gemm_workspace", "check_device_error", "linear_decode", "decode_gemm_workspace",
 ]
 
 _WORKSPACES: dict[int, torch.Tensor] = {}
@@ -269,6 +269,22 @@ def gelu_tanh(x):
     if not x.is_cuda:
         return x.copy_(ref.gelu_tanh(x))
     _lib().gelu_tanh(x)
+    return x
+
+
+def xielu(x, up: float, down: float):
+    """``up z^2 + z / 2`` for z > 0, ``down (exp(z) - 1 - z) + z / 2`` otherwise, in place; rows of a multiple of 8 values."""
+    if not x.is_cuda:
+        return x.copy_(ref.xielu(x, up, down))
+    _lib().xielu(x, float(up), float(down))
+    return x
+
+
+def tanh(x):
+    """In place over a matrix view (unit column stride, a multiple of 8 columns)."""
+    if not x.is_cuda:
+        return x.copy_(torch.tanh(x.float()))
+    _lib().tanh_cols(x)
     return x
 
 

@@ -46,6 +46,12 @@ def silu_mul(gate_up):
     return (F.silu(g) * u).to(gate_up.dtype)
 
 
+def xielu(x, up: float, down: float):
+    z = x.float()
+    low = z.clamp(max=0.0)
+    return torch.where(z > 0, up * z * z, down * (torch.expm1(low) - low)).add(0.5 * z).to(x.dtype)
+
+
 def gelu_tanh(x):
     return F.gelu(x.float(), approximate="tanh").to(x.dtype)
 

@@ -369,6 +369,13 @@ def _register_builtin() -> None:
         name="Mavidra", config_class=MavidraConfig, weights_class=MavidraWeights, model_class=MavidraModel,
         default_encoding="bfloat16", supported_encodings=("bfloat16", "float32"), example_repo_ids=(),
         preset_configs={"tiny-mavidra": MavidraConfig.tiny}), allow_override=True)
+    from ..models.vobosun import VobosunConfig, VobosunModel, VobosunWeights
+
+    # softmax attention and generalized delta-rule layers with elementwise norms and a token shift, dense or routed feed-forwards
+    PIPELINE_REGISTRY.register(SupportedArchitecture(
+        name="Vobosun", config_class=VobosunConfig, weights_class=VobosunWeights, model_class=VobosunModel,
+        default_encoding="bfloat16", supported_encodings=("bfloat16", "float32"), example_repo_ids=(),
+        preset_configs={"tiny-vobosun": VobosunConfig.tiny}), allow_override=True)
     from ..models.bert import BertConfig, BertModel, BertWeights
 
     # encoder-only embedding models (bidirectional attention; MPNet adds relative-position biases); embeddings only
