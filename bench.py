@@ -310,6 +310,7 @@ DESIGNS = {
     "gotunex": ("gotunex_bench", "Gotunex", "layers", lambda model: model.startswith("gotunex (delta")),
     "vipotar": ("vipotar_bench", "Vipotar", "layer runs", lambda model: model == "vipotar"),
     "mavidra": ("mavidra_bench", "Mavidra", "layers", lambda model: model == "mavidra"),
+    "vobosun": ("vobosun_bench", "Vobosun", "layers", lambda model: model == "vobosun"),
 }
 
 
@@ -366,7 +367,8 @@ def main() -> int:
                          "concurrency 128 unless given); deepseek-v3: DeepSeek-V3 shapes, fp8 routed experts, "
                          "expert parallel over --gpus with data-parallel attention (concurrency 256 over all ranks); gotunex: "
                          "prefill / decode throughput and kernels of that design beside DeepSeek-V3 layers of equal size; vipotar: "
-                         "the same beside Gotunex and Llama layers of equal size; mavidra: the same beside Gotunex layers")
+                         "the same beside Gotunex and Llama layers of equal size; mavidra: the same beside Gotunex layers; vobosun: the "
+                         "same beside Mavidra and Gotunex layers")
     args = ap.parse_args()
     if args.model == "deepseek-v3":
         if args.impl == "reference":

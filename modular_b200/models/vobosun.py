@@ -289,7 +289,7 @@ class VobosunWeights:
         g = torch.Generator(device=device).manual_seed(seed)
         sd = {}
         for name, shape in cfg.tensor_shapes().items():
-            leaf, t = name.rsplit(".", 1)[-1], torch.randn(*shape, generator=g, device=device)
+            leaf, t = name.rsplit(".", 1)[-1], torch.randn(shape, generator=g, device=device)
             if leaf == "alpha":
                 t = 0.7 + 0.1 * t
             elif leaf in ("b", "correction"):
