@@ -35,19 +35,32 @@ __device__ __forceinline__ float4 affine_tanh(float4 y, float alpha, float4 w, f
                      fmaf(tanh_of<T>(alpha * y.z), w.z, b.z), fmaf(tanh_of<T>(alpha * y.w), w.w, b.w));
 }
 
+// One pair of a token: the row of its expert's output (negative: none) and its weight.
+struct __align__(8) Pair { int at; float w; };
+
+// Many small CTAs per SM keep more rows in flight than several rows per thread would.
 template <typename T, bool SHIFT, bool EXPERTS>
-__global__ void __launch_bounds__(256) tanh_seam_kernel(const MbTanhSeam p, int tile) {
-  constexpr int U = 4;                           // rows whose loads are in flight together
+__global__ void __launch_bounds__(256, sizeof(T) == 4 ? 2 : EXPERTS ? 3 : SHIFT ? 6 : 8) tanh_seam_kernel(const MbTanhSeam p, int tile) {
+  extern __shared__ Pair pairs[];                // EXPERTS: of the row before the tile, then of its rows
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+  const int tb = blockIdx.x * tile, te = min(tb + tile, p.n_rows), K = p.top_k;
+  if (EXPERTS) {
+    for (int i = threadIdx.x; i < (te - tb + 1) * K; i += blockDim.x) {
+      const int t = tb - 1 + i / K;
+      if (t < 0) continue;
+      const size_t at = static_cast<size_t>(p.rows && t >= tb ? p.rows[t] : t) * K + i % K;
+      pairs[i] = Pair{p.inverse[at], p.pair_w[at]};
+    }
+    __syncthreads();
+  }
   if (c >= p.cols_pad) return;
-  const int tb = blockIdx.x * tile, te = min(tb + tile, p.n_rows);
   const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
   auto weight = [&](const void* w) { return w ? ld4(static_cast<const T*>(w) + c) : zero; };
   const float4 wu = weight(p.w_u), bu = weight(p.b_u), w1 = weight(p.w1), b1 = weight(p.b1);
   const float4 mix = SHIFT ? weight(p.shift) : zero;
   const bool update = p.a != nullptr || EXPERTS;
-  // the stream and the branch of one row
-  auto load = [&](int row, float4& x, float4& u) {
+  // the stream and the branch of one row; `own`: its pairs, where they are staged
+  auto load = [&](int row, const Pair* own, float4& x, float4& u) {
     x = u = zero;
     if (p.table) {
       const int64_t id = p.ids[row];
@@ -60,15 +73,14 @@ __global__ void __launch_bounds__(256) tanh_seam_kernel(const MbTanhSeam p, int 
     }
     if (p.a) u = ld4(static_cast<const T*>(p.a) + static_cast<size_t>(row) * p.lda + c);
     if (EXPERTS) {
-      const size_t pair = static_cast<size_t>(row) * p.top_k;
+      // a pair without a row reads the token's own one: that of an identity expert, or any at weight zero
+      const T* none = p.self ? static_cast<const T*>(p.self) + static_cast<size_t>(row) * p.ld_self + c : static_cast<const T*>(p.e) + c;
+      const T* e = static_cast<const T*>(p.e) + c;
 #pragma unroll 4
-      for (int k = 0; k < p.top_k; ++k) {
-        const int at = p.inverse[pair + k];
-        if (at < 0 && !p.self) continue;
-        const float w = p.pair_w[pair + k];
-        const T* src = at >= 0 ? static_cast<const T*>(p.e) + static_cast<size_t>(at) * p.lde
-                               : static_cast<const T*>(p.self) + static_cast<size_t>(row) * p.ld_self;
-        const float4 y = ld4(src + c);
+      for (int k = 0; k < K; ++k) {
+        const Pair q = own ? own[k] : Pair{p.inverse[static_cast<size_t>(row) * K + k], p.pair_w[static_cast<size_t>(row) * K + k]};
+        const float w = q.at >= 0 || p.self ? q.w : 0.f;
+        const float4 y = ld4(q.at >= 0 ? e + static_cast<size_t>(q.at) * p.lde : none);
         u.x = fmaf(w, y.x, u.x); u.y = fmaf(w, y.y, u.y); u.z = fmaf(w, y.z, u.z); u.w = fmaf(w, y.w, u.w);
       }
     }
@@ -78,15 +90,16 @@ __global__ void __launch_bounds__(256) tanh_seam_kernel(const MbTanhSeam p, int 
     const float4 y = affine_tanh<T>(u, p.alpha_u, wu, bu);
     x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
   };
-  auto row_h = [&](int row) {
+  auto row_h = [&](int row, const Pair* own) {
     float4 x, u;
-    load(row, x, u);
+    load(row, own, x, u);
     add(x, u);
     return affine_tanh<T>(x, p.alpha_1, w1, b1);
   };
-  int s = 0, next = 0;                           // SHIFT: the sequence of the current row, the first row behind it
-  float4 prev = zero;
+  int s = 0, first = 0, next = 0;                // SHIFT: the sequence of the current row, its first row and the one behind it
+  float4 prev = zero, hx, hu;
   if (SHIFT) {
+    load(max(tb - 1, 0), pairs + (tb > 0 ? 0 : K), hx, hu);
     s = tb;
     if (!p.one_token) {
       int lo = 0, hi = p.B - 1;                  // the last sequence that starts at or before the first row
@@ -96,53 +109,52 @@ __global__ void __launch_bounds__(256) tanh_seam_kernel(const MbTanhSeam p, int 
       }
       s = lo;
     }
-    next = p.q_start[s] + p.q_len[s];
-    if (tb > p.q_start[s] && tb < next) prev = row_h(tb - 1);
+    first = p.q_start[s];
+    next = first + p.q_len[s];
   }
-  for (int t0 = tb; t0 < te; t0 += U) {
-    float4 x[U], u[U];
-#pragma unroll
-    for (int i = 0; i < U; ++i)
-      if (t0 + i < te) load(p.rows ? p.rows[t0 + i] : t0 + i, x[i], u[i]);
-#pragma unroll
-    for (int i = 0; i < U; ++i) {
-      const int t = t0 + i;
-      if (t >= te) break;
-      add(x[i], u[i]);
-      if (p.x_out) *reinterpret_cast<float4*>(p.x_out + static_cast<size_t>(p.rows ? p.rows[t] : t) * p.ldx + c) = x[i];
-      if (!p.w1) continue;
-      float4 h = affine_tanh<T>(x[i], p.alpha_1, w1, b1);
-      if (SHIFT) {
-        while (t >= next && s + 1 < p.B) { ++s; next = p.q_start[s] + p.q_len[s]; }
-        if (t == p.q_start[s] && p.q_len[s] > 0) {
-          const int n = p.q_len[s], slot = p.state_idx[s];
-          prev = zero;
-          if (slot >= 0) {
-            float* keep = p.prev + static_cast<size_t>(slot) * p.cols_pad + c;
-            if (p.kv_len[s] > n) prev = *reinterpret_cast<const float4*>(keep);
-            *reinterpret_cast<float4*>(keep) = n == 1 ? h : row_h(t + n - 1);
-          }
-        }
-        const float4 d = make_float4(prev.x - h.x, prev.y - h.y, prev.z - h.z, prev.w - h.w);
-        prev = h;
-        h = make_float4(fmaf(d.x, mix.x, h.x), fmaf(d.y, mix.y, h.y), fmaf(d.z, mix.z, h.z), fmaf(d.w, mix.w, h.w));
-      }
-      st4(static_cast<T*>(p.n1) + static_cast<size_t>(t) * p.ld1 + c, h);
+  for (int t = tb; t < te; ++t) {
+    const int row = p.rows ? p.rows[t] : t;
+    float4 x, u;
+    load(row, pairs + (t - tb + 1) * K, x, u);
+    if (SHIFT && t == tb && tb > first && tb < next) {
+      add(hx, hu);
+      prev = affine_tanh<T>(hx, p.alpha_1, w1, b1);
     }
+    add(x, u);
+    if (p.x_out) *reinterpret_cast<float4*>(p.x_out + static_cast<size_t>(row) * p.ldx + c) = x;
+    if (!p.w1) continue;
+    float4 h = affine_tanh<T>(x, p.alpha_1, w1, b1);
+    if (SHIFT) {
+      while (t >= next && s + 1 < p.B) { ++s; first = p.q_start[s]; next = first + p.q_len[s]; }
+      if (t == first && t < next) {
+        const int n = next - first, slot = p.state_idx[s];
+        prev = zero;
+        if (slot >= 0) {
+          float* keep = p.prev + static_cast<size_t>(slot) * p.cols_pad + c;
+          if (p.kv_len[s] > n) prev = *reinterpret_cast<const float4*>(keep);
+          *reinterpret_cast<float4*>(keep) = n > 1 ? row_h(next - 1, nullptr) : h;
+        }
+      }
+      const float4 d = make_float4(prev.x - h.x, prev.y - h.y, prev.z - h.z, prev.w - h.w);
+      prev = h;
+      h = make_float4(fmaf(d.x, mix.x, h.x), fmaf(d.y, mix.y, h.y), fmaf(d.z, mix.z, h.z), fmaf(d.w, mix.w, h.w));
+    }
+    st4(static_cast<T*>(p.n1) + static_cast<size_t>(t) * p.ld1 + c, h);
   }
 }
 
 template <typename T>
 static int run(const MbTanhSeam& p, cudaStream_t stream) {
   // few rows: small CTAs over the columns of one row; many rows: each thread walks over some
-  const int vec = p.cols_pad / 4, tile = p.n_rows <= 592 ? 1 : p.n_rows <= 4096 ? 4 : 8;
+  const int vec = p.cols_pad / 4, tile = p.n_rows <= 592 ? 1 : p.n_rows <= 4096 ? 4 : p.e ? 16 : 8;
   const int most = tile == 1 ? 128 : 256, threads = vec >= most ? most : (vec + 31) / 32 * 32;
   const dim3 grid((p.n_rows + tile - 1) / tile, (vec + threads - 1) / threads), block(threads);
+  const size_t smem = p.e ? static_cast<size_t>(tile + 1) * p.top_k * sizeof(Pair) : 0;      // at most 4.3 KiB
   cudaError_t e;
-  if (p.shift) e = p.e ? launch_plain(tanh_seam_kernel<T, true, true>, grid, block, 0, stream, p, tile)
-                       : launch_plain(tanh_seam_kernel<T, true, false>, grid, block, 0, stream, p, tile);
-  else e = p.e ? launch_plain(tanh_seam_kernel<T, false, true>, grid, block, 0, stream, p, tile)
-               : launch_plain(tanh_seam_kernel<T, false, false>, grid, block, 0, stream, p, tile);
+  if (p.shift) e = p.e ? launch_plain(tanh_seam_kernel<T, true, true>, grid, block, smem, stream, p, tile)
+                       : launch_plain(tanh_seam_kernel<T, true, false>, grid, block, smem, stream, p, tile);
+  else e = p.e ? launch_plain(tanh_seam_kernel<T, false, true>, grid, block, smem, stream, p, tile)
+               : launch_plain(tanh_seam_kernel<T, false, false>, grid, block, smem, stream, p, tile);
   return e == cudaSuccess ? MB_OK : MB_ERR_LAUNCH;
 }
 
@@ -210,7 +222,7 @@ using namespace mb::tanhseam;
 extern "C" int mb_tanh_seam(const MbTanhSeam* p, int dtype, cudaStream_t stream) {
   if (p->n_rows <= 0) return MB_OK;
   if (p->cols_pad <= 0 || p->cols_pad % 4 || p->ldx % 4 || p->lda % 4 || p->lde % 4 || p->ld_self % 4 || p->ld1 % 4 || p->ld_table % 4 ||
-      (p->e && p->top_k <= 0) || ((p->a || p->e) && !(p->w_u && p->b_u)) || (p->w1 && !(p->b1 && p->n1)))
+      (p->e && (p->top_k <= 0 || p->top_k > 32)) || ((p->a || p->e) && !(p->w_u && p->b_u)) || (p->w1 && !(p->b1 && p->n1)))
     return MB_ERR_SHAPE;
   // a shifted seam reads rows that another thread has already updated, unless the update goes elsewhere
   if (p->shift && (!p->w1 || p->rows || !p->prev || p->B <= 0 || p->x_out == p->x)) return MB_ERR_SHAPE;
