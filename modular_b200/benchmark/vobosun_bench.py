@@ -65,7 +65,7 @@ def run_kernels(s: dict, name: str, prefill: int = 2048, seqs: int = 4, batch: i
     """Every kernel of the design beside the like kernel of an existing family, same shapes, L2 flushed."""
     from ..nn.delta_rule import DeltaRule, DeltaRuleConfig, delta_rule_cuda
     from ..nn.general_delta import GeneralDelta, GeneralDeltaConfig
-    from ..nn.residual import residual_norm, sandwich_norm, tanh_seam
+    from ..nn.residual import sandwich_norm, tanh_seam
     from ..nn.rotary_embedding import cos_sin_table
     from ..nn.window_attention import block_prep, tensor_core_plan, window_attention
 

@@ -5,10 +5,11 @@
 //                             best `topk_group` groups, top-k experts inside them, weights from
 //                             the un-biased scores, optional normalisation, times a scaling factor.
 //   moe_router_softmax_topk   plain softmax top-k routing (Mixtral / Qwen style).
-//   moe_score_route           the group-limited choice (sigmoid or softmax scores, groups by their best or two best, identity
-//                             experts without weights among the candidates) with one warp per token, which also counts the pairs of every
-//   moe_place_rows            expert; the second kernel scans the counts and copies token rows into expert order, so a
-//                             routed layer costs two launches between its router product and its experts.
+//   moe_score_route           the group-limited choice with one warp per token (sigmoid or softmax scores, groups by their
+//   moe_place_rows            best or their two best, identity experts without weights among the candidates), which also
+//                             counts the pairs of every expert; the second kernel scans the counts and copies token rows
+//                             into expert order, so a routed layer costs two launches between its router product and its
+//                             experts.
 //   moe_table_route           routing by token id: a table names every id's experts, so the expert order of
 //                             all layers of a step is known before the first layer runs (one launch).
 //   moe_create_indices        counting sort of (token, slot) pairs by expert: CSR offsets per

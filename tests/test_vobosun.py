@@ -544,7 +544,7 @@ def test_router_config_checks():
 
 # ---------------------------------------------------------------------------------- whole models
 MIXED = config(attention(), (delta(), moe()), (attention(4, 4, 24, 56, 16, 700.0, 1.0), moe(5, 2, 0, None, 40, 0)), 1, (delta(2, 72), None),
-               (attention(heads=8, kv_heads=1, dim=48, vdim=40, dims=48, factor=0.5), None), (delta(5, 16), dense(64)), 0, 1)
+               (attention(heads=7, kv_heads=1, dim=56, vdim=40, dims=56, factor=0.5), None), (delta(5, 16), dense(64)), 0, 1)
 
 
 def clear_choices(t, dtype):
